@@ -38,6 +38,12 @@
  *                        one or two weight vectors, for layers whose sublayers run side by side on the same input
  *   pcs_gru_scan         element-wise gated recurrence whose gates read only the current token, S_t = (1 - z_t) S_(t-1) + z_t c_t,
  *                        with its silu output gate
+ *   pcs_group_norm_conv  residual sum of a sublayer result normed in groups of channels, then a short causal convolution over time
+ *                        of the NEW stream (its last inputs are carried in the slot pool) or a grouped norm of it
+ *   pcs_short_conv       per-channel causal convolution over time + silu of projections, query / key heads made unit vectors
+ *   pcs_delta_scan       gated delta rule with a decay per key channel, token by token;  pcs_delta_chunk_*: in chunks (prompts)
+ *   pcs_head_norm_gate   per-head RMS norm of a recurrence's result times an element-wise sigmoid gate
+ *   pcs_soft_cap         cap * tanh(z / cap)
  *   (pcs_attn with `talk`: every (query, key) pair's scores of all heads are mixed by an [H, H] matrix before the softmax)
  *
  * All tensor arguments are DEVICE pointers; `dtype` selects the compute / storage type of activations, weights and K/V
@@ -59,7 +65,7 @@
 extern "C" {
 #endif
 
-#define PCS_ABI_VERSION 4
+#define PCS_ABI_VERSION 5
 #define PCS_BF16 0
 #define PCS_F32 1
 
@@ -158,7 +164,18 @@ typedef struct pcs_attn_params {
   const void* out_gate;     /* [n_tokens, out_gate_stride] `dtype` or NULL: out[t, c] *= sigmoid(out_gate[t, c]) over all H * vdim columns
                                (an element-wise output gate, applied where the result is normalised; only with `talk`) */
   int64_t out_gate_stride;
-} pcs_attn_params;
+  const float* head_scale;  /* [H] or NULL: the scaled score of head h is multiplied by head_scale[h] (before a bias) */
+  const float* bias_table;  /* [H, bias_len] or NULL: score += bias_table[h, min(i - j, bias_len - 1)] (any function of the distance,
+                               tabulated by the caller).  Not with bias_r1. */
+  int32_t bias_len;
+  int32_t chunk;            /* > 0: query i sees key j only if floor(i / chunk) == floor(j / chunk), positions counted from the
+                               sequence's start.  Not with a window. */
+  const void* head_gate;    /* [n_tokens, head_gate_stride] `dtype` or NULL: head h's result *= sigmoid(head_gate[t, h]) */
+  int64_t head_gate_stride;
+  float out_scale;          /* the result is multiplied by this before it is rounded (0 counts as 1) */
+  int32_t reserved;
+  int64_t out_stride;       /* elements between the result rows of neighbouring tokens (0: H * vdim) */
+} pcs_attn_params;        /* (head_scale to out_stride: not with `talk`) */
 /* scratch the key split of pcs_attn needs for n_tokens tokens */
 int64_t pcs_attn_workspace_floats(int n_tokens, int n_heads, int vdim);
 int pcs_attn(const pcs_attn_params* p, void* stream);
@@ -200,10 +217,10 @@ typedef struct pcs_mlstm_params {
 } pcs_mlstm_params;
 int pcs_mlstm_scan(const pcs_mlstm_params* p, void* stream);
 
-/* out[t, :] = table[ids[t], :] + pair[r, :], r = (prev_ids[t] * mul_prev + ids[t] * mul_cur) mod buckets, or r = buckets (the
+/* out[t, :] = table[ids[t], :] * scale + pair[r, :], r = (prev_ids[t] * mul_prev + ids[t] * mul_cur) mod buckets, or r = buckets (the
  * table's last row) where prev_ids[t] < 0 (a sequence's first token).  out fp32 [n, width]; pair [buckets + 1, width]. */
 int pcs_embed_bigram(const void* table, const void* pair, const int64_t* ids, const int64_t* prev_ids, float* out, int n_tokens,
-                     int width, int vocab, int64_t buckets, int64_t mul_prev, int64_t mul_cur, int dtype, void* stream);
+                     int width, int vocab, float scale, int64_t buckets, int64_t mul_prev, int64_t mul_cur, int dtype, void* stream);
 
 /* Per token t:  x[t] += y_mult * y[t]  (y may be NULL),  u[t] = x[t] / sqrt(mean(x[t]^2) + eps) * g,
  *               h_out[t] = u[t] + sum_{j < taps} conv_w[j, :] * u[t - taps + 1 + j]        (conv_w NULL: h_out = u)
@@ -253,6 +270,9 @@ typedef struct pcs_rope_params {
   int32_t n_tokens, dtype;
   const void* q_norm_w;     /* [dim] `dtype` or NULL: every query head is divided by sqrt(mean(q^2) + eps) and multiplied by this, */
   const void* k_norm_w;     /* [dim] or NULL: the same for every key head; both before the rotation, in 32-bit */
+  int32_t norm_whole;       /* 1: the norms run over the WHOLE query and the whole key projection instead of head by head, and the
+                               weights are [n_heads * dim] and [n_kv_heads * dim] */
+  int32_t impl;             /* 0 = automatic, 1 = the element-wise kernel */
 } pcs_rope_params;
 int pcs_rope_kv_prep(const pcs_rope_params* p, void* stream);
 
@@ -285,6 +305,8 @@ int pcs_moe_route(const pcs_route_params* p, void* stream);
  * u' = clamp(u, -limit, limit), g' * sigmoid(alpha * g') * (u' + 1).  A NULL pointer means PCS_GLU_SILU. */
 #define PCS_GLU_SILU 0
 #define PCS_GLU_CLAMPED_SWISH 1
+/* PCS_GLU_GELU_TANH  g/2 * (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))) * u */
+#define PCS_GLU_GELU_TANH 4
 /* Activations of a feed-forward WITHOUT a gate branch (one up-projection): the weights are [n_experts, ff, width], a "gu" matrix
  * holds ff columns, and the second argument of the activation does not exist.
  *   PCS_ACT_RELU2     max(z, 0)^2            PCS_ACT_GELU_ERF   z/2 * (1 + erf(z / sqrt 2)) */
@@ -439,9 +461,11 @@ int pcs_head_gate(const void* o, int64_t o_tok_stride, int64_t o_head_stride, co
                   int n_heads, int vdim, int dtype, void* stream);
 
 /* Gated linear attention.  log decay per key channel: ld[t, c] = logsigmoid(sum_r a2[c, r] * a[t, r] + a2_b[c]) / tau   (fp32
- * [n_tokens, n_channels]); `a` is `dtype` [n_tokens, a_stride] with `rank` numbers per token, a2 `dtype` [n_channels, rank]. */
+ * [n_tokens, n_channels]); `a` is `dtype` [n_tokens, a_stride] with `rank` numbers per token, a2 `dtype` [n_channels, rank].
+ * With `rate` (fp32, one per `rate_dim` neighbouring channels): ld[t, c] = -rate[c / rate_dim] * softplus(the same sum) instead.
+ * `expo` 1: the decay exp(ld) itself is written. */
 int pcs_gla_decay(const void* a, int64_t a_stride, const void* a2, const float* a2_b, float* ld, int n_tokens, int n_channels, int rank,
-                  float tau, int dtype, void* stream);
+                  float tau, const float* rate, int rate_dim, int expo, int dtype, void* stream);
 
 /* Per entry and head, token by token:  S <- diag(exp(ld_t)) S + k_t v_t^T,  o_t = S^T (q_t * q_scale);  then
  * out[t, h, :] = o_t / sqrt(mean(o_t^2) + eps) * norm_w * silu(g[t, h, :])   (norm_w [vdim], shared by the heads).
@@ -508,7 +532,141 @@ typedef struct pcs_gru_params {
 } pcs_gru_params;
 int pcs_gru_scan(const pcs_gru_params* p, void* stream);
 
-/* The same recurrence in chunks of `chunk` tokens (prompts).  The step's entries are cut into chunks (an entry's last one may
+/* Residual sum with a norm in groups of channels, and what the next sublayer reads.  gn(z) divides each of `groups` equal runs of
+ * neighbouring channels by its own sqrt(mean(z^2) + eps).  Per output row r (row = rows ? rows[r] : r):
+ *   s[row]  = x[row] + gn(y[row]) * w                      (y NULL: s = x), stored to x_out[row] unless x_out is NULL
+ *   conv_w given:  h_out[row] = s[row] + sum_{j < taps} conv_w[j, :] * s[row's token - taps + 1 + j]      (not with `rows`)
+ *   next_w given:  h_out[r] = gn(s[row]) * next_w
+ * s of tokens before the sequence's start is zero; s of earlier steps' tokens comes from `tail`, which is kept twice and used as
+ * pcs_norm_conv does.  With conv_w a block forms the neighbours' sums again from x and y, so x_out must not alias x (unless y is NULL
+ * and x_out too). */
+typedef struct pcs_gnconv_params {
+  const float* x;           /* [*, width] */
+  float* x_out;             /* [*, width] or NULL */
+  const void* y;            /* [*, y_stride] `dtype` or NULL */
+  int64_t y_stride;
+  const void* w;            /* [width] `dtype` */
+  const void* next_w;       /* [width] `dtype` or NULL */
+  const void* conv_w;       /* [taps, width] `dtype` or NULL */
+  float* tail;              /* [slots, 2, taps - 1, width] fp32 */
+  void* h_out;              /* [n_rows, width] `dtype` or NULL */
+  const int32_t* rows;      /* [n_rows] or NULL */
+  const int32_t* tok_seq;
+  const int32_t* tok_pos;
+  const int32_t* seq_slot;
+  const int32_t* seq_pos0;
+  const int32_t* seq_len;
+  const int32_t* seq_par;
+  int32_t n_rows, width, groups, taps;
+  float eps;
+  int32_t dtype;
+  int32_t impl;             /* 0 = automatic, 1 = the element-wise kernel */
+  int32_t reserved;
+} pcs_gnconv_params;
+int pcs_group_norm_conv(const pcs_gnconv_params* p, void* stream);
+
+/* out[r, c] = cap * tanh(z[r, c] / cap), fp32 (cap <= 0: a copy);  z `dtype` [n_rows, z_stride] */
+int pcs_soft_cap(const void* z, int64_t z_stride, float* out, int n_rows, int width, float cap, int dtype, void* stream);
+
+/* Short causal convolution over time with silu, per channel c of proj[t, c_off + c], c < 2 * kv_heads * dim + v_width:
+ *   a[t, c] = silu(sum_{j < taps} conv_w[j, c] * proj[token t - taps + 1 + j, c_off + c])      (zeros before the sequence's start)
+ * The first kv_heads * dim channels are query heads, the next as many key heads: every head becomes a unit vector,
+ * a / sqrt(sum(a^2) + unit_eps) (queries also times q_scale), written in 32-bit to qk_out [n_tokens, 2 * kv_heads * dim]; the
+ * rest goes to v_out [n_tokens, v_width] in `dtype`.  Inputs of earlier steps come from `tail` (kept twice, as in pcs_norm_conv). */
+typedef struct pcs_shortconv_params {
+  const void* proj;
+  int64_t row_stride;
+  int32_t c_off, kv_heads, dim, v_width, taps;
+  float q_scale, unit_eps;
+  const void* conv_w;       /* [taps, 2 * kv_heads * dim + v_width] `dtype` */
+  float* tail;              /* [slots, 2, taps - 1, 2 * kv_heads * dim + v_width] fp32 */
+  float* qk_out;
+  void* v_out;
+  const int32_t* tok_seq;
+  const int32_t* tok_pos;
+  const int32_t* seq_slot;
+  const int32_t* seq_pos0;
+  const int32_t* seq_len;
+  const int32_t* seq_par;
+  int32_t n_tokens, dtype;
+  int32_t impl;             /* 0 = automatic, 1 = the element-wise kernel */
+  int32_t reserved;
+} pcs_shortconv_params;
+int pcs_short_conv(const pcs_shortconv_params* p, void* stream);
+
+/* Gated delta rule, token by token.  Per entry and head h (query / key head h / (heads / kv_heads)):
+ *   S <- diag(decay_t) S;  u = sigmoid(b[t, h]) * (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t
+ * S is fp32 [slots, heads, dim, vdim] in the slot pool; an entry whose slot holds no tokens starts from zero. */
+typedef struct pcs_delta_params {
+  const float* qk;          /* [n_tokens, 2 * kv_heads * dim]: queries, then keys (already normed and scaled) */
+  const void* v;            /* [n_tokens, heads * vdim] `dtype` */
+  const float* decay;       /* [n_tokens, heads * dim]: the decays themselves */
+  const void* b;            /* [n_tokens, b_stride] `dtype` */
+  int64_t b_stride;
+  float* o;                 /* fp32 [n_tokens, heads * vdim] */
+  float* s_pool;
+  int32_t heads, kv_heads, dim, vdim;
+  const int32_t* seq_slot;
+  const int32_t* seq_pos0;
+  const int32_t* seq_len;
+  const int32_t* seq_off;
+  int32_t n_seqs, n_tokens, dtype;
+  int32_t impl;             /* 0 = automatic, 1 = the kernel with the state in shared memory */
+} pcs_delta_params;
+int pcs_delta_scan(const pcs_delta_params* p, void* stream);
+
+/* The same in chunks of PCS_DELTA_CHUNK tokens (prompts; dim <= 256).  With B_i the running sum of the log decays inside a chunk,
+ * e its last token, A[i, s] = sum_d k_i k_s exp(B_i - B_s) (s < i), M = I + diag(beta) A, and L = round up dim to a multiple of 64:
+ *   pcs_delta_chunk_prep   qd[c, h, i, :] = q_i exp(B_i);  g[c, h, :] = exp(B_e);  a[c, h, i, s] = sum_d q_i k_s exp(B_i - B_s) for s <= i, else 0
+ *                          w[c, h, d, :]  = column d of M^-1 diag(beta) K exp(B)        (element 4 (i % 16) + i / 16 belongs to token i)
+ *                          kd[c, h, i, :] = k_i exp(B_e - B_i), padded to L               (element 64 t + 4 r + n belongs to channel 64 t + r + 16 n)
+ *                          u[c, h, i, :]  = row i of M^-1 diag(beta) V                    (every exponent formed is <= 0)
+ *   pcs_delta_chunk_scan   per entry, over its chunks in order, S from the pool:  u[c] <- u[c] - w[c] S;  s[c] = S;  S <- g S + kd[c]^T u[c]
+ *   (the caller forms o[c, h] = qd[c, h] s[c, h] + a[c, h] u[c, h], fp32 [chunks, heads, 64, vdim]) */
+#define PCS_DELTA_CHUNK 64
+typedef struct pcs_delta_chunk_params {
+  const float* qk;
+  const void* v;
+  const float* ld;             /* [n_tokens, heads * dim] log decays */
+  const void* b;
+  int64_t b_stride;
+  int32_t heads, kv_heads, dim, vdim;
+  const int32_t* chunk_first;  /* [n_chunks] */
+  const int32_t* chunk_len;    /* [n_chunks] */
+  int32_t n_chunks, n_tokens, dtype, n_seqs;
+  float* qd;                   /* [chunks, heads, 64, dim] */
+  float* kd;                   /* [chunks, heads, 64, L] */
+  float* w;                    /* [chunks, heads, dim, 64] */
+  float* g;                    /* [chunks, heads, dim] */
+  float* u;                    /* [chunks, heads, 64, vdim] */
+  float* a;                    /* [chunks, heads, 64, 64] */
+  float* s;                    /* [chunks, heads, dim, vdim] */
+  float* s_pool;
+  const int32_t* seq_slot;
+  const int32_t* seq_pos0;
+  const int32_t* seq_chunk0;   /* [n_seqs] first chunk of the entry */
+  const int32_t* seq_chunks;   /* [n_seqs] number of its chunks */
+} pcs_delta_chunk_params;
+int pcs_delta_chunk_prep(const pcs_delta_chunk_params* p, void* stream);
+int pcs_delta_chunk_scan(const pcs_delta_chunk_params* p, void* stream);
+
+/* out[t * out_stride + h * vdim + c] = o / sqrt(mean_c(o^2) + eps) * w[c] * sigmoid(g[t * g_stride + h * vdim + c]) * out_scale, o fp32: row
+ * (t, h) of [n_tokens, heads, vdim], or with tok_row (token -> chunk * chunk_size + place) of [chunks, heads, chunk_size, vdim] */
+typedef struct pcs_headnorm_params {
+  const float* o;
+  const int32_t* tok_row;   /* [n_tokens] or NULL */
+  const void* w;            /* [vdim] `dtype` */
+  const void* g;            /* `dtype` */
+  int64_t g_stride;
+  void* out;                /* `dtype` */
+  int64_t out_stride;
+  int32_t n_tokens, heads, vdim, chunk_size;
+  float eps, out_scale;
+  int32_t dtype, reserved;
+} pcs_headnorm_params;
+int pcs_head_norm_gate(const pcs_headnorm_params* p, void* stream);
+
+/* The recurrence of pcs_gla_scan in chunks of `chunk` tokens (prompts).  The step's entries are cut into chunks (an entry's last one may
  * be short); chunk c holds tokens chunk_first[c] .. chunk_first[c] + chunk_len[c] - 1 of the concatenated matrix.  With B_i the
  * running sum of the log decays inside a chunk (per key channel) and e its last token:
  *   pcs_gla_chunk_prep   qd[c, h, i, :] = q_i * q_scale * exp(B_i)        kd[c, h, i, :] = k_i * exp(B_e - B_i)     (fp32 [chunks, H, chunk, dim])

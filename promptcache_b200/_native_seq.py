@@ -20,8 +20,9 @@ EXPORTS = ("pcs_version", "pcs_last_error", "pcs_launch_count", "pcs_attn_worksp
            "pcs_qk_prep", "pcs_attn", "pcs_mlstm_gates", "pcs_mlstm_scan", "pcs_embed_bigram", "pcs_norm_conv", "pcs_rope_kv_prep", "pcs_moe_route",
            "pcs_moe_rows_up", "pcs_moe_rows_down", "pcs_moe_plan", "pcs_moe_gather", "pcs_moe_gemm", "pcs_moe_combine", "pcs_silu_mul", "pcs_glu_mul",
            "pcs_depth_mix", "pcs_latent_prep", "pcs_latent_q", "pcs_latent_gather", "pcs_latent_expand", "pcs_head_gate", "pcs_gla_decay", "pcs_gla_scan", "pcs_gla_chunk_prep", "pcs_gla_chunk_scan", "pcs_gla_chunk_out",
-           "pcs_add_layer_norm", "pcs_gru_scan")
-GLU_SILU, GLU_CLAMPED_SWISH = 0, 1
+           "pcs_add_layer_norm", "pcs_gru_scan", "pcs_group_norm_conv", "pcs_soft_cap", "pcs_short_conv", "pcs_delta_scan", "pcs_delta_chunk_prep", "pcs_delta_chunk_scan",
+           "pcs_head_norm_gate")
+GLU_SILU, GLU_CLAMPED_SWISH, GLU_GELU_TANH = 0, 1, 4
 ACT_RELU2, ACT_GELU_ERF = 2, 3          # activations of a feed-forward without a gate branch
 ROUTE_SOFTMAX, ROUTE_SIGMOID = 0, 1
 
@@ -54,7 +55,9 @@ class pcs_attn_params(C.Structure):
                 ("impl", C.c_int32), ("max_keys", C.c_int32), ("workspace", C.c_void_p), ("workspace_floats", C.c_int64),
                 ("softcap", C.c_float), ("window", C.c_int32), ("keep_first", C.c_int32), ("v_row_stride", C.c_int32),
                 ("sink_logit", C.c_void_p), ("pool_slot", C.c_void_p), ("talk", C.c_void_p),
-                ("out_gate", C.c_void_p), ("out_gate_stride", C.c_int64)]
+                ("out_gate", C.c_void_p), ("out_gate_stride", C.c_int64), ("head_scale", C.c_void_p), ("bias_table", C.c_void_p), ("bias_len", C.c_int32),
+                ("chunk", C.c_int32), ("head_gate", C.c_void_p), ("head_gate_stride", C.c_int64), ("out_scale", C.c_float), ("reserved", C.c_int32),
+                ("out_stride", C.c_int64)]
 
 
 class pcs_normconv_params(C.Structure):
@@ -70,7 +73,7 @@ class pcs_rope_params(C.Structure):
                 ("freqs", C.c_void_p), ("rot_dims", C.c_int32), ("interleaved", C.c_int32), ("v_unit_rms", C.c_int32), ("eps", C.c_float),
                 ("q_out", C.c_void_p), ("k_pool", C.c_void_p), ("v_pool", C.c_void_p), ("cap", C.c_int32),
                 ("tok_seq", C.c_void_p), ("tok_pos", C.c_void_p), ("seq_slot", C.c_void_p), ("n_tokens", C.c_int32), ("dtype", C.c_int32),
-                ("q_norm_w", C.c_void_p), ("k_norm_w", C.c_void_p)]
+                ("q_norm_w", C.c_void_p), ("k_norm_w", C.c_void_p), ("norm_whole", C.c_int32), ("impl", C.c_int32)]
 
 
 class pcs_route_params(C.Structure):
@@ -148,6 +151,40 @@ class pcs_gru_params(C.Structure):
                 ("seq_off", C.c_void_p), ("n_seqs", C.c_int32), ("n_tokens", C.c_int32), ("max_len", C.c_int32), ("dtype", C.c_int32)]
 
 
+class pcs_gnconv_params(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("x_out", C.c_void_p), ("y", C.c_void_p), ("y_stride", C.c_int64), ("w", C.c_void_p), ("next_w", C.c_void_p),
+                ("conv_w", C.c_void_p), ("tail", C.c_void_p), ("h_out", C.c_void_p), ("rows", C.c_void_p), ("tok_seq", C.c_void_p), ("tok_pos", C.c_void_p),
+                ("seq_slot", C.c_void_p), ("seq_pos0", C.c_void_p), ("seq_len", C.c_void_p), ("seq_par", C.c_void_p), ("n_rows", C.c_int32), ("width", C.c_int32),
+                ("groups", C.c_int32), ("taps", C.c_int32), ("eps", C.c_float), ("dtype", C.c_int32), ("impl", C.c_int32), ("reserved", C.c_int32)]
+
+
+class pcs_shortconv_params(C.Structure):
+    _fields_ = [("proj", C.c_void_p), ("row_stride", C.c_int64), ("c_off", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("v_width", C.c_int32),
+                ("taps", C.c_int32), ("q_scale", C.c_float), ("unit_eps", C.c_float), ("conv_w", C.c_void_p), ("tail", C.c_void_p), ("qk_out", C.c_void_p),
+                ("v_out", C.c_void_p), ("tok_seq", C.c_void_p), ("tok_pos", C.c_void_p), ("seq_slot", C.c_void_p), ("seq_pos0", C.c_void_p), ("seq_len", C.c_void_p),
+                ("seq_par", C.c_void_p), ("n_tokens", C.c_int32), ("dtype", C.c_int32), ("impl", C.c_int32), ("reserved", C.c_int32)]
+
+
+class pcs_delta_params(C.Structure):
+    _fields_ = [("qk", C.c_void_p), ("v", C.c_void_p), ("decay", C.c_void_p), ("b", C.c_void_p), ("b_stride", C.c_int64), ("o", C.c_void_p), ("s_pool", C.c_void_p),
+                ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("seq_slot", C.c_void_p), ("seq_pos0", C.c_void_p),
+                ("seq_len", C.c_void_p), ("seq_off", C.c_void_p), ("n_seqs", C.c_int32), ("n_tokens", C.c_int32), ("dtype", C.c_int32), ("impl", C.c_int32)]
+
+
+class pcs_delta_chunk_params(C.Structure):
+    _fields_ = [("qk", C.c_void_p), ("v", C.c_void_p), ("ld", C.c_void_p), ("b", C.c_void_p), ("b_stride", C.c_int64), ("heads", C.c_int32), ("kv_heads", C.c_int32),
+                ("dim", C.c_int32), ("vdim", C.c_int32), ("chunk_first", C.c_void_p), ("chunk_len", C.c_void_p), ("n_chunks", C.c_int32), ("n_tokens", C.c_int32),
+                ("dtype", C.c_int32), ("n_seqs", C.c_int32), ("qd", C.c_void_p), ("kd", C.c_void_p), ("w", C.c_void_p), ("g", C.c_void_p), ("u", C.c_void_p),
+                ("a", C.c_void_p), ("s", C.c_void_p), ("s_pool", C.c_void_p), ("seq_slot", C.c_void_p), ("seq_pos0", C.c_void_p), ("seq_chunk0", C.c_void_p),
+                ("seq_chunks", C.c_void_p)]
+
+
+class pcs_headnorm_params(C.Structure):
+    _fields_ = [("o", C.c_void_p), ("tok_row", C.c_void_p), ("w", C.c_void_p), ("g", C.c_void_p), ("g_stride", C.c_int64), ("out", C.c_void_p), ("out_stride", C.c_int64),
+                ("n_tokens", C.c_int32), ("heads", C.c_int32), ("vdim", C.c_int32), ("chunk_size", C.c_int32), ("eps", C.c_float), ("out_scale", C.c_float),
+                ("dtype", C.c_int32), ("reserved", C.c_int32)]
+
+
 class pcs_mlstm_params(C.Structure):
     _fields_ = [("proj", C.c_void_p), ("row_stride", C.c_int64),
                 ("q_off", C.c_int32), ("k_off", C.c_int32), ("v_off", C.c_int32), ("g_off", C.c_int32),
@@ -190,7 +227,7 @@ def load() -> C.CDLL:
     lib.pcs_mlstm_scan.argtypes = [C.POINTER(pcs_mlstm_params), C.c_void_p]
     lib.pcs_attn_workspace_floats.argtypes = [C.c_int, C.c_int, C.c_int]
     lib.pcs_attn_workspace_floats.restype = C.c_int64
-    lib.pcs_embed_bigram.argtypes = [C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_int64, C.c_int64,
+    lib.pcs_embed_bigram.argtypes = [C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_float, C.c_int64, C.c_int64,
                                      C.c_int64, C.c_int, C.c_void_p]
     lib.pcs_norm_conv.argtypes = [C.POINTER(pcs_normconv_params), C.c_void_p]
     lib.pcs_rope_kv_prep.argtypes = [C.POINTER(pcs_rope_params), C.c_void_p]
@@ -216,12 +253,20 @@ def load() -> C.CDLL:
     lib.pcs_latent_gather.argtypes = [C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_void_p, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_void_p]
     lib.pcs_latent_expand.argtypes = [C.POINTER(pcs_latent_expand_params), C.c_void_p]
     lib.pcs_head_gate.argtypes = [C.c_void_p, C.c_int64, C.c_int64, C.c_void_p, C.c_int64, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_int, C.c_void_p]
-    lib.pcs_gla_decay.argtypes = [C.c_void_p, C.c_int64, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_float, C.c_int, C.c_void_p]
+    lib.pcs_gla_decay.argtypes = [C.c_void_p, C.c_int64, C.c_void_p, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_float, C.c_void_p, C.c_int,
+                                  C.c_int, C.c_int, C.c_void_p]
     lib.pcs_gla_scan.argtypes = [C.POINTER(pcs_gla_params), C.c_void_p]
     for name in ("pcs_gla_chunk_prep", "pcs_gla_chunk_scan", "pcs_gla_chunk_out"):
         getattr(lib, name).argtypes = [C.POINTER(pcs_gla_chunk_params), C.c_void_p]
     lib.pcs_add_layer_norm.argtypes = [C.POINTER(pcs_addln_params), C.c_void_p]
     lib.pcs_gru_scan.argtypes = [C.POINTER(pcs_gru_params), C.c_void_p]
+    lib.pcs_group_norm_conv.argtypes = [C.POINTER(pcs_gnconv_params), C.c_void_p]
+    lib.pcs_soft_cap.argtypes = [C.c_void_p, C.c_int64, C.c_void_p, C.c_int, C.c_int, C.c_float, C.c_int, C.c_void_p]
+    lib.pcs_short_conv.argtypes = [C.POINTER(pcs_shortconv_params), C.c_void_p]
+    lib.pcs_delta_scan.argtypes = [C.POINTER(pcs_delta_params), C.c_void_p]
+    for name in ("pcs_delta_chunk_prep", "pcs_delta_chunk_scan"):
+        getattr(lib, name).argtypes = [C.POINTER(pcs_delta_chunk_params), C.c_void_p]
+    lib.pcs_head_norm_gate.argtypes = [C.POINTER(pcs_headnorm_params), C.c_void_p]
     for name in EXPORTS[4:]:
         getattr(lib, name).restype = C.c_int
     _lib = lib
@@ -391,7 +436,9 @@ def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: 
               r1: Optional[torch.Tensor], r2: Optional[torch.Tensor], sink: bool, batch: Batch, impl: int = 0,
               max_keys: int = 0, workspace: Optional[torch.Tensor] = None, softcap: float = 0.0, window: int = 0,
               keep_first: int = 0, sink_logit: Optional[torch.Tensor] = None, v_row_stride: int = 0,
-              pool_slot: Optional[torch.Tensor] = None, talk: Optional[torch.Tensor] = None, out_gate: Optional[torch.Tensor] = None) -> None:
+              pool_slot: Optional[torch.Tensor] = None, talk: Optional[torch.Tensor] = None, out_gate: Optional[torch.Tensor] = None,
+              head_scale: Optional[torch.Tensor] = None, bias_table: Optional[torch.Tensor] = None, chunk: int = 0,
+              head_gate: Optional[torch.Tensor] = None, out_scale: float = 1.0) -> None:
     """q [T, H*dim], out [T, H*vdim]; causal over each entry's own slot rows; r1 / r2 float32 [H] or None.  With a float32
     `workspace` (attn_workspace) and `max_keys` (upper bound of the keys a token sees) few tokens over many keys are run
     as several splits of the keys that a second launch merges.  `softcap` > 0 caps the scaled score by softcap * tanh(s /
@@ -400,8 +447,11 @@ def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: 
     elements after the previous key's (the values may be a leading part of the key rows: pass the key pool as v_pool too; vdim is
     then out's width per head).  `pool_slot` (int32 [entries]) replaces the batch's slots.  `talk` (float32 [H, H]): every (query, key)
     pair's scaled scores are mixed across heads, s'[h] = sum_g talk[h, g] s[g], before the mask and the softmax; with it, `out_gate`
-    ([T, H * vdim], row stride free): out *= sigmoid(out_gate), element by element."""
-    _cuda(q, k_pool, v_pool, out, r1, r2, sink_logit, pool_slot, talk)
+    ([T, H * vdim], row stride free): out *= sigmoid(out_gate), element by element.  `head_scale` (float32 [H]) multiplies the scaled
+    scores per head; `bias_table` (float32 [H, L]) adds bias_table[h, min(i - j, L - 1)]; `chunk` > 0 limits query i to the keys of
+    its own run of `chunk` positions; `head_gate` ([T, H], row stride free): out[t, h] *= sigmoid(head_gate[t, h]); `out_scale`
+    multiplies the result before it is rounded.  `out` may be a column range of a wider matrix."""
+    _cuda(q, k_pool, v_pool, out, r1, r2, sink_logit, pool_slot, talk, head_scale, bias_table, head_gate)
     if talk is not None and (talk.dtype != torch.float32 or tuple(talk.shape) != (n_heads, n_heads) or not talk.is_contiguous()):
         raise NativeError("attention: talk must be contiguous float32 [H, H]")
     if sink_logit is not None and (sink_logit.dtype != torch.float32 or sink_logit.numel() != n_heads or not sink_logit.is_contiguous()):
@@ -409,9 +459,9 @@ def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: 
     if pool_slot is not None and (pool_slot.dtype != torch.int32 or pool_slot.numel() != batch.n_seqs or not pool_slot.is_contiguous()):
         raise NativeError("attention: pool_slot must be int32 [entries]")
     dt = q.dtype
-    if not (q.is_contiguous() and out.is_contiguous() and k_pool.is_contiguous() and v_pool.is_contiguous()) or out.dtype != dt \
-            or k_pool.dtype != dt or v_pool.dtype != dt:
-        raise NativeError("attention: q, out and the pools must be contiguous tensors of one compute type")
+    _rows2d(out, dt, "attention: out")
+    if not (q.is_contiguous() and k_pool.is_contiguous() and v_pool.is_contiguous()) or k_pool.dtype != dt or v_pool.dtype != dt:
+        raise NativeError("attention: q and the pools must be contiguous tensors of one compute type")
     for r in (r1, r2):
         if r is not None and (r.dtype != torch.float32 or r.numel() != n_heads or not r.is_contiguous()):
             raise NativeError("attention: the distance-bias numbers must be float32 [H]")
@@ -425,6 +475,15 @@ def attention(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, out: 
         if out_gate.dtype != dt or out_gate.dim() != 2 or out_gate.stride(1) != 1 or tuple(out_gate.shape) != tuple(out.shape):
             raise NativeError("attention: out_gate must be [T, H * vdim] in the compute type with a contiguous inner dimension")
         p.out_gate, p.out_gate_stride = out_gate.data_ptr(), out_gate.stride(0)
+    if head_scale is not None and (head_scale.dtype != torch.float32 or head_scale.numel() != n_heads or not head_scale.is_contiguous()):
+        raise NativeError("attention: head_scale must be float32 [H]")
+    if bias_table is not None and (bias_table.dtype != torch.float32 or bias_table.dim() != 2 or bias_table.shape[0] != n_heads or not bias_table.is_contiguous()):
+        raise NativeError("attention: bias_table must be contiguous float32 [H, distances]")
+    if head_gate is not None and (head_gate.dtype != dt or head_gate.dim() != 2 or head_gate.stride(1) != 1 or tuple(head_gate.shape) != (q.shape[0], n_heads)):
+        raise NativeError("attention: head_gate must be [T, H] in the compute type with a contiguous inner dimension")
+    p.head_scale, p.bias_table, p.bias_len, p.chunk = _ptr(head_scale), _ptr(bias_table), bias_table.shape[1] if bias_table is not None else 0, int(chunk)
+    p.head_gate, p.head_gate_stride, p.out_scale = _ptr(head_gate), head_gate.stride(0) if head_gate is not None else 0, float(out_scale)
+    p.out_stride = out.stride(0) if out.shape[0] > 1 and out.stride(0) != out.shape[1] else 0
     p.scale, p.bias_r1, p.bias_r2, p.sink = float(scale), _ptr(r1), _ptr(r2), 1 if sink else 0
     p.tok_seq, p.tok_pos, p.seq_slot = batch.tok_seq.data_ptr(), batch.tok_pos.data_ptr(), batch.seq_slot.data_ptr()
     p.seq_pos0, p.seq_len, p.seq_off = batch.seq_pos0.data_ptr(), batch.seq_len.data_ptr(), batch.seq_off.data_ptr()
@@ -480,8 +539,8 @@ def mlstm_scan(proj: torch.Tensor, offs, ig: torch.Tensor, fg: torch.Tensor, nor
 
 
 def embed_bigram(table: torch.Tensor, pair: torch.Tensor, ids: torch.Tensor, prev_ids: torch.Tensor, out: torch.Tensor, buckets: int,
-                 mul_prev: int, mul_cur: int) -> None:
-    """out = table[ids] + pair[(prev * mul_prev + id * mul_cur) mod buckets], the pair table's last row where prev < 0."""
+                 mul_prev: int, mul_cur: int, scale: float = 1.0) -> None:
+    """out = table[ids] * scale + pair[(prev * mul_prev + id * mul_cur) mod buckets], the pair table's last row where prev < 0."""
     _cuda(table, pair, ids, prev_ids, out)
     if ids.dtype != torch.int64 or prev_ids.dtype != torch.int64 or not ids.is_contiguous() or not prev_ids.is_contiguous() \
             or prev_ids.numel() != ids.numel() or out.dtype != torch.float32 or not out.is_contiguous():
@@ -489,7 +548,7 @@ def embed_bigram(table: torch.Tensor, pair: torch.Tensor, ids: torch.Tensor, pre
     if not (table.is_contiguous() and pair.is_contiguous()) or pair.dtype != table.dtype or pair.shape[0] != buckets + 1 or pair.shape[1] != table.shape[1]:
         raise NativeError("embed_bigram: the pair table must be [buckets + 1, width] in the embedding's type")
     _check(load().pcs_embed_bigram(table.data_ptr(), pair.data_ptr(), ids.data_ptr(), prev_ids.data_ptr(), out.data_ptr(), ids.numel(),
-                                   table.shape[1], table.shape[0], int(buckets), int(mul_prev), int(mul_cur), dtype_code(table.dtype), _stream()),
+                                   table.shape[1], table.shape[0], float(scale), int(buckets), int(mul_prev), int(mul_cur), dtype_code(table.dtype), _stream()),
            "pcs_embed_bigram")
 
 
@@ -527,15 +586,17 @@ def norm_conv(x: torch.Tensor, g: Optional[torch.Tensor], eps: float, h_out: Opt
 
 def rope_kv_prep(qkv: torch.Tensor, offs, n_heads: int, n_kv_heads: int, dim: int, vdim: int, freqs: Optional[torch.Tensor], rot_dims: int,
                  interleaved: bool, v_unit_rms: bool, eps: float, q_out: torch.Tensor, k_pool: Optional[torch.Tensor],
-                 v_pool: Optional[torch.Tensor], batch: Batch, q_norm_w: Optional[torch.Tensor] = None, k_norm_w: Optional[torch.Tensor] = None) -> None:
+                 v_pool: Optional[torch.Tensor], batch: Batch, q_norm_w: Optional[torch.Tensor] = None, k_norm_w: Optional[torch.Tensor] = None,
+                 norm_whole: bool = False, impl: int = 0) -> None:
     """qkv [T, *] with q / k / v at the column offsets `offs` (k and v offsets None: the layer appends no rows).  freqs: float64
     [rot_dims / 2] on the device.  `q_norm_w` / `k_norm_w` ([dim], shared by the heads): every query / key head is first divided by
-    its root mean square (eps inside the root) and multiplied by the weight."""
+    its root mean square (eps inside the root) and multiplied by the weight; with `norm_whole` the whole query and the whole key
+    projection are, and the weights are [H * dim] and [Hkv * dim].  impl 1: the element-wise kernel."""
     _cuda(qkv, q_out, k_pool, v_pool, freqs, q_norm_w, k_norm_w)
     dt = qkv.dtype
-    for w in (q_norm_w, k_norm_w):
-        if w is not None and (w.dtype != dt or not w.is_contiguous() or w.numel() != dim):
-            raise NativeError("rope_kv_prep: a head norm's weight must be contiguous [dim] in the compute type")
+    for w, n in ((q_norm_w, n_heads), (k_norm_w, n_kv_heads)):
+        if w is not None and (w.dtype != dt or not w.is_contiguous() or w.numel() != dim * (n if norm_whole else 1)):
+            raise NativeError("rope_kv_prep: a norm's weight must be contiguous [dim] (or [heads * dim], whole) in the compute type")
     _rows2d(qkv, dt, "rope_kv_prep: qkv")
     if not q_out.is_contiguous() or q_out.dtype != dt:
         raise NativeError("rope_kv_prep: q_out must be contiguous in the compute type")
@@ -554,7 +615,7 @@ def rope_kv_prep(qkv: torch.Tensor, offs, n_heads: int, n_kv_heads: int, dim: in
         p.k_pool, p.v_pool, p.cap = k_pool.data_ptr(), v_pool.data_ptr(), k_pool.shape[2]
     p.tok_seq, p.tok_pos, p.seq_slot = batch.tok_seq.data_ptr(), batch.tok_pos.data_ptr(), batch.seq_slot.data_ptr()
     p.n_tokens, p.dtype = batch.n_tokens, dtype_code(dt)
-    p.q_norm_w, p.k_norm_w = _ptr(q_norm_w), _ptr(k_norm_w)
+    p.q_norm_w, p.k_norm_w, p.norm_whole, p.impl = _ptr(q_norm_w), _ptr(k_norm_w), 1 if norm_whole else 0, int(impl)
     _check(load().pcs_rope_kv_prep(C.byref(p), _stream()), "pcs_rope_kv_prep")
 
 
@@ -618,7 +679,7 @@ def moe_experts(h: torch.Tensor, idx: torch.Tensor, w_gu: torch.Tensor, w_down: 
     dt = h.dtype
     _rows2d(h, dt, "moe_experts: h")
     E, ff2, W = w_gu.shape
-    gated = act is None or int(act[0]) in (GLU_SILU, GLU_CLAMPED_SWISH)
+    gated = act is None or int(act[0]) in (GLU_SILU, GLU_CLAMPED_SWISH, GLU_GELU_TANH)
     ff = ff2 // 2 if gated else ff2
     if w_gu.dtype != dt or w_down.dtype != dt or not (w_gu.is_contiguous() and w_down.is_contiguous()) or tuple(w_down.shape) != (E, W, ff) \
             or idx.dtype != torch.int32 or not idx.is_contiguous() or W != h.shape[1]:
@@ -826,15 +887,18 @@ def head_gate(o: torch.Tensor, g: torch.Tensor, out: torch.Tensor) -> None:
            "pcs_head_gate")
 
 
-def gla_decay(a: torch.Tensor, a2: torch.Tensor, a2_b: Optional[torch.Tensor], tau: float) -> torch.Tensor:
-    """float32 [T, channels]: logsigmoid(a2 a + a2_b) / tau; a [T, rank] (row stride free), a2 [channels, rank]."""
-    _cuda(a, a2, a2_b)
+def gla_decay(a: torch.Tensor, a2: torch.Tensor, a2_b: Optional[torch.Tensor], tau: float, rate: Optional[torch.Tensor] = None, expo: bool = False) -> torch.Tensor:
+    """float32 [T, channels]: logsigmoid(a2 a + a2_b) / tau; a [T, rank] (row stride free), a2 [channels, rank].  With `rate` (float32,
+    one per equal run of channels): -rate * softplus(a2 a + a2_b) instead.  `expo`: the decay itself, exp of it."""
+    _cuda(a, a2, a2_b, rate)
+    if rate is not None and (rate.dtype != torch.float32 or not rate.is_contiguous() or a2.shape[0] % rate.numel()):
+        raise NativeError("gla_decay: rate must be float32, one per equal run of channels")
     _rows2d(a, a2.dtype, "gla_decay: a")
     if not a2.is_contiguous() or a2.shape[1] != a.shape[1] or (a2_b is not None and (a2_b.dtype != torch.float32 or a2_b.numel() != a2.shape[0])):
         raise NativeError("gla_decay: a2 contiguous [channels, rank], the bias float32 [channels]")
     ld = torch.empty(a.shape[0], a2.shape[0], dtype=torch.float32, device=a.device)
     _check(load().pcs_gla_decay(a.data_ptr(), a.stride(0), a2.data_ptr(), _ptr(a2_b), ld.data_ptr(), a.shape[0], a2.shape[0], a2.shape[1], float(tau),
-                                dtype_code(a2.dtype), _stream()), "pcs_gla_decay")
+                                _ptr(rate), a2.shape[0] // rate.numel() if rate is not None else 0, 1 if expo else 0, dtype_code(a2.dtype), _stream()), "pcs_gla_decay")
     return ld
 
 
@@ -968,3 +1032,139 @@ def gru_scan(proj: torch.Tensor, offs, width: int, out: torch.Tensor, s_pool: to
                                                     batch.seq_off.data_ptr())
     p.n_seqs, p.n_tokens, p.max_len, p.dtype = batch.n_seqs, batch.n_tokens, batch.max_len, dtype_code(dt)
     _check(load().pcs_gru_scan(C.byref(p), _stream()), "pcs_gru_scan")
+
+
+def group_norm_conv(x: torch.Tensor, groups: int, eps: float, dtype: torch.dtype, x_out: Optional[torch.Tensor] = None, y: Optional[torch.Tensor] = None,
+                    w: Optional[torch.Tensor] = None, conv_w: Optional[torch.Tensor] = None, tail: Optional[torch.Tensor] = None, next_w: Optional[torch.Tensor] = None,
+                    h_out: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, batch: Optional[Batch] = None, impl: int = 0) -> None:
+    """s = x + gn(y) * w (y None: s = x) with gn a norm in `groups` equal runs of channels; x_out gets s.  Then with conv_w [taps, width] (the last
+    tap weighs the token itself): h_out = s + causal_conv(s), whose inputs of earlier steps sit in `tail` [slots, 2, taps - 1, width];
+    x_out must be another tensor than x.  Or with next_w: h_out = gn(s) * next_w, at `rows` (int32) only when given.  impl 1: the
+    element-wise kernel."""
+    _cuda(x, x_out, y, w, conv_w, tail, next_w, h_out, rows)
+    if x.dtype != torch.float32 or not x.is_contiguous() or x.dim() != 2:
+        raise NativeError("group_norm_conv: x must be a contiguous float32 matrix")
+    W = x.shape[1]
+    p = pcs_gnconv_params()
+    R = rows.numel() if rows is not None else x.shape[0]
+    if x_out is not None and (x_out.dtype != torch.float32 or not x_out.is_contiguous() or x_out.shape != x.shape):
+        raise NativeError("group_norm_conv: x_out must be contiguous float32 of x's shape")
+    if y is not None:
+        _rows2d(y, dtype, "group_norm_conv: y")
+        if y.shape != x.shape or w is None:
+            raise NativeError("group_norm_conv: y must have x's shape, with its norm weight given")
+        p.y, p.y_stride = y.data_ptr(), y.stride(0)
+    for v in (w, next_w):
+        if v is not None and (v.dtype != dtype or not v.is_contiguous() or v.numel() != W):
+            raise NativeError("group_norm_conv: norm weights must be contiguous [width] in the compute type")
+    if h_out is not None and (h_out.dtype != dtype or not h_out.is_contiguous() or tuple(h_out.shape) != (R, W)):
+        raise NativeError("group_norm_conv: h_out must be contiguous [rows, width] in the compute type")
+    if rows is not None and (rows.dtype != torch.int32 or not rows.is_contiguous()):
+        raise NativeError("group_norm_conv: rows must be contiguous int32")
+    if conv_w is not None:
+        taps = conv_w.shape[0]
+        if conv_w.dtype != dtype or not conv_w.is_contiguous() or conv_w.shape[1] != W or batch is None:
+            raise NativeError("group_norm_conv: conv_w must be contiguous [taps, width] in the compute type, with the batch given")
+        if taps > 1 and (tail is None or tail.dtype != torch.float32 or not tail.is_contiguous() or tuple(tail.shape[1:]) != (2, taps - 1, W)):
+            raise NativeError("group_norm_conv: tail must be contiguous float32 [slots, 2, taps - 1, width]")
+        p.conv_w, p.taps, p.tail = conv_w.data_ptr(), taps, _ptr(tail)
+        p.tok_seq, p.tok_pos, p.seq_slot = batch.tok_seq.data_ptr(), batch.tok_pos.data_ptr(), batch.seq_slot.data_ptr()
+        p.seq_pos0, p.seq_len, p.seq_par = batch.seq_pos0.data_ptr(), batch.seq_len.data_ptr(), batch.seq_par.data_ptr()
+    p.x, p.x_out, p.w, p.next_w, p.h_out, p.rows = x.data_ptr(), _ptr(x_out), _ptr(w), _ptr(next_w), _ptr(h_out), _ptr(rows)
+    p.n_rows, p.width, p.groups, p.eps, p.dtype, p.impl = R, W, int(groups), float(eps), dtype_code(dtype), int(impl)
+    _check(load().pcs_group_norm_conv(C.byref(p), _stream()), "pcs_group_norm_conv")
+
+
+def soft_cap(z: torch.Tensor, cap: float) -> torch.Tensor:
+    """float32 cap * tanh(z / cap); cap <= 0: z in float32."""
+    _cuda(z)
+    _rows2d(z, z.dtype, "soft_cap: z")
+    out = torch.empty(z.shape, dtype=torch.float32, device=z.device)
+    _check(load().pcs_soft_cap(z.data_ptr(), z.stride(0), out.data_ptr(), z.shape[0], z.shape[1], float(cap), dtype_code(z.dtype), _stream()), "pcs_soft_cap")
+    return out
+
+
+def short_conv(proj: torch.Tensor, c_off: int, kv_heads: int, dim: int, v_width: int, conv_w: torch.Tensor, tail: Optional[torch.Tensor], q_scale: float, unit_eps: float,
+               batch: Batch, impl: int = 0):
+    """(qk float32 [T, 2 * kv_heads * dim], v [T, v_width]): silu of a causal convolution over time of the projection columns from c_off on
+    (queries | keys | values), query and key heads as unit vectors, queries times q_scale.  conv_w [taps, channels]; `tail`
+    [slots, 2, taps - 1, channels] float32 carries the last inputs from step to step.  impl 1: the element-wise kernel."""
+    _cuda(proj, conv_w, tail)
+    dt = proj.dtype
+    _rows2d(proj, dt, "short_conv: proj")
+    U = 2 * kv_heads * dim
+    ch, taps, T = U + v_width, conv_w.shape[0], proj.shape[0]
+    if conv_w.dtype != dt or not conv_w.is_contiguous() or conv_w.shape[1] != ch or c_off + ch > proj.shape[1]:
+        raise NativeError("short_conv: conv_w must be contiguous [taps, channels] in the compute type, the channels inside proj")
+    if taps > 1 and (tail is None or tail.dtype != torch.float32 or not tail.is_contiguous() or tuple(tail.shape[1:]) != (2, taps - 1, ch)):
+        raise NativeError("short_conv: tail must be contiguous float32 [slots, 2, taps - 1, channels]")
+    qk, v = torch.empty(T, U, dtype=torch.float32, device=proj.device), torch.empty(T, v_width, dtype=dt, device=proj.device)
+    p = pcs_shortconv_params()
+    p.proj, p.row_stride, p.c_off, p.kv_heads, p.dim, p.v_width, p.taps = proj.data_ptr(), proj.stride(0), int(c_off), int(kv_heads), int(dim), int(v_width), taps
+    p.q_scale, p.unit_eps, p.conv_w, p.tail, p.qk_out, p.v_out = float(q_scale), float(unit_eps), conv_w.data_ptr(), _ptr(tail), qk.data_ptr(), v.data_ptr()
+    p.tok_seq, p.tok_pos, p.seq_slot = batch.tok_seq.data_ptr(), batch.tok_pos.data_ptr(), batch.seq_slot.data_ptr()
+    p.seq_pos0, p.seq_len, p.seq_par = batch.seq_pos0.data_ptr(), batch.seq_len.data_ptr(), batch.seq_par.data_ptr()
+    p.n_tokens, p.dtype, p.impl = T, dtype_code(dt), int(impl)
+    _check(load().pcs_short_conv(C.byref(p), _stream()), "pcs_short_conv")
+    return qk, v
+
+
+DELTA_CHUNK = 64          # PCS_DELTA_CHUNK
+DELTA_CHUNK_MIN_LEN = 32  # steps whose longest entry brings fewer tokens go token by token
+DELTA_CHUNK_MAX_DIM = 256
+
+
+def delta_takes_chunks(batch: Batch, dim: int, impl: int = 0) -> bool:
+    """Whether `delta_scan` runs a step in chunks (and wants log decays) or token by token (and wants the decays themselves)."""
+    if impl:
+        return impl == 3
+    return batch.max_len >= DELTA_CHUNK_MIN_LEN and dim <= DELTA_CHUNK_MAX_DIM and not torch.cuda.is_current_stream_capturing()
+
+
+def delta_scan(qk: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, b: torch.Tensor, kv_heads: int, s_pool: torch.Tensor, norm_w: torch.Tensor, gate: torch.Tensor,
+               out: torch.Tensor, eps: float, batch: Batch, out_scale: float = 1.0, impl: int = 0) -> None:
+    """The gated delta rule with its per-head norm and sigmoid gate.  qk float32 [T, 2 * kv_heads * dim] (unit vectors, queries scaled), v [T, H * vdim],
+    decay float32 [T, H * dim] (log decays where `delta_takes_chunks`, else the decays), b [T, H] pre-activations of the step sizes, gate
+    [T, H * vdim] pre-activations, state pool float32 [slots, H, dim, vdim]; out [T, H * vdim] (row stride free).  impl 0: by step;
+    1: token by token with the state in shared memory; 2: token by token (registers where the sizes allow); 3: in chunks."""
+    _cuda(qk, v, decay, b, s_pool, norm_w, gate, out)
+    dt = v.dtype
+    for t, what in ((b, "b"), (gate, "gate"), (out, "out")):
+        _rows2d(t, dt, f"delta_scan: {what}")
+    if s_pool.dtype != torch.float32 or not s_pool.is_contiguous() or s_pool.dim() != 4:
+        raise NativeError("delta_scan: the state pool must be contiguous float32 [slots, H, dim, vdim]")
+    H, D, V = s_pool.shape[1:]
+    T, dev = v.shape[0], v.device
+    if qk.dtype != torch.float32 or decay.dtype != torch.float32 or not (qk.is_contiguous() and v.is_contiguous() and decay.is_contiguous()) \
+            or tuple(qk.shape) != (T, 2 * kv_heads * D) or tuple(decay.shape) != (T, H * D) or tuple(v.shape) != (T, H * V) or tuple(b.shape) != (T, H):
+        raise NativeError("delta_scan: qk float32 [T, 2 * kv_heads * dim], decay float32 [T, H * dim], v [T, H * vdim], b [T, H]")
+    if norm_w.dtype != dt or norm_w.numel() != V or tuple(gate.shape) != (T, H * V) or tuple(out.shape) != (T, H * V):
+        raise NativeError("delta_scan: norm_w [vdim], gate and out [T, H * vdim] in the compute type")
+    n = pcs_headnorm_params()
+    if delta_takes_chunks(batch, D, impl):
+        ch = DELTA_CHUNK
+        plan = _gla_chunk_plan(batch, ch)
+        nc, L = plan["n_chunks"], (D + 63) // 64 * 64
+        new = lambda *s: torch.empty(*s, dtype=torch.float32, device=dev)
+        qd, kd, w, g, u, a, s = new(nc * H, ch, D), new(nc * H, ch, L), new(nc * H, D, ch), new(nc * H, D), new(nc * H, ch, V), new(nc * H, ch, ch), new(nc * H, D, V)
+        p = pcs_delta_chunk_params()
+        p.qk, p.v, p.ld, p.b, p.b_stride = qk.data_ptr(), v.data_ptr(), decay.data_ptr(), b.data_ptr(), b.stride(0)
+        p.heads, p.kv_heads, p.dim, p.vdim = H, int(kv_heads), D, V
+        p.chunk_first, p.chunk_len, p.n_chunks, p.n_tokens, p.dtype, p.n_seqs = plan["first"].data_ptr(), plan["len"].data_ptr(), nc, T, dtype_code(dt), batch.n_seqs
+        p.qd, p.kd, p.w, p.g, p.u, p.a, p.s, p.s_pool = (t.data_ptr() for t in (qd, kd, w, g, u, a, s, s_pool))
+        p.seq_slot, p.seq_pos0, p.seq_chunk0, p.seq_chunks = batch.seq_slot.data_ptr(), batch.seq_pos0.data_ptr(), plan["seq0"].data_ptr(), plan["seqn"].data_ptr()
+        _check(load().pcs_delta_chunk_prep(C.byref(p), _stream()), "pcs_delta_chunk_prep")
+        _check(load().pcs_delta_chunk_scan(C.byref(p), _stream()), "pcs_delta_chunk_scan")   # u: every token's correction; s: the chunks' start states
+        o = torch.baddbmm(torch.bmm(a, u), qd, s)             # [chunks * H, chunk, vdim]
+        n.tok_row, n.chunk_size = plan["tok_row"].data_ptr(), ch
+    else:
+        o = torch.empty(T, H * V, dtype=torch.float32, device=dev)
+        p = pcs_delta_params()
+        p.qk, p.v, p.decay, p.b, p.b_stride, p.o, p.s_pool = qk.data_ptr(), v.data_ptr(), decay.data_ptr(), b.data_ptr(), b.stride(0), o.data_ptr(), s_pool.data_ptr()
+        p.heads, p.kv_heads, p.dim, p.vdim = H, int(kv_heads), D, V
+        p.seq_slot, p.seq_pos0, p.seq_len, p.seq_off = (batch.seq_slot.data_ptr(), batch.seq_pos0.data_ptr(), batch.seq_len.data_ptr(), batch.seq_off.data_ptr())
+        p.n_seqs, p.n_tokens, p.dtype, p.impl = batch.n_seqs, T, dtype_code(dt), 1 if impl == 1 else 0
+        _check(load().pcs_delta_scan(C.byref(p), _stream()), "pcs_delta_scan")
+    n.o, n.w, n.g, n.g_stride, n.out, n.out_stride = o.data_ptr(), norm_w.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(), out.stride(0)
+    n.n_tokens, n.heads, n.vdim, n.eps, n.out_scale, n.dtype = T, H, V, float(eps), float(out_scale), dtype_code(dt)
+    _check(load().pcs_head_norm_gate(C.byref(n), _stream()), "pcs_head_norm_gate")

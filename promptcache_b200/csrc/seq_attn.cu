@@ -177,16 +177,28 @@ constexpr int kAttnThreads = 128;
 constexpr int kAttnMaxVPT = 4;  // value columns per thread: vdim <= 512
 
 // The keys a query at position `pos` sees, as one dense index range: with a window, the kept first keys [0, n_first) and
-// then the window [lo, pos]; without one (or when the two touch), all of [0, pos].
+// then the window [lo, pos]; without one (or when the two touch), all of [0, pos].  With chunks, the keys of the query's own chunk.
 struct VisibleKeys {
   int n_first, lo, count;
-  __device__ __forceinline__ VisibleKeys(int pos, int window, int keep_first) {
-    lo = window > 0 ? max(0, pos - window + 1) : 0;
-    n_first = min(max(keep_first, 0), lo);
+  __device__ __forceinline__ VisibleKeys(int pos, int window, int keep_first, int chunk) {
+    lo = window > 0 ? max(0, pos - window + 1) : (chunk > 0 ? pos / chunk * chunk : 0);
+    n_first = chunk > 0 ? 0 : min(max(keep_first, 0), lo);
     count = n_first + (pos + 1 - lo);
   }
   __device__ __forceinline__ int key(int v) const { return v < n_first ? v : lo + (v - n_first); }
 };
+
+// where head h of token t is written, and what its normalised result is multiplied by: the constant and the head's gate
+template <typename T>
+__device__ __forceinline__ T* out_row(const pcs_attn_params& p, int t, int h) {
+  return static_cast<T*>(p.out) + static_cast<long long>(t) * (p.out_stride > 0 ? p.out_stride : static_cast<long long>(p.n_heads) * p.vdim) + h * p.vdim;
+}
+template <typename T>
+__device__ __forceinline__ float out_factor(const pcs_attn_params& p, int t, int h) {
+  float f = p.out_scale != 0.f ? p.out_scale : 1.f;
+  if (p.head_gate) f *= sigmoidf_(ldf(static_cast<const T*>(p.head_gate) + static_cast<long long>(t) * p.head_gate_stride + h));
+  return f;
+}
 
 template <typename T>
 __global__ void __launch_bounds__(kAttnThreads) attn_plain_kernel(const pcs_attn_params p) {
@@ -204,8 +216,10 @@ __global__ void __launch_bounds__(kAttnThreads) attn_plain_kernel(const pcs_attn
   const T* Vp = static_cast<const T*>(p.v_pool) + (static_cast<long long>(slot) * p.n_kv_heads + g) * p.cap * VS;
   for (int i = tid; i < D; i += kAttnThreads) qs[i] = ldf(q + i);
   const float r1 = p.bias_r1 ? p.bias_r1[h] : 0.f, r2 = p.bias_r1 ? p.bias_r2[h] : 0.f;
+  const float scale = p.scale * (p.head_scale ? p.head_scale[h] : 1.f);
+  const float* tab = p.bias_table ? p.bias_table + static_cast<long long>(h) * p.bias_len : nullptr;
   // keys are cut into gridDim.z splits of whole tiles; the sink belongs to split 0
-  const VisibleKeys vis(pos, p.window, p.keep_first);
+  const VisibleKeys vis(pos, p.window, p.keep_first, p.chunk);
   const int n_keys = vis.count, S = gridDim.z, sp = blockIdx.z;
   const int chunk = ((n_keys + S - 1) / S + kAttnThreads - 1) / kAttnThreads * kAttnThreads;
   const int k_begin = sp * chunk, k_end = min(n_keys, k_begin + chunk);
@@ -230,9 +244,10 @@ __global__ void __launch_bounds__(kAttnThreads) attn_plain_kernel(const pcs_attn
       } else {
         for (int d = 0; d < D; ++d) a = fmaf(qs[d], ldf(kr + d), a);
       }
-      s = a * p.scale;
+      s = a * scale;
       if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
       if (p.bias_r1) s -= r1 * log1pf(r2 * static_cast<float>(pos - j));
+      if (tab) s += tab[min(pos - j, p.bias_len - 1)];
     }
     const float tmax = block_max(s, red);
     const float m_new = fmaxf(m, tmax);
@@ -264,8 +279,8 @@ __global__ void __launch_bounds__(kAttnThreads) attn_plain_kernel(const pcs_attn
     }
     return;
   }
-  T* o = static_cast<T*>(p.out) + (static_cast<long long>(t) * p.n_heads + h) * V;
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  T* o = out_row<T>(p, t, h);
+  const float inv = (l > 0.f ? 1.f / l : 0.f) * out_factor<T>(p, t, h);
 #pragma unroll
   for (int u = 0; u < kAttnMaxVPT; ++u) {
     const int c = tid + u * kAttnThreads;
@@ -298,7 +313,9 @@ __global__ void __launch_bounds__(kAttnThreads) attn_decode_kernel(const pcs_att
   const T* Vp = static_cast<const T*>(p.v_pool) + (static_cast<long long>(slot) * p.n_kv_heads + g) * p.cap * VS;
   for (int i = tid; i < D; i += kAttnThreads) qs[i] = ldf(q + i);
   const float r1 = p.bias_r1 ? p.bias_r1[h] : 0.f, r2 = p.bias_r1 ? p.bias_r2[h] : 0.f;
-  const VisibleKeys vis(pos, p.window, p.keep_first);
+  const float scale = p.scale * (p.head_scale ? p.head_scale[h] : 1.f);
+  const float* tab = p.bias_table ? p.bias_table + static_cast<long long>(h) * p.bias_len : nullptr;
+  const VisibleKeys vis(pos, p.window, p.keep_first, p.chunk);
   const int n_keys = vis.count, S = gridDim.z, sp = blockIdx.z;
   const int chunk = ((n_keys + S - 1) / S + kAttnThreads - 1) / kAttnThreads * kAttnThreads;
   const int k_begin = sp * chunk, k_end = min(n_keys, k_begin + chunk);
@@ -339,9 +356,10 @@ __global__ void __launch_bounds__(kAttnThreads) attn_decode_kernel(const pcs_att
 #pragma unroll
         for (int e = 0; e < N; ++e) a0 = fmaf(qs[d + e], k0[e], a0);
       }
-      s = (a0 + a1) * p.scale;
+      s = (a0 + a1) * scale;
       if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
       if (p.bias_r1) s -= r1 * log1pf(r2 * static_cast<float>(pos - j));
+      if (tab) s += tab[min(pos - j, p.bias_len - 1)];
     }
     const float wm = warp_max(s);
     if ((tid & 31) == 0) red[tid >> 5] = wm;
@@ -394,8 +412,8 @@ __global__ void __launch_bounds__(kAttnThreads) attn_decode_kernel(const pcs_att
   for (int i = 0; i < kAttnThreads; ++i) l += lred[i];
   float* part = (S > 1) ? p.workspace + ((static_cast<long long>(t) * p.n_heads + h) * S + sp) * (V + 2) : nullptr;
   if (part && tid == 0) { part[0] = m; part[1] = l; }
-  T* o = static_cast<T*>(p.out) + (static_cast<long long>(t) * p.n_heads + h) * V;
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  T* o = out_row<T>(p, t, h);
+  const float inv = (l > 0.f ? 1.f / l : 0.f) * out_factor<T>(p, t, h);
   for (int col = tid; col < V; col += kAttnThreads) {
     float a = 0.f;
     for (int rr = 0; rr < R; ++rr) a += part_s[rr * V + col];
@@ -431,8 +449,8 @@ __global__ void __launch_bounds__(kAttnThreads) attn_combine_kernel(const pcs_at
     inv_s = L > 0.f ? 1.f / L : 0.f;
   }
   __syncthreads();
-  const float inv = inv_s;
-  T* o = static_cast<T*>(p.out) + (static_cast<long long>(t) * p.n_heads + h) * V;
+  const float inv = inv_s * out_factor<T>(p, t, h);
+  T* o = out_row<T>(p, t, h);
   // a block takes every gridDim.z-th group of 128 columns; a column's S values are requested together, then summed in order
   for (int c = blockIdx.z * blockDim.x + threadIdx.x; c < V; c += gridDim.z * blockDim.x) {
     float v[kAttnMaxSplits];
@@ -495,6 +513,12 @@ PCS_API int pcs_attn(const pcs_attn_params* p, void* stream) {
   PCS_REQUIRE((p->bias_r1 == nullptr) == (p->bias_r2 == nullptr), "pcs_attn: the distance bias needs both r1 and r2");
   PCS_REQUIRE(p->v_row_stride == 0 || p->v_row_stride >= p->vdim, "pcs_attn: the value row stride %d is below vdim %d", p->v_row_stride, p->vdim);
   PCS_REQUIRE(p->out_gate == nullptr || p->talk != nullptr, "pcs_attn: the element-wise output gate comes with mixed head scores only");
+  PCS_REQUIRE(p->bias_table == nullptr || (p->bias_len > 0 && p->bias_r1 == nullptr), "pcs_attn: a tabulated bias needs its length and excludes the logarithmic one");
+  PCS_REQUIRE(p->chunk <= 0 || p->window <= 0, "pcs_attn: chunks and a window exclude each other");
+  PCS_REQUIRE(p->out_stride == 0 || p->out_stride >= static_cast<int64_t>(p->n_heads) * p->vdim, "pcs_attn: the output row stride is below a row");
+  PCS_REQUIRE(p->talk == nullptr || (!p->head_scale && !p->bias_table && p->chunk <= 0 && !p->head_gate && (p->out_scale == 0.f || p->out_scale == 1.f) &&
+                                     (p->out_stride == 0 || p->out_stride == static_cast<int64_t>(p->n_heads) * p->vdim)),
+              "pcs_attn: mixed head scores come without per-head scales, tabulated biases, chunks, head gates and output scales or strides");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (p->talk) {  // scores mixed across heads: kernels of their own (a block needs all heads of a pair), the same split merge
     int talk_splits = 1;

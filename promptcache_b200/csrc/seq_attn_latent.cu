@@ -198,7 +198,7 @@ int launch_nt(const pcs_attn_params& p, cudaStream_t st, int DKP, int splits, si
 int launch_attn_latent(const pcs_attn_params& p, cudaStream_t st, int* splits_out) {
   *splits_out = 0;
   if (p.dtype != PCS_BF16 || p.n_kv_heads != 1 || p.v_pool != p.k_pool || p.v_row_stride != p.dim || p.workspace == nullptr) return PCS_OK;
-  if (p.bias_r1 || p.softcap > 0.f || p.window > 0 || p.dim % 8 != 0 || p.vdim % 8 != 0 || p.vdim > 512 || p.vdim > p.dim) return PCS_OK;
+  if (p.bias_r1 || p.bias_table || p.head_scale || p.softcap > 0.f || p.window > 0 || p.chunk > 0 || p.dim % 8 != 0 || p.vdim % 8 != 0 || p.vdim > 512 || p.vdim > p.dim) return PCS_OK;
   if ((reinterpret_cast<uintptr_t>(p.k_pool) | reinterpret_cast<uintptr_t>(p.q)) & 15) return PCS_OK;
   const int DKP = (p.dim + 31) / 32 * 32;
   const size_t smem = static_cast<size_t>(LB_HEADS + 2 * LB_N) * (DKP + LB_PAD) * sizeof(__nv_bfloat16);

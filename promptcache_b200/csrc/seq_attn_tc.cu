@@ -79,17 +79,19 @@ __global__ void __launch_bounds__(TC_THREADS, (DP <= 128 && VP <= 128) ? 3 : 1) 
   const int total_keys = pos0 + len;
   const int n_keys = min(total_keys, pos0 + q0 + BM);  // the last row of this tile sees keys below this bound
   const float r1 = p.bias_r1 ? p.bias_r1[h] : 0.f, r2 = p.bias_r1 ? p.bias_r2[h] : 0.f;
-  const bool bias = p.bias_r1 != nullptr;
+  const float* tab = p.bias_table ? p.bias_table + static_cast<long long>(h) * p.bias_len : nullptr;
+  const bool bias = p.bias_r1 != nullptr || tab != nullptr;
   // this thread's two query rows (grp, grp + 8 of the warp's 16) and their positions
   const int row_a = warp * 16 + grp, row_b = row_a + 8;
   const int pq_a = pos0 + q0 + row_a, pq_b = pos0 + q0 + row_b;
   // the bias r1 ln(1 + r2 d) depends on the distance d = i - j alone: 127 distances per tile, computed once per tile into
-  // shared memory in the base-2 domain (r1 log2(1 + r2 d)).  A thread's two scores of an 8-key group are neighbours in
+  // shared memory in the base-2 domain (r1 log2(1 + r2 d), or the caller's tabulated bias with its sign turned).  A thread's two scores of an 8-key group are neighbours in
   // the table; two copies, one shifted by an entry, keep every thread's float2 read aligned whatever its row's parity.
   float* T0 = reinterpret_cast<float*>(Vbuf + BN * (VP + PAD));
   float* T1 = T0 + 144;  // 16 banks away from T0: the odd and the even rows of a warp read different banks
   const float* tp_a = (row_a & 1) ? T0 + (63 - row_a + qd * 2) : T1 + (62 - row_a + qd * 2);
-  const float scale2 = p.scale * 1.4426950408889634f;
+  const float scale = p.scale * (p.head_scale ? p.head_scale[h] : 1.f);
+  const float scale2 = scale * 1.4426950408889634f;
   float m_a = p.sink ? (p.sink_logit ? p.sink_logit[h] * 1.4426950408889634f : 0.f) : -INFINITY, m_b = m_a;  // base-2 domain
   float l_a = (p.sink && qd == 0) ? 1.f : 0.f, l_b = l_a;  // per-thread share of the row sums; the sink's 1 sits in one lane
   float o[VP / 8][4];
@@ -109,8 +111,17 @@ __global__ void __launch_bounds__(TC_THREADS, (DP <= 128 && VP <= 128) ? 3 : 1) 
     n_first = (min(max(p.keep_first, 0), total_keys) + BN - 1) / BN;
     if (n_first >= lo_tile) { n_first = 0; lo_tile = 0; }
   }
+  // with chunks a row sees the keys from its own chunk's first position on; the walk starts at the first row's
+  const bool chunked = p.chunk > 0;
+  int lo_a = 0, lo_b = 0, lo_warp = 0;   // this thread's two rows, and the warp's last row
+  if (chunked) {
+    lo_tile = (pos0 + q0) / p.chunk * p.chunk / BN;
+    lo_a = pq_a / p.chunk * p.chunk;
+    lo_b = pq_b / p.chunk * p.chunk;
+    lo_warp = (pos0 + q0 + warp * 16 + 15) / p.chunk * p.chunk;
+  }
   const int n_it = n_first + (n_keys + BN - 1) / BN - lo_tile;
-  const float cap_in = p.softcap > 0.f ? p.scale / p.softcap * 2.885390081777927f : 0.f;  // 2 log2(e) scale / cap
+  const float cap_in = p.softcap > 0.f ? scale / p.softcap * 2.885390081777927f : 0.f;  // 2 log2(e) scale / cap
   const float cap_out = p.softcap * 1.4426950408889634f;
   load_tile_async<DP>(Kbuf, Kg, D, (n_first > 0 ? 0 : lo_tile) * BN, total_keys, D);
   cp_async_commit();
@@ -127,7 +138,8 @@ __global__ void __launch_bounds__(TC_THREADS, (DP <= 128 && VP <= 128) ? 3 : 1) 
     cp_async_commit();  // (an empty group after the last tile keeps the counts the same)
     if (bias) {  // this tile's distance biases, one per thread: entry y belongs to distance (q0 - k0) + 63 - y
       const int y = threadIdx.x, d = pos0 + q0 - k0 + 63 - y;
-      const float v = d >= 0 ? r1 * __log2f(fmaf(r2, static_cast<float>(d), 1.f)) : 0.f;
+      float v = 0.f;
+      if (d >= 0) v = tab ? -1.4426950408889634f * tab[min(d, p.bias_len - 1)] : r1 * __log2f(fmaf(r2, static_cast<float>(d), 1.f));
       T0[y] = v;
       if (y > 0) T1[y - 1] = v;
     }
@@ -156,7 +168,7 @@ __global__ void __launch_bounds__(TC_THREADS, (DP <= 128 && VP <= 128) ? 3 : 1) 
     // ---- scores in the base-2 domain: s * scale * log2(e) - bias (from the tile's table); causal mask only where a tile
     //      reaches past the warp's first row or the last key; row maxima ----
     const bool need_mask = (k0 + BN - 1 > pos0 + q0 + warp * 16) || (k0 + BN > total_keys) ||
-                           (windowed && pos0 + q0 + warp * 16 + 15 - k0 >= p.window);
+                           (windowed && pos0 + q0 + warp * 16 + 15 - k0 >= p.window) || (chunked && k0 < lo_warp);
     float mx_a = -INFINITY, mx_b = -INFINITY;
 #pragma unroll
     for (int nt = 0; nt < BN / 8; ++nt) {
@@ -186,6 +198,12 @@ __global__ void __launch_bounds__(TC_THREADS, (DP <= 128 && VP <= 128) ? 3 : 1) 
           if (pq_a - pk - 1 >= p.window && pk + 1 >= p.keep_first) s[nt][1] = -INFINITY;
           if (pq_b - pk >= p.window && pk >= p.keep_first) s[nt][2] = -INFINITY;
           if (pq_b - pk - 1 >= p.window && pk + 1 >= p.keep_first) s[nt][3] = -INFINITY;
+        }
+        if (chunked) {
+          if (pk < lo_a) s[nt][0] = -INFINITY;
+          if (pk + 1 < lo_a) s[nt][1] = -INFINITY;
+          if (pk < lo_b) s[nt][2] = -INFINITY;
+          if (pk + 1 < lo_b) s[nt][3] = -INFINITY;
         }
       }
       mx_a = fmaxf(mx_a, fmaxf(s[nt][0], s[nt][1]));
@@ -251,16 +269,23 @@ __global__ void __launch_bounds__(TC_THREADS, (DP <= 128 && VP <= 128) ? 3 : 1) 
   l_a += __shfl_xor_sync(0xffffffffu, l_a, 2);
   l_b += __shfl_xor_sync(0xffffffffu, l_b, 1);
   l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
-  const float inv_a = l_a > 0.f ? 1.f / l_a : 0.f, inv_b = l_b > 0.f ? 1.f / l_b : 0.f;
-  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + static_cast<long long>(off) * p.n_heads * V + h * V;
+  float inv_a = l_a > 0.f ? 1.f / l_a : 0.f, inv_b = l_b > 0.f ? 1.f / l_b : 0.f;
+  if (p.out_scale != 0.f) { inv_a *= p.out_scale; inv_b *= p.out_scale; }
+  if (p.head_gate) {
+    const __nv_bfloat16* hg = static_cast<const __nv_bfloat16*>(p.head_gate) + h;
+    if (q0 + row_a < len) inv_a *= sigmoidf_(ldf(hg + static_cast<long long>(off + q0 + row_a) * p.head_gate_stride));
+    if (q0 + row_b < len) inv_b *= sigmoidf_(ldf(hg + static_cast<long long>(off + q0 + row_b) * p.head_gate_stride));
+  }
+  const long long os = p.out_stride > 0 ? p.out_stride : static_cast<long long>(p.n_heads) * V;
+  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + static_cast<long long>(off) * os + h * V;
 #pragma unroll
   for (int vn = 0; vn < VP / 8; ++vn) {
     const int c = vn * 8 + qd * 2;
     if (c < V) {
       if (q0 + row_a < len)
-        *reinterpret_cast<uint32_t*>(out + static_cast<long long>(q0 + row_a) * p.n_heads * V + c) = pack_bf16(o[vn][0] * inv_a, o[vn][1] * inv_a);
+        *reinterpret_cast<uint32_t*>(out + static_cast<long long>(q0 + row_a) * os + c) = pack_bf16(o[vn][0] * inv_a, o[vn][1] * inv_a);
       if (q0 + row_b < len)
-        *reinterpret_cast<uint32_t*>(out + static_cast<long long>(q0 + row_b) * p.n_heads * V + c) = pack_bf16(o[vn][2] * inv_b, o[vn][3] * inv_b);
+        *reinterpret_cast<uint32_t*>(out + static_cast<long long>(q0 + row_b) * os + c) = pack_bf16(o[vn][2] * inv_b, o[vn][3] * inv_b);
     }
   }
 }
@@ -294,6 +319,7 @@ int launch_attn_tc(const pcs_attn_params& p, cudaStream_t st, bool* handled) {
   *handled = false;
   if (p.dtype != PCS_BF16 || p.max_len < 16 || (p.v_row_stride != 0 && p.v_row_stride != p.vdim) || p.dim % 8 != 0 || p.vdim % 8 != 0 || p.dim > 256 || p.vdim > 256) return PCS_OK;
   if (!p.seq_pos0 || !p.seq_len || !p.seq_off) return PCS_OK;
+  if (p.out_stride % 2 != 0 || (reinterpret_cast<uintptr_t>(p.out) & 3) != 0) return PCS_OK;
   if (static_cast<long long>((p.max_len + BM - 1) / BM) * p.n_seqs * p.n_heads > 0x7fffffffLL) return PCS_OK;
   *handled = true;
   if (p.dim <= 64) return launch_v<64>(p, st);

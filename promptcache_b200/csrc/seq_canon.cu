@@ -1,6 +1,6 @@
 // Embedding with a hashed token-pair table, and the residual sum + RMS norm + short causal convolution over time.
 //
-// pcs_embed_bigram  one block per token: the token's embedding row plus the row (prev * a + cur * b) mod buckets of a second
+// pcs_embed_bigram  one block per token: the token's embedding row times a scale plus the row (prev * a + cur * b) mod buckets of a second
 //                   table (its last row for a sequence's first token), summed in 32-bit into the residual stream.
 // pcs_norm_conv     one block per token.  u = norm(x) is needed for the token and for its taps - 1 predecessors: rows of the
 //                   same step are normed again from x (they are in L2; a row's statistics cost one reduction), rows of
@@ -15,7 +15,7 @@ namespace pcs {
 template <typename T>
 __global__ void __launch_bounds__(256) embed_bigram_kernel(const T* __restrict__ table, const T* __restrict__ pair,
                                                            const int64_t* __restrict__ ids, const int64_t* __restrict__ prev_ids,
-                                                           float* __restrict__ out, int width, int vocab, long long buckets,
+                                                           float* __restrict__ out, int width, int vocab, float scale, long long buckets,
                                                            long long mul_prev, long long mul_cur) {
   const int t = blockIdx.x;
   long long id = ids[t];
@@ -26,7 +26,7 @@ __global__ void __launch_bounds__(256) embed_bigram_kernel(const T* __restrict__
   const T* e = table + id * width;
   const T* b = pair + r * width;
   float* o = out + static_cast<long long>(t) * width;
-  for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = ldf(e + i) + ldf(b + i);
+  for (int i = threadIdx.x; i < width; i += blockDim.x) o[i] = fmaf(ldf(e + i), scale, ldf(b + i));
 }
 
 constexpr int kMaxTaps = 16;
@@ -209,7 +209,7 @@ __global__ void __launch_bounds__(256) norm_conv_vec_kernel(const pcs_normconv_p
 }  // namespace pcs
 
 PCS_API int pcs_embed_bigram(const void* table, const void* pair, const int64_t* ids, const int64_t* prev_ids, float* out, int n_tokens,
-                             int width, int vocab, int64_t buckets, int64_t mul_prev, int64_t mul_cur, int dtype, void* stream) {
+                             int width, int vocab, float scale, int64_t buckets, int64_t mul_prev, int64_t mul_cur, int dtype, void* stream) {
   if (n_tokens == 0) return PCS_OK;
   PCS_REQUIRE(table && pair && ids && prev_ids && out && n_tokens > 0 && width > 0 && vocab > 0, "pcs_embed_bigram: bad arguments");
   PCS_REQUIRE(buckets > 0 && buckets < (1LL << 31), "pcs_embed_bigram: buckets %lld out of range", static_cast<long long>(buckets));
@@ -217,7 +217,7 @@ PCS_API int pcs_embed_bigram(const void* table, const void* pair, const int64_t*
   const long long mp = ((mul_prev % buckets) + buckets) % buckets, mc = ((mul_cur % buckets) + buckets) % buckets;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   PCS_DISPATCH(dtype, pcs::embed_bigram_kernel<T><<<n_tokens, 256, 0, st>>>(static_cast<const T*>(table), static_cast<const T*>(pair), ids, prev_ids,
-                                                                            out, width, vocab, buckets, mp, mc));
+                                                                            out, width, vocab, scale, buckets, mp, mc));
   PCS_CHECK_CUDA(cudaGetLastError());
   pcs::count_launch();
   return PCS_OK;

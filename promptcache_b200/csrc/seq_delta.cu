@@ -1,0 +1,858 @@
+// Gated delta rule over the slot pool.
+//
+// Per head, with a decay per key channel and a step size beta in (0, 1):
+//     S <- diag(decay_t) S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t          (S: dim x vdim, 32-bit)
+// q, k and v come out of a short causal convolution with silu; q and k are unit vectors per head.
+//
+// pcs_short_conv        the convolution over time per channel, silu, unit vectors.  Inputs of earlier steps sit in the slot's tail,
+//                       kept twice so that the copy a step reads is never the one it writes.
+// pcs_delta_scan        token by token.  The columns of S evolve independently given k, q and the decays, so the grid covers
+//                       (sequence, head, slice of columns): state in registers (dim <= 256, aligned) or in shared memory.
+// pcs_delta_chunk_prep  prompts: everything about a chunk of 64 tokens that does not need the state it starts from.
+// pcs_delta_chunk_scan  prompts: the chunks in order, two products per chunk on a slice of columns held in shared memory.
+// pcs_head_norm_gate    per-head norm and sigmoid gate of the recurrence's result.
+#include "seq_common.cuh"
+#include "seq_mma.cuh"
+
+namespace pcs {
+
+// ---- short convolution ---------------------------------------------------------------------------------------------------------
+constexpr int kScMaxTaps = 16;
+
+struct ConvPlace {
+  int pos, pos0, len;
+  const float* rd;   // tail rows: positions pos0 - R .. pos0 - 1
+  float* wr;         // tail rows: positions pos0 + len - R .. pos0 + len - 1
+};
+__device__ __forceinline__ ConvPlace conv_place(const pcs_shortconv_params& p, int t, int R, int C) {
+  ConvPlace v;
+  const int b = p.tok_seq[t];
+  v.pos = p.tok_pos[t];
+  v.pos0 = p.seq_pos0[b];
+  v.len = p.seq_len[b];
+  const int par = p.seq_par[b] & 1;
+  float* base = p.tail + static_cast<long long>(p.seq_slot[b]) * 2 * R * C;
+  v.rd = base + static_cast<long long>(par) * R * C;
+  v.wr = base + static_cast<long long>(par ^ 1) * R * C;
+  return v;
+}
+
+__device__ __forceinline__ float silu_(float z) { return z * sigmoidf_(z); }
+
+// Any sizes: one block per token; a warp per query / key head, then the value channels.
+template <typename T>
+__global__ void __launch_bounds__(256) short_conv_kernel(const pcs_shortconv_params p) {
+  const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int D = p.dim, U = 2 * p.kv_heads * D, C = U + p.v_width, R = p.taps - 1;
+  const ConvPlace cp = conv_place(p, t, R, C);
+  const T* x = static_cast<const T*>(p.proj) + static_cast<long long>(t) * p.row_stride + p.c_off;
+  const T* cw = static_cast<const T*>(p.conv_w);
+  const int last_row = cp.pos - (cp.pos0 + cp.len - R);
+  auto value = [&](int c) {
+    float acc = ldf(cw + static_cast<long long>(R) * C + c) * ldf(x + c);
+    for (int j = 1; j <= R; ++j) {
+      if (cp.pos - j < 0) break;
+      const float v = cp.pos - j >= cp.pos0 ? ldf(x - static_cast<long long>(j) * p.row_stride + c)
+                                            : cp.rd[static_cast<long long>(R - (cp.pos0 - (cp.pos - j))) * C + c];
+      acc = fmaf(ldf(cw + static_cast<long long>(R - j) * C + c), v, acc);
+    }
+    return silu_(acc);
+  };
+  float* qk = p.qk_out + static_cast<long long>(t) * U;
+  for (int hd = warp; hd < 2 * p.kv_heads; hd += 8) {
+    float ss = 0.f;
+    for (int d = lane; d < D; d += 32) { const float v = value(hd * D + d); ss = fmaf(v, v, ss); }
+    ss = warp_sum(ss);
+    const float f = (hd < p.kv_heads ? p.q_scale : 1.f) / sqrtf(ss + p.unit_eps);
+    for (int d = lane; d < D; d += 32) qk[hd * D + d] = value(hd * D + d) * f;
+  }
+  T* vo = static_cast<T*>(p.v_out) + static_cast<long long>(t) * p.v_width;
+  for (int c = tid; c < p.v_width; c += 256) stf(vo + c, value(U + c));
+  if (R > 0 && last_row >= 0)
+    for (int c = tid; c < C; c += 256) cp.wr[static_cast<long long>(last_row) * C + c] = ldf(x + c);
+  if (R > 0 && cp.pos == cp.pos0 + cp.len - 1 && cp.len < R)
+    for (int q = 0; q < R - cp.len; ++q)
+      for (int c = tid; c < C; c += 256) cp.wr[static_cast<long long>(q) * C + c] = cp.rd[static_cast<long long>(q + cp.len) * C + c];
+}
+
+// 16-byte pieces, at most MR + 1 taps: a thread owns one piece of the channels [blockIdx.y * CB, ...) for TB neighbouring tokens, whose
+// rows and predecessors are requested together.  CB is a multiple of dim, so a head's pieces meet in this block's shared memory.
+template <typename T, int TB, int MR>
+__global__ void __launch_bounds__(256) short_conv_vec_kernel(const pcs_shortconv_params p, int CB) {
+  constexpr int N = Vec<T>::n, RN = TB + MR;
+  __shared__ float ssq[TB][256];
+  __shared__ float fac[TB][256];
+  const int t0 = blockIdx.x * TB, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int D = p.dim, U = 2 * p.kv_heads * D, C = U + p.v_width, R = p.taps - 1;
+  const int c_lo = blockIdx.y * CB, c = c_lo + tid * N;
+  const bool active = tid * N < CB && c < C;
+  const T* cw = static_cast<const T*>(p.conv_w);
+  ConvPlace cp[TB];
+  bool need[RN];
+#pragma unroll
+  for (int k = 0; k < RN; ++k) need[k] = false;
+#pragma unroll
+  for (int i = 0; i < TB; ++i) {
+    cp[i] = ConvPlace{0, 0, 1, nullptr, nullptr};
+    if (t0 + i < p.n_tokens) {
+      cp[i] = conv_place(p, t0 + i, R, C);
+      need[MR + i] = true;
+#pragma unroll
+      for (int j = 1; j <= MR; ++j)
+        if (j <= R && cp[i].pos - j >= cp[i].pos0) need[MR + i - j] = true;
+    }
+  }
+  uint4 xv[RN];
+  const T* x = static_cast<const T*>(p.proj) + p.c_off + c;
+  if (active) {
+#pragma unroll
+    for (int k = 0; k < RN; ++k)
+      if (need[k]) xv[k] = *reinterpret_cast<const uint4*>(x + static_cast<long long>(t0 - MR + k) * p.row_stride);
+  }
+  float o[TB][N];
+  if (active) {
+#pragma unroll
+    for (int i = 0; i < TB; ++i)
+#pragma unroll
+      for (int e = 0; e < N; ++e) o[i][e] = 0.f;
+#pragma unroll
+    for (int j = 0; j <= MR; ++j)
+      if (j <= R) {
+        float wv[N];
+        ld16(cw + static_cast<long long>(R - j) * C + c, wv);
+#pragma unroll
+        for (int i = 0; i < TB; ++i)
+          if (need[MR + i] && cp[i].pos - j >= 0) {
+            float v[N];
+            if (cp[i].pos - j >= cp[i].pos0) ld16(reinterpret_cast<const T*>(&xv[MR + i - j]), v);
+            else ldx(cp[i].rd + static_cast<long long>(R - (cp[i].pos0 - (cp[i].pos - j))) * C + c, v);
+#pragma unroll
+            for (int e = 0; e < N; ++e) o[i][e] = fmaf(wv[e], v[e], o[i][e]);
+          }
+      }
+#pragma unroll
+    for (int i = 0; i < TB; ++i) {
+      float a = 0.f;
+#pragma unroll
+      for (int e = 0; e < N; ++e) {
+        o[i][e] = silu_(o[i][e]);
+        a = fmaf(o[i][e], o[i][e], a);
+      }
+      ssq[i][tid] = a;
+      if (need[MR + i]) {
+        const int last_row = cp[i].pos - (cp[i].pos0 + cp[i].len - R);
+        if (R > 0 && last_row >= 0) {
+          float v[N];
+          ld16(reinterpret_cast<const T*>(&xv[MR + i]), v);
+          stx(cp[i].wr + static_cast<long long>(last_row) * C + c, v);
+        }
+        if (R > 0 && cp[i].pos == cp[i].pos0 + cp[i].len - 1 && cp[i].len < R)
+          for (int q = 0; q < R - cp[i].len; ++q) {
+            float v[N];
+            ldx(cp[i].rd + static_cast<long long>(q + cp[i].len) * C + c, v);
+            stx(cp[i].wr + static_cast<long long>(q) * C + c, v);
+          }
+      }
+    }
+  }
+  __syncthreads();
+  // heads of this block's channels: a warp adds the pieces of one (token, head)
+  const int PD = D / N, heads = max(0, min(CB, U - c_lo)) / D;
+  for (int e = warp; e < TB * heads; e += 8) {
+    const int i = e / heads, hd = e - i * heads;
+    float a = 0.f;
+    for (int k = lane; k < PD; k += 32) a += ssq[i][hd * PD + k];
+    a = warp_sum(a);
+    if (lane == 0) fac[i][hd] = (c_lo / D + hd < p.kv_heads ? p.q_scale : 1.f) / sqrtf(a + p.unit_eps);
+  }
+  __syncthreads();
+  if (!active) return;
+#pragma unroll
+  for (int i = 0; i < TB; ++i)
+    if (need[MR + i]) {
+      if (c < U) {
+        const float f = fac[i][(c - c_lo) / D];
+#pragma unroll
+        for (int e = 0; e < N; ++e) o[i][e] *= f;
+        stx(p.qk_out + static_cast<long long>(t0 + i) * U + c, o[i]);
+      } else {
+        st16(static_cast<T*>(p.v_out) + static_cast<long long>(t0 + i) * p.v_width + (c - U), o[i]);
+      }
+    }
+}
+
+template <typename T>
+static int launch_short_conv(const pcs_shortconv_params& p, cudaStream_t st, bool vec) {
+  if (vec) {
+    const int per = 256 * Vec<T>::n, C = 2 * p.kv_heads * p.dim + p.v_width;
+    // few tokens: narrow channel blocks, so that the launch covers more SMs
+    int CB = per / p.dim * p.dim;
+    if (p.n_tokens < 64) {
+      const int small = (32 * Vec<T>::n + p.dim - 1) / p.dim * p.dim;
+      if (small < CB) CB = small;
+    }
+    const int ny = (C + CB - 1) / CB;
+    if (p.n_tokens >= 4 * 148) short_conv_vec_kernel<T, 4, 3><<<dim3((p.n_tokens + 3) / 4, ny), 256, 0, st>>>(p, CB);
+    else short_conv_vec_kernel<T, 1, 3><<<dim3(p.n_tokens, ny), 256, 0, st>>>(p, CB);
+  } else {
+    short_conv_kernel<T><<<p.n_tokens, 256, 0, st>>>(p);
+  }
+  PCS_CHECK_CUDA(cudaGetLastError());
+  count_launch();
+  return PCS_OK;
+}
+
+// ---- token by token --------------------------------------------------------------------------------------------------------------
+// Any sizes: S of VS columns in shared memory, thread (r, c) owns rows r, r + R, ... of column c.
+template <typename T>
+__global__ void __launch_bounds__(1024) delta_scan_kernel(const pcs_delta_params p, int VS, int R) {
+  extern __shared__ float sm[];
+  const int D = p.dim, V = p.vdim, H = p.heads, U = 2 * p.kv_heads * D;
+  const int v0 = blockIdx.z * VS, vs = min(VS, V - v0);
+  float* S = sm;               // [D][VS]
+  float* ks = S + D * VS;      // [D]
+  float* qs = ks + D;          // [D]
+  float* as = qs + D;          // [D]
+  float* us = as + D;          // [VS]
+  float* part = us + VS;       // [R][VS]
+  const int b = blockIdx.x, head = blockIdx.y, hk = head / (H / p.kv_heads), tid = threadIdx.x, nthr = blockDim.x;
+  const int slot = p.seq_slot[b], len = p.seq_len[b], off = p.seq_off[b];
+  if (len <= 0) return;
+  const bool fresh = p.seq_pos0[b] == 0;
+  float* Sg = p.s_pool + (static_cast<long long>(slot) * H + head) * D * V;
+  for (int e = tid; e < D * vs; e += nthr) {
+    const int d = e / vs, c = e - d * vs;
+    S[d * VS + c] = fresh ? 0.f : Sg[static_cast<long long>(d) * V + v0 + c];
+  }
+  const int c = tid % VS, r = tid / VS;
+  const bool active = r < R && c < vs;
+  __syncthreads();
+  for (int i = 0; i < len; ++i) {
+    const long long t = off + i;
+    for (int d = tid; d < D; d += nthr) {
+      qs[d] = p.qk[t * U + hk * D + d];
+      ks[d] = p.qk[t * U + (p.kv_heads + hk) * D + d];
+      as[d] = p.decay[t * (static_cast<long long>(H) * D) + head * D + d];
+    }
+    __syncthreads();
+    if (active) {
+      float num = 0.f;
+      for (int d = r; d < D; d += R) {
+        const float sv = as[d] * S[d * VS + c];
+        S[d * VS + c] = sv;
+        num = fmaf(sv, ks[d], num);
+      }
+      part[r * VS + c] = num;
+    }
+    __syncthreads();
+    if (tid < vs) {
+      float a = 0.f;
+      for (int rr = 0; rr < R; ++rr) a += part[rr * VS + tid];
+      const float beta = sigmoidf_(ldf(static_cast<const T*>(p.b) + t * p.b_stride + head));
+      us[tid] = beta * (ldf(static_cast<const T*>(p.v) + t * (static_cast<long long>(H) * V) + head * V + v0 + tid) - a);
+    }
+    __syncthreads();
+    if (active) {
+      const float u = us[c];
+      float num = 0.f;
+      for (int d = r; d < D; d += R) {
+        const float sv = fmaf(ks[d], u, S[d * VS + c]);
+        S[d * VS + c] = sv;
+        num = fmaf(sv, qs[d], num);
+      }
+      part[r * VS + c] = num;
+    }
+    __syncthreads();
+    if (tid < vs) {
+      float o = 0.f;
+      for (int rr = 0; rr < R; ++rr) o += part[rr * VS + tid];
+      p.o[t * (static_cast<long long>(H) * V) + head * V + v0 + tid] = o;
+    }
+    __syncthreads();
+  }
+  for (int e = tid; e < D * vs; e += nthr) {
+    const int d = e / vs, cc = e - d * vs;
+    Sg[static_cast<long long>(d) * V + v0 + cc] = S[d * VS + cc];
+  }
+}
+
+constexpr int kDsRing = 12;   // shared-memory slots of tokens whose q / k / decays are in flight or waiting
+constexpr int kDsAhead = 8;   // tokens requested ahead of the arithmetic
+constexpr int kDsGroup = 4;   // tokens computed between two block barriers
+
+// State in registers.  A warp owns 8 columns; lane = 8 * rg + c: column c, rows 4 (rg + 4 m) + e for m < M, e < 4 (four row groups
+// share a column, so a column's sums are two shuffles).  One pass over the decayed state gives both S^T k and S^T q; the read-out
+// after the write is then S^T q + (k . q) u.  Rows past dim hold zeros.  The order of every sum is fixed by M alone.
+template <typename T, int M>
+__global__ void __launch_bounds__(256) delta_scan_reg_kernel(const pcs_delta_params p, int W) {
+  extern __shared__ __align__(16) float ring[];   // per slot: q[16 M] k[16 M] decay[16 M]
+  constexpr int DP = 16 * M;
+  const int D = p.dim, V = p.vdim, H = p.heads, U = 2 * p.kv_heads * D;
+  const int b = blockIdx.x, head = blockIdx.y, hk = head / (H / p.kv_heads), v0 = blockIdx.z * 8 * W;
+  const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, rg = lane >> 3;
+  const int slot = p.seq_slot[b], len = p.seq_len[b], off = p.seq_off[b];
+  if (len <= 0) return;
+  const bool fresh = p.seq_pos0[b] == 0;
+  const int col = v0 + warp * 8 + (lane & 7);
+  const bool okc = col < V;
+  const int cd = D / 4;
+  auto issue = [&](int i) {
+    const long long t = off + i;
+    float* s = ring + (i % kDsRing) * 3 * DP;
+    for (int e = tid; e < 3 * (DP / 4); e += nthr) {
+      const int which = e / (DP / 4), c = e - which * (DP / 4);
+      float* dst = s + which * DP + c * 4;
+      if (c < cd) {
+        const float* src = which == 0 ? p.qk + t * U + hk * D : which == 1 ? p.qk + t * U + (p.kv_heads + hk) * D : p.decay + t * (static_cast<long long>(H) * D) + head * D;
+        cp_async16(dst, src + c * 4);
+      } else {
+        *reinterpret_cast<float4*>(dst) = make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+    }
+  };
+  for (int i = 0; i < kDsAhead; ++i) {
+    if (i < len) issue(i);
+    cp_async_commit();
+  }
+  float* Sg = p.s_pool + (static_cast<long long>(slot) * H + head) * D * V;
+  float S[M][4];
+#pragma unroll
+  for (int m = 0; m < M; ++m)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int d = 4 * (rg + 4 * m) + e;
+      S[m][e] = (!fresh && d < D && okc) ? Sg[static_cast<long long>(d) * V + col] : 0.f;
+    }
+  const T* vg = static_cast<const T*>(p.v) + static_cast<long long>(off) * H * V + head * V + col;
+  const T* bg = static_cast<const T*>(p.b) + static_cast<long long>(off) * p.b_stride + head;
+  float vn[kDsGroup], bn[kDsGroup];   // the next group's values and step sizes, requested a group ahead
+#pragma unroll
+  for (int u = 0; u < kDsGroup; ++u) {
+    vn[u] = (u < len && okc) ? ldf(vg + static_cast<long long>(u) * H * V) : 0.f;
+    bn[u] = u < len ? ldf(bg + u * p.b_stride) : 0.f;
+  }
+  for (int i0 = 0; i0 < len; i0 += kDsGroup) {
+    cp_async_wait<kDsAhead - kDsGroup>();
+    __syncthreads();
+    float vc[kDsGroup], bc[kDsGroup];
+#pragma unroll
+    for (int u = 0; u < kDsGroup; ++u) {
+      vc[u] = vn[u];
+      bc[u] = bn[u];
+      const int nx = i0 + kDsGroup + u;
+      vn[u] = (nx < len && okc) ? ldf(vg + static_cast<long long>(nx) * H * V) : 0.f;
+      bn[u] = nx < len ? ldf(bg + nx * p.b_stride) : 0.f;
+      if (i0 + kDsAhead + u < len) issue(i0 + kDsAhead + u);
+      cp_async_commit();
+    }
+#pragma unroll
+    for (int u = 0; u < kDsGroup; ++u) {
+      const int i = i0 + u;
+      if (i >= len) break;
+      const float* cur = ring + (i % kDsRing) * 3 * DP;
+      float pk = 0.f, pq = 0.f, kq = 0.f;
+#pragma unroll
+      for (int m = 0; m < M; ++m) {
+        const int d = 4 * (rg + 4 * m);
+        const float4 q = *reinterpret_cast<const float4*>(cur + d), k = *reinterpret_cast<const float4*>(cur + DP + d),
+                     a = *reinterpret_cast<const float4*>(cur + 2 * DP + d);
+        S[m][0] *= a.x; S[m][1] *= a.y; S[m][2] *= a.z; S[m][3] *= a.w;
+        pk = fmaf(S[m][0], k.x, fmaf(S[m][1], k.y, fmaf(S[m][2], k.z, fmaf(S[m][3], k.w, pk))));
+        pq = fmaf(S[m][0], q.x, fmaf(S[m][1], q.y, fmaf(S[m][2], q.z, fmaf(S[m][3], q.w, pq))));
+        kq = fmaf(k.x, q.x, fmaf(k.y, q.y, fmaf(k.z, q.z, fmaf(k.w, q.w, kq))));
+      }
+#pragma unroll
+      for (int o = 8; o <= 16; o <<= 1) {
+        pk += __shfl_xor_sync(0xffffffffu, pk, o);
+        pq += __shfl_xor_sync(0xffffffffu, pq, o);
+        kq += __shfl_xor_sync(0xffffffffu, kq, o);
+      }
+      const float un = sigmoidf_(bc[u]) * (vc[u] - pk);
+#pragma unroll
+      for (int m = 0; m < M; ++m) {
+        const float4 k = *reinterpret_cast<const float4*>(cur + DP + 4 * (rg + 4 * m));
+        S[m][0] = fmaf(k.x, un, S[m][0]); S[m][1] = fmaf(k.y, un, S[m][1]); S[m][2] = fmaf(k.z, un, S[m][2]); S[m][3] = fmaf(k.w, un, S[m][3]);
+      }
+      if (rg == 0 && okc) p.o[(static_cast<long long>(off) + i) * H * V + head * V + col] = fmaf(kq, un, pq);
+    }
+  }
+#pragma unroll
+  for (int m = 0; m < M; ++m)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int d = 4 * (rg + 4 * m) + e;
+      if (d < D && okc) Sg[static_cast<long long>(d) * V + col] = S[m][e];
+    }
+}
+
+// ---- in chunks -------------------------------------------------------------------------------------------------------------------
+// A chunk's 64 rows form four blocks of 16.  With B the running sums of the log decays, r(I) the row before block I:
+//   pairs inside a block take the exact factor exp(B_i - B_s) channel by channel;
+//   pairs across blocks (row i of block I, row s of block J < I) factor it into exp(B_i - B_r(I)) * exp(B_r(I) - B_r(J+1)) * exp(B_r(J+1) - B_s):
+//   every exponent is <= 0, and each factor is at least their product, so nothing is lost that the product does not lose.
+// So q and k are scaled in place to their block's start and the keys to their block's end, and the pairs across blocks are plain products.
+constexpr int kC = PCS_DELTA_CHUNK, kCB = 16, kNB = kC / kCB;
+constexpr int kDpThreads = 512;
+
+__device__ __forceinline__ int delta_kd_slot(int d) { return (d & ~63) + 4 * (d & 15) + ((d & 63) >> 4); }
+
+template <typename T>
+__global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_delta_chunk_params p) {
+  extern __shared__ __align__(16) float sm[];
+  const int D = p.dim, V = p.vdim, H = p.heads, D4 = (D + 3) & ~3, DP = D4 + 4, U = 2 * p.kv_heads * D, L = (D + 63) & ~63;
+  float* qs = sm;              // [64][DP]: q, later scaled to its block's start
+  float* ks = qs + kC * DP;    // [64][DP]: k, later scaled to its block's start
+  float* Bs = ks + kC * DP;    // [64][DP]: running sums, later the keys scaled to their block's end
+  float* f1 = Bs + kC * DP;    // [D4] each: the running sums at the blocks' ends, later exp(B_r(1)), exp(B_r(2) - B_r(1)), exp(B_r(3) - B_r(2))
+  float* f2 = f1 + D4;
+  float* f3 = f2 + D4;
+  float* fe = f3 + D4;
+  float* As = fe + D4;         // [64][64] beta_i A[i, s]
+  float* beta = As + kC * kC;  // [64]
+  const int cn = blockIdx.x, head = blockIdx.y, hk = head / (H / p.kv_heads), tid = threadIdx.x;
+  const int first = p.chunk_first[cn], n = p.chunk_len[cn];
+  const long long base = static_cast<long long>(cn) * H + head;
+  for (int e = tid; e < kC * D4; e += kDpThreads) {
+    const int i = e / D4, d = e - i * D4;
+    float q = 0.f, k = 0.f, l = 0.f;
+    if (i < n && d < D) {
+      const float* row = p.qk + static_cast<long long>(first + i) * U;
+      q = row[hk * D + d];
+      k = row[(p.kv_heads + hk) * D + d];
+      l = p.ld[static_cast<long long>(first + i) * (static_cast<long long>(H) * D) + head * D + d];
+    }
+    qs[i * DP + d] = q;
+    ks[i * DP + d] = k;
+    Bs[i * DP + d] = l;
+  }
+  if (tid < kC) beta[tid] = tid < n ? sigmoidf_(ldf(static_cast<const T*>(p.b) + static_cast<long long>(first + tid) * p.b_stride + head)) : 0.f;
+  for (int e = tid; e < kC * kC; e += kDpThreads) As[e] = 0.f;
+  float* ag = p.a + base * kC * kC;
+  for (int e = tid; e < kC * kC; e += kDpThreads)
+    if ((e & 63) > (e >> 6)) ag[e] = 0.f;   // above the diagonal
+  __syncthreads();
+  for (int d = tid; d < D4; d += kDpThreads) {
+    float acc = 0.f;
+#pragma unroll 8
+    for (int i = 0; i < kC; ++i) {
+      acc += Bs[i * DP + d];
+      Bs[i * DP + d] = acc;
+    }
+  }
+  __syncthreads();
+  // pairs inside the blocks: (block, i, s <= i), 136 per block, every pair by four neighbouring threads that split the channels
+  constexpr bool kFast = sizeof(T) == 2;   // bfloat16 runs: base-2 exponential unit (relative error near 2^-22)
+  for (int e = tid >> 2; e < kNB * 136; e += kDpThreads / 4) {
+    const int blk = e / 136, pr = e - blk * 136;
+    int i = static_cast<int>((sqrtf(8.f * pr + 1.f) - 1.f) * 0.5f);
+    while ((i + 1) * (i + 2) / 2 <= pr) ++i;
+    while (i * (i + 1) / 2 > pr) --i;
+    const int s = blk * kCB + (pr - i * (i + 1) / 2);
+    i += blk * kCB;
+    float aq = 0.f, ak = 0.f;
+    for (int d = (tid & 3) * 4; d < D4; d += 16) {
+      const float4 bi = *reinterpret_cast<const float4*>(Bs + i * DP + d), bs = *reinterpret_cast<const float4*>(Bs + s * DP + d);
+      const float4 qi = *reinterpret_cast<const float4*>(qs + i * DP + d), ki = *reinterpret_cast<const float4*>(ks + i * DP + d);
+      const float4 k4 = *reinterpret_cast<const float4*>(ks + s * DP + d);
+      auto ex = [](float x) { return kFast ? ex2(x * 1.4426950408889634f) : expf(x); };
+      const float x0 = k4.x * ex(bi.x - bs.x), x1 = k4.y * ex(bi.y - bs.y), x2 = k4.z * ex(bi.z - bs.z), x3 = k4.w * ex(bi.w - bs.w);
+      aq = fmaf(qi.x, x0, fmaf(qi.y, x1, fmaf(qi.z, x2, fmaf(qi.w, x3, aq))));
+      ak = fmaf(ki.x, x0, fmaf(ki.y, x1, fmaf(ki.z, x2, fmaf(ki.w, x3, ak))));
+    }
+    const unsigned grp = 0xfu << (tid & 28);
+    aq += __shfl_xor_sync(grp, aq, 1);
+    ak += __shfl_xor_sync(grp, ak, 1);
+    aq += __shfl_xor_sync(grp, aq, 2);
+    ak += __shfl_xor_sync(grp, ak, 2);
+    if ((tid & 3) == 0) {
+      ag[i * kC + s] = aq;
+      if (s < i) As[i * kC + s] = beta[i] * ak;
+    }
+  }
+  __syncthreads();
+  // the running sums at the blocks' ends, then per (token, channel): what leaves the chunk, q and k scaled to their block's start, and in
+  // place of the running sums the keys scaled to their block's end (the last block's keys meet no later block)
+  for (int d = tid; d < D4; d += kDpThreads) {
+    f1[d] = Bs[15 * DP + d];
+    f2[d] = Bs[31 * DP + d];
+    f3[d] = Bs[47 * DP + d];
+    fe[d] = Bs[63 * DP + d];
+  }
+  __syncthreads();
+  {
+    float* qd = p.qd + base * kC * D;
+    float* kd = p.kd + base * kC * L;
+    for (int e = tid; e < kC * D4; e += kDpThreads) {
+      const int i = e / D4, d = e - i * D4, o = i * DP + d;
+      const float bv = Bs[o], q = qs[o], k = ks[o];
+      const float br = i < 16 ? 0.f : i < 32 ? f1[d] : i < 48 ? f2[d] : f3[d];
+      const float bn = i < 16 ? f1[d] : i < 32 ? f2[d] : i < 48 ? f3[d] : bv;
+      const float es = expf(bv - br);
+      if (d < D) {
+        qd[i * D + d] = q * expf(bv);
+        kd[static_cast<long long>(i) * L + delta_kd_slot(d)] = k * expf(fe[d] - bv);
+      }
+      qs[o] = q * es;
+      ks[o] = k * es;
+      Bs[o] = k * expf(bn - bv);
+    }
+    for (int e = tid; e < kC * (L - D); e += kDpThreads) {   // the padding of the outgoing keys
+      const int i = e / (L - D), d = D + (e - i * (L - D));
+      kd[static_cast<long long>(i) * L + delta_kd_slot(d)] = 0.f;
+    }
+  }
+  __syncthreads();
+  for (int d = tid; d < D4; d += kDpThreads) {
+    const float b1 = f1[d], b2 = f2[d], b3 = f3[d];
+    f1[d] = expf(b1);
+    f2[d] = expf(b2 - b1);
+    f3[d] = expf(b3 - b2);
+    if (d < D) p.g[base * D + d] = expf(fe[d]);
+  }
+  __syncthreads();
+  // pairs across blocks: six (I, J) pairs of 16 x 16, 2 x 2 pairs per thread
+  for (int e = tid; e < 6 * 64; e += kDpThreads) {
+    const int pr = e >> 6, q4 = e & 63;
+    const int I = pr == 0 ? 1 : pr < 3 ? 2 : 3, J = pr == 0 ? 0 : pr < 3 ? pr - 1 : pr - 3;
+    const int i = I * kCB + (q4 >> 3), s = J * kCB + (q4 & 7);   // rows i, i + 8 and keys s, s + 8
+    const float* g1 = J + 1 < I ? (J == 0 ? f2 : f3) : nullptr;   // from the end of J to the start of I: one block between
+    const float* g2 = J + 2 < I ? f3 : nullptr;                    // or two
+    float q00 = 0.f, q01 = 0.f, q10 = 0.f, q11 = 0.f, k00 = 0.f, k01 = 0.f, k10 = 0.f, k11 = 0.f;
+    for (int d = 0; d < D4; d += 4) {
+      float4 ka = *reinterpret_cast<const float4*>(Bs + s * DP + d), kb = *reinterpret_cast<const float4*>(Bs + (s + 8) * DP + d);
+      if (g1) {
+        const float4 f = *reinterpret_cast<const float4*>(g1 + d);
+        ka.x *= f.x; ka.y *= f.y; ka.z *= f.z; ka.w *= f.w;
+        kb.x *= f.x; kb.y *= f.y; kb.z *= f.z; kb.w *= f.w;
+      }
+      if (g2) {
+        const float4 f = *reinterpret_cast<const float4*>(g2 + d);
+        ka.x *= f.x; ka.y *= f.y; ka.z *= f.z; ka.w *= f.w;
+        kb.x *= f.x; kb.y *= f.y; kb.z *= f.z; kb.w *= f.w;
+      }
+      auto dot = [](const float4& a, const float4& b, float c) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, fmaf(a.w, b.w, c)))); };
+      const float4 qa = *reinterpret_cast<const float4*>(qs + i * DP + d), qb = *reinterpret_cast<const float4*>(qs + (i + 8) * DP + d);
+      q00 = dot(qa, ka, q00); q01 = dot(qa, kb, q01); q10 = dot(qb, ka, q10); q11 = dot(qb, kb, q11);
+      const float4 xa = *reinterpret_cast<const float4*>(ks + i * DP + d), xb = *reinterpret_cast<const float4*>(ks + (i + 8) * DP + d);
+      k00 = dot(xa, ka, k00); k01 = dot(xa, kb, k01); k10 = dot(xb, ka, k10); k11 = dot(xb, kb, k11);
+    }
+    ag[i * kC + s] = q00; ag[i * kC + s + 8] = q01; ag[(i + 8) * kC + s] = q10; ag[(i + 8) * kC + s + 8] = q11;
+    As[i * kC + s] = beta[i] * k00; As[i * kC + s + 8] = beta[i] * k01;
+    As[(i + 8) * kC + s] = beta[i + 8] * k10; As[(i + 8) * kC + s + 8] = beta[i + 8] * k11;
+  }
+  __syncthreads();
+  // M x = rhs by forward substitution, one column per thread, the column in registers: first the dim columns of diag(beta) K exp(B), then
+  // the vdim columns of diag(beta) V
+  float* wg = p.w + base * D * kC;
+  float* ug = p.u + base * kC * V;
+  for (int col = tid; col < D + V; col += kDpThreads) {
+    float x[kC];
+    if (col < D) {
+      const float e1 = f1[col], e2 = e1 * f2[col], e3 = e2 * f3[col];
+#pragma unroll
+      for (int i = 0; i < kC; ++i) x[i] = beta[i] * ks[i * DP + col] * (i < 16 ? 1.f : i < 32 ? e1 : i < 48 ? e2 : e3);
+    } else {
+      const T* v = static_cast<const T*>(p.v) + static_cast<long long>(first) * H * V + head * V + (col - D);
+#pragma unroll
+      for (int i = 0; i < kC; ++i) x[i] = i < n ? beta[i] * ldf(v + static_cast<long long>(i) * H * V) : 0.f;
+    }
+#pragma unroll
+    for (int i = 1; i < kC; ++i) {
+      float a0 = 0.f, a1 = 0.f;
+#pragma unroll
+      for (int j = 0; j < i; j += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(As + i * kC + j);   // (entries from i on are zero)
+        a0 = fmaf(a.x, x[j], a0);
+        if (j + 1 < i) a1 = fmaf(a.y, x[j + 1], a1);
+        if (j + 2 < i) a0 = fmaf(a.z, x[j + 2], a0);
+        if (j + 3 < i) a1 = fmaf(a.w, x[j + 3], a1);
+      }
+      x[i] -= a0 + a1;
+    }
+    if (col < D) {
+      float* o = wg + static_cast<long long>(col) * kC;
+#pragma unroll
+      for (int r = 0; r < 16; ++r) *reinterpret_cast<float4*>(o + 4 * r) = make_float4(x[r], x[r + 16], x[r + 32], x[r + 48]);
+    } else {
+#pragma unroll
+      for (int i = 0; i < kC; ++i) ug[static_cast<long long>(i) * V + (col - D)] = x[i];
+    }
+  }
+}
+
+// Block = (8 value columns, head, entry), 8 warps.  Both products split their sum over the warps and meet in `red`: u = u0 - w S over
+// the channels, kd^T u over the tokens; a lane owns rows r, r + 16, r + 32, r + 48 (one 16-byte piece in the layouts the
+// preparation writes) and four columns.  w and kd of a chunk have one shared-memory buffer each: kd travels under the first product,
+// the next chunk's w under the second.
+constexpr int kDcThreads = 256, kDcV = 8;
+
+__global__ void __launch_bounds__(kDcThreads) delta_chunk_scan_kernel(const pcs_delta_chunk_params p) {
+  extern __shared__ __align__(16) float sm[];
+  const int D = p.dim, V = p.vdim, H = p.heads, L = (D + 63) & ~63, NT = L / 64;
+  float* ws = sm;                   // [D][64]
+  float* kds = ws + D * kC;         // [64][L]
+  float* S = kds + kC * L;          // [L][8]
+  float* us = S + L * kDcV;         // [64][8]
+  float* red = us + kC * kDcV;      // 4096
+  const int v0 = blockIdx.x * kDcV, head = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int r = lane & 15, c4 = (lane >> 4) * 4;
+  const int n_chunks = p.seq_chunks[b];
+  if (n_chunks <= 0) return;
+  const long long c0 = p.seq_chunk0[b];
+  const int vs = min(kDcV, V - v0);
+  float* Sg = p.s_pool + (static_cast<long long>(p.seq_slot[b]) * H + head) * D * V;
+  const bool fresh = p.seq_pos0[b] == 0;
+  for (int e = tid; e < L * kDcV; e += kDcThreads) {
+    const int d = e >> 3, c = e & 7;
+    S[e] = (!fresh && d < D && c < vs) ? Sg[static_cast<long long>(d) * V + v0 + c] : 0.f;
+  }
+  auto load_w = [&](int c) {
+    const float* src = p.w + ((c0 + c) * H + head) * D * kC;
+    for (int e = tid; e < D * (kC / 4); e += kDcThreads) cp_async16(ws + e * 4, src + e * 4);
+  };
+  auto load_kd = [&](int c) {
+    const float* src = p.kd + ((c0 + c) * H + head) * kC * L;
+    for (int e = tid; e < kC * (L / 4); e += kDcThreads) cp_async16(kds + e * 4, src + e * 4);
+  };
+  load_w(0);
+  cp_async_commit();
+  load_kd(0);
+  cp_async_commit();
+  // phase 1: warp -> channels [d_lo, d_hi); phase 2: warp -> (64-channel tile, part of the tokens)
+  const int dw = (D + 7) / 8, d_lo = min(D, warp * dw), d_hi = min(D, d_lo + dw);
+  const int parts = 8 / NT, tile = warp % NT, part = warp / NT, tw = kC / parts;
+  const int i_lo = part * tw;
+  const bool busy2 = part < parts;
+  constexpr int kMaxOut = 8;   // L * 8 / 256 outputs of phase 2 per thread
+  for (int c = 0; c < n_chunks; ++c) {
+    const long long base = (c0 + c) * H + head;
+    float* ug = p.u + base * kC * V + v0;
+    float u0[2], gd[kMaxOut];
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+      const int e = tid + m * kDcThreads;
+      u0[m] = (e & 7) < vs ? ug[static_cast<long long>(e >> 3) * V + (e & 7)] : 0.f;
+    }
+#pragma unroll
+    for (int m = 0; m < kMaxOut; ++m) {
+      const int d = (tid + m * kDcThreads) >> 3;
+      gd[m] = d < D ? p.g[base * D + d] : 0.f;
+    }
+    cp_async_wait<1>();
+    __syncthreads();   // w of this chunk, and the state
+    {
+      float acc[4][4];
+#pragma unroll
+      for (int x = 0; x < 4; ++x) acc[x][0] = acc[x][1] = acc[x][2] = acc[x][3] = 0.f;
+#pragma unroll 4
+      for (int d = d_lo; d < d_hi; ++d) {
+        const float4 w4 = *reinterpret_cast<const float4*>(ws + d * kC + 4 * r), s4 = *reinterpret_cast<const float4*>(S + d * kDcV + c4);
+        const float wv[4] = {w4.x, w4.y, w4.z, w4.w};
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          acc[x][0] = fmaf(wv[x], s4.x, acc[x][0]);
+          acc[x][1] = fmaf(wv[x], s4.y, acc[x][1]);
+          acc[x][2] = fmaf(wv[x], s4.z, acc[x][2]);
+          acc[x][3] = fmaf(wv[x], s4.w, acc[x][3]);
+        }
+      }
+#pragma unroll
+      for (int x = 0; x < 4; ++x)
+        *reinterpret_cast<float4*>(red + warp * (kC * kDcV) + (r + 16 * x) * kDcV + c4) = make_float4(acc[x][0], acc[x][1], acc[x][2], acc[x][3]);
+    }
+    __syncthreads();
+    if (c + 1 < n_chunks) load_w(c + 1);
+    cp_async_commit();
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+      const int e = tid + m * kDcThreads;
+      float a = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) a += red[w * (kC * kDcV) + e];
+      const float u = u0[m] - a;
+      us[e] = u;
+      if ((e & 7) < vs) ug[static_cast<long long>(e >> 3) * V + (e & 7)] = u;
+    }
+    cp_async_wait<1>();
+    __syncthreads();   // kd of this chunk, and u; `red` is free again
+    if (busy2) {
+      float acc[4][4];
+#pragma unroll
+      for (int x = 0; x < 4; ++x) acc[x][0] = acc[x][1] = acc[x][2] = acc[x][3] = 0.f;
+#pragma unroll 4
+      for (int i = i_lo; i < i_lo + tw; ++i) {
+        const float4 k4 = *reinterpret_cast<const float4*>(kds + i * L + tile * 64 + 4 * r), u4 = *reinterpret_cast<const float4*>(us + i * kDcV + c4);
+        const float kv[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          acc[x][0] = fmaf(kv[x], u4.x, acc[x][0]);
+          acc[x][1] = fmaf(kv[x], u4.y, acc[x][1]);
+          acc[x][2] = fmaf(kv[x], u4.z, acc[x][2]);
+          acc[x][3] = fmaf(kv[x], u4.w, acc[x][3]);
+        }
+      }
+#pragma unroll
+      for (int x = 0; x < 4; ++x)
+        *reinterpret_cast<float4*>(red + part * (L * kDcV) + (tile * 64 + r + 16 * x) * kDcV + c4) = make_float4(acc[x][0], acc[x][1], acc[x][2], acc[x][3]);
+    }
+    __syncthreads();
+    if (c + 1 < n_chunks) load_kd(c + 1);
+    cp_async_commit();
+    float* sg = p.s + base * D * V + v0;
+#pragma unroll
+    for (int m = 0; m < kMaxOut; ++m) {
+      const int e = tid + m * kDcThreads;
+      if (e < L * kDcV) {
+        float a = 0.f;
+        for (int w = 0; w < parts; ++w) a += red[w * (L * kDcV) + e];
+        const int d = e >> 3, cc = e & 7;
+        const float old = S[e];
+        if (d < D && cc < vs) sg[static_cast<long long>(d) * V + cc] = old;
+        S[e] = fmaf(gd[m], old, a);
+      }
+    }
+  }
+  __syncthreads();
+  for (int e = tid; e < D * kDcV; e += kDcThreads)
+    if ((e & 7) < vs) Sg[static_cast<long long>(e >> 3) * V + v0 + (e & 7)] = S[e];
+}
+
+// ---- per-head norm and gate ------------------------------------------------------------------------------------------------------
+template <typename T>
+__global__ void __launch_bounds__(256) head_norm_gate_kernel(const pcs_headnorm_params p) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, V = p.vdim, H = p.heads;
+  const long long e = static_cast<long long>(blockIdx.x) * 8 + warp;
+  if (e >= static_cast<long long>(p.n_tokens) * H) return;
+  const long long t = e / H;
+  const int h = static_cast<int>(e - t * H);
+  long long row = e;
+  if (p.tok_row) {
+    const int tr = p.tok_row[t];
+    row = (static_cast<long long>(tr / p.chunk_size) * H + h) * p.chunk_size + tr % p.chunk_size;
+  }
+  const float* o = p.o + row * V;
+  const T* g = static_cast<const T*>(p.g) + t * p.g_stride + h * V;
+  const T* w = static_cast<const T*>(p.w);
+  T* out = static_cast<T*>(p.out) + t * p.out_stride + h * V;
+  constexpr int KEEP = 16;   // columns of a lane that stay in registers
+  float ov[KEEP], gv[KEEP];
+  float ss = 0.f;
+#pragma unroll
+  for (int u = 0; u < KEEP; ++u) {
+    const int c = lane + u * 32;
+    ov[u] = c < V ? o[c] : 0.f;
+    gv[u] = c < V ? ldf(g + c) : 0.f;
+  }
+#pragma unroll
+  for (int u = 0; u < KEEP; ++u) ss = fmaf(ov[u], ov[u], ss);
+  for (int c = lane + KEEP * 32; c < V; c += 32) ss = fmaf(o[c], o[c], ss);
+  ss = warp_sum(ss);
+  const float inv = p.out_scale / sqrtf(ss / static_cast<float>(V) + p.eps);
+#pragma unroll
+  for (int u = 0; u < KEEP; ++u) {
+    const int c = lane + u * 32;
+    if (c < V) stf(out + c, ov[u] * inv * ldf(w + c) * sigmoidf_(gv[u]));
+  }
+  for (int c = lane + KEEP * 32; c < V; c += 32) stf(out + c, o[c] * inv * ldf(w + c) * sigmoidf_(ldf(g + c)));
+}
+
+}  // namespace pcs
+
+PCS_API int pcs_short_conv(const pcs_shortconv_params* p, void* stream) {
+  PCS_REQUIRE(p, "pcs_short_conv: null params");
+  if (p->n_tokens == 0) return PCS_OK;
+  PCS_REQUIRE(p->proj && p->conv_w && p->qk_out && p->v_out && p->tok_seq && p->tok_pos && p->seq_slot && p->seq_pos0 && p->seq_len && p->seq_par,
+              "pcs_short_conv: null tensor");
+  PCS_REQUIRE(p->kv_heads > 0 && p->dim > 0 && p->v_width > 0 && p->c_off >= 0 && p->taps >= 1 && p->taps <= pcs::kScMaxTaps && (p->tail || p->taps == 1),
+              "pcs_short_conv: bad sizes (taps %d of at most %d)", p->taps, pcs::kScMaxTaps);
+  const int piece = p->dtype == PCS_BF16 ? 8 : 4;
+  auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  const bool vec = p->impl != 1 && p->taps <= 4 && p->dim % piece == 0 && p->v_width % piece == 0 && p->c_off % piece == 0 && p->row_stride % piece == 0 &&
+                   p->dim <= 256 * piece && al(p->proj) && al(p->conv_w) && al(p->tail) && al(p->qk_out) && al(p->v_out);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  PCS_DISPATCH(p->dtype, return pcs::launch_short_conv<T>(*p, st, vec));
+}
+
+PCS_API int pcs_delta_scan(const pcs_delta_params* p, void* stream) {
+  PCS_REQUIRE(p, "pcs_delta_scan: null params");
+  if (p->n_seqs == 0 || p->n_tokens == 0) return PCS_OK;
+  PCS_REQUIRE(p->qk && p->v && p->decay && p->b && p->o && p->s_pool && p->seq_slot && p->seq_pos0 && p->seq_len && p->seq_off, "pcs_delta_scan: null tensor");
+  PCS_REQUIRE(p->heads > 0 && p->heads <= 65535 && p->kv_heads > 0 && p->heads % p->kv_heads == 0 && p->dim > 0 && p->vdim > 0, "pcs_delta_scan: bad sizes");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool aligned = p->dim % 4 == 0 && ((reinterpret_cast<uintptr_t>(p->qk) | reinterpret_cast<uintptr_t>(p->decay)) & 15) == 0;
+  if (p->impl != 1 && p->dim <= 256 && aligned) {
+    // warps per block halve until the launch has two blocks per SM (or one warp is left)
+    int W = 8;
+    while (W > 1 && 8 * (W / 2) >= p->vdim) W /= 2;
+    auto blocks = [&](int w) { return static_cast<long long>(p->n_seqs) * p->heads * ((p->vdim + 8 * w - 1) / (8 * w)); };
+    while (W > 1 && blocks(W) < 2 * 148) W /= 2;
+    dim3 grid(p->n_seqs, p->heads, (p->vdim + 8 * W - 1) / (8 * W));
+#define PCS_DELTA_REG(MV) \
+  PCS_DISPATCH(p->dtype, (pcs::delta_scan_reg_kernel<T, MV><<<grid, 32 * W, static_cast<size_t>(pcs::kDsRing) * 3 * 16 * MV * sizeof(float), st>>>(*p, W)))
+    if (p->dim <= 32) PCS_DELTA_REG(2);
+    else if (p->dim <= 64) PCS_DELTA_REG(4);
+    else if (p->dim <= 128) PCS_DELTA_REG(8);
+    else PCS_DELTA_REG(16);
+#undef PCS_DELTA_REG
+  } else {
+    int VS = p->vdim < 128 ? p->vdim : 128;
+    while (VS > 8 && static_cast<size_t>(p->dim) * VS * sizeof(float) > 160 * 1024) VS /= 2;
+    int R = 512 / VS;
+    if (R < 1) R = 1;
+    if (R > p->dim) R = p->dim;
+    const int threads = ((VS * R + 31) / 32) * 32;
+    const size_t smem = (static_cast<size_t>(p->dim) * VS + 3 * p->dim + VS + static_cast<size_t>(R) * VS) * sizeof(float);
+    PCS_REQUIRE(smem <= 220 * 1024, "pcs_delta_scan: a state of %d rows exceeds shared memory", p->dim);
+    if (smem > 48 * 1024)
+      PCS_DISPATCH(p->dtype, PCS_CHECK_CUDA(cudaFuncSetAttribute(pcs::delta_scan_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024)));
+    dim3 grid(p->n_seqs, p->heads, (p->vdim + VS - 1) / VS);
+    PCS_DISPATCH(p->dtype, pcs::delta_scan_kernel<T><<<grid, threads, smem, st>>>(*p, VS, R));
+  }
+  PCS_CHECK_CUDA(cudaGetLastError());
+  pcs::count_launch();
+  return PCS_OK;
+}
+
+PCS_API int pcs_delta_chunk_prep(const pcs_delta_chunk_params* p, void* stream) {
+  PCS_REQUIRE(p, "pcs_delta_chunk_prep: null params");
+  if (p->n_chunks == 0) return PCS_OK;
+  PCS_REQUIRE(p->qk && p->v && p->ld && p->b && p->chunk_first && p->chunk_len && p->qd && p->kd && p->w && p->g && p->u && p->a, "pcs_delta_chunk_prep: null tensor");
+  PCS_REQUIRE(p->heads > 0 && p->heads <= 65535 && p->kv_heads > 0 && p->heads % p->kv_heads == 0 && p->dim > 0 && p->dim <= 256 && p->vdim > 0,
+              "pcs_delta_chunk_prep: bad sizes (dim %d of at most 256)", p->dim);
+  const int D4 = (p->dim + 3) & ~3;
+  const size_t smem = (static_cast<size_t>(3) * pcs::kC * (D4 + 4) + 4 * D4 + pcs::kC * pcs::kC + pcs::kC) * sizeof(float);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  PCS_DISPATCH(p->dtype, PCS_CHECK_CUDA(cudaFuncSetAttribute(pcs::delta_chunk_prep_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024)));
+  PCS_DISPATCH(p->dtype, pcs::delta_chunk_prep_kernel<T><<<dim3(p->n_chunks, p->heads), pcs::kDpThreads, smem, st>>>(*p));
+  PCS_CHECK_CUDA(cudaGetLastError());
+  pcs::count_launch();
+  return PCS_OK;
+}
+
+PCS_API int pcs_delta_chunk_scan(const pcs_delta_chunk_params* p, void* stream) {
+  PCS_REQUIRE(p, "pcs_delta_chunk_scan: null params");
+  if (p->n_seqs == 0 || p->n_chunks == 0) return PCS_OK;
+  PCS_REQUIRE(p->kd && p->w && p->g && p->u && p->s && p->s_pool && p->seq_slot && p->seq_pos0 && p->seq_chunk0 && p->seq_chunks, "pcs_delta_chunk_scan: null tensor");
+  PCS_REQUIRE(p->heads > 0 && p->heads <= 65535 && p->n_seqs <= 65535 && p->dim > 0 && p->dim <= 256 && p->vdim > 0, "pcs_delta_chunk_scan: bad sizes");
+  PCS_REQUIRE(((reinterpret_cast<uintptr_t>(p->kd) | reinterpret_cast<uintptr_t>(p->w)) & 15) == 0, "pcs_delta_chunk_scan: kd and w must be 16-byte aligned");
+  const int L = (p->dim + 63) & ~63;
+  const size_t smem = (static_cast<size_t>(p->dim) * pcs::kC + static_cast<size_t>(pcs::kC) * L + static_cast<size_t>(L) * pcs::kDcV + pcs::kC * pcs::kDcV + 4096) * sizeof(float);
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  PCS_CHECK_CUDA(cudaFuncSetAttribute(pcs::delta_chunk_scan_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+  pcs::delta_chunk_scan_kernel<<<dim3((p->vdim + pcs::kDcV - 1) / pcs::kDcV, p->heads, p->n_seqs), pcs::kDcThreads, smem, st>>>(*p);
+  PCS_CHECK_CUDA(cudaGetLastError());
+  pcs::count_launch();
+  return PCS_OK;
+}
+
+PCS_API int pcs_head_norm_gate(const pcs_headnorm_params* p, void* stream) {
+  PCS_REQUIRE(p, "pcs_head_norm_gate: null params");
+  if (p->n_tokens == 0) return PCS_OK;
+  PCS_REQUIRE(p->o && p->w && p->g && p->out && p->heads > 0 && p->vdim > 0 && (p->tok_row == nullptr || p->chunk_size > 0), "pcs_head_norm_gate: bad arguments");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const long long rows = static_cast<long long>(p->n_tokens) * p->heads;
+  PCS_DISPATCH(p->dtype, pcs::head_norm_gate_kernel<T><<<static_cast<unsigned>((rows + 7) / 8), 256, 0, st>>>(*p));
+  PCS_CHECK_CUDA(cudaGetLastError());
+  pcs::count_launch();
+  return PCS_OK;
+}

@@ -15,10 +15,22 @@
 
 namespace pcs {
 
+// From a channel's pre-activation z to its log decay: logsigmoid(z) / tau, or -rate * softplus(z) with one rate per rate_dim
+// neighbouring channels; optionally the decay itself.
+struct DecayForm {
+  float inv_tau;
+  const float* rate;
+  int rate_dim, expo;
+  __device__ __forceinline__ float operator()(float z, int c) const {
+    const float l = rate ? -rate[c / rate_dim] * softplusf_(z) : logsigmoidf_(z) * inv_tau;
+    return expo ? expf(l) : l;
+  }
+};
+
 template <typename T>
 __global__ void __launch_bounds__(256) gla_decay_kernel(const T* __restrict__ a, long long a_stride, const T* __restrict__ a2,
                                                         const float* __restrict__ a2_b, float* __restrict__ ld, int n_channels, int rank,
-                                                        float inv_tau) {
+                                                        const DecayForm form) {
   extern __shared__ float as[];  // the token's low-rank input
   const long long t = blockIdx.x;
   for (int r = threadIdx.x; r < rank; r += blockDim.x) as[r] = ldf(a + t * a_stride + r);
@@ -28,7 +40,7 @@ __global__ void __launch_bounds__(256) gla_decay_kernel(const T* __restrict__ a,
     float z = 0.f;
     for (int r = 0; r < rank; ++r) z = fmaf(ldf(w + r), as[r], z);
     z += a2_b ? a2_b[c] : 0.f;
-    ld[t * n_channels + c] = logsigmoidf_(z) * inv_tau;
+    ld[t * n_channels + c] = form(z, c);
   }
 }
 
@@ -40,7 +52,7 @@ constexpr int kDecayTokens = 32;
 template <typename T>
 __global__ void __launch_bounds__(256) gla_decay_tile_kernel(const T* __restrict__ a, long long a_stride, const T* __restrict__ a2,
                                                              const float* __restrict__ a2_b, float* __restrict__ ld, int n_tokens, int n_channels,
-                                                             int rank, float inv_tau) {
+                                                             int rank, const DecayForm form) {
   extern __shared__ float sm[];
   float* w = sm;                 // [rank][256]
   float* as = sm + rank * 256;   // [kDecayTokens][rank]
@@ -60,7 +72,7 @@ __global__ void __launch_bounds__(256) gla_decay_tile_kernel(const T* __restrict
   for (int i = 0; i < nt; ++i) {
     float z = 0.f;
     for (int r = 0; r < rank; ++r) z = fmaf(w[r * 256 + threadIdx.x], as[i * rank + r], z);
-    ld[static_cast<long long>(t0 + i) * n_channels + c] = logsigmoidf_(z + bias) * inv_tau;
+    ld[static_cast<long long>(t0 + i) * n_channels + c] = form(z + bias, c);
   }
 }
 
@@ -504,18 +516,19 @@ PCS_API int pcs_gla_chunk_out(const pcs_gla_chunk_params* p, void* stream) {
 }
 
 PCS_API int pcs_gla_decay(const void* a, int64_t a_stride, const void* a2, const float* a2_b, float* ld, int n_tokens, int n_channels, int rank,
-                          float tau, int dtype, void* stream) {
+                          float tau, const float* rate, int rate_dim, int expo, int dtype, void* stream) {
   if (n_tokens == 0) return PCS_OK;
-  PCS_REQUIRE(a && a2 && ld && n_channels > 0 && rank > 0 && rank <= 8192 && tau > 0.f, "pcs_gla_decay: bad arguments");
+  PCS_REQUIRE(a && a2 && ld && n_channels > 0 && rank > 0 && rank <= 8192 && (rate ? rate_dim > 0 : tau > 0.f), "pcs_gla_decay: bad arguments");
+  const pcs::DecayForm form{rate ? 0.f : 1.f / tau, rate, rate_dim, expo};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const size_t tile_smem = static_cast<size_t>(rank) * (256 + pcs::kDecayTokens) * sizeof(float);
   if (n_tokens >= 2 * pcs::kDecayTokens && tile_smem <= 48 * 1024) {
     dim3 grid((n_channels + 255) / 256, (n_tokens + pcs::kDecayTokens - 1) / pcs::kDecayTokens);
     PCS_DISPATCH(dtype, pcs::gla_decay_tile_kernel<T><<<grid, 256, tile_smem, st>>>(static_cast<const T*>(a), a_stride, static_cast<const T*>(a2), a2_b, ld,
-                                                                                   n_tokens, n_channels, rank, 1.f / tau));
+                                                                                   n_tokens, n_channels, rank, form));
   } else
   PCS_DISPATCH(dtype, pcs::gla_decay_kernel<T><<<dim3(n_tokens, (n_channels + 255) / 256 > 64 ? 64 : (n_channels + 255) / 256), 256, rank * sizeof(float), st>>>(static_cast<const T*>(a), a_stride, static_cast<const T*>(a2),
-                                                                                           a2_b, ld, n_channels, rank, 1.f / tau));
+                                                                                           a2_b, ld, n_channels, rank, form));
   PCS_CHECK_CUDA(cudaGetLastError());
   pcs::count_launch();
   return PCS_OK;

@@ -420,7 +420,7 @@ PCS_API int pcs_silu_mul(const void* gu, int64_t gu_stride, void* out, int n_row
 PCS_API int pcs_glu_mul(const void* gu, int64_t gu_stride, void* out, int n_rows, int ff, const pcs_glu_act* glu, int dtype, void* stream) {
   if (n_rows == 0 || ff == 0) return PCS_OK;
   PCS_REQUIRE(gu && out && n_rows > 0 && ff > 0, "pcs_glu_mul: bad arguments");
-  PCS_REQUIRE(glu == nullptr || (glu->kind >= PCS_GLU_SILU && glu->kind <= PCS_ACT_GELU_ERF), "pcs_glu_mul: unknown activation %d", glu->kind);
+  PCS_REQUIRE(glu == nullptr || (glu->kind >= PCS_GLU_SILU && glu->kind <= PCS_GLU_GELU_TANH), "pcs_glu_mul: unknown activation %d", glu->kind);
   const pcs::GluAct act(glu);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const int piece = dtype == PCS_BF16 ? 8 : 4;

@@ -189,6 +189,16 @@ __global__ void __launch_bounds__(256) xielu_kernel(const T* __restrict__ z, lon
   }
 }
 
+template <typename T>
+__global__ void __launch_bounds__(256) soft_cap_kernel(const T* __restrict__ z, long long z_stride, float* __restrict__ out, int width, float cap) {
+  const long long r = blockIdx.x;
+  const float inv = cap > 0.f ? 1.f / cap : 0.f;
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < width; i += gridDim.y * blockDim.x) {
+    const float v = ldf(z + r * z_stride + i);
+    out[r * width + i] = cap > 0.f ? cap * tanhf(v * inv) : v;
+  }
+}
+
 // One block per row: the weighted sum of the terms' rows in shared memory, then the norm.
 template <typename T>
 __global__ void __launch_bounds__(256) depth_mix_kernel(const pcs_depthmix_params p) {
@@ -262,6 +272,17 @@ PCS_API int pcs_depth_mix(const pcs_depthmix_params* p, void* stream) {
   if (smem > 48 * 1024)
     PCS_DISPATCH(p->dtype, PCS_CHECK_CUDA(cudaFuncSetAttribute(pcs::depth_mix_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024)));
   PCS_DISPATCH(p->dtype, pcs::depth_mix_kernel<T><<<p->n_rows, 256, smem, st>>>(*p));
+  PCS_CHECK_CUDA(cudaGetLastError());
+  pcs::count_launch();
+  return PCS_OK;
+}
+
+PCS_API int pcs_soft_cap(const void* z, int64_t z_stride, float* out, int n_rows, int width, float cap, int dtype, void* stream) {
+  if (n_rows == 0) return PCS_OK;
+  PCS_REQUIRE(z && out && n_rows > 0 && width > 0, "pcs_soft_cap: bad arguments");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  dim3 grid(n_rows, (width + 1023) / 1024 > 64 ? 64 : (width + 1023) / 1024);
+  PCS_DISPATCH(dtype, pcs::soft_cap_kernel<T><<<grid, 256, 0, st>>>(static_cast<const T*>(z), z_stride, out, width, cap));
   PCS_CHECK_CUDA(cudaGetLastError());
   pcs::count_launch();
   return PCS_OK;

@@ -279,12 +279,34 @@ class Tevilix(LanguageModel):
         raise NotImplementedError("Tevilix keeps recurrent state next to K/V rows: there is no per-module K/V to cache and splice")
 
 
+class Zovolorn(LanguageModel):
+    """Adapter of the Zovolorn design (model/zovolorn.py) for the generation engine.  Its convolutions and its recurrent branches carry
+    state from token to token beside the K/V rows, so a prompt's state cannot be cut at module boundaries and spliced: pass
+    `cache=None` to `GenerationEngine.generate`, or batch requests with `BatchEngine`."""
+
+    def __init__(self, name: str, model=None, tokenizer=None, **kwargs):
+        from .zovolorn import ZovolornForCausalLM
+        if model is None:
+            model = ZovolornForCausalLM.from_pretrained(name, **kwargs)
+        if tokenizer is None:
+            from ..synthetic import IdTokenizer
+            tokenizer = IdTokenizer(model.vocab_size)
+        super().__init__(name, model, tokenizer, [tokenizer.eos_token_id], [])
+
+    def get_formatter(self) -> Callable[[str], str]:
+        return lambda prompt: prompt
+
+    def get_cache_shape(self) -> Tuple[int, int, int]:
+        raise NotImplementedError("Zovolorn keeps recurrent state next to K/V rows: there is no per-module K/V to cache and splice")
+
+
 # config.json "architecture" (or transformers' "architectures"/"model_type") -> loader of the bare model
 MODEL_REGISTRY = {
     "Mutolix": lambda path, **kw: _mutolix(path, **kw),
     "Raritar": lambda path, **kw: _lazy("raritar", "RaritarForCausalLM").from_pretrained(path, **kw),
     "Safilorn": lambda path, **kw: _lazy("safilorn", "SafilornForCausalLM").from_pretrained(path, **kw),
     "Tevilix": lambda path, **kw: _lazy("tevilix", "TevilixForCausalLM").from_pretrained(path, **kw),
+    "Zovolorn": lambda path, **kw: _lazy("zovolorn", "ZovolornForCausalLM").from_pretrained(path, **kw),
     "LlamaForCausalLM": lambda path, dtype=None, **kw: LlamaForCausalLM.from_pretrained(path, **kw),
     "FalconForCausalLM": lambda path, dtype=None, **kw: _lazy("falcon", "FalconForCausalLM").from_pretrained(path, **kw),
     "MptForCausalLM": lambda path, dtype=None, **kw: _lazy("mpt", "MptForCausalLM").from_pretrained(path, **kw),
@@ -316,5 +338,5 @@ def load_model(path: str, device="cuda", dtype=None, **kwargs):
     return loader(path, device=device, **kwargs)
 
 
-__all__ = ["LanguageModel", "Mutolix", "Raritar", "Safilorn", "Tevilix", "MODEL_REGISTRY", "load_model", "Llama2", "CodeLlama", "Falcon", "Mpt", "FormatConversation",
+__all__ = ["LanguageModel", "Mutolix", "Raritar", "Safilorn", "Tevilix", "Zovolorn", "MODEL_REGISTRY", "load_model", "Llama2", "CodeLlama", "Falcon", "Mpt", "FormatConversation",
            "FormatLlama2Conversation", "LlamaForCausalLM", "LlamaConfigLite"]

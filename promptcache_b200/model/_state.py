@@ -9,7 +9,7 @@ layer has pool tensors whose first dimension is the slot,
     low-rank attention  CKV [slots, 1, cap, rank + rot_dim]                        (compute type)
     decaying matrix   S [slots, H, dim, vdim]                                      (float32)
     matrix memory     S [slots, H, dim, vdim]    n [slots, H, dim]    m [slots, H]  (float32)
-    short convolution tail [slots, 2, taps - 1, width]                             (float32, double-buffered)
+    short convolution tail [slots, 2, taps - 1, width]                             (float32, double-buffered; a layer may have several, by name)
     vector state      vec [slots, width]                                            (float32)
 
 (a layer's spec may be a tuple of these, or None for a layer that reads another layer's rows)
@@ -65,6 +65,7 @@ class ConvTailSpec:
     and writes the other (the sequence's step parity says which), so that one launch can do both for a whole batch."""
     taps: int
     width: int
+    name: str = "tail"   # a layer with several convolutions names each one's tensor
 
 
 @dataclass(frozen=True)
@@ -99,7 +100,7 @@ class SlotPool:
                 out.update(self._alloc(part, n_slots, cap))
             return out
         if isinstance(spec, ConvTailSpec):
-            return {"tail": torch.zeros(n_slots, 2, max(spec.taps - 1, 1), spec.width, dtype=torch.float32, device=self.device)}
+            return {spec.name: torch.zeros(n_slots, 2, max(spec.taps - 1, 1), spec.width, dtype=torch.float32, device=self.device)}
         if isinstance(spec, KVSpec):
             return {"k": torch.zeros(n_slots, spec.n_kv_heads, cap, spec.dim, dtype=self.dtype, device=self.device),
                     "v": torch.zeros(n_slots, spec.n_kv_heads, cap, spec.vdim, dtype=self.dtype, device=self.device)}
