@@ -2,7 +2,8 @@
 (against the Llama prompt-cache path), `bench.py --design raritar` (against Mutolix's attention layers with a dense
 feed-forward of the same active size, which share the step function, the pool and the attention kernels) and
 `bench.py --design safilorn` (against Mutolix with the same order and sizes of recurrent and attention layers) and
-`bench.py --design tevilix` (against the same Mutolix model; its four layers run as a loop where Mutolix repeats them).  Random weights, synthetic token ids.  Prefill and decode tokens/s of both models through their own
+`bench.py --design tevilix` (against the same Mutolix model; its four layers run as a loop where Mutolix repeats them) and `bench.py --design
+zovolorn` (against the same Mutolix model).  Random weights, synthetic token ids.  Prefill and decode tokens/s of both models through their own
 step / forward, then every kernel of the new design alone against its roofline, next to the like kernel of the Llama path.
 
 Timing: CUDA events on the launching stream, >= 3 warm-up iterations, a 256 MiB write between timed iterations (flushes the
@@ -794,7 +795,215 @@ def run_tevilix(args, load_peaks, ClockSampler) -> None:
     print(json.dumps(line), flush=True)
 
 
+# ---- Zovolorn ---------------------------------------------------------------------------------------------------------
+ZOVOLORN_SIZES = {
+    # the recurrent and attention sizes of SIZES; attention chunks, buckets / reach of the distance bias, taps of the short convolution, low ranks;
+    # the gated feed-forward (three matrices) has the parameters of SIZES' feed-forward (two)
+    "w1024": dict(SIZES["w1024"], chunk=512, buckets=32, far=400, conv=4, taps=3, groups=8, rank=64, gff=2752),
+    "w2048": dict(SIZES["w2048"], chunk=512, buckets=32, far=400, conv=4, taps=3, groups=8, rank=128, gff=5504),
+}
+
+
+def zovolorn_config(s: dict) -> dict:
+    mlp = {"kind": "dense", "ff": s["gff"]}
+    att = {"type": "attention", "mlp": mlp, "mixer": {"heads": s["H"], "kv_heads": s["G"], "dim": s["D"], "vdim": s["V"], "scale": s["D"] ** -0.5,
+                                                      "rot": {"base": 10000.0, "dims": s["D"]}}}
+    par = {"type": "parallel", "mlp": mlp,
+           "mixer": {"left": {"heads": s["H"], "kv_heads": s["G"], "dim": s["D"], "vdim": s["D"], "scale": s["D"] ** -0.5, "bias_max": s["far"], "mask": {"size": s["chunk"]}},
+                     "right": {"heads": s["mH"], "kv_heads": s["mH"], "dim": s["mD"], "vdim": s["mV"], "conv": s["conv"]}, "left_scale": 0.7, "right_scale": 0.8}}
+    return {"architecture": "Zovolorn", "vocab": s["vocab"], "width": s["width"], "embedding": {"scale": 1.0, "bigram": {"buckets": 4093, "mul_prev": 29, "mul_cur": 5}},
+            "norm": {"eps": 1e-5, "groups": s["groups"]}, "canon": {"taps": s["taps"]}, "logit_softcap": 30.0, "layers": [par, att, att, par] * s["repeat"]}
+
+
+def zovolorn_tensors(cfg: dict, s: dict, device, seed: int = 0) -> Dict[str, torch.Tensor]:
+    g = torch.Generator(device=device).manual_seed(seed)
+    W, t = cfg["width"], {}
+    rnd = lambda *shape, std=1.0, mean=0.0: (torch.randn(*shape, generator=g, device=device) * std + mean).to(torch.bfloat16)
+    lin = lambda o, i: rnd(o, i, std=i ** -0.5)
+    t["embed"], t["bigram"], t["final.norm"] = rnd(cfg["vocab"], W), rnd(cfg["embedding"]["bigram"]["buckets"] + 1, W, std=0.5), rnd(W, std=0.05, mean=1.0)
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, ff = f"l{i}.", layer["mixer"], layer["mlp"]["ff"]
+        for n in ("1", "2"):
+            t[p + "norm" + n], t[p + "canon" + n] = rnd(W, std=0.05, mean=1.0), rnd(W, s["taps"], std=0.3)
+        if layer["type"] == "attention":
+            H, G, D, V = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            t[p + "mix.q"], t[p + "mix.k"], t[p + "mix.v"] = lin(H * D, W), lin(G * D, W), lin(G * V, W)
+            t[p + "mix.q.norm"], t[p + "mix.k.norm"] = rnd(H * D, std=0.1, mean=1.0), rnd(G * D, std=0.1, mean=1.0)
+            t[p + "mix.sink"], t[p + "mix.g"], t[p + "mix.o"] = rnd(H), lin(H, W), lin(W, H * V)
+        else:
+            a, r, q, k = m["left"], m["right"], p + "mix.left.", p + "mix.right."
+            H, G, D = a["heads"], a["kv_heads"], a["dim"]
+            t[q + "q"], t[q + "k"], t[q + "o"] = lin(H * D, W), lin(G * D, W), lin(W, H * D)
+            t[q + "q.norm"], t[q + "k.norm"] = rnd(D, std=0.1, mean=1.0), rnd(D, std=0.1, mean=1.0)
+            t[q + "rel"], t[q + "temp"] = rnd(s["buckets"], H), rnd(H, std=0.1, mean=1.0)
+            H, G, D, V = r["heads"], r["kv_heads"], r["dim"], r["vdim"]
+            for n, rows in (("q", G * D), ("k", G * D), ("v", H * V)):
+                t[k + n], t[k + n + ".conv"] = lin(rows, W), rnd(rows, r["conv"], std=0.4)
+            t[k + "b"], t[k + "A_log"], t[k + "dt_bias"] = lin(H, W), rnd(H, std=0.3, mean=-2.0), rnd(H * D)
+            t[k + "a1"], t[k + "a2"], t[k + "g1"], t[k + "g2"] = lin(s["rank"], W), lin(H * D, s["rank"]), lin(s["rank"], W), lin(H * V, s["rank"])
+            t[k + "norm"], t[k + "o"] = rnd(V, std=0.05, mean=1.0), lin(W, H * V)
+        t[p + "mlp.gate"], t[p + "mlp.up"], t[p + "mlp.down"] = lin(ff, W), lin(ff, W), lin(W, ff)
+        t[p + "mlp.gate.b"], t[p + "mlp.up.b"], t[p + "mlp.down.b"] = rnd(ff, std=0.1), rnd(ff, std=0.1), rnd(W, std=0.1)
+    return t
+
+
+def zovolorn_block(s: dict, dev, timer: Timer, prompt: int, batch: int, ctx: int) -> dict:
+    from .model.mutolix import MutolixConfig, MutolixForCausalLM
+    from .model.zovolorn import ZovolornConfig, ZovolornForCausalLM
+    cfg = zovolorn_config(s)
+    out = {"layers": len(cfg["layers"]), "width": s["width"]}
+    m = ZovolornForCausalLM(ZovolornConfig(cfg), zovolorn_tensors(cfg, s, dev), device=dev, dtype=torch.bfloat16)
+    _throughput(m, s, timer, prompt, batch, ctx, out)
+    del m
+    torch.cuda.empty_cache()
+    mc = mutolix_config(s)   # the closest existing model: recurrent and attention layers in the same order, at the same sizes
+    mm = MutolixForCausalLM(MutolixConfig(mc), random_tensors(mc, dev), device=dev, dtype=torch.bfloat16)
+    _throughput(mm, s, timer, prompt, batch, ctx, out, prefix="mutolix_")
+    del mm
+    torch.cuda.empty_cache()
+    return out
+
+
+def zovolorn_kernels(s: dict, dev, timer: Timer, prompt: int, ctx: int, hbm_gbs: float, tflops: float) -> dict:
+    """Every kernel of the design alone at this size, achieved / peak, beside the like kernel of the closest model (for the recurrence also
+    Safilorn's, whose state decays per key channel too)."""
+    from . import _native_seq as nsq
+    from .model.zovolorn import distance_bias_table
+    bf, H, G, D, V, W, chunk = torch.bfloat16, s["H"], s["G"], s["D"], s["V"], s["width"], s["chunk"]
+    out = {}
+    gb = lambda by, ms: {"us": round(ms * 1e3, 2), "gb_s": round(by / ms / 1e6, 1), "of_measured_hbm_peak": round(by / ms / 1e6 / hbm_gbs, 4)}
+    tf = lambda fl, ms: {"ms": round(ms, 4), "tflops": round(fl / ms / 1e9, 1), "of_measured_bf16_peak": round(fl / ms / 1e9 / tflops, 3)}
+    ones = lambda *n: torch.ones(*n, device=dev, dtype=bf)
+    cap = ((max(prompt, ctx + 1) + 127) // 128) * 128
+    b, b1 = nsq.Batch([0], [0], [prompt], dev), nsq.Batch([0], [ctx], [1], dev)
+    kp, vp = torch.randn(1, G, cap, D, device=dev).to(bf), torch.randn(1, G, cap, V, device=dev).to(bf)
+    q, o = torch.randn(prompt, H * D, device=dev).to(bf), torch.empty(prompt, H * V, device=dev, dtype=bf)
+    sink, temp, gt = torch.randn(H, device=dev), torch.rand(H, device=dev) + 0.5, torch.randn(prompt, H, device=dev).to(bf)
+    r1, r2 = torch.full((H,), 0.5, device=dev), torch.full((H,), 0.5, device=dev)
+    table = distance_bias_table(torch.randn(s["buckets"], H, device=dev), s["far"], chunk - 1)
+    # prompt attention: FLOPs = 2 (D + V) per (query, visible key) pair and head
+    full = prompt * (prompt + 1) / 2
+    pairs = sum(i % chunk + 1 for i in range(prompt))
+    ms = timer(lambda: nsq.attention(q, kp, vp, o, H, D ** -0.5, None, None, True, b, sink_logit=sink, head_gate=gt))
+    out["attn_prompt_sink_gate"] = tf(2.0 * (D + V) * H * full, ms)
+    ms = timer(lambda: nsq.attention(q, kp, vp, o, H, D ** -0.5, r1, r2, True, b))
+    out["like_attn_prompt"] = tf(2.0 * (D + V) * H * full, ms)
+    ms = timer(lambda: nsq.attention(q, kp, vp, o, H, D ** -0.5, None, None, False, b, head_scale=temp, bias_table=table, chunk=chunk, out_scale=0.7))
+    out["attn_prompt_chunked"] = tf(2.0 * (D + V) * H * pairs, ms)
+    win = chunk // 2     # a window of half a chunk sees as many keys per query on average
+    wpairs = sum(min(i + 1, win) for i in range(prompt))
+    ms = timer(lambda: nsq.attention(q, kp, vp, o, H, D ** -0.5, r1, r2, True, b, window=win))
+    out["like_attn_prompt_window"] = tf(2.0 * (D + V) * H * wpairs, ms)
+    # one decoded token: bytes = visible K and V rows of every key/value head (a chunk that is nearly full)
+    q1, o1, ws = torch.randn(1, H * D, device=dev).to(bf), torch.empty(1, H * V, device=dev, dtype=bf), nsq.attn_workspace(1, H, V, dev)
+    ms = timer(lambda: nsq.attention(q1, kp, vp, o1, H, D ** -0.5, None, None, True, b1, max_keys=cap, workspace=ws, sink_logit=sink, head_gate=gt[:1]), steps=15)
+    out["attn_decode_sink_gate"] = gb(2.0 * G * (ctx + 1) * (D + V), ms)
+    ms = timer(lambda: nsq.attention(q1, kp, vp, o1, H, D ** -0.5, r1, r2, True, b1, max_keys=cap, workspace=ws), steps=15)
+    out["like_attn_decode"] = gb(2.0 * G * (ctx + 1) * (D + V), ms)
+    be = nsq.Batch([0], [chunk * 3 - 1], [1], dev)
+    ms = timer(lambda: nsq.attention(q1, kp, vp, o1, H, D ** -0.5, None, None, False, be, max_keys=chunk, workspace=ws, head_scale=temp, bias_table=table, chunk=chunk), steps=15)
+    out["attn_decode_chunked"] = gb(2.0 * G * chunk * (D + V), ms)
+    ms = timer(lambda: nsq.attention(q1, kp, vp, o1, H, D ** -0.5, r1, r2, True, be, max_keys=chunk, workspace=ws, window=chunk), steps=15)
+    out["like_attn_decode_window"] = gb(2.0 * G * chunk * (D + V), ms)
+    # norms + rotation + append: reads the projection row, writes q, k, v; like: Mutolix's whole-projection norms + append
+    nq, nk = H * D, G * (D + V)
+    pj = torch.randn(prompt, nq + nk, device=dev).to(bf)
+    fr = torch.tensor([10000.0 ** (-2.0 * i / D) for i in range(D // 2)], dtype=torch.float64, device=dev)
+    offs = (0, nq, nq + G * D)
+    qn, kn, hn = ones(nq), ones(G * D), ones(D)
+    ms = timer(lambda: nsq.rope_kv_prep(pj, offs, H, G, D, V, fr, D, True, False, 1e-5, q, kp, vp, b, q_norm_w=qn, k_norm_w=kn, norm_whole=True))
+    out["whole_norm_rope_append"] = gb(prompt * (nq + nk) * 4.0, ms)
+    ms = timer(lambda: nsq.rope_kv_prep(pj, (0, nq, nq), H, G, D, D, None, 0, True, False, 1e-5, q, kp, vp, b, q_norm_w=hn, k_norm_w=hn))
+    out["head_norm_append_values_are_keys"] = gb(prompt * (nq + G * D) * 2.0 + prompt * (nq + 2 * G * D) * 2.0, ms)
+    ms = timer(lambda: nsq.qk_prep(pj, offs, qn, kn, 1e-5, H, G, D, V, 0.0, 0, q, kp, vp, None, None, b))
+    out["like_qk_prep"] = gb(prompt * (nq + nk) * 4.0, ms)
+    # layer boundary: reads x (4 B) and y (2 B), writes x (4 B) and h (2 B), neighbours from L2; like: output norm + residual + next norm
+    x, x2, y, h = torch.randn(prompt, W, device=dev), torch.empty(prompt, W, device=dev), torch.randn(prompt, W, device=dev).to(bf), torch.empty(prompt, W, device=dev, dtype=bf)
+    wn, cw, tail = ones(W), (torch.randn(s["taps"], W, device=dev) * 0.3).to(bf), torch.zeros(1, 2, s["taps"] - 1, W, device=dev)
+    ms = timer(lambda: nsq.group_norm_conv(x, s["groups"], 1e-5, bf, x_out=x2, y=y, w=wn, conv_w=cw, tail=tail, h_out=h, batch=b))
+    out["group_norm_add_conv"] = gb(prompt * W * 12.0, ms)
+    ms = timer(lambda: nsq.gate_norm_add(x, y, None, wn, None, 1e-5, wn, h))
+    out["like_norm_add_norm"] = gb(prompt * W * 12.0, ms)
+    ms = timer(lambda: nsq.norm_conv(x, wn, 1e-5, h, conv_w=cw, tail=tail, batch=b))
+    out["like_norm_conv"] = gb(prompt * W * 6.0, ms)
+    y1, h1 = y[:1].contiguous(), h[:1].contiguous()
+    ms = timer(lambda: nsq.group_norm_conv(x[:1], s["groups"], 1e-5, bf, x_out=x2[:1], y=y1, w=wn, conv_w=cw, tail=tail, h_out=h1, batch=b1), steps=15)
+    out["group_norm_add_conv_decode_us"] = round(ms * 1e3, 2)
+    ms = timer(lambda: nsq.gate_norm_add(x[:1], y1, None, wn, None, 1e-5, wn, h1), steps=15)
+    out["like_norm_add_norm_decode_us"] = round(ms * 1e3, 2)
+    # the delta rule's inputs: reads the projection columns (2 B), writes unit vectors (4 B) and values (2 B)
+    mH, mD, mV, rk = s["mH"], s["mD"], s["mV"], s["rank"]
+    ch = 2 * mH * mD + mH * mV
+    pr = (torch.randn(prompt, ch + 2 * rk + 8, device=dev) * 0.5).to(bf)
+    cv, ctail = (torch.randn(s["conv"], ch, device=dev) * 0.4).to(bf), torch.zeros(1, 2, s["conv"] - 1, ch, device=dev)
+    ms = timer(lambda: nsq.short_conv(pr, 0, mH, mD, mH * mV, cv, ctail, mD ** -0.5, 1e-6, b))
+    out["short_conv"] = gb(prompt * (2.0 * ch + 8.0 * mH * mD + 2.0 * mH * mV), ms)
+    a2, dtb, rate = (torch.randn(mH * mD, rk, device=dev) * rk ** -0.5).to(bf), torch.randn(mH * mD, device=dev), torch.full((mH,), 0.1, device=dev)
+    ms = timer(lambda: nsq.gla_decay(pr[:, ch:ch + rk], a2, dtb, 1.0, rate=rate))
+    out["delta_decay"] = gb(prompt * mH * mD * 4.0, ms)
+    ms = timer(lambda: nsq.gla_decay(pr[:, ch:ch + rk], a2, dtb, 16.0))
+    out["like_gla_decay"] = gb(prompt * mH * mD * 4.0, ms)
+    # the recurrence over a prompt and of one decoded token (state read and written once)
+    qk, v = nsq.short_conv(pr, 0, mH, mD, mH * mV, cv, ctail, mD ** -0.5, 1e-6, b)
+    ld = nsq.gla_decay(pr[:, ch:ch + rk], a2, dtb, 1.0, rate=rate)
+    sp, nw, og, gate = torch.zeros(1, mH, mD, mV, device=dev), ones(mV), torch.empty(prompt, mH * mV, device=dev, dtype=bf), torch.randn(prompt, mH * mV, device=dev).to(bf)
+    bt = pr[:, ch + 2 * rk:ch + 2 * rk + mH]
+    rec = lambda ms, n=prompt: {"ms": round(ms, 3), "us_per_token": round(ms * 1e3 / n, 3), "gflops": round(4.0 * mH * mD * mV * n / ms / 1e6, 1)}
+    out["delta_scan_prompt"] = rec(timer(lambda: nsq.delta_scan(qk, v, ld, bt, mH, sp, nw, gate, og, 1e-5, b), steps=5))
+    dec = torch.exp(ld)
+    out["delta_scan_prompt_token_by_token"] = rec(timer(lambda: nsq.delta_scan(qk, v, dec, bt, mH, sp, nw, gate, og, 1e-5, b, impl=2), steps=5))
+    ms = timer(lambda: nsq.delta_scan(qk[:1], v[:1], dec[:1], bt[:1], mH, sp, nw, gate[:1], og[:1], 1e-5, b1), steps=15)
+    out["delta_scan_decode"] = gb(8.0 * mH * mD * mV, ms)
+    pm = (torch.randn(prompt, 2 * mH * mD + 2 * mH * mV, device=dev) * 0.3).to(bf)
+    goffs = (0, mH * mD, 2 * mH * mD, 2 * mH * mD + mH * mV)
+    out["like_gla_scan_prompt"] = rec(timer(lambda: nsq.gla_scan(pm, goffs, ld, nw, og, sp, 1e-5, b), steps=5))
+    ms = timer(lambda: nsq.gla_scan(pm[:1], goffs, ld[:1], nw, og[:1], sp, 1e-5, b1), steps=15)
+    out["like_gla_scan_decode"] = gb(8.0 * mH * mD * mV, ms)
+    ig, fg = torch.randn(prompt, mH, device=dev), -torch.rand(prompt, mH, device=dev) * 0.1
+    npool, mp, nwm = torch.zeros(1, mH, mD, device=dev), torch.zeros(1, mH, device=dev), ones(mH * mV)
+    out["like_mlstm_scan_prompt"] = rec(timer(lambda: nsq.mlstm_scan(pm, goffs, ig, fg, nwm, og, sp, npool, mp, 1e-5, b), steps=5))
+    ms = timer(lambda: nsq.mlstm_scan(pm[:1], goffs, ig[:1], fg[:1], nwm, og[:1], sp, npool, mp, 1e-5, b1), steps=15)
+    out["like_mlstm_scan_decode"] = gb(8.0 * mH * mD * mV, ms)
+    # feed-forward activation and the cap on the logits
+    ff = s["gff"]
+    u = torch.randn(prompt, 2 * ff, device=dev).to(bf)
+    ms = timer(lambda: nsq.glu_mul(u, ff, (nsq.GLU_GELU_TANH, 0.0, 0.0)))
+    out["gelu_tanh_mul"] = gb(prompt * ff * 6.0, ms)
+    z, zo, av = torch.randn(prompt, s["ff"], device=dev).to(bf), torch.empty(prompt, s["ff"], device=dev, dtype=bf), torch.randn(2, device=dev).to(bf)
+    ms = timer(lambda: nsq.xielu(z, zo, av))
+    out["like_xielu"] = gb(prompt * s["ff"] * 4.0, ms)
+    lg = torch.randn(1, s["vocab"], device=dev).to(bf)
+    out["soft_cap_us"] = round(timer(lambda: nsq.soft_cap(lg, 30.0), steps=15) * 1e3, 2)
+    return out
+
+
+def run_zovolorn(args, load_peaks, ClockSampler) -> None:
+    from . import _native_seq as nsq
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    nsq.load()
+    hbm, kind, tfl = load_peaks()
+    timer = Timer(dev)
+    sampler = ClockSampler(0)
+    sampler.start()
+    sampler.mark()
+    before = nsq.launch_count()
+    line = {"design": "zovolorn", "compared_with": "mutolix (recurrent and attention layers in the same order, at the same sizes) on the same step function, "
+                                                   "pool and kernels; this design's recurrent layers run chunked attention beside the recurrence",
+            "dtype": "bf16", "data": "synthetic", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tfl, "kind": kind},
+            "timing": "CUDA events, 3 warm-up iterations, 256 MiB L2 flush between iterations, median", "sizes": {}}
+    prompt, batch, ctx = 2048, 4, 2048
+    for name, s in ZOVOLORN_SIZES.items():
+        blk = zovolorn_block(s, dev, timer, prompt, batch, ctx)
+        blk["kernels"] = zovolorn_kernels(s, dev, timer, prompt, ctx, hbm, tfl)
+        line["sizes"][name] = blk
+    line["gpu_launches"] = nsq.launch_count() - before
+    line["clocks"] = sampler.stop()
+    print(json.dumps(line), flush=True)
+
 def run(args, load_peaks, ClockSampler) -> None:
+    if args.design == "zovolorn":
+        return run_zovolorn(args, load_peaks, ClockSampler)
     if args.design == "tevilix":
         return run_tevilix(args, load_peaks, ClockSampler)
     if args.design == "raritar":

@@ -75,103 +75,123 @@ __global__ void __launch_bounds__(256) short_conv_kernel(const pcs_shortconv_par
       for (int c = tid; c < C; c += 256) cp.wr[static_cast<long long>(q) * C + c] = cp.rd[static_cast<long long>(q + cp.len) * C + c];
 }
 
-// 16-byte pieces, at most MR + 1 taps: a thread owns one piece of the channels [blockIdx.y * CB, ...) for TB neighbouring tokens, whose
-// rows and predecessors are requested together.  CB is a multiple of dim, so a head's pieces meet in this block's shared memory.
-template <typename T, int TB, int MR>
-__global__ void __launch_bounds__(256) short_conv_vec_kernel(const pcs_shortconv_params p, int CB) {
-  constexpr int N = Vec<T>::n, RN = TB + MR;
+// 16-byte pieces: a thread owns one piece of the channels [blockIdx.y * CB, ...) for TB neighbouring tokens, whose rows and R predecessors are
+// requested before the block knows which of them its tokens need.  CB is a multiple of dim, so a head's pieces meet in this block: by
+// shuffles where a head is a power of two up to 32 pieces, else through shared memory.
+template <typename T, int TB, int R>
+__global__ void __launch_bounds__(256, 2) short_conv_vec_kernel(const pcs_shortconv_params p, int CB) {
+  constexpr int N = Vec<T>::n, RN = TB + R;
   __shared__ float ssq[TB][256];
-  __shared__ float fac[TB][256];
-  const int t0 = blockIdx.x * TB, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int D = p.dim, U = 2 * p.kv_heads * D, C = U + p.v_width, R = p.taps - 1;
+  const int t0 = blockIdx.x * TB, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;   // (warp, lane: shared-memory sums)
+  const int D = p.dim, U = 2 * p.kv_heads * D, C = U + p.v_width;
   const int c_lo = blockIdx.y * CB, c = c_lo + tid * N;
   const bool active = tid * N < CB && c < C;
   const T* cw = static_cast<const T*>(p.conv_w);
-  ConvPlace cp[TB];
-  bool need[RN];
-#pragma unroll
-  for (int k = 0; k < RN; ++k) need[k] = false;
-#pragma unroll
-  for (int i = 0; i < TB; ++i) {
-    cp[i] = ConvPlace{0, 0, 1, nullptr, nullptr};
-    if (t0 + i < p.n_tokens) {
-      cp[i] = conv_place(p, t0 + i, R, C);
-      need[MR + i] = true;
-#pragma unroll
-      for (int j = 1; j <= MR; ++j)
-        if (j <= R && cp[i].pos - j >= cp[i].pos0) need[MR + i - j] = true;
-    }
-  }
   uint4 xv[RN];
   const T* x = static_cast<const T*>(p.proj) + p.c_off + c;
-  if (active) {
 #pragma unroll
-    for (int k = 0; k < RN; ++k)
-      if (need[k]) xv[k] = *reinterpret_cast<const uint4*>(x + static_cast<long long>(t0 - MR + k) * p.row_stride);
+  for (int k = 0; k < RN; ++k) {
+    const int r = t0 - R + k;
+    xv[k] = active && r >= 0 && r < p.n_tokens ? *reinterpret_cast<const uint4*>(x + static_cast<long long>(r) * p.row_stride) : make_uint4(0u, 0u, 0u, 0u);
   }
-  float o[TB][N];
+  // the tokens' places in their entries (see the boundary kernel): predecessors in this step and at all, tail row to write, rows that stay
+  int here[TB], before[TB], last_row[TB], shift[TB], par[TB];
+  long long tail0[TB];
+#pragma unroll
+  for (int i = 0; i < TB; ++i) {
+    here[i] = before[i] = shift[i] = par[i] = 0;
+    last_row[i] = -1;
+    tail0[i] = 0;
+    if (R > 0 && t0 + i < p.n_tokens) {
+      const int b = p.tok_seq[t0 + i], pos = p.tok_pos[t0 + i], pos0 = p.seq_pos0[b], len = p.seq_len[b];
+      here[i] = min(R, pos - pos0);
+      before[i] = min(R, pos);
+      last_row[i] = pos - (pos0 + len - R);
+      if (pos == pos0 + len - 1 && len < R) shift[i] = len;
+      par[i] = p.seq_par[b] & 1;
+      tail0[i] = (static_cast<long long>(p.seq_slot[b]) * 2 + par[i]) * R * C + c;
+    }
+  }
+  float o[TB][N], ss[TB];
+#pragma unroll
+  for (int i = 0; i < TB; ++i) {
+    ss[i] = 0.f;
+#pragma unroll
+    for (int e = 0; e < N; ++e) o[i][e] = 0.f;
+  }
   if (active) {
 #pragma unroll
-    for (int i = 0; i < TB; ++i)
+    for (int j = 0; j <= R; ++j) {
+      float wv[N];
+      ld16(cw + static_cast<long long>(R - j) * C + c, wv);
 #pragma unroll
-      for (int e = 0; e < N; ++e) o[i][e] = 0.f;
+      for (int i = 0; i < TB; ++i)
+        if (j <= before[i]) {
+          float v[N];
+          if (j <= here[i]) ld16(reinterpret_cast<const T*>(&xv[R + i - j]), v);
+          else ldx(p.tail + tail0[i] + static_cast<long long>(R - (j - here[i])) * C, v);
 #pragma unroll
-    for (int j = 0; j <= MR; ++j)
-      if (j <= R) {
-        float wv[N];
-        ld16(cw + static_cast<long long>(R - j) * C + c, wv);
-#pragma unroll
-        for (int i = 0; i < TB; ++i)
-          if (need[MR + i] && cp[i].pos - j >= 0) {
-            float v[N];
-            if (cp[i].pos - j >= cp[i].pos0) ld16(reinterpret_cast<const T*>(&xv[MR + i - j]), v);
-            else ldx(cp[i].rd + static_cast<long long>(R - (cp[i].pos0 - (cp[i].pos - j))) * C + c, v);
-#pragma unroll
-            for (int e = 0; e < N; ++e) o[i][e] = fmaf(wv[e], v[e], o[i][e]);
-          }
-      }
+          for (int e = 0; e < N; ++e) o[i][e] = fmaf(wv[e], v[e], o[i][e]);
+        }
+    }
 #pragma unroll
     for (int i = 0; i < TB; ++i) {
-      float a = 0.f;
 #pragma unroll
       for (int e = 0; e < N; ++e) {
         o[i][e] = silu_(o[i][e]);
-        a = fmaf(o[i][e], o[i][e], a);
+        ss[i] = fmaf(o[i][e], o[i][e], ss[i]);
       }
-      ssq[i][tid] = a;
-      if (need[MR + i]) {
-        const int last_row = cp[i].pos - (cp[i].pos0 + cp[i].len - R);
-        if (R > 0 && last_row >= 0) {
-          float v[N];
-          ld16(reinterpret_cast<const T*>(&xv[MR + i]), v);
-          stx(cp[i].wr + static_cast<long long>(last_row) * C + c, v);
+      if (R > 0) {
+        float* wr = p.tail + tail0[i] + (par[i] ? -1LL : 1LL) * R * C;
+        float v[N];
+        if (last_row[i] >= 0) {
+          ld16(reinterpret_cast<const T*>(&xv[R + i]), v);
+          stx(wr + static_cast<long long>(last_row[i]) * C, v);
         }
-        if (R > 0 && cp[i].pos == cp[i].pos0 + cp[i].len - 1 && cp[i].len < R)
-          for (int q = 0; q < R - cp[i].len; ++q) {
-            float v[N];
-            ldx(cp[i].rd + static_cast<long long>(q + cp[i].len) * C + c, v);
-            stx(cp[i].wr + static_cast<long long>(q) * C + c, v);
+        if (shift[i] > 0)
+          for (int q = 0; q < R - shift[i]; ++q) {
+            ldx(p.tail + tail0[i] + static_cast<long long>(q + shift[i]) * C, v);
+            stx(wr + static_cast<long long>(q) * C, v);
           }
       }
     }
   }
-  __syncthreads();
-  // heads of this block's channels: a warp adds the pieces of one (token, head)
-  const int PD = D / N, heads = max(0, min(CB, U - c_lo)) / D;
-  for (int e = warp; e < TB * heads; e += 8) {
-    const int i = e / heads, hd = e - i * heads;
-    float a = 0.f;
-    for (int k = lane; k < PD; k += 32) a += ssq[i][hd * PD + k];
-    a = warp_sum(a);
-    if (lane == 0) fac[i][hd] = (c_lo / D + hd < p.kv_heads ? p.q_scale : 1.f) / sqrtf(a + p.unit_eps);
+  // every piece's head sum
+  const int PD = D / N;
+  if (c_lo < U) {   // (uniform) this block holds query or key heads
+    if (PD <= 32 && (PD & (PD - 1)) == 0) {
+#pragma unroll
+      for (int q = 1; q < 32; q <<= 1)
+        if (q < PD) {
+#pragma unroll
+          for (int i = 0; i < TB; ++i) ss[i] += __shfl_xor_sync(0xffffffffu, ss[i], q);
+        }
+    } else {
+#pragma unroll
+      for (int i = 0; i < TB; ++i) ssq[i][tid] = ss[i];
+      __syncthreads();
+      const int heads = min(CB, U - c_lo) / D;
+      // a warp adds the pieces of one (token, head); the sum goes to the head's first piece
+      for (int e = warp; e < TB * heads; e += static_cast<int>(blockDim.x) >> 5) {
+        const int i = e / heads, hd = e - i * heads;
+        float a = 0.f;
+        for (int k = lane; k < PD; k += 32) a += ssq[i][hd * PD + k];
+        a = warp_sum(a);
+        if (lane == 0) ssq[i][hd * PD] = a;
+      }
+      __syncthreads();
+      if (c < U) {
+#pragma unroll
+        for (int i = 0; i < TB; ++i) ss[i] = ssq[i][tid / PD * PD];
+      }
+    }
   }
-  __syncthreads();
   if (!active) return;
 #pragma unroll
   for (int i = 0; i < TB; ++i)
-    if (need[MR + i]) {
+    if (t0 + i < p.n_tokens) {
       if (c < U) {
-        const float f = fac[i][(c - c_lo) / D];
+        const float f = (c < U / 2 ? p.q_scale : 1.f) / sqrtf(ss[i] + p.unit_eps);
 #pragma unroll
         for (int e = 0; e < N; ++e) o[i][e] *= f;
         stx(p.qk_out + static_cast<long long>(t0 + i) * U + c, o[i]);
@@ -181,22 +201,26 @@ __global__ void __launch_bounds__(256) short_conv_vec_kernel(const pcs_shortconv
     }
 }
 
+template <typename T, int R>
+static void launch_short_conv_taps(const pcs_shortconv_params& p, cudaStream_t st) {
+  const int per = 256 * Vec<T>::n, C = 2 * p.kv_heads * p.dim + p.v_width;
+  int CB = per / p.dim * p.dim;
+  if (p.n_tokens < 64) {   // few tokens: narrow channel blocks, so that the launch covers more SMs
+    const int small = (32 * Vec<T>::n + p.dim - 1) / p.dim * p.dim;
+    if (small < CB) CB = small;
+  }
+  const int ny = (C + CB - 1) / CB, thr = (CB / Vec<T>::n + 31) / 32 * 32;
+  if (R > 0 && p.n_tokens >= 4 * 148) short_conv_vec_kernel<T, (R > 0 ? 4 : 1), R><<<dim3((p.n_tokens + 3) / 4, ny), thr, 0, st>>>(p, CB);
+  else short_conv_vec_kernel<T, 1, R><<<dim3(p.n_tokens, ny), thr, 0, st>>>(p, CB);
+}
+
 template <typename T>
 static int launch_short_conv(const pcs_shortconv_params& p, cudaStream_t st, bool vec) {
-  if (vec) {
-    const int per = 256 * Vec<T>::n, C = 2 * p.kv_heads * p.dim + p.v_width;
-    // few tokens: narrow channel blocks, so that the launch covers more SMs
-    int CB = per / p.dim * p.dim;
-    if (p.n_tokens < 64) {
-      const int small = (32 * Vec<T>::n + p.dim - 1) / p.dim * p.dim;
-      if (small < CB) CB = small;
-    }
-    const int ny = (C + CB - 1) / CB;
-    if (p.n_tokens >= 4 * 148) short_conv_vec_kernel<T, 4, 3><<<dim3((p.n_tokens + 3) / 4, ny), 256, 0, st>>>(p, CB);
-    else short_conv_vec_kernel<T, 1, 3><<<dim3(p.n_tokens, ny), 256, 0, st>>>(p, CB);
-  } else {
-    short_conv_kernel<T><<<p.n_tokens, 256, 0, st>>>(p);
-  }
+  if (!vec) short_conv_kernel<T><<<p.n_tokens, 256, 0, st>>>(p);
+  else if (p.taps == 1) launch_short_conv_taps<T, 0>(p, st);
+  else if (p.taps == 2) launch_short_conv_taps<T, 1>(p, st);
+  else if (p.taps == 3) launch_short_conv_taps<T, 2>(p, st);
+  else launch_short_conv_taps<T, 3>(p, st);
   PCS_CHECK_CUDA(cudaGetLastError());
   count_launch();
   return PCS_OK;

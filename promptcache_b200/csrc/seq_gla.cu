@@ -44,35 +44,62 @@ __global__ void __launch_bounds__(256) gla_decay_kernel(const T* __restrict__ a,
   }
 }
 
-// Many tokens: block = (256 channels, kDecayTokens tokens).  The block's rows of A2 sit in shared memory transposed (a thread reads
-// its own channel's numbers without bank conflicts) and the tokens' low-rank inputs beside them (broadcast reads); a thread
-// owns one channel and walks the tokens, so the stores of a token are contiguous over the threads.  The sum runs over r in
-// increasing order as in the kernel above: both give the same bits.
-constexpr int kDecayTokens = 32;
+// Many tokens: block = 128 channels x 32 tokens, a thread owns 4 channels of 4 tokens.  The low rank is walked in pieces of kDecayR: the block's
+// rows of A2 and its tokens' low-rank inputs sit in shared memory, rank first, so a step is two 16-byte reads for 16 multiply-adds.
+// The sum runs over r in increasing order as in the kernel above: both give the same bits.
+constexpr int kDecayTokens = 32, kDecayChannels = 128, kDecayR = 32;
 template <typename T>
 __global__ void __launch_bounds__(256) gla_decay_tile_kernel(const T* __restrict__ a, long long a_stride, const T* __restrict__ a2,
                                                              const float* __restrict__ a2_b, float* __restrict__ ld, int n_tokens, int n_channels,
                                                              int rank, const DecayForm form) {
-  extern __shared__ float sm[];
-  float* w = sm;                 // [rank][256]
-  float* as = sm + rank * 256;   // [kDecayTokens][rank]
-  const int c = blockIdx.x * 256 + threadIdx.x, t0 = blockIdx.y * kDecayTokens;
-  const int nt = min(kDecayTokens, n_tokens - t0);
-  for (int e = threadIdx.x; e < 256 * rank; e += 256) {
-    const int cc = e / rank, r = e - cc * rank, ch = blockIdx.x * 256 + cc;
-    w[r * 256 + cc] = ch < n_channels ? ldf(a2 + static_cast<long long>(ch) * rank + r) : 0.f;
+  __shared__ __align__(16) float w[kDecayR][kDecayChannels + 4];
+  __shared__ __align__(16) float as[kDecayR][kDecayTokens + 4];
+  const int c0 = blockIdx.x * kDecayChannels, t0 = blockIdx.y * kDecayTokens, tid = threadIdx.x;
+  const int cq = (tid & 31) * 4, tq = (tid >> 5) * 4;
+  float acc[4][4];   // [token][channel]
+#pragma unroll
+  for (int i = 0; i < 4; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+  for (int r0 = 0; r0 < rank; r0 += kDecayR) {
+    const int rn = min(kDecayR, rank - r0);
+    for (int e = tid; e < kDecayChannels * kDecayR; e += 256) {
+      const int c = e / kDecayR, r = e - c * kDecayR;
+      w[r][c] = (r < rn && c0 + c < n_channels) ? ldf(a2 + static_cast<long long>(c0 + c) * rank + r0 + r) : 0.f;
+    }
+    for (int e = tid; e < kDecayTokens * kDecayR; e += 256) {
+      const int t = e / kDecayR, r = e - t * kDecayR;
+      as[r][t] = (r < rn && t0 + t < n_tokens) ? ldf(a + static_cast<long long>(t0 + t) * a_stride + r0 + r) : 0.f;
+    }
+    __syncthreads();
+#pragma unroll 8
+    for (int r = 0; r < rn; ++r) {
+      const float4 wv = *reinterpret_cast<const float4*>(&w[r][cq]), av = *reinterpret_cast<const float4*>(&as[r][tq]);
+      const float at[4] = {av.x, av.y, av.z, av.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        acc[i][0] = fmaf(wv.x, at[i], acc[i][0]);
+        acc[i][1] = fmaf(wv.y, at[i], acc[i][1]);
+        acc[i][2] = fmaf(wv.z, at[i], acc[i][2]);
+        acc[i][3] = fmaf(wv.w, at[i], acc[i][3]);
+      }
+    }
+    __syncthreads();
   }
-  for (int e = threadIdx.x; e < nt * rank; e += 256) {
-    const int i = e / rank, r = e - i * rank;
-    as[e] = ldf(a + static_cast<long long>(t0 + i) * a_stride + r);
-  }
-  __syncthreads();
-  if (c >= n_channels) return;
-  const float bias = a2_b ? a2_b[c] : 0.f;
-  for (int i = 0; i < nt; ++i) {
-    float z = 0.f;
-    for (int r = 0; r < rank; ++r) z = fmaf(w[r * 256 + threadIdx.x], as[i * rank + r], z);
-    ld[static_cast<long long>(t0 + i) * n_channels + c] = form(z + bias, c);
+  float bias[4];
+#pragma unroll
+  for (int j = 0; j < 4; ++j) bias[j] = (a2_b && c0 + cq + j < n_channels) ? a2_b[c0 + cq + j] : 0.f;
+  const bool vec = (n_channels & 3) == 0 && (reinterpret_cast<uintptr_t>(ld) & 15) == 0;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    if (t0 + tq + i >= n_tokens) break;
+    float* o = ld + static_cast<long long>(t0 + tq + i) * n_channels + c0 + cq;
+    if (vec && c0 + cq < n_channels) {
+      *reinterpret_cast<float4*>(o) = make_float4(form(acc[i][0] + bias[0], c0 + cq), form(acc[i][1] + bias[1], c0 + cq + 1), form(acc[i][2] + bias[2], c0 + cq + 2),
+                                                  form(acc[i][3] + bias[3], c0 + cq + 3));
+    } else {
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (c0 + cq + j < n_channels) o[j] = form(acc[i][j] + bias[j], c0 + cq + j);
+    }
   }
 }
 
@@ -521,11 +548,10 @@ PCS_API int pcs_gla_decay(const void* a, int64_t a_stride, const void* a2, const
   PCS_REQUIRE(a && a2 && ld && n_channels > 0 && rank > 0 && rank <= 8192 && (rate ? rate_dim > 0 : tau > 0.f), "pcs_gla_decay: bad arguments");
   const pcs::DecayForm form{rate ? 0.f : 1.f / tau, rate, rate_dim, expo};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const size_t tile_smem = static_cast<size_t>(rank) * (256 + pcs::kDecayTokens) * sizeof(float);
-  if (n_tokens >= 2 * pcs::kDecayTokens && tile_smem <= 48 * 1024) {
-    dim3 grid((n_channels + 255) / 256, (n_tokens + pcs::kDecayTokens - 1) / pcs::kDecayTokens);
-    PCS_DISPATCH(dtype, pcs::gla_decay_tile_kernel<T><<<grid, 256, tile_smem, st>>>(static_cast<const T*>(a), a_stride, static_cast<const T*>(a2), a2_b, ld,
-                                                                                   n_tokens, n_channels, rank, form));
+  if (n_tokens >= 2 * pcs::kDecayTokens) {
+    dim3 grid((n_channels + pcs::kDecayChannels - 1) / pcs::kDecayChannels, (n_tokens + pcs::kDecayTokens - 1) / pcs::kDecayTokens);
+    PCS_DISPATCH(dtype, pcs::gla_decay_tile_kernel<T><<<grid, 256, 0, st>>>(static_cast<const T*>(a), a_stride, static_cast<const T*>(a2), a2_b, ld, n_tokens, n_channels,
+                                                                           rank, form));
   } else
   PCS_DISPATCH(dtype, pcs::gla_decay_kernel<T><<<dim3(n_tokens, (n_channels + 255) / 256 > 64 ? 64 : (n_channels + 255) / 256), 256, rank * sizeof(float), st>>>(static_cast<const T*>(a), a_stride, static_cast<const T*>(a2),
                                                                                            a2_b, ld, n_channels, rank, form));

@@ -98,216 +98,234 @@ __global__ void __launch_bounds__(256) gnconv_kernel(const pcs_gnconv_params p) 
   for (int i = tid; i < W; i += 256) stf(h + i, s0[i] * inv[i / S] * ldf(nw + i));
 }
 
-// 16-byte pieces (the width, a group's width, strides and pointers are multiples of a piece; at most 256 * PPT pieces per row, at
-// most MR + 1 taps).  `ssq` holds a piece's sum of squares per row; a warp adds the pieces of one (row, group).
-template <typename T, int PPT, int TB, int MR>
-__global__ void __launch_bounds__(256) gnconv_vec_kernel(const pcs_gnconv_params p) {
-  constexpr int N = Vec<T>::n, RN = TB + MR;   // rows a block may form: MR predecessors, then its TB tokens
-  extern __shared__ float sm[];
-  const int W = p.width, G = p.groups, NP = W / N, PG = NP / G, R = p.conv_w ? p.taps - 1 : 0;
-  const int t0 = blockIdx.x * TB, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  float* ssq = sm;            // [RN][NP]
-  float* inv = sm + RN * NP;  // [RN][G]
-  const T* w = static_cast<const T*>(p.w);
-  const T* cw = static_cast<const T*>(p.conv_w);
-  // row k of the block is step row t0 - MR + k; it is formed when one of the block's tokens is it or has it as a predecessor in
-  // the same entry and step
-  bool need[RN];
-  long long rowi[RN];
-  TailView tv[TB];
+// Sums over the runs of PG neighbouring pieces that form a norm group, for K rows at once: v[k] is this thread's piece of row k.  With
+// one piece per thread and PG a power of two up to 32 the runs lie inside a warp and no shared memory is touched.
+template <int K, int PPT>
+__device__ __forceinline__ void group_sums(float (&v)[K][PPT], int NP, int PG, int G, float* ssq, float* tot) {
+  const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31;
+  if (PPT == 1 && PG <= 32 && (PG & (PG - 1)) == 0) {
 #pragma unroll
-  for (int k = 0; k < RN; ++k) need[k] = false;
+    for (int o = 1; o < 32; o <<= 1)
+      if (o < PG) {
 #pragma unroll
-  for (int i = 0; i < TB; ++i) {
-    tv[i] = TailView{0, 0, 1, nullptr, nullptr};
-    if (t0 + i < p.n_rows) {
-      need[MR + i] = true;
-      if (cw) {
-        tv[i] = tail_view(p, t0 + i, R);
-#pragma unroll
-        for (int j = 1; j <= MR; ++j)
-          if (j <= R && tv[i].pos - j >= tv[i].pos0) need[MR + i - j] = true;
+        for (int k = 0; k < K; ++k) v[k][0] += __shfl_xor_sync(0xffffffffu, v[k][0], o);
       }
-    }
-  }
-#pragma unroll
-  for (int k = 0; k < RN; ++k) {
-    rowi[k] = t0 - MR + k;
-    if (p.rows && k >= MR && need[k]) rowi[k] = p.rows[t0 + k - MR];
-  }
-  float s[RN][PPT][N];
-  uint4 yv[RN][PPT];
-#pragma unroll
-  for (int k = 0; k < RN; ++k)
-#pragma unroll
-    for (int u = 0; u < PPT; ++u) {
-      const int pc = tid + u * 256;
-      if (need[k] && pc < NP) {
-        ldx(p.x + rowi[k] * W + pc * N, s[k][u]);
-        if (p.y) yv[k][u] = *reinterpret_cast<const uint4*>(static_cast<const T*>(p.y) + rowi[k] * p.y_stride + pc * N);
-      }
-    }
-  auto unpack = [](const uint4& q, float (&o)[N]) { ld16(reinterpret_cast<const T*>(&q), o); };
-  if (p.y) {
-#pragma unroll
-    for (int k = 0; k < RN; ++k)
-#pragma unroll
-      for (int u = 0; u < PPT; ++u) {
-        const int pc = tid + u * 256;
-        if (need[k] && pc < NP) {
-          float v[N], a = 0.f;
-          unpack(yv[k][u], v);
-#pragma unroll
-          for (int e = 0; e < N; ++e) a = fmaf(v[e], v[e], a);
-          ssq[k * NP + pc] = a;
-        }
-      }
-    __syncthreads();
-    for (int e = warp; e < RN * G; e += 8) {
-      const int k = e / G, g = e - k * G;
-      float a = 0.f;
-      for (int i = lane; i < PG; i += 32) a += ssq[k * NP + g * PG + i];   // (rows that are not needed give numbers nobody reads)
-      a = warp_sum(a);
-      if (lane == 0) inv[e] = 1.f / sqrtf(a / static_cast<float>(PG * N) + p.eps);
-    }
-    __syncthreads();
-#pragma unroll
-    for (int u = 0; u < PPT; ++u) {
-      const int pc = tid + u * 256;
-      if (pc < NP) {
-        float wv[N];
-        ld16(w + pc * N, wv);
-        const int g = pc / PG;
-#pragma unroll
-        for (int k = 0; k < RN; ++k)
-          if (need[k]) {
-            float v[N];
-            unpack(yv[k][u], v);
-            const float f = inv[k * G + g];
-#pragma unroll
-            for (int e = 0; e < N; ++e) s[k][u][e] = fmaf(v[e] * f, wv[e], s[k][u][e]);
-          }
-      }
-    }
-  }
-#pragma unroll
-  for (int u = 0; u < PPT; ++u) {
-    const int pc = tid + u * 256;
-    if (pc < NP) {
-      if (p.x_out) {
-#pragma unroll
-        for (int i = 0; i < TB; ++i)
-          if (need[MR + i]) stx(p.x_out + rowi[MR + i] * W + pc * N, s[MR + i][u]);
-      }
-      if (cw) {
-        float o[TB][N], wv[N];
-        ld16(cw + static_cast<long long>(R) * W + pc * N, wv);
-#pragma unroll
-        for (int i = 0; i < TB; ++i)
-#pragma unroll
-          for (int e = 0; e < N; ++e) o[i][e] = fmaf(s[MR + i][u][e], wv[e], s[MR + i][u][e]);
-#pragma unroll
-        for (int j = 1; j <= MR; ++j)
-          if (j <= R) {
-            ld16(cw + static_cast<long long>(R - j) * W + pc * N, wv);
-#pragma unroll
-            for (int i = 0; i < TB; ++i)
-              if (need[MR + i] && tv[i].pos - j >= 0) {
-                if (tv[i].pos - j >= tv[i].pos0) {
-#pragma unroll
-                  for (int e = 0; e < N; ++e) o[i][e] = fmaf(wv[e], s[MR + i - j][u][e], o[i][e]);
-                } else {
-                  float q[N];
-                  ldx(tv[i].rd + static_cast<long long>(R - (tv[i].pos0 - (tv[i].pos - j))) * W + pc * N, q);
-#pragma unroll
-                  for (int e = 0; e < N; ++e) o[i][e] = fmaf(wv[e], q[e], o[i][e]);
-                }
-              }
-          }
-#pragma unroll
-        for (int i = 0; i < TB; ++i)
-          if (need[MR + i]) {
-            st16(static_cast<T*>(p.h_out) + static_cast<long long>(t0 + i) * W + pc * N, o[i]);
-            const int last_row = tv[i].pos - (tv[i].pos0 + tv[i].len - R);
-            if (R > 0 && last_row >= 0) stx(tv[i].wr + static_cast<long long>(last_row) * W + pc * N, s[MR + i][u]);
-          }
-      }
-    }
-  }
-  if (cw) {
-#pragma unroll
-    for (int i = 0; i < TB; ++i)
-      if (R > 0 && need[MR + i] && tv[i].pos == tv[i].pos0 + tv[i].len - 1 && tv[i].len < R)
-        for (int q = 0; q < R - tv[i].len; ++q)
-          for (int c = tid; c < W; c += 256) tv[i].wr[static_cast<long long>(q) * W + c] = tv[i].rd[static_cast<long long>(q + tv[i].len) * W + c];
     return;
   }
-  if (p.next_w == nullptr) return;
-  // the grouped norm of the new stream
+  __syncthreads();   // `ssq` may still be read from an earlier call
+#pragma unroll
+  for (int k = 0; k < K; ++k)
+#pragma unroll
+    for (int u = 0; u < PPT; ++u)
+      if (tid + u * nthr < NP) ssq[k * NP + tid + u * nthr] = v[k][u];
   __syncthreads();
-#pragma unroll
-  for (int i = 0; i < TB; ++i)
-#pragma unroll
-    for (int u = 0; u < PPT; ++u) {
-      const int pc = tid + u * 256;
-      if (need[MR + i] && pc < NP) {
-        float a = 0.f;
-#pragma unroll
-        for (int e = 0; e < N; ++e) a = fmaf(s[MR + i][u][e], s[MR + i][u][e], a);
-        ssq[i * NP + pc] = a;
-      }
-    }
-  __syncthreads();
-  for (int e = warp; e < TB * G; e += 8) {
+  for (int e = warp; e < K * G; e += nthr >> 5) {
     const int k = e / G, g = e - k * G;
     float a = 0.f;
     for (int i = lane; i < PG; i += 32) a += ssq[k * NP + g * PG + i];
     a = warp_sum(a);
-    if (lane == 0) inv[e] = 1.f / sqrtf(a / static_cast<float>(PG * N) + p.eps);
+    if (lane == 0) tot[e] = a;
   }
   __syncthreads();
 #pragma unroll
   for (int u = 0; u < PPT; ++u) {
-    const int pc = tid + u * 256;
+    const int pc = tid + u * nthr;
+    if (pc < NP) {
+#pragma unroll
+      for (int k = 0; k < K; ++k) v[k][u] = tot[k * G + pc / PG];
+    }
+  }
+}
+
+// 16-byte pieces (the width, a group's width, strides and pointers are multiples of a piece; at most blockDim.x * PPT pieces per row).
+// The block's rows are requested before it knows which of them its tokens need.
+template <typename T, int PPT, int TB, int R>
+__global__ void __launch_bounds__(256, (PPT == 1 ? 2 : 1)) gnconv_vec_kernel(const pcs_gnconv_params p) {
+  constexpr int N = Vec<T>::n, RN = TB + R;   // rows a block may form: R predecessors, then its TB tokens
+  extern __shared__ float sm[];
+  const int W = p.width, G = p.groups, NP = W / N, PG = NP / G;
+  const int t0 = blockIdx.x * TB, tid = threadIdx.x, nthr = blockDim.x;
+  float* ssq = sm;            // [RN][NP]
+  float* tot = sm + RN * NP;  // [RN][G]
+  const T* cw = static_cast<const T*>(p.conv_w);
+  // row k of the block is step row t0 - R + k (with `rows`: the listed row)
+  float s[RN][PPT][N];
+  uint4 yv[RN][PPT];
+#pragma unroll
+  for (int k = 0; k < RN; ++k) {
+    const int r = t0 - R + k;
+    const bool in = r >= 0 && r < p.n_rows;
+    const long long row = in ? (p.rows ? p.rows[r] : r) : 0;
+#pragma unroll
+    for (int u = 0; u < PPT; ++u) {
+      const int pc = tid + u * nthr;
+      if (in && pc < NP) {
+        ldx(p.x + row * W + pc * N, s[k][u]);
+        if (p.y) yv[k][u] = *reinterpret_cast<const uint4*>(static_cast<const T*>(p.y) + row * p.y_stride + pc * N);
+      } else {
+#pragma unroll
+        for (int e = 0; e < N; ++e) s[k][u][e] = 0.f;
+        yv[k][u] = make_uint4(0u, 0u, 0u, 0u);
+      }
+    }
+  }
+  // the tokens' places in their entries: how many of the R predecessors are rows of this step, and the tails
+  int here[TB], before[TB], last_row[TB], shift[TB];   // predecessors in this step; predecessors at all; tail row to write; rows that stay move by this
+  long long tail0[TB];                                 // element offset of the slot's copy that is read
+  int par[TB];
+  const T* w = static_cast<const T*>(p.w);
+#pragma unroll
+  for (int i = 0; i < TB; ++i) {
+    here[i] = before[i] = 0;
+    last_row[i] = -1;
+    shift[i] = 0;
+    tail0[i] = 0;
+    par[i] = 0;
+    if (R > 0 && cw && t0 + i < p.n_rows) {
+      const int b = p.tok_seq[t0 + i], pos = p.tok_pos[t0 + i], pos0 = p.seq_pos0[b], len = p.seq_len[b];
+      here[i] = min(R, pos - pos0);
+      before[i] = min(R, pos);
+      last_row[i] = pos - (pos0 + len - R);
+      if (pos == pos0 + len - 1 && len < R) shift[i] = len;
+      par[i] = p.seq_par[b] & 1;
+      tail0[i] = (static_cast<long long>(p.seq_slot[b]) * 2 + par[i]) * R * W;
+    }
+  }
+  auto unpack = [](const uint4& q, float (&o)[N]) { ld16(reinterpret_cast<const T*>(&q), o); };
+  const float inv_n = 1.f / static_cast<float>(PG * N);
+  if (p.y) {
+    float ss[RN][PPT];
+#pragma unroll
+    for (int k = 0; k < RN; ++k)
+#pragma unroll
+      for (int u = 0; u < PPT; ++u) {
+        float v[N], a = 0.f;
+        unpack(yv[k][u], v);
+#pragma unroll
+        for (int e = 0; e < N; ++e) a = fmaf(v[e], v[e], a);
+        ss[k][u] = a;
+      }
+    group_sums<RN, PPT>(ss, NP, PG, G, ssq, tot);
+#pragma unroll
+    for (int u = 0; u < PPT; ++u) {
+      const int pc = tid + u * nthr;
+      if (pc < NP) {
+        float wv[N];
+        ld16(w + pc * N, wv);
+#pragma unroll
+        for (int k = 0; k < RN; ++k) {
+          float v[N];
+          unpack(yv[k][u], v);
+          const float f = 1.f / sqrtf(fmaf(ss[k][u], inv_n, p.eps));
+#pragma unroll
+          for (int e = 0; e < N; ++e) s[k][u][e] = fmaf(v[e] * f, wv[e], s[k][u][e]);
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int u = 0; u < PPT; ++u) {
+    const int pc = tid + u * nthr;
+    if (pc < NP) {
+#pragma unroll
+      for (int i = 0; i < TB; ++i)
+        if (t0 + i < p.n_rows) {
+          if (p.x_out) stx(p.x_out + static_cast<long long>(p.rows ? p.rows[t0 + i] : t0 + i) * W + pc * N, s[R + i][u]);
+          if (cw) {
+            float o[N], wv[N];
+            ld16(cw + static_cast<long long>(R) * W + pc * N, wv);
+#pragma unroll
+            for (int e = 0; e < N; ++e) o[e] = fmaf(s[R + i][u][e], wv[e], s[R + i][u][e]);
+#pragma unroll
+            for (int j = 1; j <= R; ++j)
+              if (j <= before[i]) {
+                ld16(cw + static_cast<long long>(R - j) * W + pc * N, wv);
+                if (j <= here[i]) {
+#pragma unroll
+                  for (int e = 0; e < N; ++e) o[e] = fmaf(wv[e], s[R + i - j][u][e], o[e]);
+                } else {   // position pos - j sits in tail row R - (pos0 - (pos - j)); pos - pos0 is `here` whenever it is below R
+                  float q[N];
+                  ldx(p.tail + tail0[i] + static_cast<long long>(R - (j - here[i])) * W + pc * N, q);
+#pragma unroll
+                  for (int e = 0; e < N; ++e) o[e] = fmaf(wv[e], q[e], o[e]);
+                }
+              }
+            st16(static_cast<T*>(p.h_out) + static_cast<long long>(t0 + i) * W + pc * N, o);
+            if (R > 0) {
+              float* wr = p.tail + tail0[i] + (par[i] ? -1LL : 1LL) * R * W + pc * N;
+              if (last_row[i] >= 0) stx(wr + static_cast<long long>(last_row[i]) * W, s[R + i][u]);
+              if (shift[i] > 0)
+                for (int q = 0; q < R - shift[i]; ++q) {
+                  float v[N];
+                  ldx(p.tail + tail0[i] + static_cast<long long>(q + shift[i]) * W + pc * N, v);
+                  stx(wr + static_cast<long long>(q) * W, v);
+                }
+            }
+          }
+        }
+    }
+  }
+  if (cw || p.next_w == nullptr) return;
+  // the grouped norm of the new stream
+  float ss[TB][PPT];
+#pragma unroll
+  for (int i = 0; i < TB; ++i)
+#pragma unroll
+    for (int u = 0; u < PPT; ++u) {
+      float a = 0.f;
+#pragma unroll
+      for (int e = 0; e < N; ++e) a = fmaf(s[R + i][u][e], s[R + i][u][e], a);
+      ss[i][u] = a;
+    }
+  group_sums<TB, PPT>(ss, NP, PG, G, ssq, tot);
+#pragma unroll
+  for (int u = 0; u < PPT; ++u) {
+    const int pc = tid + u * nthr;
     if (pc < NP) {
       float nv[N];
       ld16(static_cast<const T*>(p.next_w) + pc * N, nv);
 #pragma unroll
       for (int i = 0; i < TB; ++i)
-        if (need[MR + i]) {
+        if (t0 + i < p.n_rows) {
           float o[N];
-          const float f = inv[i * G + pc / PG];
+          const float f = 1.f / sqrtf(fmaf(ss[i][u], inv_n, p.eps));
 #pragma unroll
-          for (int e = 0; e < N; ++e) o[e] = s[MR + i][u][e] * f * nv[e];
+          for (int e = 0; e < N; ++e) o[e] = s[R + i][u][e] * f * nv[e];
           st16(static_cast<T*>(p.h_out) + static_cast<long long>(t0 + i) * W + pc * N, o);
         }
     }
   }
 }
 
-template <typename T, int PPT, int TB, int MR>
+template <typename T, int PPT, int TB, int R>
 static int launch_gnconv_vec(const pcs_gnconv_params& p, cudaStream_t st) {
-  const size_t smem = static_cast<size_t>(TB + MR) * (p.width / Vec<T>::n + p.groups) * sizeof(float);
-  gnconv_vec_kernel<T, PPT, TB, MR><<<(p.n_rows + TB - 1) / TB, 256, smem, st>>>(p);
+  const int np = p.width / Vec<T>::n, thr = PPT == 1 ? (np + 31) / 32 * 32 : 256;
+  const size_t smem = static_cast<size_t>(TB + R) * (np + p.groups) * sizeof(float);
+  gnconv_vec_kernel<T, PPT, TB, R><<<(p.n_rows + TB - 1) / TB, thr, smem, st>>>(p);
   PCS_CHECK_CUDA(cudaGetLastError());
   count_launch();
   return PCS_OK;
 }
 
+template <typename T, int R>
+static int launch_gnconv_taps(const pcs_gnconv_params& p, cudaStream_t st) {
+  const int np = p.width / Vec<T>::n;
+  if (np > 256) return launch_gnconv_vec<T, 2, 1, R>(p, st);
+  // four tokens per block where that leaves two blocks per SM
+  if (R > 0 && p.n_rows >= 4 * 2 * 148) return launch_gnconv_vec<T, 1, (R > 0 ? 4 : 1), R>(p, st);
+  return launch_gnconv_vec<T, 1, 1, R>(p, st);
+}
+
 template <typename T>
 static int launch_gnconv(const pcs_gnconv_params& p, cudaStream_t st, bool vec) {
-  constexpr int N = Vec<T>::n;
+  const int R = p.conv_w ? p.taps - 1 : 0;
   if (vec) {
-    const int np = p.width / N, R = p.conv_w ? p.taps - 1 : 0;
-    // tokens per block: as many as keep two blocks per SM busy
-    const bool tile = p.conv_w && R > 0 && p.n_rows >= 4 * 2 * 148 && np <= 256;
-    if (R == 0) return np <= 256 ? launch_gnconv_vec<T, 1, 1, 0>(p, st) : launch_gnconv_vec<T, 2, 1, 0>(p, st);
-    if (R <= 3) {
-      if (tile) return launch_gnconv_vec<T, 1, 4, 3>(p, st);
-      return np <= 256 ? launch_gnconv_vec<T, 1, 1, 3>(p, st) : launch_gnconv_vec<T, 2, 1, 3>(p, st);
-    }
+    if (R == 0) return launch_gnconv_taps<T, 0>(p, st);
+    if (R == 1) return launch_gnconv_taps<T, 1>(p, st);
+    if (R == 2) return launch_gnconv_taps<T, 2>(p, st);
+    if (R == 3) return launch_gnconv_taps<T, 3>(p, st);
   }
-  const size_t smem = (static_cast<size_t>(p.conv_w ? p.taps : 1) * p.groups + p.width) * sizeof(float);
+  const size_t smem = (static_cast<size_t>(R + 1) * p.groups + p.width) * sizeof(float);
   PCS_REQUIRE(smem <= 200 * 1024, "pcs_group_norm_conv: width %d with %d groups exceeds shared memory", p.width, p.groups);
   if (smem > 48 * 1024) PCS_CHECK_CUDA(cudaFuncSetAttribute(gnconv_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
   gnconv_kernel<T><<<p.n_rows, 256, smem, st>>>(p);
