@@ -41,6 +41,7 @@
  *   pcs_group_norm_conv  residual sum of a sublayer result normed in groups of channels, then a short causal convolution over time
  *                        of the NEW stream (its last inputs are carried in the slot pool) or a grouped norm of it
  *   pcs_short_conv       per-channel causal convolution over time + silu of projections, query / key heads made unit vectors
+ *   pcs_delta_inputs     the same for few tokens with the delta rule's two low-rank products (decays, output gate) in one launch
  *   pcs_delta_scan       gated delta rule with a decay per key channel, token by token;  pcs_delta_chunk_*: in chunks (prompts)
  *   pcs_head_norm_gate   per-head RMS norm of a recurrence's result times an element-wise sigmoid gate
  *   pcs_soft_cap         cap * tanh(z / cap)
@@ -593,6 +594,21 @@ typedef struct pcs_shortconv_params {
   int32_t reserved;
 } pcs_shortconv_params;
 int pcs_short_conv(const pcs_shortconv_params* p, void* stream);
+
+/* For few tokens: pcs_short_conv and, in the same launch, two low-rank products of the same projection rows:
+ *   decay_out[t, c] = exp(-rate[c / dim] * softplus(sum_r a2[c, r] * proj[t, a_off + r] + dt_bias[c]))     (c < heads * dim)
+ *   gate_out[t, c]  = sum_r g2[c, r] * proj[t, g_off + r]                                                     (c < gate_width, `dtype`)
+ * Sizes off the 16-byte pieces, or more than four taps, give PCS_ERR_UNSUPPORTED. */
+typedef struct pcs_lowrank_params {
+  const void* a2;           /* [heads * dim, decay_rank] `dtype` */
+  const float* dt_bias;     /* [heads * dim] */
+  const float* rate;        /* [heads] */
+  float* decay_out;         /* [n_tokens, heads * dim] */
+  const void* g2;           /* [gate_width, gate_rank] `dtype` */
+  void* gate_out;           /* [n_tokens, gate_width] `dtype` */
+  int32_t a_off, g_off, decay_rank, gate_rank, heads, dim, gate_width, reserved;
+} pcs_lowrank_params;
+int pcs_delta_inputs(const pcs_shortconv_params* p, const pcs_lowrank_params* q, void* stream);
 
 /* Gated delta rule, token by token.  Per entry and head h (query / key head h / (heads / kv_heads)):
  *   S <- diag(decay_t) S;  u = sigmoid(b[t, h]) * (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t

@@ -20,7 +20,7 @@ EXPORTS = ("pcs_version", "pcs_last_error", "pcs_launch_count", "pcs_attn_worksp
            "pcs_qk_prep", "pcs_attn", "pcs_mlstm_gates", "pcs_mlstm_scan", "pcs_embed_bigram", "pcs_norm_conv", "pcs_rope_kv_prep", "pcs_moe_route",
            "pcs_moe_rows_up", "pcs_moe_rows_down", "pcs_moe_plan", "pcs_moe_gather", "pcs_moe_gemm", "pcs_moe_combine", "pcs_silu_mul", "pcs_glu_mul",
            "pcs_depth_mix", "pcs_latent_prep", "pcs_latent_q", "pcs_latent_gather", "pcs_latent_expand", "pcs_head_gate", "pcs_gla_decay", "pcs_gla_scan", "pcs_gla_chunk_prep", "pcs_gla_chunk_scan", "pcs_gla_chunk_out",
-           "pcs_add_layer_norm", "pcs_gru_scan", "pcs_group_norm_conv", "pcs_soft_cap", "pcs_short_conv", "pcs_delta_scan", "pcs_delta_chunk_prep", "pcs_delta_chunk_scan",
+           "pcs_add_layer_norm", "pcs_gru_scan", "pcs_group_norm_conv", "pcs_soft_cap", "pcs_short_conv", "pcs_delta_inputs", "pcs_delta_scan", "pcs_delta_chunk_prep", "pcs_delta_chunk_scan",
            "pcs_head_norm_gate")
 GLU_SILU, GLU_CLAMPED_SWISH, GLU_GELU_TANH = 0, 1, 4
 ACT_RELU2, ACT_GELU_ERF = 2, 3          # activations of a feed-forward without a gate branch
@@ -165,6 +165,12 @@ class pcs_shortconv_params(C.Structure):
                 ("seq_par", C.c_void_p), ("n_tokens", C.c_int32), ("dtype", C.c_int32), ("impl", C.c_int32), ("reserved", C.c_int32)]
 
 
+class pcs_lowrank_params(C.Structure):
+    _fields_ = [("a2", C.c_void_p), ("dt_bias", C.c_void_p), ("rate", C.c_void_p), ("decay_out", C.c_void_p), ("g2", C.c_void_p), ("gate_out", C.c_void_p),
+                ("a_off", C.c_int32), ("g_off", C.c_int32), ("decay_rank", C.c_int32), ("gate_rank", C.c_int32), ("heads", C.c_int32), ("dim", C.c_int32),
+                ("gate_width", C.c_int32), ("reserved", C.c_int32)]
+
+
 class pcs_delta_params(C.Structure):
     _fields_ = [("qk", C.c_void_p), ("v", C.c_void_p), ("decay", C.c_void_p), ("b", C.c_void_p), ("b_stride", C.c_int64), ("o", C.c_void_p), ("s_pool", C.c_void_p),
                 ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("seq_slot", C.c_void_p), ("seq_pos0", C.c_void_p),
@@ -263,6 +269,7 @@ def load() -> C.CDLL:
     lib.pcs_group_norm_conv.argtypes = [C.POINTER(pcs_gnconv_params), C.c_void_p]
     lib.pcs_soft_cap.argtypes = [C.c_void_p, C.c_int64, C.c_void_p, C.c_int, C.c_int, C.c_float, C.c_int, C.c_void_p]
     lib.pcs_short_conv.argtypes = [C.POINTER(pcs_shortconv_params), C.c_void_p]
+    lib.pcs_delta_inputs.argtypes = [C.POINTER(pcs_shortconv_params), C.POINTER(pcs_lowrank_params), C.c_void_p]
     lib.pcs_delta_scan.argtypes = [C.POINTER(pcs_delta_params), C.c_void_p]
     for name in ("pcs_delta_chunk_prep", "pcs_delta_chunk_scan"):
         getattr(lib, name).argtypes = [C.POINTER(pcs_delta_chunk_params), C.c_void_p]
@@ -1084,11 +1091,7 @@ def soft_cap(z: torch.Tensor, cap: float) -> torch.Tensor:
     return out
 
 
-def short_conv(proj: torch.Tensor, c_off: int, kv_heads: int, dim: int, v_width: int, conv_w: torch.Tensor, tail: Optional[torch.Tensor], q_scale: float, unit_eps: float,
-               batch: Batch, impl: int = 0):
-    """(qk float32 [T, 2 * kv_heads * dim], v [T, v_width]): silu of a causal convolution over time of the projection columns from c_off on
-    (queries | keys | values), query and key heads as unit vectors, queries times q_scale.  conv_w [taps, channels]; `tail`
-    [slots, 2, taps - 1, channels] float32 carries the last inputs from step to step.  impl 1: the element-wise kernel."""
+def _short_conv_params(proj, c_off, kv_heads, dim, v_width, conv_w, tail, q_scale, unit_eps, batch, impl):
     _cuda(proj, conv_w, tail)
     dt = proj.dtype
     _rows2d(proj, dt, "short_conv: proj")
@@ -1105,8 +1108,50 @@ def short_conv(proj: torch.Tensor, c_off: int, kv_heads: int, dim: int, v_width:
     p.tok_seq, p.tok_pos, p.seq_slot = batch.tok_seq.data_ptr(), batch.tok_pos.data_ptr(), batch.seq_slot.data_ptr()
     p.seq_pos0, p.seq_len, p.seq_par = batch.seq_pos0.data_ptr(), batch.seq_len.data_ptr(), batch.seq_par.data_ptr()
     p.n_tokens, p.dtype, p.impl = T, dtype_code(dt), int(impl)
+    return p, qk, v
+
+
+def short_conv(proj: torch.Tensor, c_off: int, kv_heads: int, dim: int, v_width: int, conv_w: torch.Tensor, tail: Optional[torch.Tensor], q_scale: float, unit_eps: float,
+               batch: Batch, impl: int = 0):
+    """(qk float32 [T, 2 * kv_heads * dim], v [T, v_width]): silu of a causal convolution over time of the projection columns from c_off on
+    (queries | keys | values), query and key heads as unit vectors, queries times q_scale.  conv_w [taps, channels]; `tail`
+    [slots, 2, taps - 1, channels] float32 carries the last inputs from step to step.  impl 1: the element-wise kernel."""
+    p, qk, v = _short_conv_params(proj, c_off, kv_heads, dim, v_width, conv_w, tail, q_scale, unit_eps, batch, impl)
     _check(load().pcs_short_conv(C.byref(p), _stream()), "pcs_short_conv")
     return qk, v
+
+
+DELTA_INPUTS_MAX_TOKENS = 32
+
+
+def delta_inputs(proj: torch.Tensor, c_off: int, kv_heads: int, heads: int, dim: int, vdim: int, conv_w: torch.Tensor, tail: Optional[torch.Tensor], q_scale: float,
+                 unit_eps: float, a1, a2: torch.Tensor, dt_bias: torch.Tensor, rate: torch.Tensor, g1, g2: torch.Tensor, batch: Batch, expo: bool, fused: Optional[bool] = None):
+    """(qk, v, decay float32 [T, heads * dim], gate [T, heads * vdim]): `short_conv`, `gla_decay` with rates (`expo`: the decays, else their logarithms)
+    of the columns `a1` = (first, last + 1) of proj, and the product of the columns `g1` with g2.  A few tokens whose sizes are multiples
+    of 16-byte pieces take one launch (`pcs_delta_inputs`); `fused` True / False forces the choice."""
+    piece = 16 // proj.element_size()
+    fits = expo and conv_w.shape[0] <= 4 and dim % piece == 0 and (heads * vdim) % piece == 0 and c_off % piece == 0 and proj.stride(0) % piece == 0 \
+        and proj.data_ptr() % 16 == 0 and conv_w.data_ptr() % 16 == 0 and dim <= 256 * piece
+    if fused is None:
+        fused = fits and proj.shape[0] <= DELTA_INPUTS_MAX_TOKENS
+    if not fused:
+        qk, v = short_conv(proj, c_off, kv_heads, dim, heads * vdim, conv_w, tail, q_scale, unit_eps, batch)
+        return qk, v, gla_decay(proj[:, a1[0]:a1[1]], a2, dt_bias, 1.0, rate=rate, expo=expo), linear(proj[:, g1[0]:g1[1]], g2)
+    if not fits:
+        raise NativeError("delta_inputs: one launch serves decays (not logarithms) at sizes that are multiples of 16-byte pieces and up to four taps")
+    _cuda(a2, dt_bias, rate, g2)
+    dt, T = proj.dtype, proj.shape[0]
+    if a2.dtype != dt or g2.dtype != dt or not (a2.is_contiguous() and g2.is_contiguous()) or tuple(a2.shape) != (heads * dim, a1[1] - a1[0]) \
+            or tuple(g2.shape) != (heads * vdim, g1[1] - g1[0]) or dt_bias.dtype != torch.float32 or dt_bias.numel() != heads * dim or rate.dtype != torch.float32 \
+            or rate.numel() != heads or not (dt_bias.is_contiguous() and rate.is_contiguous()) or max(a1[1], g1[1]) > proj.shape[1]:
+        raise NativeError("delta_inputs: a2 [heads * dim, rank] and g2 [heads * vdim, rank] in the compute type, dt_bias and rate float32")
+    p, qk, v = _short_conv_params(proj, c_off, kv_heads, dim, heads * vdim, conv_w, tail, q_scale, unit_eps, batch, 0)
+    decay, gate = torch.empty(T, heads * dim, dtype=torch.float32, device=proj.device), torch.empty(T, heads * vdim, dtype=dt, device=proj.device)
+    q = pcs_lowrank_params()
+    q.a2, q.dt_bias, q.rate, q.decay_out, q.g2, q.gate_out = (t.data_ptr() for t in (a2, dt_bias, rate, decay, g2, gate))
+    q.a_off, q.g_off, q.decay_rank, q.gate_rank, q.heads, q.dim, q.gate_width = int(a1[0]), int(g1[0]), a2.shape[1], g2.shape[1], int(heads), int(dim), heads * vdim
+    _check(load().pcs_delta_inputs(C.byref(p), C.byref(q), _stream()), "pcs_delta_inputs")
+    return qk, v, decay, gate
 
 
 DELTA_CHUNK = 64          # PCS_DELTA_CHUNK

@@ -943,6 +943,14 @@ def zovolorn_kernels(s: dict, dev, timer: Timer, prompt: int, ctx: int, hbm_gbs:
     out["delta_decay"] = gb(prompt * mH * mD * 4.0, ms)
     ms = timer(lambda: nsq.gla_decay(pr[:, ch:ch + rk], a2, dtb, 16.0))
     out["like_gla_decay"] = gb(prompt * mH * mD * 4.0, ms)
+    # one decoded token's inputs in one launch: bytes = the two low-rank matrices
+    g2 = (torch.randn(mH * mV, rk, device=dev) * rk ** -0.5).to(bf)
+    ms = timer(lambda: nsq.delta_inputs(pr[:1], 0, mH, mH, mD, mV, cv, ctail, mD ** -0.5, 1e-6, (ch, ch + rk), a2, dtb, rate, (ch + rk, ch + 2 * rk), g2, b1, True), steps=15)
+    out["delta_inputs_decode"] = gb(2.0 * rk * mH * (mD + mV), ms)
+    wl = (torch.randn(mH * (mD + mV), rk, device=dev) * rk ** -0.5).to(bf)
+    xl = torch.randn(1, rk, device=dev).to(bf)
+    ms = timer(lambda: nsq.linear(xl, wl, kernel=True), steps=15)
+    out["like_linear_rows_same_bytes"] = gb(2.0 * rk * mH * (mD + mV), ms)
     # the recurrence over a prompt and of one decoded token (state read and written once)
     qk, v = nsq.short_conv(pr, 0, mH, mD, mH * mV, cv, ctail, mD ** -0.5, 1e-6, b)
     ld = nsq.gla_decay(pr[:, ch:ch + rk], a2, dtb, 1.0, rate=rate)

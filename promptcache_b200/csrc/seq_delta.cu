@@ -6,6 +6,7 @@
 //
 // pcs_short_conv        the convolution over time per channel, silu, unit vectors.  Inputs of earlier steps sit in the slot's tail,
 //                       kept twice so that the copy a step reads is never the one it writes.
+// pcs_delta_inputs      decoding: the convolution and the two low-rank products beside it (decays, output gate) in one launch.
 // pcs_delta_scan        token by token.  The columns of S evolve independently given k, q and the decays, so the grid covers
 //                       (sequence, head, slice of columns): state in registers (dim <= 256, aligned) or in shared memory.
 // pcs_delta_chunk_prep  prompts: everything about a chunk of 64 tokens that does not need the state it starts from.
@@ -79,7 +80,7 @@ __global__ void __launch_bounds__(256) short_conv_kernel(const pcs_shortconv_par
 // requested before the block knows which of them its tokens need.  CB is a multiple of dim, so a head's pieces meet in this block: by
 // shuffles where a head is a power of two up to 32 pieces, else through shared memory.
 template <typename T, int TB, int R>
-__global__ void __launch_bounds__(256, 2) short_conv_vec_kernel(const pcs_shortconv_params p, int CB) {
+__device__ __forceinline__ void short_conv_tile(const pcs_shortconv_params& p, int CB) {
   constexpr int N = Vec<T>::n, RN = TB + R;
   __shared__ float ssq[TB][256];
   const int t0 = blockIdx.x * TB, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;   // (warp, lane: shared-memory sums)
@@ -93,6 +94,11 @@ __global__ void __launch_bounds__(256, 2) short_conv_vec_kernel(const pcs_shortc
   for (int k = 0; k < RN; ++k) {
     const int r = t0 - R + k;
     xv[k] = active && r >= 0 && r < p.n_tokens ? *reinterpret_cast<const uint4*>(x + static_cast<long long>(r) * p.row_stride) : make_uint4(0u, 0u, 0u, 0u);
+  }
+  uint4 cq[R + 1];   // (many tokens: other blocks hide these loads)
+  if (TB == 1 && active) {
+#pragma unroll
+    for (int j = 0; j <= R; ++j) cq[j] = *reinterpret_cast<const uint4*>(cw + static_cast<long long>(R - j) * C + c);
   }
   // the tokens' places in their entries (see the boundary kernel): predecessors in this step and at all, tail row to write, rows that stay
   int here[TB], before[TB], last_row[TB], shift[TB], par[TB];
@@ -123,7 +129,8 @@ __global__ void __launch_bounds__(256, 2) short_conv_vec_kernel(const pcs_shortc
 #pragma unroll
     for (int j = 0; j <= R; ++j) {
       float wv[N];
-      ld16(cw + static_cast<long long>(R - j) * C + c, wv);
+      if (TB == 1) ld16(reinterpret_cast<const T*>(&cq[j]), wv);
+      else ld16(cw + static_cast<long long>(R - j) * C + c, wv);
 #pragma unroll
       for (int i = 0; i < TB; ++i)
         if (j <= before[i]) {
@@ -201,26 +208,76 @@ __global__ void __launch_bounds__(256, 2) short_conv_vec_kernel(const pcs_shortc
     }
 }
 
+template <typename T, int TB, int R>
+__global__ void __launch_bounds__(256, 2) short_conv_vec_kernel(const pcs_shortconv_params p, int CB) {
+  short_conv_tile<T, TB, R>(p, CB);
+}
+
+// Few tokens (decoding): the convolution, and behind its blocks in blockIdx.y the two low-rank products that read the same projection
+// row, the decays and the output gate's pre-activation: 8 lanes per output, 16-byte pieces of the matrix row where it is aligned.
 template <typename T, int R>
-static void launch_short_conv_taps(const pcs_shortconv_params& p, cudaStream_t st) {
+__global__ void __launch_bounds__(256) delta_inputs_kernel(const pcs_shortconv_params p, const pcs_lowrank_params q, int CB, int ny) {
+  if (static_cast<int>(blockIdx.y) < ny) {
+    short_conv_tile<T, 1, R>(p, CB);
+    return;
+  }
+  constexpr int N = Vec<T>::n;
+  const int t = blockIdx.x, lane8 = threadIdx.x & 7, HD = q.heads * q.dim, n_out = HD + q.gate_width;
+  const int o = (static_cast<int>(blockIdx.y) - ny) * (blockDim.x >> 3) + (threadIdx.x >> 3);
+  const bool ok = o < n_out, dec = o < HD;
+  const int rank = dec ? q.decay_rank : q.gate_rank, row = dec ? o : o - HD;
+  const T* w = static_cast<const T*>(dec ? q.a2 : q.g2) + static_cast<long long>(row) * rank;
+  const T* x = static_cast<const T*>(p.proj) + static_cast<long long>(t) * p.row_stride + (dec ? q.a_off : q.g_off);
+  float acc = 0.f;
+  if (ok) {
+    const bool vec = rank % N == 0 && ((reinterpret_cast<uintptr_t>(w) | reinterpret_cast<uintptr_t>(x)) & 15) == 0;
+    if (vec) {
+      for (int r = lane8 * N; r < rank; r += 8 * N) {
+        float a[N], b[N];
+        ld16(w + r, a);
+        ld16(x + r, b);
+#pragma unroll
+        for (int e = 0; e < N; ++e) acc = fmaf(a[e], b[e], acc);
+      }
+    } else {
+      for (int r = lane8; r < rank; r += 8) acc = fmaf(ldf(w + r), ldf(x + r), acc);
+    }
+  }
+#pragma unroll
+  for (int m = 1; m < 8; m <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, m);
+  if (!ok || lane8 != 0) return;
+  if (dec) q.decay_out[static_cast<long long>(t) * HD + o] = expf(-q.rate[o / q.dim] * softplusf_(acc + q.dt_bias[o]));
+  else stf(static_cast<T*>(q.gate_out) + static_cast<long long>(t) * q.gate_width + row, acc);
+}
+
+template <typename T, int R>
+static void launch_short_conv_taps(const pcs_shortconv_params& p, const pcs_lowrank_params* q, cudaStream_t st) {
   const int per = 256 * Vec<T>::n, C = 2 * p.kv_heads * p.dim + p.v_width;
   int CB = per / p.dim * p.dim;
-  if (p.n_tokens < 64) {   // few tokens: narrow channel blocks, so that the launch covers more SMs
+  if (p.n_tokens < 64 || q) {   // few tokens: narrow channel blocks, so that the launch covers more SMs
     const int small = (32 * Vec<T>::n + p.dim - 1) / p.dim * p.dim;
     if (small < CB) CB = small;
   }
-  const int ny = (C + CB - 1) / CB, thr = (CB / Vec<T>::n + 31) / 32 * 32;
-  if (R > 0 && p.n_tokens >= 4 * 148) short_conv_vec_kernel<T, (R > 0 ? 4 : 1), R><<<dim3((p.n_tokens + 3) / 4, ny), thr, 0, st>>>(p, CB);
-  else short_conv_vec_kernel<T, 1, R><<<dim3(p.n_tokens, ny), thr, 0, st>>>(p, CB);
+  const int ny = (C + CB - 1) / CB;
+  int thr = (CB / Vec<T>::n + 31) / 32 * 32;
+  if (q) {
+    if (thr < 128) thr = 128;
+    const int outs = q->heads * q->dim + q->gate_width, extra = (outs + thr / 8 - 1) / (thr / 8);
+    delta_inputs_kernel<T, R><<<dim3(p.n_tokens, ny + extra), thr, 0, st>>>(p, *q, CB, ny);
+  } else if (R > 0 && p.n_tokens >= 4 * 148) {
+    short_conv_vec_kernel<T, (R > 0 ? 4 : 1), R><<<dim3((p.n_tokens + 3) / 4, ny), thr, 0, st>>>(p, CB);
+  } else {
+    short_conv_vec_kernel<T, 1, R><<<dim3(p.n_tokens, ny), thr, 0, st>>>(p, CB);
+  }
 }
 
 template <typename T>
-static int launch_short_conv(const pcs_shortconv_params& p, cudaStream_t st, bool vec) {
+static int launch_short_conv(const pcs_shortconv_params& p, const pcs_lowrank_params* q, cudaStream_t st, bool vec) {
   if (!vec) short_conv_kernel<T><<<p.n_tokens, 256, 0, st>>>(p);
-  else if (p.taps == 1) launch_short_conv_taps<T, 0>(p, st);
-  else if (p.taps == 2) launch_short_conv_taps<T, 1>(p, st);
-  else if (p.taps == 3) launch_short_conv_taps<T, 2>(p, st);
-  else launch_short_conv_taps<T, 3>(p, st);
+  else if (p.taps == 1) launch_short_conv_taps<T, 0>(p, q, st);
+  else if (p.taps == 2) launch_short_conv_taps<T, 1>(p, q, st);
+  else if (p.taps == 3) launch_short_conv_taps<T, 2>(p, q, st);
+  else launch_short_conv_taps<T, 3>(p, q, st);
   PCS_CHECK_CUDA(cudaGetLastError());
   count_launch();
   return PCS_OK;
@@ -436,18 +493,44 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_
   const int cn = blockIdx.x, head = blockIdx.y, hk = head / (H / p.kv_heads), tid = threadIdx.x;
   const int first = p.chunk_first[cn], n = p.chunk_len[cn];
   const long long base = static_cast<long long>(cn) * H + head;
-  for (int e = tid; e < kC * D4; e += kDpThreads) {
-    const int i = e / D4, d = e - i * D4;
-    float q = 0.f, k = 0.f, l = 0.f;
-    if (i < n && d < D) {
-      const float* row = p.qk + static_cast<long long>(first + i) * U;
-      q = row[hk * D + d];
-      k = row[(p.kv_heads + hk) * D + d];
-      l = p.ld[static_cast<long long>(first + i) * (static_cast<long long>(H) * D) + head * D + d];
+  // bfloat16 runs work in the base-2 domain (exponential unit, relative error near 2^-22), float32 runs with the library exponential
+  constexpr bool kFast = sizeof(T) == 2;
+  constexpr float kLog = kFast ? 1.4426950408889634f : 1.f;
+  auto ex = [](float x) { return kFast ? ex2(x) : expf(x); };
+  const int warp = tid >> 5, lane = tid & 31;
+  constexpr int kWarps = kDpThreads / 32;
+  {
+    const float* qb = p.qk + hk * D;
+    const float* kb = p.qk + (p.kv_heads + hk) * D;
+    const float* lb = p.ld + head * D;
+    const bool vec = D == D4 && ((reinterpret_cast<uintptr_t>(p.qk) | reinterpret_cast<uintptr_t>(p.ld)) & 15) == 0;
+    if (vec) {   // a warp takes a row at a time, the rows' loads overlap
+      for (int d = lane * 4; d < D; d += 128) {
+#pragma unroll
+        for (int it = 0; it < kC / kWarps; ++it) {
+          const int i = warp + it * kWarps;
+          float4 q = make_float4(0.f, 0.f, 0.f, 0.f), k = q, l = q;
+          if (i < n) {
+            const long long t = first + i;
+            q = *reinterpret_cast<const float4*>(qb + t * U + d);
+            k = *reinterpret_cast<const float4*>(kb + t * U + d);
+            l = *reinterpret_cast<const float4*>(lb + t * (static_cast<long long>(H) * D) + d);
+          }
+          *reinterpret_cast<float4*>(qs + i * DP + d) = q;
+          *reinterpret_cast<float4*>(ks + i * DP + d) = k;
+          *reinterpret_cast<float4*>(Bs + i * DP + d) = make_float4(l.x * kLog, l.y * kLog, l.z * kLog, l.w * kLog);
+        }
+      }
+    } else {
+      for (int i = warp; i < kC; i += kWarps)
+        for (int d = lane; d < D4; d += 32) {
+          const long long t = first + i;
+          const bool ok = i < n && d < D;
+          qs[i * DP + d] = ok ? qb[t * U + d] : 0.f;
+          ks[i * DP + d] = ok ? kb[t * U + d] : 0.f;
+          Bs[i * DP + d] = ok ? lb[t * (static_cast<long long>(H) * D) + d] * kLog : 0.f;
+        }
     }
-    qs[i * DP + d] = q;
-    ks[i * DP + d] = k;
-    Bs[i * DP + d] = l;
   }
   if (tid < kC) beta[tid] = tid < n ? sigmoidf_(ldf(static_cast<const T*>(p.b) + static_cast<long long>(first + tid) * p.b_stride + head)) : 0.f;
   for (int e = tid; e < kC * kC; e += kDpThreads) As[e] = 0.f;
@@ -465,7 +548,6 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_
   }
   __syncthreads();
   // pairs inside the blocks: (block, i, s <= i), 136 per block, every pair by four neighbouring threads that split the channels
-  constexpr bool kFast = sizeof(T) == 2;   // bfloat16 runs: base-2 exponential unit (relative error near 2^-22)
   for (int e = tid >> 2; e < kNB * 136; e += kDpThreads / 4) {
     const int blk = e / 136, pr = e - blk * 136;
     int i = static_cast<int>((sqrtf(8.f * pr + 1.f) - 1.f) * 0.5f);
@@ -478,7 +560,6 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_
       const float4 bi = *reinterpret_cast<const float4*>(Bs + i * DP + d), bs = *reinterpret_cast<const float4*>(Bs + s * DP + d);
       const float4 qi = *reinterpret_cast<const float4*>(qs + i * DP + d), ki = *reinterpret_cast<const float4*>(ks + i * DP + d);
       const float4 k4 = *reinterpret_cast<const float4*>(ks + s * DP + d);
-      auto ex = [](float x) { return kFast ? ex2(x * 1.4426950408889634f) : expf(x); };
       const float x0 = k4.x * ex(bi.x - bs.x), x1 = k4.y * ex(bi.y - bs.y), x2 = k4.z * ex(bi.z - bs.z), x3 = k4.w * ex(bi.w - bs.w);
       aq = fmaf(qi.x, x0, fmaf(qi.y, x1, fmaf(qi.z, x2, fmaf(qi.w, x3, aq))));
       ak = fmaf(ki.x, x0, fmaf(ki.y, x1, fmaf(ki.z, x2, fmaf(ki.w, x3, ak))));
@@ -506,19 +587,22 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_
   {
     float* qd = p.qd + base * kC * D;
     float* kd = p.kd + base * kC * L;
-    for (int e = tid; e < kC * D4; e += kDpThreads) {
-      const int i = e / D4, d = e - i * D4, o = i * DP + d;
-      const float bv = Bs[o], q = qs[o], k = ks[o];
-      const float br = i < 16 ? 0.f : i < 32 ? f1[d] : i < 48 ? f2[d] : f3[d];
-      const float bn = i < 16 ? f1[d] : i < 32 ? f2[d] : i < 48 ? f3[d] : bv;
-      const float es = expf(bv - br);
-      if (d < D) {
-        qd[i * D + d] = q * expf(bv);
-        kd[static_cast<long long>(i) * L + delta_kd_slot(d)] = k * expf(fe[d] - bv);
+    for (int i = warp; i < kC; i += kWarps) {
+#pragma unroll 4
+      for (int d = lane; d < D4; d += 32) {
+        const int o = i * DP + d;
+        const float bv = Bs[o], q = qs[o], k = ks[o];
+        const float br = i < 16 ? 0.f : i < 32 ? f1[d] : i < 48 ? f2[d] : f3[d];
+        const float bn = i < 16 ? f1[d] : i < 32 ? f2[d] : i < 48 ? f3[d] : bv;
+        const float es = ex(bv - br);
+        if (d < D) {
+          qd[i * D + d] = q * ex(bv);
+          kd[static_cast<long long>(i) * L + delta_kd_slot(d)] = k * ex(fe[d] - bv);
+        }
+        qs[o] = q * es;
+        ks[o] = k * es;
+        Bs[o] = k * ex(bn - bv);
       }
-      qs[o] = q * es;
-      ks[o] = k * es;
-      Bs[o] = k * expf(bn - bv);
     }
     for (int e = tid; e < kC * (L - D); e += kDpThreads) {   // the padding of the outgoing keys
       const int i = e / (L - D), d = D + (e - i * (L - D));
@@ -528,10 +612,10 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_
   __syncthreads();
   for (int d = tid; d < D4; d += kDpThreads) {
     const float b1 = f1[d], b2 = f2[d], b3 = f3[d];
-    f1[d] = expf(b1);
-    f2[d] = expf(b2 - b1);
-    f3[d] = expf(b3 - b2);
-    if (d < D) p.g[base * D + d] = expf(fe[d]);
+    f1[d] = ex(b1);
+    f2[d] = ex(b2 - b1);
+    f3[d] = ex(b3 - b2);
+    if (d < D) p.g[base * D + d] = ex(fe[d]);
   }
   __syncthreads();
   // pairs across blocks: six (I, J) pairs of 16 x 16, 2 x 2 pairs per thread
@@ -604,148 +688,192 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_
   }
 }
 
-// Block = (8 value columns, head, entry), 8 warps.  Both products split their sum over the warps and meet in `red`: u = u0 - w S over
-// the channels, kd^T u over the tokens; a lane owns rows r, r + 16, r + 32, r + 48 (one 16-byte piece in the layouts the
-// preparation writes) and four columns.  w and kd of a chunk have one shared-memory buffer each: kd travels under the first product,
-// the next chunk's w under the second.
-constexpr int kDcThreads = 256, kDcV = 8;
+// Block = (VS value columns, head, entry), 8 warps.  Both products split their sum over the warps and meet in `red`: u = u0 - w S over the
+// channels, kd^T u over the tokens; a lane owns rows r, r + 16, r + 32, r + 48 (one 16-byte piece in the layouts the preparation writes) and
+// half of the columns.  With NB = 2 the next chunk's w and kd travel under the whole of this chunk; with NB = 1 (wide heads) kd travels under
+// the first product and the next chunk's w under the second.
+constexpr int kDcThreads = 256;
 
+template <int VS, int NB>
 __global__ void __launch_bounds__(kDcThreads) delta_chunk_scan_kernel(const pcs_delta_chunk_params p) {
   extern __shared__ __align__(16) float sm[];
+  constexpr int CW = VS / 2;        // columns of a lane
+  constexpr int LV = VS == 8 ? 3 : 4;
   const int D = p.dim, V = p.vdim, H = p.heads, L = (D + 63) & ~63, NT = L / 64;
-  float* ws = sm;                   // [D][64]
-  float* kds = ws + D * kC;         // [64][L]
-  float* S = kds + kC * L;          // [L][8]
-  float* us = S + L * kDcV;         // [64][8]
-  float* red = us + kC * kDcV;      // 4096
-  const int v0 = blockIdx.x * kDcV, head = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int r = lane & 15, c4 = (lane >> 4) * 4;
+  float* ws = sm;                        // [NB][D][64]
+  float* kds = ws + NB * D * kC;         // [NB][64][L]
+  float* S = kds + NB * kC * L;          // [L][VS]
+  float* us = S + L * VS;                // [64][VS]
+  float* red = us + kC * VS;             // [8][64][VS]
+  const int v0 = blockIdx.x * VS, head = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int r = lane & 15, c4 = (lane >> 4) * CW;
   const int n_chunks = p.seq_chunks[b];
   if (n_chunks <= 0) return;
   const long long c0 = p.seq_chunk0[b];
-  const int vs = min(kDcV, V - v0);
+  const int vs = min(VS, V - v0);
   float* Sg = p.s_pool + (static_cast<long long>(p.seq_slot[b]) * H + head) * D * V;
   const bool fresh = p.seq_pos0[b] == 0;
-  for (int e = tid; e < L * kDcV; e += kDcThreads) {
-    const int d = e >> 3, c = e & 7;
-    S[e] = (!fresh && d < D && c < vs) ? Sg[static_cast<long long>(d) * V + v0 + c] : 0.f;
-  }
   auto load_w = [&](int c) {
     const float* src = p.w + ((c0 + c) * H + head) * D * kC;
-    for (int e = tid; e < D * (kC / 4); e += kDcThreads) cp_async16(ws + e * 4, src + e * 4);
+    float* dst = ws + (NB == 2 ? (c & 1) * D * kC : 0);
+    for (int e = tid; e < D * (kC / 4); e += kDcThreads) cp_async16(dst + e * 4, src + e * 4);
   };
   auto load_kd = [&](int c) {
     const float* src = p.kd + ((c0 + c) * H + head) * kC * L;
-    for (int e = tid; e < kC * (L / 4); e += kDcThreads) cp_async16(kds + e * 4, src + e * 4);
+    float* dst = kds + (NB == 2 ? (c & 1) * kC * L : 0);
+    for (int e = tid; e < kC * (L / 4); e += kDcThreads) cp_async16(dst + e * 4, src + e * 4);
   };
   load_w(0);
   cp_async_commit();
   load_kd(0);
   cp_async_commit();
+  for (int e = tid; e < L * VS; e += kDcThreads) {
+    const int d = e >> LV, c = e & (VS - 1);
+    S[e] = (!fresh && d < D && c < vs) ? Sg[static_cast<long long>(d) * V + v0 + c] : 0.f;
+  }
   // phase 1: warp -> channels [d_lo, d_hi); phase 2: warp -> (64-channel tile, part of the tokens)
   const int dw = (D + 7) / 8, d_lo = min(D, warp * dw), d_hi = min(D, d_lo + dw);
   const int parts = 8 / NT, tile = warp % NT, part = warp / NT, tw = kC / parts;
   const int i_lo = part * tw;
   const bool busy2 = part < parts;
-  constexpr int kMaxOut = 8;   // L * 8 / 256 outputs of phase 2 per thread
+  constexpr int kOut1 = kC * VS / kDcThreads;        // outputs of phase 1 per thread
+  constexpr int kOut2 = 256 * VS / kDcThreads;       // of phase 2, at most
   for (int c = 0; c < n_chunks; ++c) {
     const long long base = (c0 + c) * H + head;
     float* ug = p.u + base * kC * V + v0;
-    float u0[2], gd[kMaxOut];
+    float u0[kOut1], gd[kOut2];
 #pragma unroll
-    for (int m = 0; m < 2; ++m) {
+    for (int m = 0; m < kOut1; ++m) {
       const int e = tid + m * kDcThreads;
-      u0[m] = (e & 7) < vs ? ug[static_cast<long long>(e >> 3) * V + (e & 7)] : 0.f;
+      u0[m] = (e & (VS - 1)) < vs ? ug[static_cast<long long>(e >> LV) * V + (e & (VS - 1))] : 0.f;
     }
 #pragma unroll
-    for (int m = 0; m < kMaxOut; ++m) {
-      const int d = (tid + m * kDcThreads) >> 3;
+    for (int m = 0; m < kOut2; ++m) {
+      const int d = (tid + m * kDcThreads) >> LV;
       gd[m] = d < D ? p.g[base * D + d] : 0.f;
     }
     cp_async_wait<1>();
-    __syncthreads();   // w of this chunk, and the state
+    __syncthreads();   // w of this chunk, and the state; the buffers of the chunk before are free
+    if (NB == 2) {
+      if (c + 1 < n_chunks) load_w(c + 1);
+      cp_async_commit();
+      if (c + 1 < n_chunks) load_kd(c + 1);
+      cp_async_commit();
+    }
     {
-      float acc[4][4];
+      const float* wc = ws + (NB == 2 ? (c & 1) * D * kC : 0);
+      float acc[4][CW];
 #pragma unroll
-      for (int x = 0; x < 4; ++x) acc[x][0] = acc[x][1] = acc[x][2] = acc[x][3] = 0.f;
+      for (int x = 0; x < 4; ++x)
+#pragma unroll
+        for (int y = 0; y < CW; ++y) acc[x][y] = 0.f;
 #pragma unroll 4
       for (int d = d_lo; d < d_hi; ++d) {
-        const float4 w4 = *reinterpret_cast<const float4*>(ws + d * kC + 4 * r), s4 = *reinterpret_cast<const float4*>(S + d * kDcV + c4);
+        const float4 w4 = *reinterpret_cast<const float4*>(wc + d * kC + 4 * r);
         const float wv[4] = {w4.x, w4.y, w4.z, w4.w};
 #pragma unroll
-        for (int x = 0; x < 4; ++x) {
-          acc[x][0] = fmaf(wv[x], s4.x, acc[x][0]);
-          acc[x][1] = fmaf(wv[x], s4.y, acc[x][1]);
-          acc[x][2] = fmaf(wv[x], s4.z, acc[x][2]);
-          acc[x][3] = fmaf(wv[x], s4.w, acc[x][3]);
+        for (int y = 0; y < CW; y += 4) {
+          const float4 s4 = *reinterpret_cast<const float4*>(S + d * VS + c4 + y);
+#pragma unroll
+          for (int x = 0; x < 4; ++x) {
+            acc[x][y] = fmaf(wv[x], s4.x, acc[x][y]);
+            acc[x][y + 1] = fmaf(wv[x], s4.y, acc[x][y + 1]);
+            acc[x][y + 2] = fmaf(wv[x], s4.z, acc[x][y + 2]);
+            acc[x][y + 3] = fmaf(wv[x], s4.w, acc[x][y + 3]);
+          }
         }
       }
 #pragma unroll
       for (int x = 0; x < 4; ++x)
-        *reinterpret_cast<float4*>(red + warp * (kC * kDcV) + (r + 16 * x) * kDcV + c4) = make_float4(acc[x][0], acc[x][1], acc[x][2], acc[x][3]);
+#pragma unroll
+        for (int y = 0; y < CW; y += 4)
+          *reinterpret_cast<float4*>(red + warp * (kC * VS) + (r + 16 * x) * VS + c4 + y) = make_float4(acc[x][y], acc[x][y + 1], acc[x][y + 2], acc[x][y + 3]);
     }
     __syncthreads();
-    if (c + 1 < n_chunks) load_w(c + 1);
-    cp_async_commit();
+    if (NB == 1) {
+      if (c + 1 < n_chunks) load_w(c + 1);
+      cp_async_commit();
+    }
 #pragma unroll
-    for (int m = 0; m < 2; ++m) {
+    for (int m = 0; m < kOut1; ++m) {
       const int e = tid + m * kDcThreads;
       float a = 0.f;
 #pragma unroll
-      for (int w = 0; w < 8; ++w) a += red[w * (kC * kDcV) + e];
+      for (int w = 0; w < 8; ++w) a += red[w * (kC * VS) + e];
       const float u = u0[m] - a;
       us[e] = u;
-      if ((e & 7) < vs) ug[static_cast<long long>(e >> 3) * V + (e & 7)] = u;
+      if ((e & (VS - 1)) < vs) ug[static_cast<long long>(e >> LV) * V + (e & (VS - 1))] = u;
     }
-    cp_async_wait<1>();
+    cp_async_wait<NB>();
     __syncthreads();   // kd of this chunk, and u; `red` is free again
     if (busy2) {
-      float acc[4][4];
+      const float* kc = kds + (NB == 2 ? (c & 1) * kC * L : 0);
+      float acc[4][CW];
 #pragma unroll
-      for (int x = 0; x < 4; ++x) acc[x][0] = acc[x][1] = acc[x][2] = acc[x][3] = 0.f;
+      for (int x = 0; x < 4; ++x)
+#pragma unroll
+        for (int y = 0; y < CW; ++y) acc[x][y] = 0.f;
 #pragma unroll 4
       for (int i = i_lo; i < i_lo + tw; ++i) {
-        const float4 k4 = *reinterpret_cast<const float4*>(kds + i * L + tile * 64 + 4 * r), u4 = *reinterpret_cast<const float4*>(us + i * kDcV + c4);
+        const float4 k4 = *reinterpret_cast<const float4*>(kc + i * L + tile * 64 + 4 * r);
         const float kv[4] = {k4.x, k4.y, k4.z, k4.w};
 #pragma unroll
-        for (int x = 0; x < 4; ++x) {
-          acc[x][0] = fmaf(kv[x], u4.x, acc[x][0]);
-          acc[x][1] = fmaf(kv[x], u4.y, acc[x][1]);
-          acc[x][2] = fmaf(kv[x], u4.z, acc[x][2]);
-          acc[x][3] = fmaf(kv[x], u4.w, acc[x][3]);
+        for (int y = 0; y < CW; y += 4) {
+          const float4 u4 = *reinterpret_cast<const float4*>(us + i * VS + c4 + y);
+#pragma unroll
+          for (int x = 0; x < 4; ++x) {
+            acc[x][y] = fmaf(kv[x], u4.x, acc[x][y]);
+            acc[x][y + 1] = fmaf(kv[x], u4.y, acc[x][y + 1]);
+            acc[x][y + 2] = fmaf(kv[x], u4.z, acc[x][y + 2]);
+            acc[x][y + 3] = fmaf(kv[x], u4.w, acc[x][y + 3]);
+          }
         }
       }
 #pragma unroll
       for (int x = 0; x < 4; ++x)
-        *reinterpret_cast<float4*>(red + part * (L * kDcV) + (tile * 64 + r + 16 * x) * kDcV + c4) = make_float4(acc[x][0], acc[x][1], acc[x][2], acc[x][3]);
+#pragma unroll
+        for (int y = 0; y < CW; y += 4)
+          *reinterpret_cast<float4*>(red + part * (L * VS) + (tile * 64 + r + 16 * x) * VS + c4 + y) = make_float4(acc[x][y], acc[x][y + 1], acc[x][y + 2], acc[x][y + 3]);
     }
     __syncthreads();
-    if (c + 1 < n_chunks) load_kd(c + 1);
-    cp_async_commit();
+    if (NB == 1) {
+      if (c + 1 < n_chunks) load_kd(c + 1);
+      cp_async_commit();
+    }
     float* sg = p.s + base * D * V + v0;
 #pragma unroll
-    for (int m = 0; m < kMaxOut; ++m) {
+    for (int m = 0; m < kOut2; ++m) {
       const int e = tid + m * kDcThreads;
-      if (e < L * kDcV) {
+      if (e < L * VS) {
         float a = 0.f;
-        for (int w = 0; w < parts; ++w) a += red[w * (L * kDcV) + e];
-        const int d = e >> 3, cc = e & 7;
+        for (int w = 0; w < parts; ++w) a += red[w * (L * VS) + e];
+        const int d = e >> LV, cc = e & (VS - 1);
         const float old = S[e];
         if (d < D && cc < vs) sg[static_cast<long long>(d) * V + cc] = old;
         S[e] = fmaf(gd[m], old, a);
       }
     }
   }
+  cp_async_wait<0>();
   __syncthreads();
-  for (int e = tid; e < D * kDcV; e += kDcThreads)
-    if ((e & 7) < vs) Sg[static_cast<long long>(e >> 3) * V + v0 + (e & 7)] = S[e];
+  for (int e = tid; e < D * VS; e += kDcThreads)
+    if ((e & (VS - 1)) < vs) Sg[static_cast<long long>(e >> LV) * V + v0 + (e & (VS - 1))] = S[e];
+}
+
+template <int VS, int NB>
+static int launch_delta_chunk_scan(const pcs_delta_chunk_params& p, size_t smem, cudaStream_t st) {
+  PCS_CHECK_CUDA(cudaFuncSetAttribute(delta_chunk_scan_kernel<VS, NB>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+  delta_chunk_scan_kernel<VS, NB><<<dim3((p.vdim + VS - 1) / VS, p.heads, p.n_seqs), kDcThreads, smem, st>>>(p);
+  PCS_CHECK_CUDA(cudaGetLastError());
+  count_launch();
+  return PCS_OK;
 }
 
 // ---- per-head norm and gate ------------------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(256) head_norm_gate_kernel(const pcs_headnorm_params p) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, V = p.vdim, H = p.heads;
-  const long long e = static_cast<long long>(blockIdx.x) * 8 + warp;
+  const long long e = static_cast<long long>(blockIdx.x) * (blockDim.x >> 5) + warp;
   if (e >= static_cast<long long>(p.n_tokens) * H) return;
   const long long t = e / H;
   const int h = static_cast<int>(e - t * H);
@@ -759,13 +887,14 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const pcs_headnorm_
   const T* w = static_cast<const T*>(p.w);
   T* out = static_cast<T*>(p.out) + t * p.out_stride + h * V;
   constexpr int KEEP = 16;   // columns of a lane that stay in registers
-  float ov[KEEP], gv[KEEP];
+  float ov[KEEP], gv[KEEP], wv[KEEP];
   float ss = 0.f;
 #pragma unroll
   for (int u = 0; u < KEEP; ++u) {
     const int c = lane + u * 32;
     ov[u] = c < V ? o[c] : 0.f;
     gv[u] = c < V ? ldf(g + c) : 0.f;
+    wv[u] = c < V ? ldf(w + c) : 0.f;
   }
 #pragma unroll
   for (int u = 0; u < KEEP; ++u) ss = fmaf(ov[u], ov[u], ss);
@@ -775,26 +904,44 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const pcs_headnorm_
 #pragma unroll
   for (int u = 0; u < KEEP; ++u) {
     const int c = lane + u * 32;
-    if (c < V) stf(out + c, ov[u] * inv * ldf(w + c) * sigmoidf_(gv[u]));
+    if (c < V) stf(out + c, ov[u] * inv * wv[u] * sigmoidf_(gv[u]));
   }
   for (int c = lane + KEEP * 32; c < V; c += 32) stf(out + c, o[c] * inv * ldf(w + c) * sigmoidf_(ldf(g + c)));
 }
 
 }  // namespace pcs
 
+static int check_short_conv(const pcs_shortconv_params* p, const char* what, bool* vec) {
+  PCS_REQUIRE(p->proj && p->conv_w && p->qk_out && p->v_out && p->tok_seq && p->tok_pos && p->seq_slot && p->seq_pos0 && p->seq_len && p->seq_par,
+              "%s: null tensor", what);
+  PCS_REQUIRE(p->kv_heads > 0 && p->dim > 0 && p->v_width > 0 && p->c_off >= 0 && p->taps >= 1 && p->taps <= pcs::kScMaxTaps && (p->tail || p->taps == 1),
+              "%s: bad sizes (taps %d of at most %d)", what, p->taps, pcs::kScMaxTaps);
+  const int piece = p->dtype == PCS_BF16 ? 8 : 4;
+  auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+  *vec = p->impl != 1 && p->taps <= 4 && p->dim % piece == 0 && p->v_width % piece == 0 && p->c_off % piece == 0 && p->row_stride % piece == 0 &&
+         p->dim <= 256 * piece && al(p->proj) && al(p->conv_w) && al(p->tail) && al(p->qk_out) && al(p->v_out);
+  return PCS_OK;
+}
+
 PCS_API int pcs_short_conv(const pcs_shortconv_params* p, void* stream) {
   PCS_REQUIRE(p, "pcs_short_conv: null params");
   if (p->n_tokens == 0) return PCS_OK;
-  PCS_REQUIRE(p->proj && p->conv_w && p->qk_out && p->v_out && p->tok_seq && p->tok_pos && p->seq_slot && p->seq_pos0 && p->seq_len && p->seq_par,
-              "pcs_short_conv: null tensor");
-  PCS_REQUIRE(p->kv_heads > 0 && p->dim > 0 && p->v_width > 0 && p->c_off >= 0 && p->taps >= 1 && p->taps <= pcs::kScMaxTaps && (p->tail || p->taps == 1),
-              "pcs_short_conv: bad sizes (taps %d of at most %d)", p->taps, pcs::kScMaxTaps);
-  const int piece = p->dtype == PCS_BF16 ? 8 : 4;
-  auto al = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
-  const bool vec = p->impl != 1 && p->taps <= 4 && p->dim % piece == 0 && p->v_width % piece == 0 && p->c_off % piece == 0 && p->row_stride % piece == 0 &&
-                   p->dim <= 256 * piece && al(p->proj) && al(p->conv_w) && al(p->tail) && al(p->qk_out) && al(p->v_out);
+  bool vec = false;
+  if (int rc = check_short_conv(p, "pcs_short_conv", &vec)) return rc;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  PCS_DISPATCH(p->dtype, return pcs::launch_short_conv<T>(*p, st, vec));
+  PCS_DISPATCH(p->dtype, return pcs::launch_short_conv<T>(*p, nullptr, st, vec));
+}
+
+PCS_API int pcs_delta_inputs(const pcs_shortconv_params* p, const pcs_lowrank_params* q, void* stream) {
+  PCS_REQUIRE(p && q, "pcs_delta_inputs: null params");
+  if (p->n_tokens == 0) return PCS_OK;
+  bool vec = false;
+  if (int rc = check_short_conv(p, "pcs_delta_inputs", &vec)) return rc;
+  if (!vec) return pcs::set_error(PCS_ERR_UNSUPPORTED, "pcs_delta_inputs: sizes off the 16-byte pieces take pcs_short_conv and products of their own");
+  PCS_REQUIRE(q->a2 && q->dt_bias && q->rate && q->decay_out && q->g2 && q->gate_out && q->heads > 0 && q->dim > 0 && q->decay_rank > 0 && q->gate_rank > 0 &&
+                  q->gate_width > 0 && q->a_off >= 0 && q->g_off >= 0, "pcs_delta_inputs: bad low-rank products");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  PCS_DISPATCH(p->dtype, return pcs::launch_short_conv<T>(*p, q, st, true));
 }
 
 PCS_API int pcs_delta_scan(const pcs_delta_params* p, void* stream) {
@@ -860,13 +1007,18 @@ PCS_API int pcs_delta_chunk_scan(const pcs_delta_chunk_params* p, void* stream) 
   PCS_REQUIRE(p->heads > 0 && p->heads <= 65535 && p->n_seqs <= 65535 && p->dim > 0 && p->dim <= 256 && p->vdim > 0, "pcs_delta_chunk_scan: bad sizes");
   PCS_REQUIRE(((reinterpret_cast<uintptr_t>(p->kd) | reinterpret_cast<uintptr_t>(p->w)) & 15) == 0, "pcs_delta_chunk_scan: kd and w must be 16-byte aligned");
   const int L = (p->dim + 63) & ~63;
-  const size_t smem = (static_cast<size_t>(p->dim) * pcs::kC + static_cast<size_t>(pcs::kC) * L + static_cast<size_t>(L) * pcs::kDcV + pcs::kC * pcs::kDcV + 4096) * sizeof(float);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  PCS_CHECK_CUDA(cudaFuncSetAttribute(pcs::delta_chunk_scan_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
-  pcs::delta_chunk_scan_kernel<<<dim3((p->vdim + pcs::kDcV - 1) / pcs::kDcV, p->heads, p->n_seqs), pcs::kDcThreads, smem, st>>>(*p);
-  PCS_CHECK_CUDA(cudaGetLastError());
-  pcs::count_launch();
-  return PCS_OK;
+  auto smem = [&](int vs, int nb) {
+    return (static_cast<size_t>(nb) * (p->dim * pcs::kC + pcs::kC * L) + static_cast<size_t>(vs) * (L + pcs::kC + 8 * pcs::kC)) * sizeof(float);
+  };
+  // 8 columns per block where that still is one block per SM, else 16 (half of the chunk traffic); two buffers where they fit
+  const long long rows = static_cast<long long>(p->heads) * p->n_seqs;
+  const bool narrow = rows * ((p->vdim + 7) / 8) <= 148;
+  const int vs = narrow ? 8 : 16;
+  const bool one_wave = rows * ((p->vdim + vs - 1) / vs) <= 148;
+  const bool two = smem(vs, 2) <= (one_wave ? 227u : 112u) * 1024u;
+  if (narrow) return two ? pcs::launch_delta_chunk_scan<8, 2>(*p, smem(8, 2), st) : pcs::launch_delta_chunk_scan<8, 1>(*p, smem(8, 1), st);
+  return two ? pcs::launch_delta_chunk_scan<16, 2>(*p, smem(16, 2), st) : pcs::launch_delta_chunk_scan<16, 1>(*p, smem(16, 1), st);
 }
 
 PCS_API int pcs_head_norm_gate(const pcs_headnorm_params* p, void* stream) {
@@ -875,7 +1027,8 @@ PCS_API int pcs_head_norm_gate(const pcs_headnorm_params* p, void* stream) {
   PCS_REQUIRE(p->o && p->w && p->g && p->out && p->heads > 0 && p->vdim > 0 && (p->tok_row == nullptr || p->chunk_size > 0), "pcs_head_norm_gate: bad arguments");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const long long rows = static_cast<long long>(p->n_tokens) * p->heads;
-  PCS_DISPATCH(p->dtype, pcs::head_norm_gate_kernel<T><<<static_cast<unsigned>((rows + 7) / 8), 256, 0, st>>>(*p));
+  const int warps = rows < 8 * 148 ? 1 : 8;   // few rows: one warp per block
+  PCS_DISPATCH(p->dtype, pcs::head_norm_gate_kernel<T><<<static_cast<unsigned>((rows + warps - 1) / warps), 32 * warps, 0, st>>>(*p));
   PCS_CHECK_CUDA(cudaGetLastError());
   pcs::count_launch();
   return PCS_OK;

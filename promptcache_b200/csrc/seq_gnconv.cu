@@ -169,6 +169,21 @@ __global__ void __launch_bounds__(256, (PPT == 1 ? 2 : 1)) gnconv_vec_kernel(con
       }
     }
   }
+  // few tokens: the weights are requested with the rows (many tokens: their loads are hidden by other blocks, the registers are not free)
+  uint4 wq[PPT], cq[PPT][R + 1];
+  if (TB == 1) {
+#pragma unroll
+    for (int u = 0; u < PPT; ++u) {
+      const int pc = tid + u * nthr;
+      if (pc < NP) {
+        if (p.y) wq[u] = *reinterpret_cast<const uint4*>(static_cast<const T*>(p.w) + pc * N);
+        if (cw) {
+#pragma unroll
+          for (int j = 0; j <= R; ++j) cq[u][j] = *reinterpret_cast<const uint4*>(cw + static_cast<long long>(R - j) * W + pc * N);
+        }
+      }
+    }
+  }
   // the tokens' places in their entries: how many of the R predecessors are rows of this step, and the tails
   int here[TB], before[TB], last_row[TB], shift[TB];   // predecessors in this step; predecessors at all; tail row to write; rows that stay move by this
   long long tail0[TB];                                 // element offset of the slot's copy that is read
@@ -211,7 +226,8 @@ __global__ void __launch_bounds__(256, (PPT == 1 ? 2 : 1)) gnconv_vec_kernel(con
       const int pc = tid + u * nthr;
       if (pc < NP) {
         float wv[N];
-        ld16(w + pc * N, wv);
+        if (TB == 1) unpack(wq[u], wv);
+        else ld16(w + pc * N, wv);
 #pragma unroll
         for (int k = 0; k < RN; ++k) {
           float v[N];
@@ -233,13 +249,15 @@ __global__ void __launch_bounds__(256, (PPT == 1 ? 2 : 1)) gnconv_vec_kernel(con
           if (p.x_out) stx(p.x_out + static_cast<long long>(p.rows ? p.rows[t0 + i] : t0 + i) * W + pc * N, s[R + i][u]);
           if (cw) {
             float o[N], wv[N];
-            ld16(cw + static_cast<long long>(R) * W + pc * N, wv);
+            if (TB == 1) unpack(cq[u][0], wv);
+            else ld16(cw + static_cast<long long>(R) * W + pc * N, wv);
 #pragma unroll
             for (int e = 0; e < N; ++e) o[e] = fmaf(s[R + i][u][e], wv[e], s[R + i][u][e]);
 #pragma unroll
             for (int j = 1; j <= R; ++j)
               if (j <= before[i]) {
-                ld16(cw + static_cast<long long>(R - j) * W + pc * N, wv);
+                if (TB == 1) unpack(cq[u][j], wv);
+                else ld16(cw + static_cast<long long>(R - j) * W + pc * N, wv);
                 if (j <= here[i]) {
 #pragma unroll
                   for (int e = 0; e < N; ++e) o[e] = fmaf(wv[e], s[R + i - j][u][e], o[e]);

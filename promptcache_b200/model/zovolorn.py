@@ -14,7 +14,8 @@ on the sublayers' RESULTS only and a short causal convolution in front of every 
                          chunk of positions only                                          (`pcs_rope_kv_prep`, `pcs_attn`)
                   right  the gated delta rule: q, k, v through a short convolution with silu, q and k unit vectors, a decay per key
                          channel, a step size per head, per-head norm and a low-rank sigmoid gate
-                                          (`pcs_short_conv`, `pcs_gla_decay`, `pcs_delta_scan` / `pcs_delta_chunk_*`, `pcs_head_norm_gate`)
+                                          (`pcs_short_conv`, `pcs_gla_decay`, `pcs_delta_scan` / `pcs_delta_chunk_*`, `pcs_head_norm_gate`;
+                         decoding takes the inputs in one launch, `pcs_delta_inputs`)
                   both write their columns of ONE matrix, already times their constants, so one product with the two output
                   projections side by side adds them in 32-bit
     feed-forward  W_down(gelu(W_gate h + b) * (W_up h + b)) + b with the tanh form of gelu                    (`pcs_glu_mul`)
@@ -250,10 +251,9 @@ class ZovolornForCausalLM(SlotPoolCausalLM):
         ws = nsq.attn_workspace(T, H, D, dev) if T <= 16 else None
         nsq.attention(q, st["k"], st["v"], mixed[:, :H * D], H, blk["scale"], None, None, False, batch, impl=self.attn_impl, max_keys=seen, workspace=ws,
                       head_scale=blk["temp"], bias_table=blk["bias"], chunk=blk["chunk"], out_scale=blk["left_scale"])
-        qk, v = nsq.short_conv(proj, blk["conv_off"], Gr, Dr, Hr * Vr, blk["conv"], st.get("conv_tail"), Dr ** -0.5, UNIT_VECTOR_EPS, batch)
-        gate = nsq.linear(proj[:, slice(*blk["g1"])], blk["w_g2"])
-        decay = nsq.gla_decay(proj[:, slice(*blk["a1"])], blk["w_a2"], blk["dt_bias"], 1.0, rate=blk["rate"],
-                              expo=not nsq.delta_takes_chunks(batch, Dr, self.scan_impl))
+        qk, v, decay, gate = nsq.delta_inputs(proj, blk["conv_off"], Gr, Hr, Dr, Vr, blk["conv"], st.get("conv_tail"), Dr ** -0.5, UNIT_VECTOR_EPS, blk["a1"],
+                                              blk["w_a2"], blk["dt_bias"], blk["rate"], blk["g1"], blk["w_g2"], batch,
+                                              expo=not nsq.delta_takes_chunks(batch, Dr, self.scan_impl))
         nsq.delta_scan(qk, v, decay, proj[:, slice(*blk["b"])], Gr, st["s"], blk["r_norm"], gate, mixed[:, H * D:], self.eps, batch, out_scale=blk["right_scale"],
                        impl=self.scan_impl)
         return nsq.linear(mixed, blk["w_o"])

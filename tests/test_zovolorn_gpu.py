@@ -422,6 +422,39 @@ def test_decays_from_softplus_rates(nsq, dtype, T, H, D, r):
     close(nsq.gla_decay(*args, rate=torch.exp(dev(a_log)), expo=True), torch.exp(want), 3e-6, "decays")
 
 
+@pytest.mark.parametrize("dtype,G,H,D,V,ra,rg,taps", [(F32, 2, 4, 8, 12, 5, 3, 4), (BF16, 2, 2, 32, 48, 24, 16, 4), (BF16, 1, 4, 64, 16, 8, 130, 3), (F32, 3, 3, 12, 4, 64, 40, 2),
+                                                         (BF16, 2, 2, 24, 8, 1, 7, 1)])
+def test_inputs_of_the_delta_rule_in_one_launch(nsq, dtype, G, H, D, V, ra, rg, taps):
+    """A few tokens of several sequences: the convolution, the decays and the gate product from one launch against the oracle, and tails that the
+    separate kernels go on from."""
+    g = torch.Generator().manual_seed(ra + rg)
+    U, vw, R = 2 * G * D, H * V, taps - 1
+    ch = U + vw
+    offs = (8, 8 + ch, 8 + ch + rg)                       # convolution | gate inputs | decay inputs
+    width = (8 + ch + rg + ra + 7) // 8 * 8
+    rq = lambda *s, sc=1.0: (torch.randn(*s, generator=g, dtype=F64) * sc).to(dtype).to(F64)
+    proj, cw, a2, g2 = rq(14, width), rq(ch, taps, sc=0.6), rq(H * D, ra), rq(H * V, rg)
+    dtb, rate = torch.randn(H * D, generator=g, dtype=F64).to(F32).to(F64), torch.rand(H, generator=g, dtype=F64).to(F32).to(F64)
+    a = O.silu(O.causal_conv(proj[:, 8:8 + ch], cw))
+    qk = O.unit_vector(a[:, :U].view(14, 2 * G, D))
+    qk[:, :G] *= 0.5
+    decay = torch.exp(O.log_decay(proj[:, offs[2]:offs[2] + ra] @ a2.T + dtb, torch.log(rate), D)).reshape(14, H * D)
+    gate = proj[:, offs[1]:offs[1] + rg] @ g2.T
+    tol = 3e-6 if dtype == F32 else 6e-3
+    pd, tail = dev(proj, dtype), torch.full((2, 2, max(R, 1), ch), 5.0, device=DEV)
+    out, p0 = [], 0
+    for k, (n, fused) in enumerate([(1, True), (1, True), (2, False), (1, True), (5, True), (4, None)]):
+        b = batch_of(nsq, [1], [p0], [n], [k & 1])
+        out.append(nsq.delta_inputs(pd[p0:p0 + n], 8, G, H, D, V, dev(cw.T, dtype), tail if R else None, 0.5, O.UNIT_EPS, (offs[2], offs[2] + ra), dev(a2, dtype), dev(dtb), dev(rate),
+                                    (offs[1], offs[1] + rg), dev(g2, dtype), b, True, fused=fused))
+        p0 += n
+    got = [torch.cat(x) for x in zip(*out)]
+    close(got[0].view(14, 2 * G, D), qk, 3e-6, "unit vectors")
+    close(got[1], a[:, U:], tol, "values")
+    close(got[2], decay, 3e-6, "decays")
+    close(got[3], gate, 3e-6 if dtype == F32 else 1e-2, "gate inputs")
+
+
 def test_gelu_with_a_gate_and_soft_cap(nsq):
     g = torch.Generator().manual_seed(1)
     gu, z = torch.randn(9, 34, generator=g, dtype=F64) * 2, torch.randn(5, 77, generator=g, dtype=F64) * 30
