@@ -634,8 +634,10 @@ int pcs_delta_scan(const pcs_delta_params* p, void* stream);
 /* The same in chunks of PCS_DELTA_CHUNK tokens (prompts; dim <= 256).  With B_i the running sum of the log decays inside a chunk,
  * e its last token, A[i, s] = sum_d k_i k_s exp(B_i - B_s) (s < i), M = I + diag(beta) A, and L = round up dim to a multiple of 64:
  *   pcs_delta_chunk_prep   qd[c, h, i, :] = q_i exp(B_i);  g[c, h, :] = exp(B_e);  a[c, h, i, s] = sum_d q_i k_s exp(B_i - B_s) for s <= i, else 0
- *                          w[c, h, d, :]  = column d of M^-1 diag(beta) K exp(B)        (element 4 (i % 16) + i / 16 belongs to token i)
- *                          kd[c, h, i, :] = k_i exp(B_e - B_i), padded to L               (element 64 t + 4 r + n belongs to channel 64 t + r + 16 n)
+ *                          w[c, h]        = M^-1 diag(beta) K exp(B)     (64 tokens x D8 channels, D8: dim rounded up to a multiple of 8)
+ *                          kd[c, h]       = K exp(B_e - B)               (64 tokens x L channels)
+ *                          in layouts of the scan's own: bfloat16 runs m16n8k8 operand fragments, float32 runs w[d][4 (i % 16) + i / 16] and
+ *                          kd[i][64 t + 4 r + n] for channel 64 t + r + 16 n
  *                          u[c, h, i, :]  = row i of M^-1 diag(beta) V                    (every exponent formed is <= 0)
  *   pcs_delta_chunk_scan   per entry, over its chunks in order, S from the pool:  u[c] <- u[c] - w[c] S;  s[c] = S;  S <- g S + kd[c]^T u[c]
  *   (the caller forms o[c, h] = qd[c, h] s[c, h] + a[c, h] u[c, h], fp32 [chunks, heads, 64, vdim]) */
@@ -651,8 +653,8 @@ typedef struct pcs_delta_chunk_params {
   const int32_t* chunk_len;    /* [n_chunks] */
   int32_t n_chunks, n_tokens, dtype, n_seqs;
   float* qd;                   /* [chunks, heads, 64, dim] */
-  float* kd;                   /* [chunks, heads, 64, L] */
-  float* w;                    /* [chunks, heads, dim, 64] */
+  float* kd;                   /* [chunks, heads, 64 * L] */
+  float* w;                    /* [chunks, heads, D8 * 64] */
   float* g;                    /* [chunks, heads, dim] */
   float* u;                    /* [chunks, heads, 64, vdim] */
   float* a;                    /* [chunks, heads, 64, 64] */

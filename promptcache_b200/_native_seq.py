@@ -1191,7 +1191,7 @@ def delta_scan(qk: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, b: torch.
         plan = _gla_chunk_plan(batch, ch)
         nc, L = plan["n_chunks"], (D + 63) // 64 * 64
         new = lambda *s: torch.empty(*s, dtype=torch.float32, device=dev)
-        qd, kd, w, g, u, a, s = new(nc * H, ch, D), new(nc * H, ch, L), new(nc * H, D, ch), new(nc * H, D), new(nc * H, ch, V), new(nc * H, ch, ch), new(nc * H, D, V)
+        qd, kd, w, g, u, a, s = new(nc * H, ch, D), new(nc * H, ch, L), new(nc * H, (D + 7) // 8 * 8, ch), new(nc * H, D), new(nc * H, ch, V), new(nc * H, ch, ch), new(nc * H, D, V)
         p = pcs_delta_chunk_params()
         p.qk, p.v, p.ld, p.b, p.b_stride = qk.data_ptr(), v.data_ptr(), decay.data_ptr(), b.data_ptr(), b.stride(0)
         p.heads, p.kv_heads, p.dim, p.vdim = H, int(kv_heads), D, V

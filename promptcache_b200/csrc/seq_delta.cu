@@ -473,7 +473,7 @@ __global__ void __launch_bounds__(256) delta_scan_reg_kernel(const pcs_delta_par
 //   every exponent is <= 0, and each factor is at least their product, so nothing is lost that the product does not lose.
 // So q and k are scaled in place to their block's start and the keys to their block's end, and the pairs across blocks are plain products.
 constexpr int kC = PCS_DELTA_CHUNK, kCB = 16, kNB = kC / kCB;
-constexpr int kDpThreads = 512;
+constexpr int kDpThreads = 384;
 
 __device__ __forceinline__ int delta_kd_slot(int d) { return (d & ~63) + 4 * (d & 15) + ((d & 63) >> 4); }
 
@@ -507,8 +507,9 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_
     if (vec) {   // a warp takes a row at a time, the rows' loads overlap
       for (int d = lane * 4; d < D; d += 128) {
 #pragma unroll
-        for (int it = 0; it < kC / kWarps; ++it) {
+        for (int it = 0; it < (kC + kWarps - 1) / kWarps; ++it) {
           const int i = warp + it * kWarps;
+          if (i >= kC) break;
           float4 q = make_float4(0.f, 0.f, 0.f, 0.f), k = q, l = q;
           if (i < n) {
             const long long t = first + i;
@@ -587,6 +588,19 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_
   {
     float* qd = p.qd + base * kC * D;
     float* kd = p.kd + base * kC * L;
+    if (kFast) {   // the outgoing keys as fragments: a warp takes (16 channels, 8 tokens) at a time and writes 512 bytes
+      for (int f = warp; f < (L / 16) * (kC / 8); f += kWarps) {
+        const int mt = f >> 3, kt = f & 7;
+        float o[4];
+#pragma unroll
+        for (int r = 0; r < 4; ++r) {
+          const int i = kt * 8 + (lane & 3) + 4 * (r >> 1), d = mt * 16 + (lane >> 2) + 8 * (r & 1);
+          o[r] = d < D ? ks[i * DP + d] * ex(fe[d] - Bs[i * DP + d]) : 0.f;
+        }
+        *reinterpret_cast<float4*>(kd + (static_cast<long long>(f) * 32 + lane) * 4) = make_float4(o[0], o[1], o[2], o[3]);
+      }
+      __syncthreads();
+    }
     for (int i = warp; i < kC; i += kWarps) {
 #pragma unroll 4
       for (int d = lane; d < D4; d += 32) {
@@ -597,14 +611,14 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_
         const float es = ex(bv - br);
         if (d < D) {
           qd[i * D + d] = q * ex(bv);
-          kd[static_cast<long long>(i) * L + delta_kd_slot(d)] = k * ex(fe[d] - bv);
+          if (!kFast) kd[static_cast<long long>(i) * L + delta_kd_slot(d)] = k * ex(fe[d] - bv);
         }
         qs[o] = q * es;
         ks[o] = k * es;
         Bs[o] = k * ex(bn - bv);
       }
     }
-    for (int e = tid; e < kC * (L - D); e += kDpThreads) {   // the padding of the outgoing keys
+    for (int e = kFast ? kC * L : tid; e < kC * (L - D); e += kDpThreads) {   // the padding of the outgoing keys
       const int i = e / (L - D), d = D + (e - i * (L - D));
       kd[static_cast<long long>(i) * L + delta_kd_slot(d)] = 0.f;
     }
@@ -651,10 +665,18 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_
   __syncthreads();
   // M x = rhs by forward substitution, one column per thread, the column in registers: first the dim columns of diag(beta) K exp(B), then
   // the vdim columns of diag(beta) V
-  float* wg = p.w + base * D * kC;
+  const int D8 = (D + 7) & ~7;
+  float* wg = p.w + base * D8 * kC;
   float* ug = p.u + base * kC * V;
+  for (int e = tid; e < (D8 - D) * kC; e += kDpThreads) {   // channels that only pad the fragments
+    const int d = D + e / kC, i = e % kC;
+    if (kFast) wg[(((d >> 3) * 4 + (i >> 4)) * 32 + (i & 7) * 4 + (d & 3)) * 4 + ((i >> 3) & 1) + 2 * ((d >> 2) & 1)] = 0.f;
+  }
+#pragma unroll 1
   for (int col = tid; col < D + V; col += kDpThreads) {
     float x[kC];
+    long long v_step = static_cast<long long>(H) * V, u_step = V;
+    asm volatile("" : "+l"(v_step), "+l"(u_step));   // (64 row offsets each, taken out of the column loop, would spill)
     if (col < D) {
       const float e1 = f1[col], e2 = e1 * f2[col], e3 = e2 * f3[col];
 #pragma unroll
@@ -662,7 +684,7 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_
     } else {
       const T* v = static_cast<const T*>(p.v) + static_cast<long long>(first) * H * V + head * V + (col - D);
 #pragma unroll
-      for (int i = 0; i < kC; ++i) x[i] = i < n ? beta[i] * ldf(v + static_cast<long long>(i) * H * V) : 0.f;
+      for (int i = 0; i < kC; ++i) x[i] = i < n ? beta[i] * ldf(v + i * v_step) : 0.f;
     }
 #pragma unroll
     for (int i = 1; i < kC; ++i) {
@@ -678,35 +700,43 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_
       x[i] -= a0 + a1;
     }
     if (col < D) {
-      float* o = wg + static_cast<long long>(col) * kC;
+      if (kFast) {
+        float* o = wg + ((col >> 3) * 4 * 32 + (col & 3)) * 4 + 2 * ((col >> 2) & 1);
 #pragma unroll
-      for (int r = 0; r < 16; ++r) *reinterpret_cast<float4*>(o + 4 * r) = make_float4(x[r], x[r + 16], x[r + 32], x[r + 48]);
+        for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+          for (int g = 0; g < 16; ++g) o[(mt * 32 + (g & 7) * 4) * 4 + (g >> 3)] = x[mt * 16 + g];   // (wider stores would pin register pairs)
+      } else {
+        float* o = wg + static_cast<long long>(col) * kC;
+#pragma unroll
+        for (int r = 0; r < 16; ++r) *reinterpret_cast<float4*>(o + 4 * r) = make_float4(x[r], x[r + 16], x[r + 32], x[r + 48]);
+      }
     } else {
 #pragma unroll
-      for (int i = 0; i < kC; ++i) ug[static_cast<long long>(i) * V + (col - D)] = x[i];
+      for (int i = 0; i < kC; ++i) ug[i * u_step + (col - D)] = x[i];
     }
   }
 }
 
-// Block = (VS value columns, head, entry), 8 warps.  Both products split their sum over the warps and meet in `red`: u = u0 - w S over the
-// channels, kd^T u over the tokens; a lane owns rows r, r + 16, r + 32, r + 48 (one 16-byte piece in the layouts the preparation writes) and
-// half of the columns.  With NB = 2 the next chunk's w and kd travel under the whole of this chunk; with NB = 1 (wide heads) kd travels under
+// Block = (VS value columns, head, entry), 16 warps.  Both products split their sum over the warps and meet in `red`: u = u0 - w S over the
+// channels, kd^T u over the tokens; a lane owns two rows, r and r + 16 of its warp's half of 64 (neighbours in
+// the layouts the preparation writes), and half of the columns.  With NB = 2 the next chunk's w and kd travel under the whole of this chunk; with NB = 1 (wide heads) kd travels under
 // the first product and the next chunk's w under the second.
-constexpr int kDcThreads = 256;
+constexpr int kDcThreads = 512;
 
 template <int VS, int NB>
 __global__ void __launch_bounds__(kDcThreads) delta_chunk_scan_kernel(const pcs_delta_chunk_params p) {
   extern __shared__ __align__(16) float sm[];
   constexpr int CW = VS / 2;        // columns of a lane
   constexpr int LV = VS == 8 ? 3 : 4;
-  const int D = p.dim, V = p.vdim, H = p.heads, L = (D + 63) & ~63, NT = L / 64;
+  const int D = p.dim, V = p.vdim, H = p.heads, L = (D + 63) & ~63, NT = L / 64, D8 = (D + 7) & ~7;
   float* ws = sm;                        // [NB][D][64]
   float* kds = ws + NB * D * kC;         // [NB][64][L]
   float* S = kds + NB * kC * L;          // [L][VS]
   float* us = S + L * VS;                // [64][VS]
   float* red = us + kC * VS;             // [8][64][VS]
   const int v0 = blockIdx.x * VS, head = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int r = lane & 15, c4 = (lane >> 4) * CW;
+  const int r = lane & 15, c4 = (lane >> 4) * CW, half = warp & 1, kp = warp >> 1;   // rows half * 32 + {r, r + 16} of 64; one of 8 parts of the sum
   const int n_chunks = p.seq_chunks[b];
   if (n_chunks <= 0) return;
   const long long c0 = p.seq_chunk0[b];
@@ -714,7 +744,7 @@ __global__ void __launch_bounds__(kDcThreads) delta_chunk_scan_kernel(const pcs_
   float* Sg = p.s_pool + (static_cast<long long>(p.seq_slot[b]) * H + head) * D * V;
   const bool fresh = p.seq_pos0[b] == 0;
   auto load_w = [&](int c) {
-    const float* src = p.w + ((c0 + c) * H + head) * D * kC;
+    const float* src = p.w + ((c0 + c) * H + head) * D8 * kC;
     float* dst = ws + (NB == 2 ? (c & 1) * D * kC : 0);
     for (int e = tid; e < D * (kC / 4); e += kDcThreads) cp_async16(dst + e * 4, src + e * 4);
   };
@@ -731,26 +761,39 @@ __global__ void __launch_bounds__(kDcThreads) delta_chunk_scan_kernel(const pcs_
     const int d = e >> LV, c = e & (VS - 1);
     S[e] = (!fresh && d < D && c < vs) ? Sg[static_cast<long long>(d) * V + v0 + c] : 0.f;
   }
-  // phase 1: warp -> channels [d_lo, d_hi); phase 2: warp -> (64-channel tile, part of the tokens)
-  const int dw = (D + 7) / 8, d_lo = min(D, warp * dw), d_hi = min(D, d_lo + dw);
-  const int parts = 8 / NT, tile = warp % NT, part = warp / NT, tw = kC / parts;
+  // phase 1: warp pair -> channels [d_lo, d_hi); phase 2: warp pair -> (64-channel tile, part of the tokens)
+  const int dw = (D + 7) / 8, d_lo = min(D, kp * dw), d_hi = min(D, d_lo + dw);
+  const int parts = 8 / NT, tile = kp % NT, part = kp / NT, tw = kC / parts;
   const int i_lo = part * tw;
   const bool busy2 = part < parts;
   constexpr int kOut1 = kC * VS / kDcThreads;        // outputs of phase 1 per thread
-  constexpr int kOut2 = 256 * VS / kDcThreads;       // of phase 2, at most
-  for (int c = 0; c < n_chunks; ++c) {
-    const long long base = (c0 + c) * H + head;
-    float* ug = p.u + base * kC * V + v0;
-    float u0[kOut1], gd[kOut2];
+  constexpr int kOut2 = 256 * VS / kDcThreads;       // of phase 2, at most (dim 256)
+  float u0[kOut1], gd[kOut2];   // this chunk's right-hand sides and decays; the next chunk's are requested a chunk ahead
+  auto load_u = [&](int c, float (&o)[kOut1]) {
+    const float* src = p.u + ((c0 + c) * H + head) * kC * V + v0;
 #pragma unroll
     for (int m = 0; m < kOut1; ++m) {
       const int e = tid + m * kDcThreads;
-      u0[m] = (e & (VS - 1)) < vs ? ug[static_cast<long long>(e >> LV) * V + (e & (VS - 1))] : 0.f;
+      o[m] = (e & (VS - 1)) < vs ? src[static_cast<long long>(e >> LV) * V + (e & (VS - 1))] : 0.f;
     }
+  };
+  auto load_g = [&](int c, float (&o)[kOut2]) {
+    const float* src = p.g + ((c0 + c) * H + head) * D;
 #pragma unroll
     for (int m = 0; m < kOut2; ++m) {
       const int d = (tid + m * kDcThreads) >> LV;
-      gd[m] = d < D ? p.g[base * D + d] : 0.f;
+      o[m] = d < D ? src[d] : 0.f;
+    }
+  };
+  load_u(0, u0);
+  load_g(0, gd);
+  for (int c = 0; c < n_chunks; ++c) {
+    const long long base = (c0 + c) * H + head;
+    float* ug = p.u + base * kC * V + v0;
+    float un[kOut1], gn[kOut2];
+    if (c + 1 < n_chunks) {
+      load_u(c + 1, un);
+      load_g(c + 1, gn);
     }
     cp_async_wait<1>();
     __syncthreads();   // w of this chunk, and the state; the buffers of the chunk before are free
@@ -762,20 +805,20 @@ __global__ void __launch_bounds__(kDcThreads) delta_chunk_scan_kernel(const pcs_
     }
     {
       const float* wc = ws + (NB == 2 ? (c & 1) * D * kC : 0);
-      float acc[4][CW];
+      float acc[2][CW];
 #pragma unroll
-      for (int x = 0; x < 4; ++x)
+      for (int x = 0; x < 2; ++x)
 #pragma unroll
         for (int y = 0; y < CW; ++y) acc[x][y] = 0.f;
-#pragma unroll 4
+#pragma unroll 8
       for (int d = d_lo; d < d_hi; ++d) {
-        const float4 w4 = *reinterpret_cast<const float4*>(wc + d * kC + 4 * r);
-        const float wv[4] = {w4.x, w4.y, w4.z, w4.w};
+        const float2 w2 = *reinterpret_cast<const float2*>(wc + d * kC + 4 * r + 2 * half);
+        const float wv[2] = {w2.x, w2.y};
 #pragma unroll
         for (int y = 0; y < CW; y += 4) {
           const float4 s4 = *reinterpret_cast<const float4*>(S + d * VS + c4 + y);
 #pragma unroll
-          for (int x = 0; x < 4; ++x) {
+          for (int x = 0; x < 2; ++x) {
             acc[x][y] = fmaf(wv[x], s4.x, acc[x][y]);
             acc[x][y + 1] = fmaf(wv[x], s4.y, acc[x][y + 1]);
             acc[x][y + 2] = fmaf(wv[x], s4.z, acc[x][y + 2]);
@@ -784,10 +827,10 @@ __global__ void __launch_bounds__(kDcThreads) delta_chunk_scan_kernel(const pcs_
         }
       }
 #pragma unroll
-      for (int x = 0; x < 4; ++x)
+      for (int x = 0; x < 2; ++x)
 #pragma unroll
         for (int y = 0; y < CW; y += 4)
-          *reinterpret_cast<float4*>(red + warp * (kC * VS) + (r + 16 * x) * VS + c4 + y) = make_float4(acc[x][y], acc[x][y + 1], acc[x][y + 2], acc[x][y + 3]);
+          *reinterpret_cast<float4*>(red + kp * (kC * VS) + (half * 32 + r + 16 * x) * VS + c4 + y) = make_float4(acc[x][y], acc[x][y + 1], acc[x][y + 2], acc[x][y + 3]);
     }
     __syncthreads();
     if (NB == 1) {
@@ -808,20 +851,20 @@ __global__ void __launch_bounds__(kDcThreads) delta_chunk_scan_kernel(const pcs_
     __syncthreads();   // kd of this chunk, and u; `red` is free again
     if (busy2) {
       const float* kc = kds + (NB == 2 ? (c & 1) * kC * L : 0);
-      float acc[4][CW];
+      float acc[2][CW];
 #pragma unroll
-      for (int x = 0; x < 4; ++x)
+      for (int x = 0; x < 2; ++x)
 #pragma unroll
         for (int y = 0; y < CW; ++y) acc[x][y] = 0.f;
-#pragma unroll 4
+#pragma unroll 8
       for (int i = i_lo; i < i_lo + tw; ++i) {
-        const float4 k4 = *reinterpret_cast<const float4*>(kc + i * L + tile * 64 + 4 * r);
-        const float kv[4] = {k4.x, k4.y, k4.z, k4.w};
+        const float2 k2 = *reinterpret_cast<const float2*>(kc + i * L + tile * 64 + 4 * r + 2 * half);
+        const float kv[2] = {k2.x, k2.y};
 #pragma unroll
         for (int y = 0; y < CW; y += 4) {
           const float4 u4 = *reinterpret_cast<const float4*>(us + i * VS + c4 + y);
 #pragma unroll
-          for (int x = 0; x < 4; ++x) {
+          for (int x = 0; x < 2; ++x) {
             acc[x][y] = fmaf(kv[x], u4.x, acc[x][y]);
             acc[x][y + 1] = fmaf(kv[x], u4.y, acc[x][y + 1]);
             acc[x][y + 2] = fmaf(kv[x], u4.z, acc[x][y + 2]);
@@ -830,10 +873,10 @@ __global__ void __launch_bounds__(kDcThreads) delta_chunk_scan_kernel(const pcs_
         }
       }
 #pragma unroll
-      for (int x = 0; x < 4; ++x)
+      for (int x = 0; x < 2; ++x)
 #pragma unroll
         for (int y = 0; y < CW; y += 4)
-          *reinterpret_cast<float4*>(red + part * (L * VS) + (tile * 64 + r + 16 * x) * VS + c4 + y) = make_float4(acc[x][y], acc[x][y + 1], acc[x][y + 2], acc[x][y + 3]);
+          *reinterpret_cast<float4*>(red + part * (L * VS) + (tile * 64 + half * 32 + r + 16 * x) * VS + c4 + y) = make_float4(acc[x][y], acc[x][y + 1], acc[x][y + 2], acc[x][y + 3]);
     }
     __syncthreads();
     if (NB == 1) {
@@ -852,12 +895,276 @@ __global__ void __launch_bounds__(kDcThreads) delta_chunk_scan_kernel(const pcs_
         if (d < D && cc < vs) sg[static_cast<long long>(d) * V + cc] = old;
         S[e] = fmaf(gd[m], old, a);
       }
+      gd[m] = gn[m];
     }
+#pragma unroll
+    for (int m = 0; m < kOut1; ++m) u0[m] = un[m];
   }
   cp_async_wait<0>();
   __syncthreads();
   for (int e = tid; e < D * VS; e += kDcThreads)
     if ((e & (VS - 1)) < vs) Sg[static_cast<long long>(e >> LV) * V + v0 + (e & (VS - 1))] = S[e];
+}
+
+// The same in bfloat16 runs, the two products on the tensor cores: m16n8k8 with every 32-bit operand split into two TF32 parts, x = hi + lo, and
+// the three products hi hi + hi lo + lo hi in 32-bit accumulators (what is dropped is 2^-22 of a product; states stay 32-bit).  Block = (8 NV
+// value columns, head, entry), 8 warps.  The preparation writes w and kd as fragments, so an operand tile is one 16-byte load per lane.
+//   u = u0 - w S      warp = (16 tokens, half of the channels); the two halves meet in shared memory
+//   S = g S + kd^T u  warp = 16 channels (and 16 more at dim > 128): no sum leaves the warp, S stays in its accumulators
+// S and u also sit in shared memory as [row][8] tiles: a B fragment is 32 neighbouring numbers.
+constexpr int kDtThreads = 256;
+
+__device__ __forceinline__ void mma_tf32(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// hi keeps the sign, the exponent and 10 bits of the fraction; the remainder is exact in 32-bit and its own leading bits are what the unit reads
+__device__ __forceinline__ void split_tf32(float x, uint32_t& hi, uint32_t& lo) {
+  hi = __float_as_uint(x) & 0xffffe000u;
+  lo = __float_as_uint(x - __uint_as_float(hi));
+}
+
+template <int NV, int NB, int MT>   // MT: 16-channel tiles per warp (dim <= 128 MT)
+__global__ void __launch_bounds__(kDtThreads) delta_chunk_scan_tc_kernel(const pcs_delta_chunk_params p) {
+  extern __shared__ __align__(16) float sm[];
+  constexpr int VS = 8 * NV;
+  const int D = p.dim, V = p.vdim, H = p.heads, L = (D + 63) & ~63, D8 = (D + 7) & ~7, KT = D8 / 8;
+  float* ws = sm;                        // [NB][D8 / 8][4][32][4]
+  float* kds = ws + NB * D8 * kC;        // [NB][L / 16][8][32][4]
+  float* S = kds + NB * kC * L;          // [NV][128 MT][8]
+  float* us = S + NV * 128 * MT * 8;     // [NV][64][8]
+  float* red = us + NV * kC * 8;         // [NV][64][8]
+  const int v0 = blockIdx.x * VS, head = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int g = lane >> 2, t = lane & 3;
+  const int n_chunks = p.seq_chunks[b];
+  if (n_chunks <= 0) return;
+  const long long c0 = p.seq_chunk0[b];
+  float* Sg = p.s_pool + (static_cast<long long>(p.seq_slot[b]) * H + head) * D * V;
+  const bool fresh = p.seq_pos0[b] == 0;
+  auto load_w = [&](int c) {
+    const float* src = p.w + ((c0 + c) * H + head) * D8 * kC;
+    float* dst = ws + (NB == 2 ? (c & 1) * D8 * kC : 0);
+    for (int e = tid; e < D8 * (kC / 4); e += kDtThreads) cp_async16(dst + e * 4, src + e * 4);
+  };
+  auto load_kd = [&](int c) {
+    const float* src = p.kd + ((c0 + c) * H + head) * kC * L;
+    float* dst = kds + (NB == 2 ? (c & 1) * kC * L : 0);
+    for (int e = tid; e < kC * (L / 4); e += kDtThreads) cp_async16(dst + e * 4, src + e * 4);
+  };
+  load_w(0);
+  cp_async_commit();
+  load_kd(0);
+  cp_async_commit();
+  // this thread's state: rows 16 (warp + 8 m) + g (+ 8), columns 8 n + 2 t (+ 1)
+  float st[MT][NV][4];
+  const bool even = (V & 1) == 0;
+  auto load2 = [&](const float* row, int col, float& x, float& y) {   // two neighbouring columns of a row, those past vdim zero
+    if (even) {
+      const float2 q = col < V ? *reinterpret_cast<const float2*>(row + col) : make_float2(0.f, 0.f);
+      x = q.x;
+      y = q.y;
+    } else {
+      x = col < V ? row[col] : 0.f;
+      y = col + 1 < V ? row[col + 1] : 0.f;
+    }
+  };
+  auto store2 = [&](float* row, int col, float x, float y) {
+    if (even) {
+      if (col < V) *reinterpret_cast<float2*>(row + col) = make_float2(x, y);
+    } else {
+      if (col < V) row[col] = x;
+      if (col + 1 < V) row[col + 1] = y;
+    }
+  };
+  auto publish = [&]() {
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int n = 0; n < NV; ++n) {
+        float* o = S + (n * 128 * MT + 16 * (warp + 8 * m) + g) * 8 + 2 * t;
+        *reinterpret_cast<float2*>(o) = make_float2(st[m][n][0], st[m][n][1]);
+        *reinterpret_cast<float2*>(o + 64) = make_float2(st[m][n][2], st[m][n][3]);
+      }
+  };
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int n = 0; n < NV; ++n)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int d = 16 * (warp + 8 * m) + g + 8 * h;
+        st[m][n][2 * h] = st[m][n][2 * h + 1] = 0.f;
+        if (!fresh && d < D) load2(Sg + static_cast<long long>(d) * V, v0 + 8 * n + 2 * t, st[m][n][2 * h], st[m][n][2 * h + 1]);
+      }
+  publish();
+  const int mi = warp & 3, kh = warp >> 2, kt_lo = kh ? (KT + 1) / 2 : 0, kt_hi = kh ? KT : (KT + 1) / 2;
+  float u0[NV][4], gd[MT][2], un[NV][4], gn[MT][2];
+  auto load_u = [&](int c, float (&o)[NV][4]) {
+    if (kh != 0) return;
+    const float* src = p.u + ((c0 + c) * H + head) * kC * V;
+#pragma unroll
+    for (int n = 0; n < NV; ++n)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) load2(src + static_cast<long long>(16 * mi + g + 8 * h) * V, v0 + 8 * n + 2 * t, o[n][2 * h], o[n][2 * h + 1]);
+  };
+  auto load_g = [&](int c, float (&o)[MT][2]) {
+    const float* src = p.g + ((c0 + c) * H + head) * D;
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int d = 16 * (warp + 8 * m) + g + 8 * h;
+        o[m][h] = d < D ? src[d] : 0.f;
+      }
+  };
+  load_u(0, u0);
+  load_g(0, gd);
+  // one k-step: the A fragment against every column tile; three accumulators per tile, so that a chain is one product per step
+  auto step = [&](const float* af, const float* bt, int b_tile, float (&hh)[NV][4], float (&hl)[NV][4], float (&lh)[NV][4]) {
+    const float4 a4 = *reinterpret_cast<const float4*>(af + lane * 4);
+    uint32_t ah[4], al[4];
+    split_tf32(a4.x, ah[0], al[0]);
+    split_tf32(a4.y, ah[1], al[1]);
+    split_tf32(a4.z, ah[2], al[2]);
+    split_tf32(a4.w, ah[3], al[3]);
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      uint32_t h0, l0, h1, l1;
+      split_tf32(bt[n * b_tile + t * 8 + g], h0, l0);
+      split_tf32(bt[n * b_tile + 32 + t * 8 + g], h1, l1);
+      mma_tf32(hh[n], ah, h0, h1);
+      mma_tf32(hl[n], ah, l0, l1);
+      mma_tf32(lh[n], al, h0, h1);
+    }
+  };
+  for (int c = 0; c < n_chunks; ++c) {
+    const long long base = (c0 + c) * H + head;
+    if (c + 1 < n_chunks) {
+      load_u(c + 1, un);
+      load_g(c + 1, gn);
+    }
+    cp_async_wait<1>();
+    __syncthreads();   // w of this chunk, and the state; the buffers of the chunk before are free
+    if (NB == 2) {
+      if (c + 1 < n_chunks) load_w(c + 1);
+      cp_async_commit();
+      if (c + 1 < n_chunks) load_kd(c + 1);
+      cp_async_commit();
+    }
+    float hh[NV][4], hl[NV][4], lh[NV][4];
+    auto zero = [&](float (&x)[NV][4]) {
+#pragma unroll
+      for (int n = 0; n < NV; ++n) x[n][0] = x[n][1] = x[n][2] = x[n][3] = 0.f;
+    };
+    zero(hh);
+    zero(hl);
+    zero(lh);
+    {
+      const float* wc = ws + (NB == 2 ? (c & 1) * D8 * kC : 0) + mi * 128;
+#pragma unroll 4
+      for (int kt = kt_lo; kt < kt_hi; ++kt) step(wc + kt * 512, S + kt * 64, 128 * MT * 8, hh, hl, lh);
+    }
+#pragma unroll
+    for (int n = 0; n < NV; ++n)
+#pragma unroll
+      for (int x = 0; x < 4; ++x) hh[n][x] += hl[n][x] + lh[n][x];
+    if (kh == 1) {
+#pragma unroll
+      for (int n = 0; n < NV; ++n) {
+        float* o = red + (n * kC + 16 * mi + g) * 8 + 2 * t;
+        *reinterpret_cast<float2*>(o) = make_float2(hh[n][0], hh[n][1]);
+        *reinterpret_cast<float2*>(o + 64) = make_float2(hh[n][2], hh[n][3]);
+      }
+    }
+    __syncthreads();
+    if (NB == 1) {
+      if (c + 1 < n_chunks) load_w(c + 1);
+      cp_async_commit();
+    }
+    if (kh == 0) {
+      float* ug = p.u + base * kC * V;
+#pragma unroll
+      for (int n = 0; n < NV; ++n)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int i = 16 * mi + g + 8 * h, o = (n * kC + i) * 8 + 2 * t;
+          const float2 r2 = *reinterpret_cast<const float2*>(red + o);
+          const float x = u0[n][2 * h] - (hh[n][2 * h] + r2.x), y = u0[n][2 * h + 1] - (hh[n][2 * h + 1] + r2.y);
+          *reinterpret_cast<float2*>(us + o) = make_float2(x, y);
+          store2(ug + static_cast<long long>(i) * V, v0 + 8 * n + 2 * t, x, y);
+        }
+    }
+    cp_async_wait<NB>();
+    __syncthreads();   // kd of this chunk, and u
+    float* sg = p.s + base * D * V;
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      const int mt = warp + 8 * m;
+      if (16 * mt < D) {
+#pragma unroll
+        for (int n = 0; n < NV; ++n)
+#pragma unroll
+          for (int h = 0; h < 2; ++h) {
+            const int d = 16 * mt + g + 8 * h;
+            if (d < D) store2(sg + static_cast<long long>(d) * V, v0 + 8 * n + 2 * t, st[m][n][2 * h], st[m][n][2 * h + 1]);   // the state this chunk starts from
+          }
+        zero(hh);
+        zero(hl);
+        zero(lh);
+        const float* kc = kds + (NB == 2 ? (c & 1) * kC * L : 0) + mt * 1024;
+#pragma unroll
+        for (int kt = 0; kt < 8; ++kt) step(kc + kt * 128, us + kt * 64, kC * 8, hh, hl, lh);
+#pragma unroll
+        for (int n = 0; n < NV; ++n)
+#pragma unroll
+          for (int x = 0; x < 4; ++x) st[m][n][x] = fmaf(gd[m][x >> 1], st[m][n][x], hh[n][x] + (hl[n][x] + lh[n][x]));
+      }
+#pragma unroll
+      for (int h = 0; h < 2; ++h) gd[m][h] = gn[m][h];
+    }
+    publish();
+#pragma unroll
+    for (int n = 0; n < NV; ++n)
+#pragma unroll
+      for (int x = 0; x < 4; ++x) u0[n][x] = un[n][x];
+    if (NB == 1) {
+      __syncthreads();   // every warp has read this chunk's kd
+      if (c + 1 < n_chunks) load_kd(c + 1);
+      cp_async_commit();
+    }
+  }
+  cp_async_wait<0>();
+#pragma unroll
+  for (int m = 0; m < MT; ++m)
+#pragma unroll
+    for (int n = 0; n < NV; ++n)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int d = 16 * (warp + 8 * m) + g + 8 * h;
+        if (d < D) store2(Sg + static_cast<long long>(d) * V, v0 + 8 * n + 2 * t, st[m][n][2 * h], st[m][n][2 * h + 1]);
+      }
+}
+
+template <int NV, int NB, int MT>
+static int launch_delta_chunk_scan_tc(const pcs_delta_chunk_params& p, size_t smem, cudaStream_t st) {
+  PCS_CHECK_CUDA(cudaFuncSetAttribute(delta_chunk_scan_tc_kernel<NV, NB, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024));
+  delta_chunk_scan_tc_kernel<NV, NB, MT><<<dim3((p.vdim + 8 * NV - 1) / (8 * NV), p.heads, p.n_seqs), kDtThreads, smem, st>>>(p);
+  PCS_CHECK_CUDA(cudaGetLastError());
+  count_launch();
+  return PCS_OK;
+}
+
+template <int MT>
+static int launch_delta_chunk_scan_tc(const pcs_delta_chunk_params& p, cudaStream_t st) {
+  const int L = (p.dim + 63) & ~63, D8 = (p.dim + 7) & ~7;
+  auto smem = [&](int nv, int nb) { return (static_cast<size_t>(nb) * kC * (D8 + L) + static_cast<size_t>(nv) * 8 * (128 * MT + 2 * kC)) * sizeof(float); };
+  // 8 columns per block where that still is one block per SM, else 16 (half of the chunk traffic); two buffers where they fit
+  const long long rows = static_cast<long long>(p.heads) * p.n_seqs;
+  const int nv = rows * ((p.vdim + 7) / 8) <= 148 ? 1 : 2;
+  const bool one_wave = rows * ((p.vdim + 8 * nv - 1) / (8 * nv)) <= 148;
+  const bool two = smem(nv, 2) <= (one_wave ? 227u : 112u) * 1024u;
+  if (nv == 1) return two ? launch_delta_chunk_scan_tc<1, 2, MT>(p, smem(1, 2), st) : launch_delta_chunk_scan_tc<1, 1, MT>(p, smem(1, 1), st);
+  return two ? launch_delta_chunk_scan_tc<2, 2, MT>(p, smem(2, 2), st) : launch_delta_chunk_scan_tc<2, 1, MT>(p, smem(2, 1), st);
 }
 
 template <int VS, int NB>
@@ -1008,6 +1315,7 @@ PCS_API int pcs_delta_chunk_scan(const pcs_delta_chunk_params* p, void* stream) 
   PCS_REQUIRE(((reinterpret_cast<uintptr_t>(p->kd) | reinterpret_cast<uintptr_t>(p->w)) & 15) == 0, "pcs_delta_chunk_scan: kd and w must be 16-byte aligned");
   const int L = (p->dim + 63) & ~63;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (p->dtype == PCS_BF16) return p->dim <= 128 ? pcs::launch_delta_chunk_scan_tc<1>(*p, st) : pcs::launch_delta_chunk_scan_tc<2>(*p, st);
   auto smem = [&](int vs, int nb) {
     return (static_cast<size_t>(nb) * (p->dim * pcs::kC + pcs::kC * L) + static_cast<size_t>(vs) * (L + pcs::kC + 8 * pcs::kC)) * sizeof(float);
   };
