@@ -83,7 +83,7 @@ template <typename T, int TB, int R>
 __device__ __forceinline__ void short_conv_tile(const pcs_shortconv_params& p, int CB) {
   constexpr int N = Vec<T>::n, RN = TB + R;
   __shared__ float ssq[TB][256];
-  const int t0 = blockIdx.x * TB, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;   // (warp, lane: shared-memory sums)
+  const int t0 = blockIdx.x * TB, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int D = p.dim, U = 2 * p.kv_heads * D, C = U + p.v_width;
   const int c_lo = blockIdx.y * CB, c = c_lo + tid * N;
   const bool active = tid * N < CB && c < C;

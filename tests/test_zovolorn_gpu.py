@@ -633,14 +633,9 @@ def test_medium_model_long_prompt(tmp_path):
                          P(heads=2, kv_heads=1, dim=128, chunk=512, bias_max=300, buckets=32, r_heads=8, r_kv_heads=4, r_dim=32, r_vdim=32, ff=0)], width=192, vocab=300, groups=6,
                         embed_scale=4.0)
     W = O.random_model(cfg, seed=21)
-    from functools import lru_cache
-    plain, O.distance_bucket = O.distance_bucket, lru_cache(None)(O.distance_bucket)
-    try:
-        toks = tokens(1320, 300, 4)
-        rows = sorted(list(range(0, 1300, 97)) + [399, 400, 511, 512, 1023, 1024, 1297, 1298, 1299])
-        want = O.forward(cfg, W, toks)
-    finally:
-        O.distance_bucket = plain
+    toks = tokens(1320, 300, 4)
+    rows = sorted(list(range(0, 1300, 97)) + [399, 400, 511, 512, 1023, 1024, 1297, 1298, 1299])
+    want = O.forward(cfg, W, toks)
     for dtype in (F32, BF16):
         m = load(tmp_path, cfg, W, dtype, str(dtype)[-4:])
         for cuts in ([1300], [700, 600]):

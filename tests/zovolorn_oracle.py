@@ -102,14 +102,17 @@ def softmax_attention(q, k, v, pos_q, pos_k, scale, sink=None, temp=None, rel=No
     seen = d >= 0
     if chunk:
         seen = seen & (pos_q[:, None] // chunk == pos_k[None, :] // chunk)
+    bucket = None
+    if rel is not None:
+        of = torch.tensor([distance_bucket(n, rel.shape[0], bias_max) for n in range(int(d.max()) + 1)])
+        bucket = of[d.clamp(min=0)]
     out = []
     for h in range(H):
         s = q[:, h] @ k[:, h // rep].T * scale
         if temp is not None:
             s = s * temp[h]
         if rel is not None:
-            b = torch.tensor([[distance_bucket(max(int(n), 0), rel.shape[0], bias_max) for n in row] for row in d])
-            s = s + rel[b, h]
+            s = s + rel[bucket, h]
         s = s.masked_fill(~seen, -float("inf"))
         m = s.max(-1, keepdim=True).values
         if sink is not None:
