@@ -395,7 +395,8 @@ int pcs_depth_mix(const pcs_depthmix_params* p, void* stream);
  * followed by the key part that is rotated (kv_rank + rot_dim numbers at ckv_off).
  *   cq_out[t]                       = rms(query latent) * cq_norm_w                              [n_tokens, q_rank]
  *   pool[slot, pos, 0:kv_rank]      = rms(key/value latent) * ckv_norm_w
- *   pool[slot, pos, kv_rank: ...]   = the rotated part turned by pos (pairs (i, i + rot_dim/2), cos and sin times rot_mult)
+ *   pool[slot, pos, kv_rank: ...]   = the rotated part turned by pos (pairs (i, i + rot_dim/2), or (2i, 2i + 1) with `interleaved`; cos and
+ *                                     sin times rot_mult)
  * pool is [slots, cap, kv_rank + rot_dim]. */
 typedef struct pcs_latent_prep_params {
   const void* proj;
@@ -413,6 +414,7 @@ typedef struct pcs_latent_prep_params {
   const int32_t* tok_pos;
   const int32_t* seq_slot;
   int32_t n_tokens, dtype;
+  int32_t interleaved, reserved;
 } pcs_latent_prep_params;
 int pcs_latent_prep(const pcs_latent_prep_params* p, void* stream);
 
@@ -420,7 +422,8 @@ int pcs_latent_prep(const pcs_latent_prep_params* p, void* stream);
  *   q_lat == NULL:  the rotated part of every head is turned by the token's position in place (q_out == q) or into q_out
  *                   (same layout, plain part copied).
  *   q_lat != NULL:  q_out [n_tokens, H * (kv_rank + rot_dim)] gets per head [q_lat[t, h, :] | rotated part], where
- *                   q_lat[t, h, c] sits at q_lat + t * lat_tok_stride + h * lat_head_stride + c. */
+ *                   q_lat[t, h, c] sits at q_lat + t * lat_tok_stride + h * lat_head_stride + c.  q_lat == q_out: already in its place.
+ *   The rotated part pairs (i, i + rot_dim / 2), or neighbours (2i, 2i + 1) with `interleaved`. */
 typedef struct pcs_latent_q_params {
   const void* q;
   void* q_out;
@@ -431,13 +434,15 @@ typedef struct pcs_latent_q_params {
   float rot_mult;
   const int32_t* tok_pos;
   int32_t n_tokens, dtype;
+  int32_t interleaved, reserved;
 } pcs_latent_q_params;
 int pcs_latent_q(const pcs_latent_q_params* p, void* stream);
 
 /* Per-head rows for attention over expanded keys and values.  kv [n_ctx, H * (dim + vdim)]: for context token n (entry
  * ctx_seq[n], position ctx_pos[n]) the plain key parts of all heads, then the values of all heads.
  *   k_dense[b, h, pos, :] = [kv[n, h * dim ...] | pool[seq_slot[b], pos, kv_rank : kv_rank + rot_dim]]     [B, H, cap_dense, dim + rot_dim]
- *   v_dense[b, h, pos, :] = kv[n, H * dim + h * vdim ...]                                                   [B, H, cap_dense, vdim] */
+ *   v_dense[b, h, pos, :] = kv[n, H * dim + h * vdim ...]                                                   [B, H, cap_dense, vdim]
+ * With seq_base the dense rows of entry b count from position seq_base[b] (a window's context starts there). */
 typedef struct pcs_latent_expand_params {
   const void* kv;
   int64_t kv_stride;
@@ -450,6 +455,7 @@ typedef struct pcs_latent_expand_params {
   const int32_t* ctx_pos;
   const int32_t* seq_slot;
   int32_t n_ctx, dtype;
+  const int32_t* seq_base;  /* [entries] or NULL */
 } pcs_latent_expand_params;
 int pcs_latent_expand(const pcs_latent_expand_params* p, void* stream);
 
@@ -491,10 +497,13 @@ typedef struct pcs_gla_params {
 } pcs_gla_params;
 int pcs_gla_scan(const pcs_gla_params* p, void* stream);
 
-/* Residual sum and layer norm (weight, no bias) of the 32-bit stream.  Per row r (row(r) = rows ? rows[r] : r):
- *   x[row, :] += sum_i y_mult[i] * y[i][row, :]          (n_addends <= 3 sublayer results, `dtype` or fp32; not with `rows`)
+/* Residual sum and norm (weight, no bias) of the 32-bit stream.  Per row r (row(r) = rows ? rows[r] : r):
+ *   x[row, :] += sum_i y_mult[i] * y[i][row, :]          (n_addends <= 3 sublayer results, `dtype` or fp32; not with `rows`; a row
+ *                                                         stride of 0 adds one vector to every row)
  *   mu = mean(x[row]), var = mean((x[row] - mu)^2)        (two passes over the row, 32-bit)
- *   h1[r, :] = (x[row] - mu) / sqrt(var + eps) * w1;  h2[r, :] likewise with w2   (each may be NULL) */
+ *   h1[r, :] = (x[row] - mu) / sqrt(var + eps) * w1;  h2[r, :] likewise with w2   (each may be NULL)
+ * rms 1: h1[r, :] = x[row] / sqrt(mean(x[row]^2) + eps) * (w_offset + w1), h2 likewise.
+ * y_norm_w: addend 0 enters as y / sqrt(mean(y^2) + eps) * y_norm_w.  copy: the new x[row] in `dtype` (not with `rows`). */
 typedef struct pcs_addln_params {
   float* x;                 /* [*, width] */
   const int32_t* rows;      /* [n_rows] or NULL */
@@ -510,8 +519,17 @@ typedef struct pcs_addln_params {
   int32_t n_rows, width;
   float eps;
   int32_t dtype;
+  int32_t rms;              /* 0: layer norm, 1: RMS norm */
+  float w_offset;           /* with rms: added to w1 and w2 */
+  const void* y_norm_w;     /* [width] `dtype` or NULL */
+  void* copy;               /* [n_rows, width] `dtype` or NULL */
 } pcs_addln_params;
 int pcs_add_layer_norm(const pcs_addln_params* p, void* stream);
+
+/* The gated token-side input: out[t, c] = gelu(u[t, c]) * table[ids[t], col + c] with the tanh form of gelu, c < dim   (out `dtype` [n_tokens, dim];
+ * table `dtype` [vocab, table_stride], ids outside [0, vocab) read row 0) */
+int pcs_side_gate(const void* u, int64_t u_stride, const void* table, int64_t table_stride, int vocab, int col, const int64_t* ids, void* out,
+                  int n_tokens, int dim, int dtype, void* stream);
 
 /* Element-wise gated recurrence whose gates read only the current token (no dependence on the state).  Per entry and channel c:
  *   z_t = sigmoid(proj[t, z_off + c]),  u_t = proj[t, x_off + c],  cand_t = u_t >= 0 ? u_t + 1/2 : sigmoid(u_t)
@@ -612,6 +630,7 @@ int pcs_delta_inputs(const pcs_shortconv_params* p, const pcs_lowrank_params* q,
 
 /* Gated delta rule, token by token.  Per entry and head h (query / key head h / (heads / kv_heads)):
  *   S <- diag(decay_t) S;  u = sigmoid(b[t, h]) * (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t
+ * decay NULL: one decay per head, exp(-rate[h] * softplus(a[t, h] + dt_bias[h])), formed in 32-bit inside the kernel.
  * S is fp32 [slots, heads, dim, vdim] in the slot pool; an entry whose slot holds no tokens starts from zero. */
 typedef struct pcs_delta_params {
   const float* qk;          /* [n_tokens, 2 * kv_heads * dim]: queries, then keys (already normed and scaled) */
@@ -628,6 +647,10 @@ typedef struct pcs_delta_params {
   const int32_t* seq_off;
   int32_t n_seqs, n_tokens, dtype;
   int32_t impl;             /* 0 = automatic, 1 = the kernel with the state in shared memory */
+  const void* a;            /* [n_tokens, a_stride] `dtype`: the pre-activations of per-head decays (decay NULL) */
+  int64_t a_stride;
+  const float* dt_bias;     /* [heads] */
+  const float* rate;        /* [heads] */
 } pcs_delta_params;
 int pcs_delta_scan(const pcs_delta_params* p, void* stream);
 
@@ -640,7 +663,8 @@ int pcs_delta_scan(const pcs_delta_params* p, void* stream);
  *                          kd[i][64 t + 4 r + n] for channel 64 t + r + 16 n
  *                          u[c, h, i, :]  = row i of M^-1 diag(beta) V                    (every exponent formed is <= 0)
  *   pcs_delta_chunk_scan   per entry, over its chunks in order, S from the pool:  u[c] <- u[c] - w[c] S;  s[c] = S;  S <- g S + kd[c]^T u[c]
- *   (the caller forms o[c, h] = qd[c, h] s[c, h] + a[c, h] u[c, h], fp32 [chunks, heads, 64, vdim]) */
+ *   (the caller forms o[c, h] = qd[c, h] s[c, h] + a[c, h] u[c, h], fp32 [chunks, heads, 64, vdim])
+ * ld NULL: one decay per head, as in pcs_delta_scan; the sums over pairs are then plain products scaled pair by pair. */
 #define PCS_DELTA_CHUNK 64
 typedef struct pcs_delta_chunk_params {
   const float* qk;
@@ -664,12 +688,17 @@ typedef struct pcs_delta_chunk_params {
   const int32_t* seq_pos0;
   const int32_t* seq_chunk0;   /* [n_seqs] first chunk of the entry */
   const int32_t* seq_chunks;   /* [n_seqs] number of its chunks */
+  const void* dec_a;           /* [n_tokens, dec_stride] `dtype`: the pre-activations of per-head decays (ld NULL) */
+  int64_t dec_stride;
+  const float* dt_bias;        /* [heads] */
+  const float* rate;           /* [heads] */
 } pcs_delta_chunk_params;
 int pcs_delta_chunk_prep(const pcs_delta_chunk_params* p, void* stream);
 int pcs_delta_chunk_scan(const pcs_delta_chunk_params* p, void* stream);
 
 /* out[t * out_stride + h * vdim + c] = o / sqrt(mean_c(o^2) + eps) * w[c] * sigmoid(g[t * g_stride + h * vdim + c]) * out_scale, o fp32: row
- * (t, h) of [n_tokens, heads, vdim], or with tok_row (token -> chunk * chunk_size + place) of [chunks, heads, chunk_size, vdim] */
+ * (t, h) of [n_tokens, heads, vdim], or with tok_row (token -> chunk * chunk_size + place) of [chunks, heads, chunk_size, vdim];
+ * with `silu` the gate is silu(g) instead of sigmoid(g) */
 typedef struct pcs_headnorm_params {
   const float* o;
   const int32_t* tok_row;   /* [n_tokens] or NULL */
@@ -680,7 +709,7 @@ typedef struct pcs_headnorm_params {
   int64_t out_stride;
   int32_t n_tokens, heads, vdim, chunk_size;
   float eps, out_scale;
-  int32_t dtype, reserved;
+  int32_t dtype, silu;
 } pcs_headnorm_params;
 int pcs_head_norm_gate(const pcs_headnorm_params* p, void* stream);
 

@@ -21,7 +21,7 @@ EXPORTS = ("pcs_version", "pcs_last_error", "pcs_launch_count", "pcs_attn_worksp
            "pcs_moe_rows_up", "pcs_moe_rows_down", "pcs_moe_plan", "pcs_moe_gather", "pcs_moe_gemm", "pcs_moe_combine", "pcs_silu_mul", "pcs_glu_mul",
            "pcs_depth_mix", "pcs_latent_prep", "pcs_latent_q", "pcs_latent_gather", "pcs_latent_expand", "pcs_head_gate", "pcs_gla_decay", "pcs_gla_scan", "pcs_gla_chunk_prep", "pcs_gla_chunk_scan", "pcs_gla_chunk_out",
            "pcs_add_layer_norm", "pcs_gru_scan", "pcs_group_norm_conv", "pcs_soft_cap", "pcs_short_conv", "pcs_delta_inputs", "pcs_delta_scan", "pcs_delta_chunk_prep", "pcs_delta_chunk_scan",
-           "pcs_head_norm_gate")
+           "pcs_head_norm_gate", "pcs_side_gate")
 GLU_SILU, GLU_CLAMPED_SWISH, GLU_GELU_TANH = 0, 1, 4
 ACT_RELU2, ACT_GELU_ERF = 2, 3          # activations of a feed-forward without a gate branch
 ROUTE_SOFTMAX, ROUTE_SIGMOID = 0, 1
@@ -99,20 +99,21 @@ class pcs_latent_prep_params(C.Structure):
     _fields_ = [("proj", C.c_void_p), ("row_stride", C.c_int64), ("cq_off", C.c_int32), ("ckv_off", C.c_int32), ("q_rank", C.c_int32),
                 ("kv_rank", C.c_int32), ("rot_dim", C.c_int32), ("cq_norm_w", C.c_void_p), ("ckv_norm_w", C.c_void_p), ("eps", C.c_float),
                 ("freqs", C.c_void_p), ("rot_mult", C.c_float), ("cq_out", C.c_void_p), ("pool", C.c_void_p), ("cap", C.c_int32),
-                ("tok_seq", C.c_void_p), ("tok_pos", C.c_void_p), ("seq_slot", C.c_void_p), ("n_tokens", C.c_int32), ("dtype", C.c_int32)]
+                ("tok_seq", C.c_void_p), ("tok_pos", C.c_void_p), ("seq_slot", C.c_void_p), ("n_tokens", C.c_int32), ("dtype", C.c_int32),
+                ("interleaved", C.c_int32), ("reserved", C.c_int32)]
 
 
 class pcs_latent_q_params(C.Structure):
     _fields_ = [("q", C.c_void_p), ("q_out", C.c_void_p), ("q_lat", C.c_void_p), ("lat_tok_stride", C.c_int64), ("lat_head_stride", C.c_int64),
                 ("n_heads", C.c_int32), ("dim", C.c_int32), ("rot_dim", C.c_int32), ("kv_rank", C.c_int32), ("freqs", C.c_void_p),
-                ("rot_mult", C.c_float), ("tok_pos", C.c_void_p), ("n_tokens", C.c_int32), ("dtype", C.c_int32)]
+                ("rot_mult", C.c_float), ("tok_pos", C.c_void_p), ("n_tokens", C.c_int32), ("dtype", C.c_int32), ("interleaved", C.c_int32), ("reserved", C.c_int32)]
 
 
 class pcs_latent_expand_params(C.Structure):
     _fields_ = [("kv", C.c_void_p), ("kv_stride", C.c_int64), ("pool", C.c_void_p), ("cap", C.c_int32), ("kv_rank", C.c_int32),
                 ("rot_dim", C.c_int32), ("n_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("k_dense", C.c_void_p),
                 ("v_dense", C.c_void_p), ("cap_dense", C.c_int32), ("ctx_seq", C.c_void_p), ("ctx_pos", C.c_void_p), ("seq_slot", C.c_void_p),
-                ("n_ctx", C.c_int32), ("dtype", C.c_int32)]
+                ("n_ctx", C.c_int32), ("dtype", C.c_int32), ("seq_base", C.c_void_p)]
 
 
 class pcs_gla_params(C.Structure):
@@ -142,7 +143,8 @@ class pcs_combine_params(C.Structure):
 class pcs_addln_params(C.Structure):
     _fields_ = [("x", C.c_void_p), ("rows", C.c_void_p), ("y", C.c_void_p * 3), ("y_stride", C.c_int64 * 3), ("y_mult", C.c_float * 3),
                 ("y_f32", C.c_int32 * 3), ("n_addends", C.c_int32), ("w1", C.c_void_p), ("h1", C.c_void_p), ("w2", C.c_void_p), ("h2", C.c_void_p),
-                ("n_rows", C.c_int32), ("width", C.c_int32), ("eps", C.c_float), ("dtype", C.c_int32)]
+                ("n_rows", C.c_int32), ("width", C.c_int32), ("eps", C.c_float), ("dtype", C.c_int32), ("rms", C.c_int32), ("w_offset", C.c_float),
+                ("y_norm_w", C.c_void_p), ("copy", C.c_void_p)]
 
 
 class pcs_gru_params(C.Structure):
@@ -174,7 +176,8 @@ class pcs_lowrank_params(C.Structure):
 class pcs_delta_params(C.Structure):
     _fields_ = [("qk", C.c_void_p), ("v", C.c_void_p), ("decay", C.c_void_p), ("b", C.c_void_p), ("b_stride", C.c_int64), ("o", C.c_void_p), ("s_pool", C.c_void_p),
                 ("heads", C.c_int32), ("kv_heads", C.c_int32), ("dim", C.c_int32), ("vdim", C.c_int32), ("seq_slot", C.c_void_p), ("seq_pos0", C.c_void_p),
-                ("seq_len", C.c_void_p), ("seq_off", C.c_void_p), ("n_seqs", C.c_int32), ("n_tokens", C.c_int32), ("dtype", C.c_int32), ("impl", C.c_int32)]
+                ("seq_len", C.c_void_p), ("seq_off", C.c_void_p), ("n_seqs", C.c_int32), ("n_tokens", C.c_int32), ("dtype", C.c_int32), ("impl", C.c_int32),
+                ("a", C.c_void_p), ("a_stride", C.c_int64), ("dt_bias", C.c_void_p), ("rate", C.c_void_p)]
 
 
 class pcs_delta_chunk_params(C.Structure):
@@ -182,13 +185,13 @@ class pcs_delta_chunk_params(C.Structure):
                 ("dim", C.c_int32), ("vdim", C.c_int32), ("chunk_first", C.c_void_p), ("chunk_len", C.c_void_p), ("n_chunks", C.c_int32), ("n_tokens", C.c_int32),
                 ("dtype", C.c_int32), ("n_seqs", C.c_int32), ("qd", C.c_void_p), ("kd", C.c_void_p), ("w", C.c_void_p), ("g", C.c_void_p), ("u", C.c_void_p),
                 ("a", C.c_void_p), ("s", C.c_void_p), ("s_pool", C.c_void_p), ("seq_slot", C.c_void_p), ("seq_pos0", C.c_void_p), ("seq_chunk0", C.c_void_p),
-                ("seq_chunks", C.c_void_p)]
+                ("seq_chunks", C.c_void_p), ("dec_a", C.c_void_p), ("dec_stride", C.c_int64), ("dt_bias", C.c_void_p), ("rate", C.c_void_p)]
 
 
 class pcs_headnorm_params(C.Structure):
     _fields_ = [("o", C.c_void_p), ("tok_row", C.c_void_p), ("w", C.c_void_p), ("g", C.c_void_p), ("g_stride", C.c_int64), ("out", C.c_void_p), ("out_stride", C.c_int64),
                 ("n_tokens", C.c_int32), ("heads", C.c_int32), ("vdim", C.c_int32), ("chunk_size", C.c_int32), ("eps", C.c_float), ("out_scale", C.c_float),
-                ("dtype", C.c_int32), ("reserved", C.c_int32)]
+                ("dtype", C.c_int32), ("silu", C.c_int32)]
 
 
 class pcs_mlstm_params(C.Structure):
@@ -274,6 +277,7 @@ def load() -> C.CDLL:
     for name in ("pcs_delta_chunk_prep", "pcs_delta_chunk_scan"):
         getattr(lib, name).argtypes = [C.POINTER(pcs_delta_chunk_params), C.c_void_p]
     lib.pcs_head_norm_gate.argtypes = [C.POINTER(pcs_headnorm_params), C.c_void_p]
+    lib.pcs_side_gate.argtypes = [C.c_void_p, C.c_int64, C.c_void_p, C.c_int64, C.c_int, C.c_int, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_void_p]
     for name in EXPORTS[4:]:
         getattr(lib, name).restype = C.c_int
     _lib = lib
@@ -336,6 +340,7 @@ class Batch:
         m = self.meta
         self.tok_seq, self.tok_pos = m[0:T], m[T:2 * T]
         self.seq_slot, self.seq_pos0, self.seq_len, self.seq_off, self.seq_par = (m[2 * T + i * B:2 * T + (i + 1) * B] for i in range(5))
+        self.wants_all = False  # the logits of every token are asked for, in order
         self.prev_ids = None  # int64 [T] on the device: every token's predecessor in its sequence, -1 for a first token
         self.n_tokens, self.n_seqs, self.max_len = T, B, max(lens) if lens else 0
         self.offsets, self.lens, self.pos0, self.slots = offs, list(lens), list(pos0), list(slots)
@@ -815,8 +820,9 @@ def depth_mix(xs: torch.Tensor, n_terms: int, coef: torch.Tensor, eps: float, x_
 
 def latent_prep(proj: torch.Tensor, cq_off: int, ckv_off: int, q_rank: int, kv_rank: int, rot_dim: int, cq_norm_w: Optional[torch.Tensor],
                 ckv_norm_w: torch.Tensor, eps: float, freqs: Optional[torch.Tensor], rot_mult: float, cq_out: Optional[torch.Tensor], pool: torch.Tensor,
-                batch: Batch) -> None:
-    """proj [T, *]: the query latent at cq_off, [key/value latent | rotated key part] at ckv_off; pool [slots, 1, cap, kv_rank + rot_dim]."""
+                batch: Batch, interleaved: bool = False) -> None:
+    """proj [T, *]: the query latent at cq_off, [key/value latent | rotated key part] at ckv_off; pool [slots, 1, cap, kv_rank + rot_dim].
+    The rotation pairs coordinates half a part apart, or neighbours (`interleaved`)."""
     _cuda(proj, cq_norm_w, ckv_norm_w, freqs, cq_out, pool)
     dt = proj.dtype
     _rows2d(proj, dt, "latent_prep: proj")
@@ -831,30 +837,35 @@ def latent_prep(proj: torch.Tensor, cq_off: int, ckv_off: int, q_rank: int, kv_r
     p.q_rank, p.kv_rank, p.rot_dim, p.cq_norm_w, p.ckv_norm_w, p.eps = int(q_rank), int(kv_rank), int(rot_dim), _ptr(cq_norm_w), ckv_norm_w.data_ptr(), float(eps)
     p.freqs, p.rot_mult, p.cq_out, p.pool, p.cap = _ptr(freqs), float(rot_mult), _ptr(cq_out), pool.data_ptr(), pool.shape[2]
     p.tok_seq, p.tok_pos, p.seq_slot = batch.tok_seq.data_ptr(), batch.tok_pos.data_ptr(), batch.seq_slot.data_ptr()
-    p.n_tokens, p.dtype = batch.n_tokens, dtype_code(dt)
+    p.n_tokens, p.dtype, p.interleaved = batch.n_tokens, dtype_code(dt), 1 if interleaved else 0
     _check(load().pcs_latent_prep(C.byref(p), _stream()), "pcs_latent_prep")
 
 
 def latent_q(q: torch.Tensor, n_heads: int, dim: int, rot_dim: int, freqs: Optional[torch.Tensor], rot_mult: float, batch: Batch,
-             q_lat: Optional[torch.Tensor] = None) -> torch.Tensor:
+             q_lat: Optional[torch.Tensor] = None, interleaved: bool = False, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """q [T, H * (dim + rot_dim)]: every head's rotated part is turned by the token's position.  Without q_lat in place (q is
     returned); with q_lat [T, H, kv_rank] (any strides, contiguous last dimension) a new [T, H * (kv_rank + rot_dim)] matrix of
-    [q_lat | rotated part] per head is returned."""
+    [q_lat | rotated part] per head is returned.  `out`: that matrix; where q_lat already is its columns, only the rotated parts are written."""
     _cuda(q, freqs, q_lat)
     dt = q.dtype
     if not q.is_contiguous() or q.dim() != 2 or q.shape[1] != n_heads * (dim + rot_dim):
         raise NativeError("latent_q: q must be contiguous [T, H * (dim + rot_dim)]")
     p = pcs_latent_q_params()
-    out = q
+    res = q
     if q_lat is not None:
         if q_lat.dtype != dt or q_lat.dim() != 3 or q_lat.stride(2) != 1 or q_lat.shape[0] != q.shape[0] or q_lat.shape[1] != n_heads:
             raise NativeError("latent_q: q_lat must be [T, H, kv_rank] with a contiguous last dimension")
-        out = torch.empty(q.shape[0], n_heads * (q_lat.shape[2] + rot_dim), dtype=dt, device=q.device)
+        row = n_heads * (q_lat.shape[2] + rot_dim)
+        res = out if out is not None else torch.empty(q.shape[0], row, dtype=dt, device=q.device)
+        if res.dtype != dt or not res.is_contiguous() or tuple(res.shape) != (q.shape[0], row) or \
+                (q_lat.data_ptr() == res.data_ptr() and (q_lat.stride(1) != row // n_heads or (q.shape[0] > 1 and q_lat.stride(0) != row))):
+            raise NativeError("latent_q: out must be contiguous [T, H * (kv_rank + rot_dim)], and a q_lat inside it its leading columns per head")
         p.q_lat, p.lat_tok_stride, p.lat_head_stride, p.kv_rank = q_lat.data_ptr(), q_lat.stride(0), q_lat.stride(1), q_lat.shape[2]
-    p.q, p.q_out, p.n_heads, p.dim, p.rot_dim = q.data_ptr(), out.data_ptr(), int(n_heads), int(dim), int(rot_dim)
+    p.q, p.q_out, p.n_heads, p.dim, p.rot_dim = q.data_ptr(), res.data_ptr(), int(n_heads), int(dim), int(rot_dim)
     p.freqs, p.rot_mult, p.tok_pos, p.n_tokens, p.dtype = _ptr(freqs), float(rot_mult), batch.tok_pos.data_ptr(), q.shape[0], dtype_code(dt)
+    p.interleaved = 1 if interleaved else 0
     _check(load().pcs_latent_q(C.byref(p), _stream()), "pcs_latent_q")
-    return out
+    return res
 
 
 def latent_gather(pool: torch.Tensor, width: int, ctx: Batch) -> torch.Tensor:
@@ -867,9 +878,9 @@ def latent_gather(pool: torch.Tensor, width: int, ctx: Batch) -> torch.Tensor:
 
 
 def latent_expand(kv: torch.Tensor, pool: torch.Tensor, kv_rank: int, rot_dim: int, n_heads: int, dim: int, vdim: int, k_dense: torch.Tensor,
-                  v_dense: torch.Tensor, ctx: Batch) -> None:
+                  v_dense: torch.Tensor, ctx: Batch, seq_base: Optional[torch.Tensor] = None) -> None:
     """kv [N, H * (dim + vdim)] (plain key parts of all heads, then values) of the context tokens -> k_dense [B, H, cap', dim + rot_dim],
-    v_dense [B, H, cap', vdim], indexed by the batch entry."""
+    v_dense [B, H, cap', vdim], indexed by the batch entry; an entry's dense rows count from position seq_base (int32 [entries]; None: 0)."""
     _cuda(kv, pool, k_dense, v_dense)
     dt = kv.dtype
     _rows2d(kv, dt, "latent_expand: kv")
@@ -880,6 +891,7 @@ def latent_expand(kv: torch.Tensor, pool: torch.Tensor, kv_rank: int, rot_dim: i
     p.kv, p.kv_stride, p.pool, p.cap, p.kv_rank, p.rot_dim = kv.data_ptr(), kv.stride(0), pool.data_ptr(), pool.shape[2], int(kv_rank), int(rot_dim)
     p.n_heads, p.dim, p.vdim, p.k_dense, p.v_dense, p.cap_dense = int(n_heads), int(dim), int(vdim), k_dense.data_ptr(), v_dense.data_ptr(), k_dense.shape[2]
     p.ctx_seq, p.ctx_pos, p.seq_slot, p.n_ctx, p.dtype = ctx.tok_seq.data_ptr(), ctx.tok_pos.data_ptr(), ctx.seq_slot.data_ptr(), ctx.n_tokens, dtype_code(dt)
+    p.seq_base = _ptr(seq_base)
     _check(load().pcs_latent_expand(C.byref(p), _stream()), "pcs_latent_expand")
 
 
@@ -998,11 +1010,24 @@ def add_layer_norm(x: torch.Tensor, addends, eps: float, w1: Optional[torch.Tens
     """x += sum_i mult_i * y_i for `addends` = [(y_i [T, width] in the compute type or float32, mult_i)] (at most three), then
     h1 = ln(x) * w1 and h2 = ln(x) * w2 with ln(x) = (x - mean) / sqrt(var + eps) (each optional).  With `rows` (int32) only
     those rows are normed (no addends) and h1 / h2 have one row per entry of `rows`."""
+    _add_norm(x, addends, eps, w1, h1, w2, h2, rows)
+
+
+def add_rms_norm(x: torch.Tensor, addends, eps: float, w1: Optional[torch.Tensor] = None, h1: Optional[torch.Tensor] = None, w2: Optional[torch.Tensor] = None,
+                 h2: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None, w_offset: float = 0.0, y_norm_w: Optional[torch.Tensor] = None,
+                 copy: Optional[torch.Tensor] = None) -> None:
+    """`add_layer_norm` with RMS norms, h = x / sqrt(mean(x^2) + eps) * (w_offset + w).  With `y_norm_w` the first addend passes such a norm
+    with that plain weight before it is added; `copy` ([T, width]) gets the new x in the compute type.  An addend of row stride 0
+    (`vector.expand(T, -1)`) is added to every row."""
+    _add_norm(x, addends, eps, w1, h1, w2, h2, rows, True, w_offset, y_norm_w, copy)
+
+
+def _add_norm(x, addends, eps, w1, h1, w2, h2, rows, rms=False, w_offset=0.0, y_norm_w=None, copy=None) -> None:
     addends = list(addends or [])
     _cuda(x, w1, h1, w2, h2, rows, *[y for y, _ in addends])
     if x.dtype != torch.float32 or not x.is_contiguous() or x.dim() != 2 or len(addends) > 3:
         raise NativeError("add_layer_norm: x must be a contiguous float32 matrix, with at most three addends")
-    wt = w1 if w1 is not None else w2
+    wt = next((w for w in (w1, w2, y_norm_w, copy) if w is not None), None)
     dt = wt.dtype if wt is not None else next((y.dtype for y, _ in addends if y.dtype != torch.float32), torch.float32)
     R = rows.numel() if rows is not None else x.shape[0]
     if rows is not None and (rows.dtype != torch.int32 or not rows.is_contiguous() or addends):
@@ -1018,8 +1043,25 @@ def add_layer_norm(x: torch.Tensor, addends, eps: float, w1: Optional[torch.Tens
                               or tuple(h.shape) != (R, x.shape[1])):
             raise NativeError("add_layer_norm: a weight [width] needs its output [rows, width], both in the compute type")
     p.w1, p.h1, p.w2, p.h2 = _ptr(w1), _ptr(h1) if w1 is not None else None, _ptr(w2), _ptr(h2) if w2 is not None else None
+    if y_norm_w is not None and (not addends or y_norm_w.dtype != dt or not y_norm_w.is_contiguous() or y_norm_w.numel() != x.shape[1]):
+        raise NativeError("add_rms_norm: y_norm_w must be contiguous [width] in the compute type, with an addend")
+    if copy is not None and (rows is not None or copy.dtype != dt or not copy.is_contiguous() or copy.shape != x.shape):
+        raise NativeError("add_rms_norm: copy must be contiguous of x's shape in the compute type, without a row subset")
+    p.rms, p.w_offset, p.y_norm_w, p.copy = 1 if rms else 0, float(w_offset), _ptr(y_norm_w), _ptr(copy)
     p.n_rows, p.width, p.eps, p.dtype = R, x.shape[1], float(eps), dtype_code(dt)
     _check(load().pcs_add_layer_norm(C.byref(p), _stream()), "pcs_add_layer_norm")
+
+
+def side_gate(u: torch.Tensor, table: torch.Tensor, col: int, ids: torch.Tensor) -> torch.Tensor:
+    """gelu(u) * table[ids, col:col + dim] with the tanh form of gelu; u [T, dim] (row stride free), table [vocab, *]."""
+    _cuda(u, table, ids)
+    _rows2d(u, table.dtype, "side_gate: u")
+    if not table.is_contiguous() or ids.dtype != torch.int64 or not ids.is_contiguous() or ids.numel() != u.shape[0] or col + u.shape[1] > table.shape[1]:
+        raise NativeError("side_gate: table contiguous [vocab, columns] with the columns inside, ids contiguous int64, one per row")
+    out = torch.empty(u.shape, dtype=u.dtype, device=u.device)
+    _check(load().pcs_side_gate(u.data_ptr(), u.stride(0), table.data_ptr(), table.stride(0), table.shape[0], int(col), ids.data_ptr(), out.data_ptr(), u.shape[0],
+                                u.shape[1], dtype_code(u.dtype), _stream()), "pcs_side_gate")
+    return out
 
 
 def gru_scan(proj: torch.Tensor, offs, width: int, out: torch.Tensor, s_pool: torch.Tensor, batch: Batch) -> None:
@@ -1166,9 +1208,10 @@ def delta_takes_chunks(batch: Batch, dim: int, impl: int = 0) -> bool:
     return batch.max_len >= DELTA_CHUNK_MIN_LEN and dim <= DELTA_CHUNK_MAX_DIM and not torch.cuda.is_current_stream_capturing()
 
 
-def delta_scan(qk: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, b: torch.Tensor, kv_heads: int, s_pool: torch.Tensor, norm_w: torch.Tensor, gate: torch.Tensor,
-               out: torch.Tensor, eps: float, batch: Batch, out_scale: float = 1.0, impl: int = 0) -> None:
-    """The gated delta rule with its per-head norm and sigmoid gate.  qk float32 [T, 2 * kv_heads * dim] (unit vectors, queries scaled), v [T, H * vdim],
+def delta_scan(qk: torch.Tensor, v: torch.Tensor, decay: Optional[torch.Tensor], b: torch.Tensor, kv_heads: int, s_pool: torch.Tensor, norm_w: torch.Tensor, gate: torch.Tensor,
+               out: torch.Tensor, eps: float, batch: Batch, out_scale: float = 1.0, impl: int = 0, head_decay=None, gate_silu: bool = False) -> None:
+    """The gated delta rule with its per-head norm and sigmoid gate (silu with `gate_silu`).  One decay per head instead of per channel: decay None
+    and head_decay = (a [T, H] pre-activations, dt_bias float32 [H], rate float32 [H]) for exp(-rate * softplus(a + dt_bias)).  qk float32 [T, 2 * kv_heads * dim] (unit vectors, queries scaled), v [T, H * vdim],
     decay float32 [T, H * dim] (log decays where `delta_takes_chunks`, else the decays), b [T, H] pre-activations of the step sizes, gate
     [T, H * vdim] pre-activations, state pool float32 [slots, H, dim, vdim]; out [T, H * vdim] (row stride free).  impl 0: by step;
     1: token by token with the state in shared memory; 2: token by token (registers where the sizes allow); 3: in chunks."""
@@ -1180,9 +1223,20 @@ def delta_scan(qk: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, b: torch.
         raise NativeError("delta_scan: the state pool must be contiguous float32 [slots, H, dim, vdim]")
     H, D, V = s_pool.shape[1:]
     T, dev = v.shape[0], v.device
-    if qk.dtype != torch.float32 or decay.dtype != torch.float32 or not (qk.is_contiguous() and v.is_contiguous() and decay.is_contiguous()) \
-            or tuple(qk.shape) != (T, 2 * kv_heads * D) or tuple(decay.shape) != (T, H * D) or tuple(v.shape) != (T, H * V) or tuple(b.shape) != (T, H):
-        raise NativeError("delta_scan: qk float32 [T, 2 * kv_heads * dim], decay float32 [T, H * dim], v [T, H * vdim], b [T, H]")
+    if qk.dtype != torch.float32 or not (qk.is_contiguous() and v.is_contiguous()) or tuple(qk.shape) != (T, 2 * kv_heads * D) or tuple(v.shape) != (T, H * V) \
+            or tuple(b.shape) != (T, H):
+        raise NativeError("delta_scan: qk float32 [T, 2 * kv_heads * dim], v [T, H * vdim], b [T, H]")
+    if (decay is None) == (head_decay is None):
+        raise NativeError("delta_scan: either decay (per channel) or head_decay")
+    if decay is not None and (decay.dtype != torch.float32 or not decay.is_contiguous() or tuple(decay.shape) != (T, H * D)):
+        raise NativeError("delta_scan: decay float32 [T, H * dim]")
+    da = dt_bias = rate = None
+    if head_decay is not None:
+        da, dt_bias, rate = head_decay
+        _cuda(da, dt_bias, rate)
+        _rows2d(da, dt, "delta_scan: head decays")
+        if tuple(da.shape) != (T, H) or any(t.dtype != torch.float32 or t.numel() != H or not t.is_contiguous() for t in (dt_bias, rate)):
+            raise NativeError("delta_scan: head_decay is (a [T, H] in the compute type, dt_bias float32 [H], rate float32 [H])")
     if norm_w.dtype != dt or norm_w.numel() != V or tuple(gate.shape) != (T, H * V) or tuple(out.shape) != (T, H * V):
         raise NativeError("delta_scan: norm_w [vdim], gate and out [T, H * vdim] in the compute type")
     n = pcs_headnorm_params()
@@ -1193,7 +1247,8 @@ def delta_scan(qk: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, b: torch.
         new = lambda *s: torch.empty(*s, dtype=torch.float32, device=dev)
         qd, kd, w, g, u, a, s = new(nc * H, ch, D), new(nc * H, ch, L), new(nc * H, (D + 7) // 8 * 8, ch), new(nc * H, D), new(nc * H, ch, V), new(nc * H, ch, ch), new(nc * H, D, V)
         p = pcs_delta_chunk_params()
-        p.qk, p.v, p.ld, p.b, p.b_stride = qk.data_ptr(), v.data_ptr(), decay.data_ptr(), b.data_ptr(), b.stride(0)
+        p.qk, p.v, p.ld, p.b, p.b_stride = qk.data_ptr(), v.data_ptr(), _ptr(decay), b.data_ptr(), b.stride(0)
+        p.dec_a, p.dec_stride, p.dt_bias, p.rate = _ptr(da), da.stride(0) if da is not None else 0, _ptr(dt_bias), _ptr(rate)
         p.heads, p.kv_heads, p.dim, p.vdim = H, int(kv_heads), D, V
         p.chunk_first, p.chunk_len, p.n_chunks, p.n_tokens, p.dtype, p.n_seqs = plan["first"].data_ptr(), plan["len"].data_ptr(), nc, T, dtype_code(dt), batch.n_seqs
         p.qd, p.kd, p.w, p.g, p.u, p.a, p.s, p.s_pool = (t.data_ptr() for t in (qd, kd, w, g, u, a, s, s_pool))
@@ -1205,11 +1260,12 @@ def delta_scan(qk: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, b: torch.
     else:
         o = torch.empty(T, H * V, dtype=torch.float32, device=dev)
         p = pcs_delta_params()
-        p.qk, p.v, p.decay, p.b, p.b_stride, p.o, p.s_pool = qk.data_ptr(), v.data_ptr(), decay.data_ptr(), b.data_ptr(), b.stride(0), o.data_ptr(), s_pool.data_ptr()
+        p.qk, p.v, p.decay, p.b, p.b_stride, p.o, p.s_pool = qk.data_ptr(), v.data_ptr(), _ptr(decay), b.data_ptr(), b.stride(0), o.data_ptr(), s_pool.data_ptr()
+        p.a, p.a_stride, p.dt_bias, p.rate = _ptr(da), da.stride(0) if da is not None else 0, _ptr(dt_bias), _ptr(rate)
         p.heads, p.kv_heads, p.dim, p.vdim = H, int(kv_heads), D, V
         p.seq_slot, p.seq_pos0, p.seq_len, p.seq_off = (batch.seq_slot.data_ptr(), batch.seq_pos0.data_ptr(), batch.seq_len.data_ptr(), batch.seq_off.data_ptr())
         p.n_seqs, p.n_tokens, p.dtype, p.impl = batch.n_seqs, T, dtype_code(dt), 1 if impl == 1 else 0
         _check(load().pcs_delta_scan(C.byref(p), _stream()), "pcs_delta_scan")
     n.o, n.w, n.g, n.g_stride, n.out, n.out_stride = o.data_ptr(), norm_w.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(), out.stride(0)
-    n.n_tokens, n.heads, n.vdim, n.eps, n.out_scale, n.dtype = T, H, V, float(eps), float(out_scale), dtype_code(dt)
+    n.n_tokens, n.heads, n.vdim, n.eps, n.out_scale, n.dtype, n.silu = T, H, V, float(eps), float(out_scale), dtype_code(dt), 1 if gate_silu else 0
     _check(load().pcs_head_norm_gate(C.byref(n), _stream()), "pcs_head_norm_gate")

@@ -29,9 +29,9 @@ __global__ void __launch_bounds__(LB_THREADS) attn_latent_kernel(const pcs_attn_
   const int b = p.tok_seq[t], pos = p.tok_pos[t], slot = p.pool_slot ? p.pool_slot[b] : p.seq_slot[b];
   const int D = p.dim, V = p.vdim, H = p.n_heads;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, grp = lane >> 2, qd = lane & 3;
-  const int n_keys = pos + 1;
+  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0, n_keys = pos + 1 - lo;   // a window's keys are the last ones
   const int chunk = ((n_keys + S - 1) / S + LB_N - 1) / LB_N * LB_N;
-  const int k_begin = sp * chunk, k_end = min(n_keys, k_begin + chunk);
+  const int k_begin = lo + sp * chunk, k_end = min(pos + 1, k_begin + chunk);
   const __nv_bfloat16* Kg = static_cast<const __nv_bfloat16*>(p.k_pool) + static_cast<long long>(slot) * p.cap * D;
   const __nv_bfloat16* Qg = static_cast<const __nv_bfloat16*>(p.q) + (static_cast<long long>(t) * H + h0) * D;
   const int pieces = DKP / 8;
@@ -193,12 +193,12 @@ int launch_nt(const pcs_attn_params& p, cudaStream_t st, int DKP, int splits, si
 
 }  // namespace
 
-// Serves bfloat16 rows shared by all heads whose values are the rows' leading numbers, without bias, cap or window, when a
+// Serves bfloat16 rows shared by all heads whose values are the rows' leading numbers, without bias, cap or kept first keys, when a
 // workspace for the partial results is given; `splits_out` tells the caller how many partial results the merge reads.
 int launch_attn_latent(const pcs_attn_params& p, cudaStream_t st, int* splits_out) {
   *splits_out = 0;
   if (p.dtype != PCS_BF16 || p.n_kv_heads != 1 || p.v_pool != p.k_pool || p.v_row_stride != p.dim || p.workspace == nullptr) return PCS_OK;
-  if (p.bias_r1 || p.bias_table || p.head_scale || p.softcap > 0.f || p.window > 0 || p.chunk > 0 || p.dim % 8 != 0 || p.vdim % 8 != 0 || p.vdim > 512 || p.vdim > p.dim) return PCS_OK;
+  if (p.bias_r1 || p.bias_table || p.head_scale || p.softcap > 0.f || (p.window > 0 && p.keep_first > 0) || p.chunk > 0 || p.dim % 8 != 0 || p.vdim % 8 != 0 || p.vdim > 512 || p.vdim > p.dim) return PCS_OK;
   if ((reinterpret_cast<uintptr_t>(p.k_pool) | reinterpret_cast<uintptr_t>(p.q)) & 15) return PCS_OK;
   const int DKP = (p.dim + 31) / 32 * 32;
   const size_t smem = static_cast<size_t>(LB_HEADS + 2 * LB_N) * (DKP + LB_PAD) * sizeof(__nv_bfloat16);

@@ -138,6 +138,7 @@ __device__ __forceinline__ void angle_sincos(int pos, double f, float* s, float*
 struct GluAct {
   int kind;
   float alpha, limit;
+  __host__ __device__ explicit GluAct(int k) : kind(k), alpha(1.f), limit(0.f) {}
   __host__ GluAct() : kind(PCS_GLU_SILU), alpha(1.f), limit(0.f) {}
   __host__ explicit GluAct(const pcs_glu_act* a) : kind(a ? a->kind : PCS_GLU_SILU), alpha(a ? a->alpha : 1.f), limit(a ? a->limit : 0.f) {}
   __host__ __device__ __forceinline__ bool gated() const { return kind == PCS_GLU_SILU || kind == PCS_GLU_CLAMPED_SWISH || kind == PCS_GLU_GELU_TANH; }

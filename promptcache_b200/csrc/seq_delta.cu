@@ -40,6 +40,9 @@ __device__ __forceinline__ ConvPlace conv_place(const pcs_shortconv_params& p, i
 
 __device__ __forceinline__ float silu_(float z) { return z * sigmoidf_(z); }
 
+// log of a head's decay from its pre-activation
+__device__ __forceinline__ float head_log_decay(float z, float rate) { return -rate * softplusf_(z); }
+
 // Any sizes: one block per token; a warp per query / key head, then the value channels.
 template <typename T>
 __global__ void __launch_bounds__(256) short_conv_kernel(const pcs_shortconv_params p) {
@@ -313,7 +316,8 @@ __global__ void __launch_bounds__(1024) delta_scan_kernel(const pcs_delta_params
     for (int d = tid; d < D; d += nthr) {
       qs[d] = p.qk[t * U + hk * D + d];
       ks[d] = p.qk[t * U + (p.kv_heads + hk) * D + d];
-      as[d] = p.decay[t * (static_cast<long long>(H) * D) + head * D + d];
+      as[d] = p.decay ? p.decay[t * (static_cast<long long>(H) * D) + head * D + d]
+                      : expf(head_log_decay(ldf(static_cast<const T*>(p.a) + t * p.a_stride + head) + p.dt_bias[head], p.rate[head]));
     }
     __syncthreads();
     if (active) {
@@ -363,11 +367,12 @@ constexpr int kDsGroup = 4;   // tokens computed between two block barriers
 
 // State in registers.  A warp owns 8 columns; lane = 8 * rg + c: column c, rows 4 (rg + 4 m) + e for m < M, e < 4 (four row groups
 // share a column, so a column's sums are two shuffles).  One pass over the decayed state gives both S^T k and S^T q; the read-out
-// after the write is then S^T q + (k . q) u.  Rows past dim hold zeros.  The order of every sum is fixed by M alone.
-template <typename T, int M>
+// after the write is then S^T q + (k . q) u.  Rows past dim hold zeros.  The order of every sum is fixed by M alone.  HD: one decay per
+// head, formed here from its pre-activation (requested a group ahead, like the step sizes).
+template <typename T, int M, bool HD>
 __global__ void __launch_bounds__(256) delta_scan_reg_kernel(const pcs_delta_params p, int W) {
-  extern __shared__ __align__(16) float ring[];   // per slot: q[16 M] k[16 M] decay[16 M]
-  constexpr int DP = 16 * M;
+  extern __shared__ __align__(16) float ring[];   // per slot: q[16 M] k[16 M] decay[16 M] (per channel)
+  constexpr int DP = 16 * M, NR = HD ? 2 : 3;
   const int D = p.dim, V = p.vdim, H = p.heads, U = 2 * p.kv_heads * D;
   const int b = blockIdx.x, head = blockIdx.y, hk = head / (H / p.kv_heads), v0 = blockIdx.z * 8 * W;
   const int tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, rg = lane >> 3;
@@ -379,8 +384,8 @@ __global__ void __launch_bounds__(256) delta_scan_reg_kernel(const pcs_delta_par
   const int cd = D / 4;
   auto issue = [&](int i) {
     const long long t = off + i;
-    float* s = ring + (i % kDsRing) * 3 * DP;
-    for (int e = tid; e < 3 * (DP / 4); e += nthr) {
+    float* s = ring + (i % kDsRing) * NR * DP;
+    for (int e = tid; e < NR * (DP / 4); e += nthr) {
       const int which = e / (DP / 4), c = e - which * (DP / 4);
       float* dst = s + which * DP + c * 4;
       if (c < cd) {
@@ -406,23 +411,28 @@ __global__ void __launch_bounds__(256) delta_scan_reg_kernel(const pcs_delta_par
     }
   const T* vg = static_cast<const T*>(p.v) + static_cast<long long>(off) * H * V + head * V + col;
   const T* bg = static_cast<const T*>(p.b) + static_cast<long long>(off) * p.b_stride + head;
-  float vn[kDsGroup], bn[kDsGroup];   // the next group's values and step sizes, requested a group ahead
+  const T* ag = HD ? static_cast<const T*>(p.a) + static_cast<long long>(off) * p.a_stride + head : nullptr;
+  const float a_bias = HD ? p.dt_bias[head] : 0.f, a_rate = HD ? p.rate[head] : 0.f;
+  float vn[kDsGroup], bn[kDsGroup], an[kDsGroup];   // the next group's values and step sizes, requested a group ahead
 #pragma unroll
   for (int u = 0; u < kDsGroup; ++u) {
     vn[u] = (u < len && okc) ? ldf(vg + static_cast<long long>(u) * H * V) : 0.f;
     bn[u] = u < len ? ldf(bg + u * p.b_stride) : 0.f;
+    an[u] = HD && u < len ? ldf(ag + u * p.a_stride) : 0.f;
   }
   for (int i0 = 0; i0 < len; i0 += kDsGroup) {
     cp_async_wait<kDsAhead - kDsGroup>();
     __syncthreads();
-    float vc[kDsGroup], bc[kDsGroup];
+    float vc[kDsGroup], bc[kDsGroup], ac[kDsGroup];
 #pragma unroll
     for (int u = 0; u < kDsGroup; ++u) {
       vc[u] = vn[u];
       bc[u] = bn[u];
+      ac[u] = an[u];
       const int nx = i0 + kDsGroup + u;
       vn[u] = (nx < len && okc) ? ldf(vg + static_cast<long long>(nx) * H * V) : 0.f;
       bn[u] = nx < len ? ldf(bg + nx * p.b_stride) : 0.f;
+      an[u] = HD && nx < len ? ldf(ag + nx * p.a_stride) : 0.f;
       if (i0 + kDsAhead + u < len) issue(i0 + kDsAhead + u);
       cp_async_commit();
     }
@@ -430,13 +440,14 @@ __global__ void __launch_bounds__(256) delta_scan_reg_kernel(const pcs_delta_par
     for (int u = 0; u < kDsGroup; ++u) {
       const int i = i0 + u;
       if (i >= len) break;
-      const float* cur = ring + (i % kDsRing) * 3 * DP;
+      const float* cur = ring + (i % kDsRing) * NR * DP;
+      const float hd = HD ? expf(head_log_decay(ac[u] + a_bias, a_rate)) : 0.f;
       float pk = 0.f, pq = 0.f, kq = 0.f;
 #pragma unroll
       for (int m = 0; m < M; ++m) {
         const int d = 4 * (rg + 4 * m);
         const float4 q = *reinterpret_cast<const float4*>(cur + d), k = *reinterpret_cast<const float4*>(cur + DP + d),
-                     a = *reinterpret_cast<const float4*>(cur + 2 * DP + d);
+                     a = HD ? make_float4(hd, hd, hd, hd) : *reinterpret_cast<const float4*>(cur + 2 * DP + d);
         S[m][0] *= a.x; S[m][1] *= a.y; S[m][2] *= a.z; S[m][3] *= a.w;
         pk = fmaf(S[m][0], k.x, fmaf(S[m][1], k.y, fmaf(S[m][2], k.z, fmaf(S[m][3], k.w, pk))));
         pq = fmaf(S[m][0], q.x, fmaf(S[m][1], q.y, fmaf(S[m][2], q.z, fmaf(S[m][3], q.w, pq))));
@@ -475,7 +486,75 @@ __global__ void __launch_bounds__(256) delta_scan_reg_kernel(const pcs_delta_par
 constexpr int kC = PCS_DELTA_CHUNK, kCB = 16, kNB = kC / kCB;
 constexpr int kDpThreads = 384;
 
+__device__ __forceinline__ void mma_tf32(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+// hi keeps the sign, the exponent and 10 bits of the fraction; the remainder is exact in 32-bit and its own leading bits are what the unit reads
+__device__ __forceinline__ void split_tf32(float x, uint32_t& hi, uint32_t& lo) {
+  hi = __float_as_uint(x) & 0xffffe000u;
+  lo = __float_as_uint(x - __uint_as_float(hi));
+}
+
 __device__ __forceinline__ int delta_kd_slot(int d) { return (d & ~63) + 4 * (d & 15) + ((d & 63) >> 4); }
+
+// M x = rhs by forward substitution, one column per thread, the column in registers: first the dim columns of diag(beta) K exp(B), then the
+// vdim columns of diag(beta) V.  `key(i, col)` gives row i of column col of K exp(B).
+template <typename T, typename Key>
+__device__ __forceinline__ void delta_chunk_solve(const pcs_delta_chunk_params& p, const float* As, const float* beta, long long base, int first, int n, int head, Key key) {
+  constexpr bool kFast = sizeof(T) == 2;
+  const int D = p.dim, V = p.vdim, H = p.heads, tid = threadIdx.x;
+  const int D8 = (D + 7) & ~7;
+  float* wg = p.w + base * D8 * kC;
+  float* ug = p.u + base * kC * V;
+  for (int e = tid; e < (D8 - D) * kC; e += kDpThreads) {   // channels that only pad the fragments
+    const int d = D + e / kC, i = e % kC;
+    if (kFast) wg[(((d >> 3) * 4 + (i >> 4)) * 32 + (i & 7) * 4 + (d & 3)) * 4 + ((i >> 3) & 1) + 2 * ((d >> 2) & 1)] = 0.f;
+  }
+#pragma unroll 1
+  for (int col = tid; col < D + V; col += kDpThreads) {
+    float x[kC];
+    long long v_step = static_cast<long long>(H) * V, u_step = V;
+    asm volatile("" : "+l"(v_step), "+l"(u_step));   // (64 row offsets each, taken out of the column loop, would spill)
+    if (col < D) {
+#pragma unroll
+      for (int i = 0; i < kC; ++i) x[i] = beta[i] * key(i, col);
+    } else {
+      const T* v = static_cast<const T*>(p.v) + static_cast<long long>(first) * H * V + head * V + (col - D);
+#pragma unroll
+      for (int i = 0; i < kC; ++i) x[i] = i < n ? beta[i] * ldf(v + i * v_step) : 0.f;
+    }
+#pragma unroll
+    for (int i = 1; i < kC; ++i) {
+      float a0 = 0.f, a1 = 0.f;
+#pragma unroll
+      for (int j = 0; j < i; j += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(As + i * kC + j);   // (entries from i on are zero)
+        a0 = fmaf(a.x, x[j], a0);
+        if (j + 1 < i) a1 = fmaf(a.y, x[j + 1], a1);
+        if (j + 2 < i) a0 = fmaf(a.z, x[j + 2], a0);
+        if (j + 3 < i) a1 = fmaf(a.w, x[j + 3], a1);
+      }
+      x[i] -= a0 + a1;
+    }
+    if (col < D) {
+      if (kFast) {
+        float* o = wg + ((col >> 3) * 4 * 32 + (col & 3)) * 4 + 2 * ((col >> 2) & 1);
+#pragma unroll
+        for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+          for (int g = 0; g < 16; ++g) o[(mt * 32 + (g & 7) * 4) * 4 + (g >> 3)] = x[mt * 16 + g];   // (wider stores would pin register pairs)
+      } else {
+        float* o = wg + static_cast<long long>(col) * kC;
+#pragma unroll
+        for (int r = 0; r < 16; ++r) *reinterpret_cast<float4*>(o + 4 * r) = make_float4(x[r], x[r + 16], x[r + 32], x[r + 48]);
+      }
+    } else {
+#pragma unroll
+      for (int i = 0; i < kC; ++i) ug[i * u_step + (col - D)] = x[i];
+    }
+  }
+}
 
 template <typename T>
 __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_delta_chunk_params p) {
@@ -663,59 +742,175 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_
     As[(i + 8) * kC + s] = beta[i + 8] * k10; As[(i + 8) * kC + s + 8] = beta[i + 8] * k11;
   }
   __syncthreads();
-  // M x = rhs by forward substitution, one column per thread, the column in registers: first the dim columns of diag(beta) K exp(B), then
-  // the vdim columns of diag(beta) V
-  const int D8 = (D + 7) & ~7;
-  float* wg = p.w + base * D8 * kC;
-  float* ug = p.u + base * kC * V;
-  for (int e = tid; e < (D8 - D) * kC; e += kDpThreads) {   // channels that only pad the fragments
-    const int d = D + e / kC, i = e % kC;
-    if (kFast) wg[(((d >> 3) * 4 + (i >> 4)) * 32 + (i & 7) * 4 + (d & 3)) * 4 + ((i >> 3) & 1) + 2 * ((d >> 2) & 1)] = 0.f;
-  }
-#pragma unroll 1
-  for (int col = tid; col < D + V; col += kDpThreads) {
-    float x[kC];
-    long long v_step = static_cast<long long>(H) * V, u_step = V;
-    asm volatile("" : "+l"(v_step), "+l"(u_step));   // (64 row offsets each, taken out of the column loop, would spill)
-    if (col < D) {
-      const float e1 = f1[col], e2 = e1 * f2[col], e3 = e2 * f3[col];
-#pragma unroll
-      for (int i = 0; i < kC; ++i) x[i] = beta[i] * ks[i * DP + col] * (i < 16 ? 1.f : i < 32 ? e1 : i < 48 ? e2 : e3);
-    } else {
-      const T* v = static_cast<const T*>(p.v) + static_cast<long long>(first) * H * V + head * V + (col - D);
-#pragma unroll
-      for (int i = 0; i < kC; ++i) x[i] = i < n ? beta[i] * ldf(v + i * v_step) : 0.f;
+  delta_chunk_solve<T>(p, As, beta, base, first, n, head, [&](int i, int col) {
+    const float e1 = f1[col];
+    return ks[i * DP + col] * (i < 16 ? 1.f : i < 32 ? e1 : i < 48 ? e1 * f2[col] : e1 * f2[col] * f3[col]);
+  });
+}
+
+// One decay per head: the factor of a pair (i, s) is one number, exp(B_i - B_s) <= 1, so the sums over pairs are plain products q k^T and k k^T
+// scaled afterwards (bfloat16 runs: m16n8k8 TF32 products of hi + lo operands, as in the scan; float32 runs: 32-bit multiply-adds).
+template <typename T>
+__global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_head_kernel(const pcs_delta_chunk_params p) {
+  extern __shared__ __align__(16) float sm[];
+  const int D = p.dim, H = p.heads, D8 = (D + 7) & ~7, DP = ((D8 + 31) & ~31) + 4, U = 2 * p.kv_heads * D, L = (D + 63) & ~63;   // (rows 4 banks apart)
+  float* qs = sm;              // [64][DP]
+  float* ks = qs + kC * DP;    // [64][DP]
+  float* As = ks + kC * DP;    // [64][64] beta_i A[i, s]
+  float* beta = As + kC * kC;  // [64] each: step sizes, running sums of the log decays, their exponentials, the exponentials of what is left to the end
+  float* Bs = beta + kC;
+  float* eB = Bs + kC;
+  float* eE = eB + kC;
+  const int cn = blockIdx.x, head = blockIdx.y, hk = head / (H / p.kv_heads), tid = threadIdx.x;
+  const int first = p.chunk_first[cn], n = p.chunk_len[cn];
+  const long long base = static_cast<long long>(cn) * H + head;
+  constexpr bool kFast = sizeof(T) == 2;
+  constexpr float kLog = kFast ? 1.4426950408889634f : 1.f;
+  auto ex = [](float x) { return kFast ? ex2(x) : expf(x); };
+  const int warp = tid >> 5, lane = tid & 31;
+  constexpr int kWarps = kDpThreads / 32;
+  const float* qb = p.qk + hk * D;
+  const float* kb = p.qk + (p.kv_heads + hk) * D;
+  const bool vec = D % 4 == 0 && (reinterpret_cast<uintptr_t>(p.qk) & 15) == 0;
+  if (vec) {
+    for (int e = tid; e < 2 * kC * (D8 / 4); e += kDpThreads) {
+      const int row = e / (D8 / 4), c = (e - row * (D8 / 4)) * 4, i = row & (kC - 1);
+      float* dst = (row < kC ? qs : ks) + i * DP + c;
+      if (i < n && c < D) cp_async16(dst, (row < kC ? qb : kb) + static_cast<long long>(first + i) * U + c);
+      else *reinterpret_cast<float4*>(dst) = make_float4(0.f, 0.f, 0.f, 0.f);
     }
-#pragma unroll
-    for (int i = 1; i < kC; ++i) {
-      float a0 = 0.f, a1 = 0.f;
-#pragma unroll
-      for (int j = 0; j < i; j += 4) {
-        const float4 a = *reinterpret_cast<const float4*>(As + i * kC + j);   // (entries from i on are zero)
-        a0 = fmaf(a.x, x[j], a0);
-        if (j + 1 < i) a1 = fmaf(a.y, x[j + 1], a1);
-        if (j + 2 < i) a0 = fmaf(a.z, x[j + 2], a0);
-        if (j + 3 < i) a1 = fmaf(a.w, x[j + 3], a1);
-      }
-      x[i] -= a0 + a1;
-    }
-    if (col < D) {
-      if (kFast) {
-        float* o = wg + ((col >> 3) * 4 * 32 + (col & 3)) * 4 + 2 * ((col >> 2) & 1);
-#pragma unroll
-        for (int mt = 0; mt < 4; ++mt)
-#pragma unroll
-          for (int g = 0; g < 16; ++g) o[(mt * 32 + (g & 7) * 4) * 4 + (g >> 3)] = x[mt * 16 + g];   // (wider stores would pin register pairs)
-      } else {
-        float* o = wg + static_cast<long long>(col) * kC;
-#pragma unroll
-        for (int r = 0; r < 16; ++r) *reinterpret_cast<float4*>(o + 4 * r) = make_float4(x[r], x[r + 16], x[r + 32], x[r + 48]);
-      }
-    } else {
-#pragma unroll
-      for (int i = 0; i < kC; ++i) ug[i * u_step + (col - D)] = x[i];
+  } else {
+    for (int e = tid; e < 2 * kC * D8; e += kDpThreads) {
+      const int row = e / D8, c = e - row * D8, i = row & (kC - 1);
+      (row < kC ? qs : ks)[i * DP + c] = i < n && c < D ? (row < kC ? qb : kb)[static_cast<long long>(first + i) * U + c] : 0.f;
     }
   }
+  cp_async_commit();
+  if (warp == 0) {   // lane owns tokens 2 lane and 2 lane + 1; tokens past the chunk's end decay nothing and write nothing
+    float l[2];
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {
+      const int i = 2 * lane + x;
+      l[x] = 0.f;
+      float bt = 0.f;
+      if (i < n) {
+        const long long t = first + i;
+        l[x] = kLog * head_log_decay(ldf(static_cast<const T*>(p.dec_a) + t * p.dec_stride + head) + p.dt_bias[head], p.rate[head]);
+        bt = sigmoidf_(ldf(static_cast<const T*>(p.b) + t * p.b_stride + head));
+      }
+      beta[i] = bt;
+    }
+    float run = l[0] + l[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+      const float up = __shfl_up_sync(0xffffffffu, run, o);
+      if (lane >= o) run += up;
+    }
+    const float end = __shfl_sync(0xffffffffu, run, 31), b1 = run, b0 = run - l[1];
+    Bs[2 * lane] = b0;
+    Bs[2 * lane + 1] = b1;
+    eB[2 * lane] = ex(b0);
+    eB[2 * lane + 1] = ex(b1);
+    eE[2 * lane] = ex(fminf(end - b0, 0.f));
+    eE[2 * lane + 1] = ex(fminf(end - b1, 0.f));
+  }
+  float* ag = p.a + base * kC * kC;
+  for (int e = tid; e < kC * kC; e += kDpThreads)
+    if ((e & 63) > (e >> 6)) { ag[e] = 0.f; As[e] = 0.f; }   // above the diagonal
+  cp_async_wait<0>();
+  __syncthreads();
+  auto put = [&](int i, int s, float qk, float kk) {
+    if (s > i) return;
+    const float f = ex(fminf(Bs[i] - Bs[s], 0.f));
+    ag[i * kC + s] = qk * f;
+    As[i * kC + s] = s < i ? beta[i] * kk * f : 0.f;
+  };
+  if (kFast) {
+    const int g = lane >> 2, t = lane & 3;
+    // 20 tiles of 16 x 8 pairs on and below the diagonal: row tile mi holds 2 (mi + 1) of them
+    for (int job = warp; job < 20; job += kWarps) {
+      const int mi = job < 2 ? 0 : job < 6 ? 1 : job < 12 ? 2 : 3, ni = job - mi * (mi + 1);
+      float q[3][4], k[3][4];
+#pragma unroll
+      for (int a = 0; a < 3; ++a)
+#pragma unroll
+        for (int x = 0; x < 4; ++x) q[a][x] = k[a][x] = 0.f;
+      const float* qa = qs + (16 * mi + g) * DP + t;
+      const float* ka = ks + (16 * mi + g) * DP + t;
+      const float* kn = ks + (8 * ni + g) * DP + t;
+#pragma unroll 2
+      for (int d = 0; d < D8; d += 8) {
+        uint32_t ah[4], al[4], h0, l0, h1, l1;
+        split_tf32(kn[d], h0, l0);
+        split_tf32(kn[d + 4], h1, l1);
+        split_tf32(qa[d], ah[0], al[0]);
+        split_tf32(qa[d + 8 * DP], ah[1], al[1]);
+        split_tf32(qa[d + 4], ah[2], al[2]);
+        split_tf32(qa[d + 8 * DP + 4], ah[3], al[3]);
+        mma_tf32(q[0], ah, h0, h1);
+        mma_tf32(q[1], ah, l0, l1);
+        mma_tf32(q[2], al, h0, h1);
+        split_tf32(ka[d], ah[0], al[0]);
+        split_tf32(ka[d + 8 * DP], ah[1], al[1]);
+        split_tf32(ka[d + 4], ah[2], al[2]);
+        split_tf32(ka[d + 8 * DP + 4], ah[3], al[3]);
+        mma_tf32(k[0], ah, h0, h1);
+        mma_tf32(k[1], ah, l0, l1);
+        mma_tf32(k[2], al, h0, h1);
+      }
+#pragma unroll
+      for (int x = 0; x < 4; ++x)
+        put(16 * mi + g + 8 * (x >> 1), 8 * ni + 2 * t + (x & 1), q[0][x] + (q[1][x] + q[2][x]), k[0][x] + (k[1][x] + k[2][x]));
+    }
+  } else {
+    for (int e = tid; e < (kC / 2) * (kC / 2 + 1) / 2; e += kDpThreads) {   // 2 x 2 pairs on and below the diagonal
+      int bi = static_cast<int>((sqrtf(8.f * e + 1.f) - 1.f) * 0.5f);
+      while ((bi + 1) * (bi + 2) / 2 <= e) ++bi;
+      while (bi * (bi + 1) / 2 > e) --bi;
+      const int i = 2 * bi, s = 2 * (e - bi * (bi + 1) / 2);
+      float q[2][2] = {}, k[2][2] = {};
+      for (int d = 0; d < D8; ++d) {
+        const float s0 = ks[s * DP + d], s1 = ks[(s + 1) * DP + d];
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const float qv = qs[(i + x) * DP + d], kv = ks[(i + x) * DP + d];
+          q[x][0] = fmaf(qv, s0, q[x][0]);
+          q[x][1] = fmaf(qv, s1, q[x][1]);
+          k[x][0] = fmaf(kv, s0, k[x][0]);
+          k[x][1] = fmaf(kv, s1, k[x][1]);
+        }
+      }
+#pragma unroll
+      for (int x = 0; x < 4; ++x) put(i + (x >> 1), s + (x & 1), q[x >> 1][x & 1], k[x >> 1][x & 1]);
+    }
+  }
+  // what leaves the chunk
+  {
+    float* qd = p.qd + base * kC * D;
+    float* kd = p.kd + base * kC * L;
+    if (kFast) {   // the outgoing keys as fragments: a warp takes (16 channels, 8 tokens) at a time and writes 512 bytes
+      for (int f = warp; f < (L / 16) * (kC / 8); f += kWarps) {
+        const int mt = f >> 3, kt = f & 7;
+        float o[4];
+#pragma unroll
+        for (int r = 0; r < 4; ++r) {
+          const int i = kt * 8 + (lane & 3) + 4 * (r >> 1), d = mt * 16 + (lane >> 2) + 8 * (r & 1);
+          o[r] = d < D ? ks[i * DP + d] * eE[i] : 0.f;
+        }
+        *reinterpret_cast<float4*>(kd + (static_cast<long long>(f) * 32 + lane) * 4) = make_float4(o[0], o[1], o[2], o[3]);
+      }
+    } else {
+      for (int e = tid; e < kC * L; e += kDpThreads) {
+        const int i = e / L, d = e - i * L;
+        kd[static_cast<long long>(i) * L + delta_kd_slot(d)] = d < D ? ks[i * DP + d] * eE[i] : 0.f;
+      }
+    }
+    for (int i = warp; i < kC; i += kWarps)
+      for (int d = lane; d < D; d += 32) qd[i * D + d] = qs[i * DP + d] * eB[i];
+    for (int d = tid; d < D; d += kDpThreads) p.g[base * D + d] = eB[kC - 1];
+  }
+  __syncthreads();
+  delta_chunk_solve<T>(p, As, beta, base, first, n, head, [&](int i, int col) { return ks[i * DP + col] * eB[i]; });
 }
 
 // Block = (VS value columns, head, entry), 16 warps.  Both products split their sum over the warps and meet in `red`: u = u0 - w S over the
@@ -913,16 +1108,6 @@ __global__ void __launch_bounds__(kDcThreads) delta_chunk_scan_kernel(const pcs_
 //   S = g S + kd^T u  warp = 16 channels (and 16 more at dim > 128): no sum leaves the warp, S stays in its accumulators
 // S and u also sit in shared memory as [row][8] tiles: a B fragment is 32 neighbouring numbers.
 constexpr int kDtThreads = 256;
-
-__device__ __forceinline__ void mma_tf32(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-// hi keeps the sign, the exponent and 10 bits of the fraction; the remainder is exact in 32-bit and its own leading bits are what the unit reads
-__device__ __forceinline__ void split_tf32(float x, uint32_t& hi, uint32_t& lo) {
-  hi = __float_as_uint(x) & 0xffffe000u;
-  lo = __float_as_uint(x - __uint_as_float(hi));
-}
 
 template <int NV, int NB, int MT>   // MT: 16-channel tiles per warp (dim <= 128 MT)
 __global__ void __launch_bounds__(kDtThreads) delta_chunk_scan_tc_kernel(const pcs_delta_chunk_params p) {
@@ -1211,9 +1396,12 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const pcs_headnorm_
 #pragma unroll
   for (int u = 0; u < KEEP; ++u) {
     const int c = lane + u * 32;
-    if (c < V) stf(out + c, ov[u] * inv * wv[u] * sigmoidf_(gv[u]));
+    if (c < V) stf(out + c, ov[u] * inv * wv[u] * sigmoidf_(gv[u]) * (p.silu ? gv[u] : 1.f));
   }
-  for (int c = lane + KEEP * 32; c < V; c += 32) stf(out + c, o[c] * inv * ldf(w + c) * sigmoidf_(ldf(g + c)));
+  for (int c = lane + KEEP * 32; c < V; c += 32) {
+    const float gc = ldf(g + c);
+    stf(out + c, o[c] * inv * ldf(w + c) * sigmoidf_(gc) * (p.silu ? gc : 1.f));
+  }
 }
 
 }  // namespace pcs
@@ -1254,7 +1442,8 @@ PCS_API int pcs_delta_inputs(const pcs_shortconv_params* p, const pcs_lowrank_pa
 PCS_API int pcs_delta_scan(const pcs_delta_params* p, void* stream) {
   PCS_REQUIRE(p, "pcs_delta_scan: null params");
   if (p->n_seqs == 0 || p->n_tokens == 0) return PCS_OK;
-  PCS_REQUIRE(p->qk && p->v && p->decay && p->b && p->o && p->s_pool && p->seq_slot && p->seq_pos0 && p->seq_len && p->seq_off, "pcs_delta_scan: null tensor");
+  PCS_REQUIRE(p->qk && p->v && p->b && p->o && p->s_pool && p->seq_slot && p->seq_pos0 && p->seq_len && p->seq_off, "pcs_delta_scan: null tensor");
+  PCS_REQUIRE(p->decay || (p->a && p->dt_bias && p->rate), "pcs_delta_scan: neither decays per channel nor what per-head decays are formed of");
   PCS_REQUIRE(p->heads > 0 && p->heads <= 65535 && p->kv_heads > 0 && p->heads % p->kv_heads == 0 && p->dim > 0 && p->vdim > 0, "pcs_delta_scan: bad sizes");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const bool aligned = p->dim % 4 == 0 && ((reinterpret_cast<uintptr_t>(p->qk) | reinterpret_cast<uintptr_t>(p->decay)) & 15) == 0;
@@ -1266,7 +1455,11 @@ PCS_API int pcs_delta_scan(const pcs_delta_params* p, void* stream) {
     while (W > 1 && blocks(W) < 2 * 148) W /= 2;
     dim3 grid(p->n_seqs, p->heads, (p->vdim + 8 * W - 1) / (8 * W));
 #define PCS_DELTA_REG(MV) \
-  PCS_DISPATCH(p->dtype, (pcs::delta_scan_reg_kernel<T, MV><<<grid, 32 * W, static_cast<size_t>(pcs::kDsRing) * 3 * 16 * MV * sizeof(float), st>>>(*p, W)))
+  PCS_DISPATCH(p->dtype, { \
+    const size_t row = static_cast<size_t>(pcs::kDsRing) * 16 * MV * sizeof(float); \
+    if (p->decay) pcs::delta_scan_reg_kernel<T, MV, false><<<grid, 32 * W, 3 * row, st>>>(*p, W); \
+    else pcs::delta_scan_reg_kernel<T, MV, true><<<grid, 32 * W, 2 * row, st>>>(*p, W); \
+  })
     if (p->dim <= 32) PCS_DELTA_REG(2);
     else if (p->dim <= 64) PCS_DELTA_REG(4);
     else if (p->dim <= 128) PCS_DELTA_REG(8);
@@ -1294,12 +1487,21 @@ PCS_API int pcs_delta_scan(const pcs_delta_params* p, void* stream) {
 PCS_API int pcs_delta_chunk_prep(const pcs_delta_chunk_params* p, void* stream) {
   PCS_REQUIRE(p, "pcs_delta_chunk_prep: null params");
   if (p->n_chunks == 0) return PCS_OK;
-  PCS_REQUIRE(p->qk && p->v && p->ld && p->b && p->chunk_first && p->chunk_len && p->qd && p->kd && p->w && p->g && p->u && p->a, "pcs_delta_chunk_prep: null tensor");
+  PCS_REQUIRE(p->ld || (p->dec_a && p->dt_bias && p->rate), "pcs_delta_chunk_prep: neither log decays per channel nor what per-head decays are formed of");
+  PCS_REQUIRE(p->qk && p->v && p->b && p->chunk_first && p->chunk_len && p->qd && p->kd && p->w && p->g && p->u && p->a, "pcs_delta_chunk_prep: null tensor");
   PCS_REQUIRE(p->heads > 0 && p->heads <= 65535 && p->kv_heads > 0 && p->heads % p->kv_heads == 0 && p->dim > 0 && p->dim <= 256 && p->vdim > 0,
               "pcs_delta_chunk_prep: bad sizes (dim %d of at most 256)", p->dim);
   const int D4 = (p->dim + 3) & ~3;
   const size_t smem = (static_cast<size_t>(3) * pcs::kC * (D4 + 4) + 4 * D4 + pcs::kC * pcs::kC + pcs::kC) * sizeof(float);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (!p->ld) {
+    const size_t smem_h = (static_cast<size_t>(2) * pcs::kC * (((p->dim + 31) & ~31) + 4) + pcs::kC * pcs::kC + 4 * pcs::kC) * sizeof(float);
+    PCS_DISPATCH(p->dtype, PCS_CHECK_CUDA(cudaFuncSetAttribute(pcs::delta_chunk_prep_head_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024)));
+    PCS_DISPATCH(p->dtype, pcs::delta_chunk_prep_head_kernel<T><<<dim3(p->n_chunks, p->heads), pcs::kDpThreads, smem_h, st>>>(*p));
+    PCS_CHECK_CUDA(cudaGetLastError());
+    pcs::count_launch();
+    return PCS_OK;
+  }
   PCS_DISPATCH(p->dtype, PCS_CHECK_CUDA(cudaFuncSetAttribute(pcs::delta_chunk_prep_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024)));
   PCS_DISPATCH(p->dtype, pcs::delta_chunk_prep_kernel<T><<<dim3(p->n_chunks, p->heads), pcs::kDpThreads, smem, st>>>(*p));
   PCS_CHECK_CUDA(cudaGetLastError());

@@ -10,10 +10,11 @@
 //                          values of every head; the result is carried back by U_v,h.
 // pcs_latent_prep   one block per token: RMS norms (32-bit statistics) of the query latent and of c, rotation of the
 //                   shared key part by the token's position, append of [c | rot] to the pool.
-// pcs_latent_q      one block per token: rotation of every head's rotated query part; optionally packs [q'_h | rotated part].
+// pcs_latent_q      one block per token: rotation of every head's rotated query part; optionally packs [q'_h | rotated part]
+//                   (q'_h already in its place, q_lat == q_out, is not copied).
 // pcs_latent_gather / pcs_latent_expand   context rows out of the pool, and per-head rows into the dense pool.
 // pcs_head_gate     the per-head output gate sigmoid(g[t, h]).
-// Rotation pairs coordinate i with i + rot_dim / 2; cos and sin carry a common multiplier (a frequency rescaling's
+// Rotation pairs coordinate i with i + rot_dim / 2, or neighbours (2i, 2i + 1); cos and sin carry a common multiplier (a frequency rescaling's
 // attention factor).  Angles are formed in 64-bit from a host-made frequency table.
 #include "seq_common.cuh"
 
@@ -53,9 +54,10 @@ __global__ void __launch_bounds__(256) latent_prep_kernel(const pcs_latent_prep_
   T* dst = static_cast<T*>(p.pool) + (static_cast<long long>(slot) * p.cap + pos) * (C + R);
   for (int i = threadIdx.x; i < C; i += blockDim.x) stf(dst + i, ldf(ckv + i) * inv * ldf(w + i));
   for (int i = threadIdx.x; i < half; i += blockDim.x) {
-    const float u = ldf(ckv + C + i), v = ldf(ckv + C + half + i);
-    stf(dst + C + i, u * sc[i].y - v * sc[i].x);
-    stf(dst + C + half + i, v * sc[i].y + u * sc[i].x);
+    const int a = p.interleaved ? 2 * i : i, c = p.interleaved ? 2 * i + 1 : half + i;
+    const float u = ldf(ckv + C + a), v = ldf(ckv + C + c);
+    stf(dst + C + a, u * sc[i].y - v * sc[i].x);
+    stf(dst + C + c, v * sc[i].y + u * sc[i].x);
   }
 }
 
@@ -78,18 +80,19 @@ __global__ void __launch_bounds__(256) latent_q_kernel(const pcs_latent_q_params
   for (int e = tid0; e < H * half; e += nthr) {
     const int h = e / half, i = e - h * half;
     const T* s = q + h * (D + R) + D;
-    const float u = ldf(s + i), v = ldf(s + half + i);
+    const int a = p.interleaved ? 2 * i : i, c = p.interleaved ? 2 * i + 1 : half + i;
+    const float u = ldf(s + a), v = ldf(s + c);
     T* d = qo + h * (lead + R) + lead;
-    stf(d + i, u * sc[i].y - v * sc[i].x);
-    stf(d + half + i, v * sc[i].y + u * sc[i].x);
+    stf(d + a, u * sc[i].y - v * sc[i].x);
+    stf(d + c, v * sc[i].y + u * sc[i].x);
   }
-  if (p.q_lat) {
+  if (p.q_lat && p.q_lat != p.q_out) {
     const T* ql = static_cast<const T*>(p.q_lat) + t * p.lat_tok_stride;
     for (int e = tid0; e < H * C; e += nthr) {
       const int h = e / C, c = e - h * C;
       qo[h * (C + R) + c] = ql[h * p.lat_head_stride + c];
     }
-  } else if (p.q_out != p.q) {
+  } else if (!p.q_lat && p.q_out != p.q) {
     for (int e = tid0; e < H * D; e += nthr) {
       const int h = e / D, c = e - h * D;
       qo[h * (D + R) + c] = q[h * (D + R) + c];
@@ -115,8 +118,9 @@ __global__ void __launch_bounds__(256) latent_expand_kernel(const pcs_latent_exp
   const int H = p.n_heads, D = p.dim, V = p.vdim, R = p.rot_dim, C = p.kv_rank;
   const T* kv = static_cast<const T*>(p.kv) + n * p.kv_stride;
   const T* rot = static_cast<const T*>(p.pool) + (static_cast<long long>(slot) * p.cap + pos) * (C + R) + C;
-  T* kd = static_cast<T*>(p.k_dense) + (static_cast<long long>(b) * H * p.cap_dense + pos) * (D + R);
-  T* vd = static_cast<T*>(p.v_dense) + (static_cast<long long>(b) * H * p.cap_dense + pos) * V;
+  const int dense = p.seq_base ? pos - p.seq_base[b] : pos;
+  T* kd = static_cast<T*>(p.k_dense) + (static_cast<long long>(b) * H * p.cap_dense + dense) * (D + R);
+  T* vd = static_cast<T*>(p.v_dense) + (static_cast<long long>(b) * H * p.cap_dense + dense) * V;
   const long long k_head = static_cast<long long>(p.cap_dense) * (D + R), v_head = static_cast<long long>(p.cap_dense) * V;
   for (int e = threadIdx.x; e < H * (D + R); e += blockDim.x) {
     const int h = e / (D + R), i = e - h * (D + R);
@@ -163,7 +167,7 @@ PCS_API int pcs_latent_q(const pcs_latent_q_params* p, void* stream) {
   PCS_REQUIRE(p->q_lat == nullptr || (p->kv_rank > 0 && p->q_out != p->q), "pcs_latent_q: latent queries need kv_rank and an output of their own");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   // few tokens (decoding): a token's copies are spread over several blocks, two elements per thread
-  const int per_token = p->n_heads * ((p->q_lat ? p->kv_rank : (p->q_out != p->q ? p->dim : 0)) + p->rot_dim / 2);
+  const int per_token = p->n_heads * ((p->q_lat ? (p->q_lat != p->q_out ? p->kv_rank : 0) : (p->q_out != p->q ? p->dim : 0)) + p->rot_dim / 2);
   int ny = p->n_tokens >= 256 ? 1 : (per_token + 511) / 512;
   if (ny > 64) ny = 64;
   if (ny < 1) ny = 1;

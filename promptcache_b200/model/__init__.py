@@ -300,6 +300,27 @@ class Zovolorn(LanguageModel):
         raise NotImplementedError("Zovolorn keeps recurrent state next to K/V rows: there is no per-module K/V to cache and splice")
 
 
+class Zepilix(LanguageModel):
+    """Adapter of the Zepilix design (model/zepilix.py) for the generation engine.  Its delta layers carry a state and its convolutions'
+    last inputs from token to token beside the attention layers' rows, so a prompt's state cannot be cut at module boundaries and
+    spliced: pass `cache=None` to `GenerationEngine.generate`, or batch requests with `BatchEngine`."""
+
+    def __init__(self, name: str, model=None, tokenizer=None, **kwargs):
+        from .zepilix import ZepilixForCausalLM
+        if model is None:
+            model = ZepilixForCausalLM.from_pretrained(name, **kwargs)
+        if tokenizer is None:
+            from ..synthetic import IdTokenizer
+            tokenizer = IdTokenizer(model.vocab_size)
+        super().__init__(name, model, tokenizer, [tokenizer.eos_token_id], [])
+
+    def get_formatter(self) -> Callable[[str], str]:
+        return lambda prompt: prompt
+
+    def get_cache_shape(self) -> Tuple[int, int, int]:
+        raise NotImplementedError("Zepilix keeps recurrent state next to K/V and latent rows: there is no per-module K/V to cache and splice")
+
+
 # config.json "architecture" (or transformers' "architectures"/"model_type") -> loader of the bare model
 MODEL_REGISTRY = {
     "Mutolix": lambda path, **kw: _mutolix(path, **kw),
@@ -307,6 +328,7 @@ MODEL_REGISTRY = {
     "Safilorn": lambda path, **kw: _lazy("safilorn", "SafilornForCausalLM").from_pretrained(path, **kw),
     "Tevilix": lambda path, **kw: _lazy("tevilix", "TevilixForCausalLM").from_pretrained(path, **kw),
     "Zovolorn": lambda path, **kw: _lazy("zovolorn", "ZovolornForCausalLM").from_pretrained(path, **kw),
+    "Zepilix": lambda path, **kw: _lazy("zepilix", "ZepilixForCausalLM").from_pretrained(path, **kw),
     "LlamaForCausalLM": lambda path, dtype=None, **kw: LlamaForCausalLM.from_pretrained(path, **kw),
     "FalconForCausalLM": lambda path, dtype=None, **kw: _lazy("falcon", "FalconForCausalLM").from_pretrained(path, **kw),
     "MptForCausalLM": lambda path, dtype=None, **kw: _lazy("mpt", "MptForCausalLM").from_pretrained(path, **kw),
@@ -338,5 +360,5 @@ def load_model(path: str, device="cuda", dtype=None, **kwargs):
     return loader(path, device=device, **kwargs)
 
 
-__all__ = ["LanguageModel", "Mutolix", "Raritar", "Safilorn", "Tevilix", "Zovolorn", "MODEL_REGISTRY", "load_model", "Llama2", "CodeLlama", "Falcon", "Mpt", "FormatConversation",
+__all__ = ["LanguageModel", "Mutolix", "Raritar", "Safilorn", "Tevilix", "Zepilix", "Zovolorn", "MODEL_REGISTRY", "load_model", "Llama2", "CodeLlama", "Falcon", "Mpt", "FormatConversation",
            "FormatLlama2Conversation", "LlamaForCausalLM", "LlamaConfigLite"]

@@ -77,14 +77,15 @@ class SlotPoolCausalLM(nn.Module):
         for seq, toks in entries:
             prev += [seq.last_token if seq.rows > 0 else -1] + [int(t) for t in list(toks)[:-1]]
         parity = [s.steps & 1 for s, _ in entries]
-        decode = max(lens) == 1 and min(pos0) > 0 and len(rows) == len(entries)
+        every = rows == list(range(len(flat)))   # every token's logits, in order
+        decode = max(lens) == 1 and min(pos0) > 0 and every
         logits = None
         if decode and self.use_cuda_graphs and not torch.cuda.is_current_stream_capturing():
             logits = self._decode_replay(flat, slots, pos0, prev, parity)
         if logits is None:
             batch = nsq.Batch(slots, pos0, lens, self._device, parity)
             both = torch.tensor(flat + prev, dtype=torch.int64).pin_memory().to(self._device, non_blocking=True)
-            ids, batch.prev_ids = both[:len(flat)], both[len(flat):]
+            ids, batch.prev_ids, batch.wants_all = both[:len(flat)], both[len(flat):], every
             rows_t = torch.tensor(rows, dtype=torch.int32).pin_memory().to(self._device, non_blocking=True) if rows else None
             logits = self._layers(ids, batch, rows_t)
         for (seq, toks), n in zip(entries, lens):
@@ -107,7 +108,7 @@ class SlotPoolCausalLM(nn.Module):
                 self._graphs.pop(next(iter(self._graphs)))
             batch = nsq.Batch(slots, pos0, [1] * B, self._device, parity)
             both = torch.tensor(flat + prev, dtype=torch.int64, device=self._device)
-            ids, batch.prev_ids = both[:B], both[B:]
+            ids, batch.prev_ids, batch.wants_all = both[:B], both[B:], True
             rows_t = torch.arange(B, dtype=torch.int32, device=self._device)
             torch.cuda.synchronize()
             graph = torch.cuda.CUDAGraph()

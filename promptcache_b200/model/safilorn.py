@@ -33,8 +33,9 @@ import torch
 
 from .. import _native_seq as nsq
 from .. import weights as wio
+from ._latent import latent_attention, load_latent
 from ._seqbase import SlotPoolCausalLM
-from ._state import DecayStateSpec, LatentKVSpec
+from ._state import DecayStateSpec
 
 SWISH_ALPHA = 1.702        # the experts' gate activation g * sigmoid(SWISH_ALPHA * g)
 ATTENTION_FACTOR_COEF = 0.1  # cos and sin are multiplied by ATTENTION_FACTOR_COEF * ln(factor) + 1 when frequencies are rescaled
@@ -122,27 +123,9 @@ class SafilornForCausalLM(SlotPoolCausalLM):
             if blk["depth"].numel() != i + 2:
                 raise ValueError(f"layer {i}: the depth average needs {i + 2} coefficients, the checkpoint has {blk['depth'].numel()}")
             if layer["type"] == "latent_attention":
-                H, D, R, V, C = (int(m[k]) for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank"))
-                rot = m.get("rot") or {}
-                if R and int(rot.get("dims", R)) != R:
-                    raise ValueError(f"layer {i}: the rotation covers {rot.get('dims')} dimensions, the rotated part has {R}")
-                dq, dkv = get(p + "mix.dq"), get(p + "mix.dkv")
-                Q = dq.shape[0]
-                if dkv.shape[0] != C + R:
-                    raise ValueError(f"layer {i}: the key/value down-projection has {dkv.shape[0]} rows, not kv_rank + rot_dim = {C + R}")
+                R, rot = int(m["rot_dim"]), m.get("rot") or {}
                 freqs, mult = ramp_scaled_frequencies(R, float(rot.get("base", 10000.0)), rot.get("scaling")) if R else ([], 1.0)
-                uk, uv = get(p + "mix.uk"), get(p + "mix.uv")
-                blk.update(heads=H, dim=D, rot_dim=R, vdim=V, kv_rank=C, q_rank=Q, scale=float(m["scale"]), rot_mult=float(mult),
-                           freqs=torch.tensor(freqs, dtype=torch.float64, device=dev) if R else None,
-                           # one product of the mixer's input: query latent, key/value latent with the rotated part, head gates
-                           w_in=torch.cat([dq, dkv, get(p + "mix.g")], 0).contiguous(), offs=(0, Q, Q + C + R),
-                           cq_norm=get(p + "mix.dq.norm"), ckv_norm=get(p + "mix.dkv.norm"), w_uq=get(p + "mix.uq"),
-                           w_ukv=torch.cat([uk, uv], 0).contiguous(),             # latents -> plain key parts of all heads, then values
-                           uk_h=uk.view(H, D, C).contiguous(),                    # per head: carries a query into the latent space
-                           uv_t=uv.view(H, V, C).transpose(1, 2).contiguous(),    # per head [C, V]: carries a latent result back
-                           sink=f32(p + "mix.sink").reshape(-1), w_o=get(p + "mix.o"), spec=LatentKVSpec(C, R),
-                           # the latent form's result per head is kv_rank wide: beyond what the decoding kernels hold, only the expanded form runs
-                           latent_ok=C <= nsq.ATTN_MAX_VDIM)
+                blk.update(load_latent(get, p + "mix.", f"layer {i}", m, freqs, rot_mult=mult, gate=get(p + "mix.g"), sink=f32(p + "mix.sink").reshape(-1), device=dev))
             else:
                 H, D, V = (int(m[k]) for k in ("heads", "dim", "vdim"))
                 a1 = get(p + "mix.a1")
@@ -192,52 +175,8 @@ class SafilornForCausalLM(SlotPoolCausalLM):
         return cls(cfg, tensors, device=device, dtype=dtype, max_tokens=max_tokens)
 
     # ---- the mixers ---------------------------------------------------------------------------------------------
-    def _context(self, batch, step):
-        """The step's context tokens (every entry's rows from its first one) as a batch description, and the entries' indices as
-        the dense pool's slots; built once per step, on the first latent-attention layer that expands."""
-        if "ctx" not in step:
-            if all(p0 == 0 for p0 in batch.pos0):
-                step["ctx"] = batch
-            else:
-                step["ctx"] = nsq.Batch(batch.slots, [0] * batch.n_seqs, [p0 + n for p0, n in zip(batch.pos0, batch.lens)], self._device)
-            step["ids"] = torch.arange(batch.n_seqs, dtype=torch.int32, device=self._device)
-        return step["ctx"], step["ids"]
-
     def _latent_attention(self, h, blk, pool, batch, step):
-        T, dt, dev = h.shape[0], self.compute_dtype, self._device
-        H, D, R, V, C, Q = blk["heads"], blk["dim"], blk["rot_dim"], blk["vdim"], blk["kv_rank"], blk["q_rank"]
-        proj = nsq.linear(h, blk["w_in"])
-        cq = torch.empty(T, Q, dtype=dt, device=dev)
-        nsq.latent_prep(proj, blk["offs"][0], blk["offs"][1], Q, C, R, blk["cq_norm"], blk["ckv_norm"], self.eps, blk["freqs"], blk["rot_mult"], cq,
-                        pool["ckv"], batch)
-        q = nsq.linear(cq, blk["w_uq"])                      # [T, H * (D + R)], per head [plain | rotated]
-        # a recorded decoding step reads everything that changes from device buffers: only the latent form does
-        form = "latent" if torch.cuda.is_current_stream_capturing() else (self.latent_form or ("expanded" if batch.max_len >= self.expand_min_len else "latent"))
-        if not blk["latent_ok"]:
-            form = "expanded"
-        if form == "expanded":
-            ctx, ids = self._context(batch, step)
-            c_ctx = nsq.latent_gather(pool["ckv"], C, ctx)
-            kv = nsq.linear(c_ctx, blk["w_ukv"])             # [N, H * D + H * V]
-            cap = ((max(p0 + n for p0, n in zip(batch.pos0, batch.lens)) + 63) // 64) * 64
-            kd = torch.empty(batch.n_seqs, H, cap, D + R, dtype=dt, device=dev)
-            vd = torch.empty(batch.n_seqs, H, cap, V, dtype=dt, device=dev)
-            nsq.latent_expand(kv, pool["ckv"], C, R, H, D, V, kd, vd, ctx)
-            nsq.latent_q(q, H, D, R, blk["freqs"], blk["rot_mult"], batch)
-            o = torch.empty(T, H * V, dtype=dt, device=dev)
-            nsq.attention(q, kd, vd, o, H, blk["scale"], None, None, True, batch, impl=self.attn_impl, sink_logit=blk["sink"], pool_slot=ids)
-            o3 = o.view(T, H, V)
-        else:
-            # q'_h = U_k,h^T q_h: [H, T, D] x [H, D, C]; the rotated parts ride along unchanged
-            q_lat = torch.bmm(q.view(T, H, D + R)[:, :, :D].transpose(0, 1), blk["uk_h"]).transpose(0, 1)   # [T, H, C]
-            ql = nsq.latent_q(q, H, D, R, blk["freqs"], blk["rot_mult"], batch, q_lat=q_lat)
-            o_lat = torch.empty(T, H * C, dtype=dt, device=dev)
-            ws = nsq.attn_workspace(T, H, C, dev) if T <= 32 else None
-            nsq.attention(ql, pool["ckv"], pool["ckv"], o_lat, H, blk["scale"], None, None, True, batch, impl=self.attn_impl, max_keys=self.pool.cap,
-                          workspace=ws, sink_logit=blk["sink"], v_row_stride=C + R)
-            o3 = torch.bmm(o_lat.view(T, H, C).transpose(0, 1), blk["uv_t"]).transpose(0, 1)                  # [T, H, V]
-        mixed = torch.empty(T, H * V, dtype=dt, device=dev)
-        nsq.head_gate(o3, proj[:, blk["offs"][2]:blk["offs"][2] + H], mixed)
+        mixed = latent_attention(h, blk, pool["ckv"], batch, step, self.eps, self.pool.cap, form=self.latent_form, expand_min_len=self.expand_min_len, impl=self.attn_impl)
         return nsq.linear(mixed, blk["w_o"])
 
     def _gla(self, h, blk, pool, batch):
