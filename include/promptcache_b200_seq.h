@@ -531,6 +531,31 @@ int pcs_add_layer_norm(const pcs_addln_params* p, void* stream);
 int pcs_side_gate(const void* u, int64_t u_stride, const void* table, int64_t table_stride, int vocab, int col, const int64_t* ids, void* out,
                   int n_tokens, int dim, int dtype, void* stream);
 
+/* A layer's end with a token-side input, for a few tokens in one launch.  Per token t, with e[c] = table[ids[t], col + c] and c < dim:
+ *   x[t] += sum of the n_y <= 2 results y[i][t];   g = gelu(gate x[t]) * e;   z = proj g;   x[t] += z / sqrt(mean(z^2) + eps) * norm_w (+ x0[t]) (+ step)
+ *   h1[t] = x[t] / sqrt(mean(x[t]^2) + eps) * (w_offset + w1), h2 likewise    (each optional)
+ * A cluster of 8 CTAs per token; everything between the results and h1 / h2 stays in 32-bit. */
+typedef struct pcs_side_params {
+  float* x;                 /* [n_tokens, width] */
+  const void* y[2];         /* `dtype` */
+  int64_t y_stride[2];
+  const int64_t* ids;
+  const void* table;        /* [vocab, table_stride] `dtype` */
+  int64_t table_stride;
+  const void* gate;         /* [dim, width] `dtype` */
+  const void* proj;         /* [width, dim] `dtype` */
+  const void* norm_w;       /* [width] `dtype` */
+  const float* x0;          /* [n_tokens, width] or NULL */
+  const void* step;         /* [width] `dtype` or NULL */
+  const void* w1;
+  void* h1;
+  const void* w2;
+  void* h2;
+  float w_offset, eps;
+  int32_t n_y, vocab, col, n_tokens, width, dim, dtype, reserved;
+} pcs_side_params;
+int pcs_side_boundary(const pcs_side_params* p, void* stream);
+
 /* Element-wise gated recurrence whose gates read only the current token (no dependence on the state).  Per entry and channel c:
  *   z_t = sigmoid(proj[t, z_off + c]),  u_t = proj[t, x_off + c],  cand_t = u_t >= 0 ? u_t + 1/2 : sigmoid(u_t)
  *   S_t = (1 - z_t) S_(t-1) + z_t cand_t                         (32-bit; an entry whose slot holds no tokens starts from zero)

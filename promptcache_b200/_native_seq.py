@@ -21,7 +21,7 @@ EXPORTS = ("pcs_version", "pcs_last_error", "pcs_launch_count", "pcs_attn_worksp
            "pcs_moe_rows_up", "pcs_moe_rows_down", "pcs_moe_plan", "pcs_moe_gather", "pcs_moe_gemm", "pcs_moe_combine", "pcs_silu_mul", "pcs_glu_mul",
            "pcs_depth_mix", "pcs_latent_prep", "pcs_latent_q", "pcs_latent_gather", "pcs_latent_expand", "pcs_head_gate", "pcs_gla_decay", "pcs_gla_scan", "pcs_gla_chunk_prep", "pcs_gla_chunk_scan", "pcs_gla_chunk_out",
            "pcs_add_layer_norm", "pcs_gru_scan", "pcs_group_norm_conv", "pcs_soft_cap", "pcs_short_conv", "pcs_delta_inputs", "pcs_delta_scan", "pcs_delta_chunk_prep", "pcs_delta_chunk_scan",
-           "pcs_head_norm_gate", "pcs_side_gate")
+           "pcs_head_norm_gate", "pcs_side_gate", "pcs_side_boundary")
 GLU_SILU, GLU_CLAMPED_SWISH, GLU_GELU_TANH = 0, 1, 4
 ACT_RELU2, ACT_GELU_ERF = 2, 3          # activations of a feed-forward without a gate branch
 ROUTE_SOFTMAX, ROUTE_SIGMOID = 0, 1
@@ -145,6 +145,13 @@ class pcs_addln_params(C.Structure):
                 ("y_f32", C.c_int32 * 3), ("n_addends", C.c_int32), ("w1", C.c_void_p), ("h1", C.c_void_p), ("w2", C.c_void_p), ("h2", C.c_void_p),
                 ("n_rows", C.c_int32), ("width", C.c_int32), ("eps", C.c_float), ("dtype", C.c_int32), ("rms", C.c_int32), ("w_offset", C.c_float),
                 ("y_norm_w", C.c_void_p), ("copy", C.c_void_p)]
+
+
+class pcs_side_params(C.Structure):
+    _fields_ = [("x", C.c_void_p), ("y", C.c_void_p * 2), ("y_stride", C.c_int64 * 2), ("ids", C.c_void_p), ("table", C.c_void_p), ("table_stride", C.c_int64),
+                ("gate", C.c_void_p), ("proj", C.c_void_p), ("norm_w", C.c_void_p), ("x0", C.c_void_p), ("step", C.c_void_p), ("w1", C.c_void_p), ("h1", C.c_void_p),
+                ("w2", C.c_void_p), ("h2", C.c_void_p), ("w_offset", C.c_float), ("eps", C.c_float), ("n_y", C.c_int32), ("vocab", C.c_int32), ("col", C.c_int32),
+                ("n_tokens", C.c_int32), ("width", C.c_int32), ("dim", C.c_int32), ("dtype", C.c_int32), ("reserved", C.c_int32)]
 
 
 class pcs_gru_params(C.Structure):
@@ -277,6 +284,7 @@ def load() -> C.CDLL:
     for name in ("pcs_delta_chunk_prep", "pcs_delta_chunk_scan"):
         getattr(lib, name).argtypes = [C.POINTER(pcs_delta_chunk_params), C.c_void_p]
     lib.pcs_head_norm_gate.argtypes = [C.POINTER(pcs_headnorm_params), C.c_void_p]
+    lib.pcs_side_boundary.argtypes = [C.POINTER(pcs_side_params), C.c_void_p]
     lib.pcs_side_gate.argtypes = [C.c_void_p, C.c_int64, C.c_void_p, C.c_int64, C.c_int, C.c_int, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_void_p]
     for name in EXPORTS[4:]:
         getattr(lib, name).restype = C.c_int
@@ -1062,6 +1070,39 @@ def side_gate(u: torch.Tensor, table: torch.Tensor, col: int, ids: torch.Tensor)
     _check(load().pcs_side_gate(u.data_ptr(), u.stride(0), table.data_ptr(), table.stride(0), table.shape[0], int(col), ids.data_ptr(), out.data_ptr(), u.shape[0],
                                 u.shape[1], dtype_code(u.dtype), _stream()), "pcs_side_gate")
     return out
+
+
+SIDE_BOUNDARY_MAX_TOKENS = 16   # more tokens read the two matrices from L2 too often
+
+
+def side_boundary(x: torch.Tensor, results, ids: torch.Tensor, table: torch.Tensor, col: int, gate: torch.Tensor, proj: torch.Tensor, norm_w: torch.Tensor, eps: float,
+                  x0: Optional[torch.Tensor] = None, step: Optional[torch.Tensor] = None, w1: Optional[torch.Tensor] = None, h1: Optional[torch.Tensor] = None,
+                  w2: Optional[torch.Tensor] = None, h2: Optional[torch.Tensor] = None, w_offset: float = 0.0) -> None:
+    """x += the (at most two) `results` [T, width]; g = gelu(gate x) * table[ids, col:col + dim]; x += rms(proj g) * norm_w (+ x0) (+ step); h1 / h2 =
+    rms(x) * (w_offset + w1 / w2).  One launch, made for a few tokens."""
+    results = list(results)
+    _cuda(x, ids, table, gate, proj, norm_w, x0, step, w1, h1, w2, h2, *results)
+    dt, (T, W), S = gate.dtype, x.shape, gate.shape[0]
+    if x.dtype != torch.float32 or not x.is_contiguous() or len(results) > 2 or ids.dtype != torch.int64 or not ids.is_contiguous() or ids.numel() != T:
+        raise NativeError("side_boundary: x contiguous float32 [T, width], at most two results, ids contiguous int64 [T]")
+    if tuple(gate.shape) != (S, W) or tuple(proj.shape) != (W, S) or any(t.dtype != dt or not t.is_contiguous() for t in (gate, proj, norm_w, table)) or norm_w.numel() != W \
+            or table.dim() != 2 or col + S > table.shape[1]:
+        raise NativeError("side_boundary: gate [dim, width], proj [width, dim], norm_w [width], table [vocab, columns], contiguous in one type")
+    if x0 is not None and (x0.dtype != torch.float32 or not x0.is_contiguous() or x0.shape != x.shape):
+        raise NativeError("side_boundary: x0 must be contiguous float32 of x's shape")
+    for w, h in ((step, None), (w1, h1), (w2, h2)):
+        if w is not None and (w.dtype != dt or not w.is_contiguous() or w.numel() != W or (w is not step and (h is None or h.dtype != dt or not h.is_contiguous() or h.shape != x.shape))):
+            raise NativeError("side_boundary: step, w1, w2 are [width], h1 and h2 [T, width], contiguous in the compute type")
+    p = pcs_side_params()
+    for j, y in enumerate(results):
+        _rows2d(y, dt, "side_boundary: a result")
+        if y.shape != x.shape:
+            raise NativeError("side_boundary: a result must have x's shape")
+        p.y[j], p.y_stride[j] = y.data_ptr(), y.stride(0)
+    p.x, p.ids, p.table, p.table_stride, p.gate, p.proj, p.norm_w = x.data_ptr(), ids.data_ptr(), table.data_ptr(), table.stride(0), gate.data_ptr(), proj.data_ptr(), norm_w.data_ptr()
+    p.x0, p.step, p.w1, p.h1, p.w2, p.h2 = _ptr(x0), _ptr(step), _ptr(w1), _ptr(h1) if w1 is not None else None, _ptr(w2), _ptr(h2) if w2 is not None else None
+    p.w_offset, p.eps, p.n_y, p.vocab, p.col, p.n_tokens, p.width, p.dim, p.dtype = float(w_offset), float(eps), len(results), table.shape[0], int(col), T, W, S, dtype_code(dt)
+    _check(load().pcs_side_boundary(C.byref(p), _stream()), "pcs_side_boundary")
 
 
 def gru_scan(proj: torch.Tensor, offs, width: int, out: torch.Tensor, s_pool: torch.Tensor, batch: Batch) -> None:

@@ -172,6 +172,7 @@ class ZepilixForCausalLM(SlotPoolCausalLM):
         self.scan_impl = 0           # delta rule: 0 by step, 1 / 2 token by token, 3 in chunks
         self.latent_form = None      # None: by step (prompts expanded, decoding in the latent space); "expanded" / "latent" force one
         self.expand_min_len = 16     # steps whose longest entry brings at least this many tokens attend over expanded keys
+        self.fused_side = None       # a layer's end in one launch: None: for a few tokens; True / False force it
         self._init_runtime(dev, max_tokens)
         if not all(b.get("latent_ok", True) for b in self.blocks):
             self.use_cuda_graphs = False   # the expanded form describes the step's context on the host: it is not recorded
@@ -257,6 +258,15 @@ class ZepilixForCausalLM(SlotPoolCausalLM):
             if nxt is not None or addends:
                 nsq.add_rms_norm(x, addends, eps, nxt["norm1"] if nxt else None, h1, nxt.get("norm2") if nxt else None, h2, w_offset=off, y_norm_w=normed)
 
+        def side_end(r: int, blk: dict, ys: list) -> None:
+            """A layer's end for a few tokens in one launch: its sublayers' sum, its side input, what enters before run r and run r's inputs."""
+            nxt = self.blocks[self.runs[r]] if r < len(self.runs) else None
+            t = self.passes.get(r)
+            nsq.side_boundary(x, [y for y, _ in ys], ids, self.side_table, blk["side_col"], blk["side_gate"], blk["side_proj"], blk["side_norm"], eps,
+                              x0=x0 if t else None, step=self.loop_step[t] if t is not None else None, w1=nxt["norm1"] if nxt else None, h1=h1,
+                              w2=nxt.get("norm2") if nxt else None, h2=h2, w_offset=off)
+
+        fused_side = self.fused_side if self.fused_side is not None else T <= nsq.SIDE_BOUNDARY_MAX_TOKENS
         boundary(0, [])
         for r, li in enumerate(self.runs):
             blk, st = self.blocks[li], self.pool.layers[r]
@@ -265,6 +275,9 @@ class ZepilixForCausalLM(SlotPoolCausalLM):
                 ys.append((self._feed_forward(h2, blk), 1.0))
             if self.side_table is None:
                 boundary(r + 1, ys)
+                continue
+            if fused_side and self.layer_trace is None:
+                side_end(r + 1, blk, ys)
                 continue
             xc = torch.empty(T, W, dtype=dt, device=dev)
             nsq.add_rms_norm(x, ys, eps, copy=xc)
