@@ -9,6 +9,7 @@ import ctypes as C
 import os
 from typing import Optional
 
+import numpy as np
 import torch
 
 from ._native import NativeError, note_replayed_launches  # noqa: F401  (one error type for both libraries)
@@ -298,7 +299,7 @@ def _check(rc: int, what: str) -> None:
 
 
 def _stream() -> int:
-    return torch.cuda.current_stream().cuda_stream
+    return torch._C._cuda_getCurrentRawStream(torch._C._cuda_getDevice())   # (the stream object itself costs the host microseconds per launch)
 
 
 def dtype_code(dtype: torch.dtype) -> int:
@@ -336,13 +337,16 @@ class Batch:
     def __init__(self, slots, pos0, lens, device, parity=None):
         n_seqs, n_tokens = len(slots), int(sum(lens))
         parity = list(parity) if parity is not None else [0] * n_seqs
-        offs, tok_seq, tok_pos, o = [], [], [], 0
+        offs, o = [], 0
+        host = np.empty(2 * n_tokens + 5 * n_seqs, dtype=np.int32)   # tok_seq | tok_pos | slots | pos0 | lens | offsets | parity
         for b, (p0, n) in enumerate(zip(pos0, lens)):
             offs.append(o)
-            tok_seq += [b] * n
-            tok_pos += range(p0, p0 + n)
+            host[o:o + n] = b
+            host[n_tokens + o:n_tokens + o + n] = np.arange(p0, p0 + n, dtype=np.int32)
             o += n
-        host = torch.tensor(tok_seq + tok_pos + list(slots) + list(pos0) + list(lens) + offs + parity, dtype=torch.int32)
+        for i, part in enumerate((slots, pos0, lens, offs, parity)):
+            host[2 * n_tokens + i * n_seqs:2 * n_tokens + (i + 1) * n_seqs] = part
+        host = torch.from_numpy(host)
         self.meta = host.pin_memory().to(device, non_blocking=True) if device.type == "cuda" else host
         T, B = n_tokens, n_seqs
         m = self.meta
@@ -940,14 +944,14 @@ def _gla_chunk_plan(batch: Batch, chunk: int):
         return plan
     first, length, seq0, seqn, tok_row = [], [], [], [], []
     for off, n in zip(batch.offsets, batch.lens):
-        seq0.append(len(first))
+        c0 = len(first)
+        seq0.append(c0)
         seqn.append((n + chunk - 1) // chunk)
-        for c in range(0, n, chunk):
-            tok_row += range(len(first) * chunk, len(first) * chunk + min(chunk, n - c))
-            first.append(off + c)
-            length.append(min(chunk, n - c))
+        tok_row.append(np.arange(c0 * chunk, c0 * chunk + n, dtype=np.int32))   # only an entry's last chunk is short
+        first += range(off, off + n, chunk)
+        length += [min(chunk, n - c) for c in range(0, n, chunk)]
     nc = len(first)
-    host = torch.tensor(first + length + seq0 + seqn + tok_row, dtype=torch.int32)
+    host = torch.from_numpy(np.concatenate([np.asarray(first + length + seq0 + seqn, dtype=np.int32)] + tok_row))
     dev = host.pin_memory().to(batch.meta.device, non_blocking=True)
     B = batch.n_seqs
     plan = {"chunk": chunk, "n_chunks": nc, "first": dev[:nc], "len": dev[nc:2 * nc], "seq0": dev[2 * nc:2 * nc + B], "seqn": dev[2 * nc + B:2 * nc + 2 * B],

@@ -3,7 +3,7 @@
 feed-forward of the same active size, which share the step function, the pool and the attention kernels) and
 `bench.py --design safilorn` (against Mutolix with the same order and sizes of recurrent and attention layers) and
 `bench.py --design tevilix` (against the same Mutolix model; its four layers run as a loop where Mutolix repeats them) and `bench.py --design
-zovolorn` (against the same Mutolix model).  Random weights, synthetic token ids.  Prefill and decode tokens/s of both models through their own
+zovolorn` (against the same Mutolix model) and `bench.py --design zepilix` (against Safilorn with dense feed-forwards).  Random weights, synthetic token ids.  Prefill and decode tokens/s of both models through their own
 step / forward, then every kernel of the new design alone against its roofline, next to the like kernel of the Llama path.
 
 Timing: CUDA events on the launching stream, >= 3 warm-up iterations, a 256 MiB write between timed iterations (flushes the
@@ -1019,7 +1019,234 @@ def run_zovolorn(args, load_peaks, ClockSampler) -> None:
     line["clocks"] = sampler.stop()
     print(json.dumps(line), flush=True)
 
+# ---- Zepilix ----------------------------------------------------------------------------------------------------------
+ZEPILIX_SIZES = {
+    # the recurrent sizes of SIZES, Safilorn's latent sizes under a window, full attention at SIZES' heads, a token-side input of width / 16
+    "w1024": dict(SIZES["w1024"], R=32, LD=96, C=256, Q=512, window=512, conv=4, side=64, gff=2752, rank=16, tau=16.0),
+    "w2048": dict(SIZES["w2048"], R=32, LD=96, C=512, Q=768, window=512, conv=4, side=128, gff=5504, rank=32, tau=16.0),
+}
+
+
+def zepilix_config(s: dict) -> dict:
+    mlp = {"kind": "dense", "ff": s["gff"]}
+    delta = {"type": "delta", "mlp": mlp, "mixer": {"heads": s["mH"], "kv_heads": s["mH"], "dim": s["mD"], "vdim": s["mV"], "conv": s["conv"]}}
+    att = {"type": "attention", "mlp": mlp, "mixer": {"heads": s["H"], "kv_heads": s["G"], "dim": s["D"], "vdim": s["D"], "scale": s["D"] ** 0.5,
+                                                      "rot": {"base": 10000.0, "dims": s["D"]}}}
+    lat = {"type": "latent_attention", "mlp": mlp,
+           "mixer": {"heads": s["H"], "dim": s["LD"], "rot_dim": s["R"], "vdim": s["V"], "kv_rank": s["C"], "q_rank": s["Q"], "scale": (s["LD"] + s["R"]) ** -0.5,
+                     "rot": {"base": 10000.0, "dims": s["R"]}, "mask": {"size": s["window"]}}}
+    return {"architecture": "Zepilix", "vocab": s["vocab"], "width": s["width"], "norm": {"eps": 1e-5}, "token_side": {"dim": s["side"]},
+            "layers": [delta, lat, att, delta] * s["repeat"]}
+
+
+def zepilix_tensors(cfg: dict, device, seed: int = 0) -> Dict[str, torch.Tensor]:
+    g = torch.Generator(device=device).manual_seed(seed)
+    W, S, t = cfg["width"], cfg["token_side"]["dim"], {}
+    rnd = lambda *shape, std=1.0, mean=0.0: (torch.randn(*shape, generator=g, device=device) * std + mean).to(torch.bfloat16)
+    lin = lambda o, i: rnd(o, i, std=i ** -0.5)
+    t["embed"], t["final.norm"], t["side.embed"] = rnd(cfg["vocab"], W), rnd(W, std=0.05), rnd(cfg["vocab"], S * len(cfg["layers"]))
+    for i, layer in enumerate(cfg["layers"]):
+        p, m, ff = f"l{i}.", layer["mixer"], layer["mlp"]["ff"]
+        q = p + "mix."
+        t[p + "norm1"], t[p + "norm2"] = rnd(W, std=0.05), rnd(W, std=0.05)
+        t[p + "side.gate"], t[p + "side.proj"], t[p + "side.norm"] = lin(S, W), lin(W, S), rnd(W, std=0.05, mean=0.3)
+        if layer["type"] == "delta":
+            H, G, D, V = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+            for n, rows in (("q", G * D), ("k", G * D), ("v", H * V)):
+                t[q + n], t[q + n + ".conv"] = lin(rows, W), rnd(rows, m["conv"], std=0.4)
+            t[q + "a"], t[q + "b"], t[q + "g"], t[q + "o"] = lin(H, W), lin(H, W), lin(H * V, W), lin(W, H * V)
+            t[q + "A_log"], t[q + "dt_bias"], t[q + "norm"] = rnd(H, std=0.3, mean=-2.0), rnd(H), rnd(V, std=0.05, mean=1.0)
+        elif layer["type"] == "attention":
+            t[q + "q"], t[q + "k"], t[q + "o"] = lin(m["heads"] * m["dim"], W), lin(m["kv_heads"] * m["dim"], W), lin(W, m["heads"] * m["dim"])
+        else:
+            H, D, R, V, C, Q = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"], m["q_rank"]
+            t[q + "dq"], t[q + "dq.norm"], t[q + "uq"] = lin(Q, W), rnd(Q, std=0.05, mean=1.0), lin(H * (D + R), Q)
+            t[q + "dkv"], t[q + "dkv.norm"], t[q + "uk"], t[q + "uv"], t[q + "o"] = lin(C + R, W), rnd(C, std=0.05, mean=1.0), lin(H * D, C), lin(H * V, C), lin(W, H * V)
+        t[p + "mlp.gate"], t[p + "mlp.up"], t[p + "mlp.down"] = lin(ff, W), lin(ff, W), lin(W, ff)
+        t[p + "mlp.gate.b"], t[p + "mlp.up.b"], t[p + "mlp.down.b"] = rnd(ff, std=0.1), rnd(ff, std=0.1), rnd(W, std=0.1)
+    return t
+
+
+def zepilix_block(s: dict, dev, timer: Timer, prompt: int, batch: int, ctx: int) -> dict:
+    from .model.safilorn import SafilornConfig, SafilornForCausalLM
+    from .model.zepilix import ZepilixConfig, ZepilixForCausalLM
+    cfg = zepilix_config(s)
+    out = {"layers": len(cfg["layers"]), "width": s["width"]}
+    m = ZepilixForCausalLM(ZepilixConfig(cfg), zepilix_tensors(cfg, dev), device=dev, dtype=torch.bfloat16)
+    _throughput(m, s, timer, prompt, batch, ctx, out)
+    del m
+    torch.cuda.empty_cache()
+    # the closest existing model: gated linear attention where this one has the delta rule, latent attention in both other layers, dense feed-forwards
+    sc = safilorn_config(dict(s, D=s["LD"], E=2, top=1, eff=8))
+    for layer in sc["layers"]:
+        layer["mlp"] = {"kind": "dense", "ff": s["gff"]}
+    mm = SafilornForCausalLM(SafilornConfig(sc), safilorn_tensors(sc, s, dev), device=dev, dtype=torch.bfloat16)
+    _throughput(mm, s, timer, prompt, batch, ctx, out, prefix="safilorn_")
+    del mm
+    torch.cuda.empty_cache()
+    return out
+
+
+def zepilix_kernels(s: dict, dev, timer: Timer, prompt: int, ctx: int, hbm_gbs: float, tflops: float) -> dict:
+    """Every kernel of the design alone at this size, achieved / peak, beside the like kernel of Safilorn, Zovolorn, Tevilix or Mutolix."""
+    from . import _native_seq as nsq
+    bf, H, G, D, W, win = torch.bfloat16, s["H"], s["G"], s["D"], s["width"], s["window"]
+    out = {}
+    gb = lambda by, ms: {"us": round(ms * 1e3, 2), "gb_s": round(by / ms / 1e6, 1), "of_measured_hbm_peak": round(by / ms / 1e6 / hbm_gbs, 4)}
+    tf = lambda fl, ms: {"ms": round(ms, 4), "tflops": round(fl / ms / 1e9, 1), "of_measured_bf16_peak": round(fl / ms / 1e9 / tflops, 3)}
+    ones = lambda *n: torch.ones(*n, device=dev, dtype=bf)
+    rnd = lambda *n: torch.randn(*n, device=dev).to(bf)
+
+    def replay(fn):
+        """Milliseconds of fn as decoding runs it: recorded once, replayed (no host work between its launches)."""
+        fn()
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            fn()
+        return timer(graph.replay, steps=15)
+
+    cap = ((max(prompt, ctx + 1) + 127) // 128) * 128
+    b, b1 = nsq.Batch([0], [0], [prompt], dev), nsq.Batch([0], [ctx], [1], dev)
+    full, wpairs = prompt * (prompt + 1) / 2, sum(min(i + 1, win) for i in range(prompt))
+    r1, r2 = torch.full((H,), 0.5, device=dev), torch.full((H,), 0.5, device=dev)
+    # full attention: FLOPs = 2 (D + V) per (query, visible key) pair and head; one decoded token: bytes = K and V rows of every key/value head
+    kp, vp, q, o = rnd(1, G, cap, D), rnd(1, G, cap, D), rnd(prompt, H * D), torch.empty(prompt, H * D, device=dev, dtype=bf)
+    ms = timer(lambda: nsq.attention(q, kp, vp, o, H, D ** -0.5, None, None, False, b))
+    out["attn_prompt"] = tf(4.0 * D * H * full, ms)
+    ms = timer(lambda: nsq.attention(q, kp, vp, o, H, D ** -0.5, r1, r2, True, b))
+    out["like_attn_prompt"] = tf(4.0 * D * H * full, ms)
+    q1, o1, ws = rnd(1, H * D), torch.empty(1, H * D, device=dev, dtype=bf), nsq.attn_workspace(1, H, D, dev)
+    ms = replay(lambda: nsq.attention(q1, kp, vp, o1, H, D ** -0.5, None, None, False, b1, max_keys=cap, workspace=ws))
+    out["attn_decode"] = gb(4.0 * G * (ctx + 1) * D, ms)
+    ms = replay(lambda: nsq.attention(q1, kp, vp, o1, H, D ** -0.5, r1, r2, True, b1, max_keys=cap, workspace=ws))
+    out["like_attn_decode"] = gb(4.0 * G * (ctx + 1) * D, ms)
+    nq, nk = H * D, G * D
+    pj, un, qn, kn = rnd(prompt, nq + 2 * nk), ones(D), ones(nq), ones(nk)
+    fr = torch.tensor([10000.0 ** (-2.0 * i / D) for i in range(D // 2)], dtype=torch.float64, device=dev)
+    ms = timer(lambda: nsq.rope_kv_prep(pj, (0, nq, nq), H, G, D, D, fr, D, True, False, 1e-5, q, kp, vp, b, q_norm_w=un, k_norm_w=un))
+    out["unit_heads_rope_append_values_are_keys"] = gb(prompt * 2.0 * (nq + nk + nq + 2 * nk), ms)
+    ms = timer(lambda: nsq.rope_kv_prep(pj, (0, nq, nq + nk), H, G, D, D, fr, D, True, False, 1e-5, q, kp, vp, b, q_norm_w=qn, k_norm_w=kn, norm_whole=True))
+    out["like_whole_norm_rope_append"] = gb(prompt * 4.0 * (nq + 2 * nk), ms)
+    # latent attention under a window: expanded for prompts, the cached rows themselves for a decoded token
+    R, LD, V, C, Q = s["R"], s["LD"], s["V"], s["C"], s["Q"]
+    kd, vd, ql, ol, ids = rnd(1, H, cap, LD + R), rnd(1, H, cap, V), rnd(prompt, H * (LD + R)), torch.empty(prompt, H * V, device=dev, dtype=bf), torch.zeros(1, dtype=torch.int32, device=dev)
+    ms = timer(lambda: nsq.attention(ql, kd, vd, ol, H, 0.1, None, None, False, b, pool_slot=ids, window=win))
+    out["latent_attn_prompt_window"] = tf(2.0 * (LD + R + V) * H * wpairs, ms)
+    kg, vg = rnd(1, G, cap, LD + R), rnd(1, G, cap, V)
+    ms = timer(lambda: nsq.attention(ql, kg, vg, ol, H, 0.1, r1, r2, True, b, window=win))
+    out["like_attn_prompt_window"] = tf(2.0 * (LD + R + V) * H * wpairs, ms)
+    pool, qz, oz, wz = rnd(1, 1, cap, C + R), rnd(1, H * (C + R)), torch.empty(1, H * C, device=dev, dtype=bf), nsq.attn_workspace(1, H, C, dev)
+    ms = replay(lambda: nsq.attention(qz, pool, pool, oz, H, 0.1, None, None, False, b1, max_keys=win, workspace=wz, v_row_stride=C + R, window=win))
+    out["latent_attn_decode_window"] = gb(2.0 * win * (C + R), ms)
+    bw, sink = nsq.Batch([0], [win - 1], [1], dev), torch.randn(H, device=dev)
+    ms = replay(lambda: nsq.attention(qz, pool, pool, oz, H, 0.1, None, None, True, bw, max_keys=win, workspace=wz, sink_logit=sink, v_row_stride=C + R))
+    out["like_latent_attn_decode_as_many_keys"] = gb(2.0 * win * (C + R), ms)
+    pl, cq, wq_, wc_ = rnd(prompt, Q + C + R), torch.empty(prompt, Q, device=dev, dtype=bf), ones(Q), ones(C)
+    fl = torch.tensor([10000.0 ** (-2.0 * i / R) for i in range(R // 2)], dtype=torch.float64, device=dev)
+    for il, name in ((True, "latent_prep_pairs"), (False, "like_latent_prep_halves")):
+        ms = timer(lambda: nsq.latent_prep(pl, 0, Q, Q, C, R, wq_, wc_, 1e-5, fl, 1.0, cq, pool, b, interleaved=il))
+        out[name] = gb(prompt * (Q + C + R) * 4.0, ms)
+    for il, name in ((True, "latent_q_pairs"), (False, "like_latent_q_halves")):
+        ms = timer(lambda: nsq.latent_q(ql, H, LD, R, fl, 1.0, b, interleaved=il))
+        out[name] = gb(prompt * H * R * 4.0, ms)
+    wukv = (torch.randn(H * (LD + V), C, device=dev) * C ** -0.5).to(bf)
+    ms = timer(lambda: nsq.latent_expand(nsq.linear(nsq.latent_gather(pool, C, b), wukv), pool, C, R, H, LD, V, kd, vd, b))
+    out["latent_expand_chain"] = tf(2.0 * prompt * C * H * (LD + V), ms)
+    # layer end: the sum with the copy (x 4 B read and written, two results, the copy 2 B each); the normed side input with both next norms
+    S = s["side"]
+    x, y, f, wn, h1, h2 = torch.randn(prompt, W, device=dev), rnd(prompt, W), rnd(prompt, W), ones(W), torch.empty(prompt, W, device=dev, dtype=bf), torch.empty(prompt, W, device=dev, dtype=bf)
+    ms = timer(lambda: nsq.add_rms_norm(x, [(y, 1.0), (f, 1.0)], 1e-5, copy=h1))
+    out["add_copy"] = gb(prompt * W * 14.0, ms)
+    ms = timer(lambda: nsq.add_rms_norm(x, [(y, 1.0)], 1e-5, wn, h1, wn, h2, w_offset=1.0, y_norm_w=wn))
+    out["side_norm_add_two_norms"] = gb(prompt * W * 14.0, ms)
+    ms = timer(lambda: nsq.add_layer_norm(x, [(y, 1.0), (f, 1.0)], 1e-5, wn, h1, wn, h2))
+    out["like_add_two_layer_norms"] = gb(prompt * W * 16.0, ms)
+    gw, pw, table, tid = (torch.randn(S, W, device=dev) * W ** -0.5).to(bf), (torch.randn(W, S, device=dev) * S ** -0.5).to(bf), rnd(s["vocab"], 4 * S), torch.randint(0, s["vocab"], (prompt,), device=dev)
+    u = rnd(prompt, S)
+    ms = timer(lambda: nsq.side_gate(u, table, S, tid))
+    out["side_gate"] = gb(prompt * S * 6.0, ms)
+    us = torch.cat([u, u], 1)
+    ms = timer(lambda: nsq.glu_mul(us, S))
+    out["like_glu_mul_same_size"] = gb(prompt * S * 6.0, ms)
+    x1, y1, f1, i1 = x[:1].contiguous(), y[:1].contiguous(), f[:1].contiguous(), tid[:1].contiguous()
+
+    def layer_end():
+        xc = torch.empty(1, W, device=dev, dtype=bf)
+        nsq.add_rms_norm(x1, [(y1, 1.0), (f1, 1.0)], 1e-5, copy=xc)
+        z = nsq.linear(nsq.side_gate(nsq.linear(xc, gw), table, S, i1), pw)
+        nsq.add_rms_norm(x1, [(z, 1.0)], 1e-5, wn, h1[:1], wn, h2[:1], w_offset=1.0, y_norm_w=wn)
+
+    ms = replay(lambda: nsq.side_boundary(x1, [y1, f1], i1, table, S, gw, pw, wn, 1e-5, w1=wn, h1=h1[:1], w2=wn, h2=h2[:1], w_offset=1.0))
+    out["side_boundary_decode"] = gb(4.0 * S * W + 18.0 * W, ms)
+    out["side_boundary_decode_as_five_launches_us"] = round(replay(layer_end) * 1e3, 2)
+    wl = (torch.randn(2 * S, W, device=dev) * W ** -0.5).to(bf)
+    ms = replay(lambda: nsq.linear(y1, wl, kernel=True))
+    out["like_linear_rows_same_bytes"] = gb(4.0 * S * W, ms)
+    ms = replay(lambda: nsq.add_layer_norm(x1, [(y1, 1.0), (f1, 1.0)], 1e-5, wn, h1[:1], wn, h2[:1]))
+    out["like_add_two_layer_norms_decode_us"] = round(ms * 1e3, 2)
+    # the delta rule: its inputs, a prompt, one decoded token (state read and written once)
+    mH, mD, mV = s["mH"], s["mD"], s["mV"]
+    ch = 2 * mH * mD + mH * mV
+    pr = (torch.randn(prompt, ch + mH * mV + 2 * mH + 8, device=dev) * 0.5).to(bf)
+    cv, ctail = (torch.randn(s["conv"], ch, device=dev) * 0.4).to(bf), torch.zeros(1, 2, s["conv"] - 1, ch, device=dev)
+    ms = timer(lambda: nsq.short_conv(pr, 0, mH, mD, mH * mV, cv, ctail, mD ** -0.5, 1e-6, b))
+    out["short_conv"] = gb(prompt * (2.0 * ch + 8.0 * mH * mD + 2.0 * mH * mV), ms)
+    out["short_conv_decode_us"] = round(replay(lambda: nsq.short_conv(pr[:1], 0, mH, mD, mH * mV, cv, ctail, mD ** -0.5, 1e-6, b1)) * 1e3, 2)
+    qk, v = nsq.short_conv(pr, 0, mH, mD, mH * mV, cv, ctail, mD ** -0.5, 1e-6, b)
+    sp, nw, og = torch.zeros(1, mH, mD, mV, device=dev), ones(mV), torch.empty(prompt, mH * mV, device=dev, dtype=bf)
+    gate, at, bt = pr[:, ch:ch + mH * mV], pr[:, ch + mH * mV:ch + mH * mV + mH], pr[:, ch + mH * mV + mH:ch + mH * mV + 2 * mH]
+    dtb, rate = torch.randn(mH, device=dev), torch.full((mH,), 0.1, device=dev)
+    rec = lambda ms, n=prompt: {"ms": round(ms, 3), "us_per_token": round(ms * 1e3 / n, 3), "gflops": round(4.0 * mH * mD * mV * n / ms / 1e6, 1)}
+    head = lambda n, bb, impl=0: nsq.delta_scan(qk[:n], v[:n], None, bt[:n], mH, sp, nw, gate[:n], og[:n], 1e-5, bb, impl=impl, head_decay=(at[:n], dtb, rate), gate_silu=True)
+    out["delta_scan_prompt"] = rec(timer(lambda: head(prompt, b), steps=5))
+    out["delta_scan_prompt_token_by_token"] = rec(timer(lambda: head(prompt, b, 2), steps=5))
+    out["delta_scan_decode"] = gb(8.0 * mH * mD * mV, replay(lambda: head(1, b1)))
+    ld = -torch.rand(prompt, mH * mD, device=dev) * 0.1
+    dec = torch.exp(ld)
+    out["like_delta_scan_prompt_decay_per_channel"] = rec(timer(lambda: nsq.delta_scan(qk, v, ld, bt, mH, sp, nw, gate, og, 1e-5, b), steps=5))
+    ms = replay(lambda: nsq.delta_scan(qk[:1], v[:1], dec[:1], bt[:1], mH, sp, nw, gate[:1], og[:1], 1e-5, b1))
+    out["like_delta_scan_decode_decay_per_channel"] = gb(8.0 * mH * mD * mV, ms)
+    pm, goffs = (torch.randn(prompt, 2 * mH * mD + 2 * mH * mV, device=dev) * 0.3).to(bf), (0, mH * mD, 2 * mH * mD, 2 * mH * mD + mH * mV)
+    out["like_gla_scan_prompt"] = rec(timer(lambda: nsq.gla_scan(pm, goffs, ld, nw, og, sp, 1e-5, b), steps=5))
+    ms = replay(lambda: nsq.gla_scan(pm[:1], goffs, ld[:1], nw, og[:1], sp, 1e-5, b1))
+    out["like_gla_scan_decode"] = gb(8.0 * mH * mD * mV, ms)
+    # feed-forward activation
+    ff = s["gff"]
+    gu = rnd(prompt, 2 * ff)
+    out["silu_mul"] = gb(prompt * ff * 6.0, timer(lambda: nsq.glu_mul(gu, ff)))
+    out["like_gelu_tanh_mul"] = gb(prompt * ff * 6.0, timer(lambda: nsq.glu_mul(gu, ff, (nsq.GLU_GELU_TANH, 0.0, 0.0))))
+    return out
+
+
+def run_zepilix(args, load_peaks, ClockSampler) -> None:
+    from . import _native_seq as nsq
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    nsq.load()
+    hbm, kind, tfl = load_peaks()
+    timer = Timer(dev)
+    sampler = ClockSampler(0)
+    sampler.start()
+    sampler.mark()
+    before = nsq.launch_count()
+    line = {"design": "zepilix", "compared_with": "safilorn (gated linear attention where this design has the delta rule, latent attention in the other layers, dense feed-forwards, at "
+                                                  "the same sizes) on the same step function, pool and kernels",
+            "dtype": "bf16", "data": "synthetic", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tfl, "kind": kind},
+            "timing": "CUDA events, 3 warm-up iterations, 256 MiB L2 flush between iterations, median", "sizes": {}}
+    prompt, batch, ctx = 2048, 4, 2048
+    for name, s in ZEPILIX_SIZES.items():
+        blk = zepilix_block(s, dev, timer, prompt, batch, ctx)
+        blk["kernels"] = zepilix_kernels(s, dev, timer, prompt, ctx, hbm, tfl)
+        line["sizes"][name] = blk
+    line["gpu_launches"] = nsq.launch_count() - before
+    line["clocks"] = sampler.stop()
+    print(json.dumps(line), flush=True)
+
+
 def run(args, load_peaks, ClockSampler) -> None:
+    if args.design == "zepilix":
+        return run_zepilix(args, load_peaks, ClockSampler)
     if args.design == "zovolorn":
         return run_zovolorn(args, load_peaks, ClockSampler)
     if args.design == "tevilix":

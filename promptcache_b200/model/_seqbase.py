@@ -8,6 +8,7 @@ from __future__ import annotations
 
 from typing import List, Optional, Sequence, Tuple
 
+import numpy as np
 import torch
 import torch.nn as nn
 
@@ -72,20 +73,23 @@ class SlotPoolCausalLM(nn.Module):
                     raise ValueError(f"wanted place {i} is outside the {n} tokens of entry {b}")
                 rows.append(off + i)
             off += n
-        flat = [int(t) for _, toks in entries for t in toks]
-        prev = []   # every token's predecessor in its own sequence (-1: none)
-        for seq, toks in entries:
-            prev += [seq.last_token if seq.rows > 0 else -1] + [int(t) for t in list(toks)[:-1]]
+        both = np.empty((2, off), dtype=np.int64)   # the tokens, and every token's predecessor in its own sequence (-1: none)
+        o = 0
+        for (seq, toks), n in zip(entries, lens):
+            both[0, o:o + n] = toks
+            both[1, o] = seq.last_token if seq.rows > 0 else -1
+            both[1, o + 1:o + n] = both[0, o:o + n - 1]
+            o += n
         parity = [s.steps & 1 for s, _ in entries]
-        every = rows == list(range(len(flat)))   # every token's logits, in order
+        every = len(rows) == off and rows == list(range(off))   # every token's logits, in order
         decode = max(lens) == 1 and min(pos0) > 0 and every
         logits = None
         if decode and self.use_cuda_graphs and not torch.cuda.is_current_stream_capturing():
-            logits = self._decode_replay(flat, slots, pos0, prev, parity)
+            logits = self._decode_replay(both, slots, pos0, parity)
         if logits is None:
             batch = nsq.Batch(slots, pos0, lens, self._device, parity)
-            both = torch.tensor(flat + prev, dtype=torch.int64).pin_memory().to(self._device, non_blocking=True)
-            ids, batch.prev_ids, batch.wants_all = both[:len(flat)], both[len(flat):], every
+            dev = torch.from_numpy(both).pin_memory().to(self._device, non_blocking=True)
+            ids, batch.prev_ids, batch.wants_all = dev[0], dev[1], every
             rows_t = torch.tensor(rows, dtype=torch.int32).pin_memory().to(self._device, non_blocking=True) if rows else None
             logits = self._layers(ids, batch, rows_t)
         for (seq, toks), n in zip(entries, lens):
@@ -94,10 +98,10 @@ class SlotPoolCausalLM(nn.Module):
             seq.last_token = int(toks[-1])
         return logits
 
-    def _decode_replay(self, flat, slots, pos0, prev, parity):
+    def _decode_replay(self, tokens, slots, pos0, parity):
         """One-token-per-sequence steps of a given batch size replay ONE captured graph: everything that changes from step
         to step (token ids, slots, positions) lives in static device buffers the kernels read at run time."""
-        B = len(flat)
+        B = tokens.shape[1]
         key = (B, self.pool.version)
         entry = self._graphs.get(key)
         if entry is None:
@@ -107,8 +111,8 @@ class SlotPoolCausalLM(nn.Module):
             if len(self._graphs) >= self.max_graphs:
                 self._graphs.pop(next(iter(self._graphs)))
             batch = nsq.Batch(slots, pos0, [1] * B, self._device, parity)
-            both = torch.tensor(flat + prev, dtype=torch.int64, device=self._device)
-            ids, batch.prev_ids, batch.wants_all = both[:B], both[B:], True
+            both = torch.from_numpy(tokens).to(self._device)
+            ids, batch.prev_ids, batch.wants_all = both[0], both[1], True
             rows_t = torch.arange(B, dtype=torch.int32, device=self._device)
             torch.cuda.synchronize()
             graph = torch.cuda.CUDAGraph()
@@ -122,7 +126,7 @@ class SlotPoolCausalLM(nn.Module):
         ar = list(range(B))
         host = torch.tensor(ar + list(pos0) + list(slots) + list(pos0) + [1] * B + ar + list(parity), dtype=torch.int32)
         batch.meta.copy_(host.pin_memory(), non_blocking=True)
-        both.copy_(torch.tensor(flat + prev, dtype=torch.int64).pin_memory(), non_blocking=True)
+        both.copy_(torch.from_numpy(tokens).pin_memory(), non_blocking=True)
         graph.replay()
         nsq.note_replayed_launches(n_native)
         return out.clone()

@@ -40,6 +40,7 @@ from .zovolorn import UNIT_VECTOR_EPS
 
 NORM_WEIGHT_OFFSET = 1.0   # the layers' norm weights are stored around zero
 ROW_ALIGN = 8              # fused projections are padded with zero rows to a multiple of this
+BRANCH_MAX_TOKENS = 64     # steps of at most this many tokens run mixer and feed-forward side by side on the device too
 MIXERS = ("delta", "attention", "latent_attention")
 
 
@@ -173,6 +174,8 @@ class ZepilixForCausalLM(SlotPoolCausalLM):
         self.latent_form = None      # None: by step (prompts expanded, decoding in the latent space); "expanded" / "latent" force one
         self.expand_min_len = 16     # steps whose longest entry brings at least this many tokens attend over expanded keys
         self.fused_side = None       # a layer's end in one launch: None: for a few tokens; True / False force it
+        self.branches = None         # mixer and feed-forward on two streams: None: for a few tokens; True / False force it
+        self._branch_stream = None
         self._init_runtime(dev, max_tokens)
         if not all(b.get("latent_ok", True) for b in self.blocks):
             self.use_cuda_graphs = False   # the expanded form describes the step's context on the host: it is not recorded
@@ -238,6 +241,9 @@ class ZepilixForCausalLM(SlotPoolCausalLM):
             nsq.embed(self.embed, ids, x0, 1.0)
         step: dict = {}
 
+        # every token's logits are asked for (decoding): the last layer's end forms the output norm of all rows
+        last = {"norm1": self.final_norm} if batch.wants_all else None
+
         def entering(r: int) -> list:
             """What joins the stream before run r."""
             t = self.passes.get(r)
@@ -248,7 +254,7 @@ class ZepilixForCausalLM(SlotPoolCausalLM):
         def boundary(r: int, results: list, normed: Optional[torch.Tensor] = None) -> None:
             """Add the results of run r - 1 (the first one through its own norm where `normed` is given) and what enters before run r, and form
             run r's inputs."""
-            nxt = self.blocks[self.runs[r]] if r < len(self.runs) else None
+            nxt = self.blocks[self.runs[r]] if r < len(self.runs) else last
             addends = results + entering(r)
             if results and (self.layer_trace is not None or len(addends) > 3):
                 nsq.add_rms_norm(x, results, eps, y_norm_w=normed)
@@ -260,7 +266,7 @@ class ZepilixForCausalLM(SlotPoolCausalLM):
 
         def side_end(r: int, blk: dict, ys: list) -> None:
             """A layer's end for a few tokens in one launch: its sublayers' sum, its side input, what enters before run r and run r's inputs."""
-            nxt = self.blocks[self.runs[r]] if r < len(self.runs) else None
+            nxt = self.blocks[self.runs[r]] if r < len(self.runs) else last
             t = self.passes.get(r)
             nsq.side_boundary(x, [y for y, _ in ys], ids, self.side_table, blk["side_col"], blk["side_gate"], blk["side_proj"], blk["side_norm"], eps,
                               x0=x0 if t else None, step=self.loop_step[t] if t is not None else None, w1=nxt["norm1"] if nxt else None, h1=h1,
@@ -268,11 +274,24 @@ class ZepilixForCausalLM(SlotPoolCausalLM):
 
         fused_side = self.fused_side if self.fused_side is not None else T <= nsq.SIDE_BOUNDARY_MAX_TOKENS
         boundary(0, [])
+        # the sublayers read the same stream: where a step is bound by its launches the feed-forward runs on a stream of its own
+        main, branch = torch.cuda.current_stream(), None
+        if self.branches if self.branches is not None else T <= BRANCH_MAX_TOKENS:
+            branch = self._branch_stream = self._branch_stream or torch.cuda.Stream(device=dev)
         for r, li in enumerate(self.runs):
             blk, st = self.blocks[li], self.pool.layers[r]
+            ff = None
+            if blk["mlp"] and branch is not None:
+                branch.wait_stream(main)
+                with torch.cuda.stream(branch):
+                    ff = self._feed_forward(h2, blk)
             ys = [(self._mixer(h1, blk, st, batch, step), 1.0)]
-            if blk["mlp"]:
-                ys.append((self._feed_forward(h2, blk), 1.0))
+            if ff is not None:
+                main.wait_stream(branch)    # the branch starts again only after the launch that reads `ff`, so its memory is free by then
+            elif blk["mlp"]:
+                ff = self._feed_forward(h2, blk)
+            if ff is not None:
+                ys.append((ff, 1.0))
             if self.side_table is None:
                 boundary(r + 1, ys)
                 continue
@@ -285,6 +304,7 @@ class ZepilixForCausalLM(SlotPoolCausalLM):
             boundary(r + 1, [(nsq.linear(g, blk["side_proj"]), 1.0)], blk["side_norm"])
         if rows is None or rows.numel() == 0:
             return torch.zeros(0, self.vocab_size, dtype=torch.float32, device=dev)
-        hw = torch.empty(rows.numel(), W, dtype=dt, device=dev)
-        nsq.add_rms_norm(x, [], eps, self.final_norm, hw, rows=rows, w_offset=off)     # only the wanted rows go on
-        return nsq.linear(hw, self.embed).float()
+        if last is None:
+            h1 = torch.empty(rows.numel(), W, dtype=dt, device=dev)
+            nsq.add_rms_norm(x, [], eps, self.final_norm, h1, rows=rows, w_offset=off)     # only the wanted rows go on
+        return nsq.linear(h1, self.embed).float()
