@@ -738,6 +738,10 @@ typedef struct pcs_headnorm_params {
 } pcs_headnorm_params;
 int pcs_head_norm_gate(const pcs_headnorm_params* p, void* stream);
 
+/* bfloat16 runs, vdim <= 512: the read-out of the chunks and pcs_head_norm_gate in one launch, without o in memory (o, tok_row, n_tokens, heads,
+ * vdim and chunk_size of `o` are not read; entry c of the chunk list is written to its tokens' rows) */
+int pcs_delta_chunk_out(const pcs_delta_chunk_params* p, const pcs_headnorm_params* o, void* stream);
+
 /* The recurrence of pcs_gla_scan in chunks of `chunk` tokens (prompts).  The step's entries are cut into chunks (an entry's last one may
  * be short); chunk c holds tokens chunk_first[c] .. chunk_first[c] + chunk_len[c] - 1 of the concatenated matrix.  With B_i the
  * running sum of the log decays inside a chunk (per key channel) and e its last token:

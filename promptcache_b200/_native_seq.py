@@ -22,7 +22,7 @@ EXPORTS = ("pcs_version", "pcs_last_error", "pcs_launch_count", "pcs_attn_worksp
            "pcs_moe_rows_up", "pcs_moe_rows_down", "pcs_moe_plan", "pcs_moe_gather", "pcs_moe_gemm", "pcs_moe_combine", "pcs_silu_mul", "pcs_glu_mul",
            "pcs_depth_mix", "pcs_latent_prep", "pcs_latent_q", "pcs_latent_gather", "pcs_latent_expand", "pcs_head_gate", "pcs_gla_decay", "pcs_gla_scan", "pcs_gla_chunk_prep", "pcs_gla_chunk_scan", "pcs_gla_chunk_out",
            "pcs_add_layer_norm", "pcs_gru_scan", "pcs_group_norm_conv", "pcs_soft_cap", "pcs_short_conv", "pcs_delta_inputs", "pcs_delta_scan", "pcs_delta_chunk_prep", "pcs_delta_chunk_scan",
-           "pcs_head_norm_gate", "pcs_side_gate", "pcs_side_boundary")
+           "pcs_head_norm_gate", "pcs_delta_chunk_out", "pcs_side_gate", "pcs_side_boundary")
 GLU_SILU, GLU_CLAMPED_SWISH, GLU_GELU_TANH = 0, 1, 4
 ACT_RELU2, ACT_GELU_ERF = 2, 3          # activations of a feed-forward without a gate branch
 ROUTE_SOFTMAX, ROUTE_SIGMOID = 0, 1
@@ -285,6 +285,7 @@ def load() -> C.CDLL:
     for name in ("pcs_delta_chunk_prep", "pcs_delta_chunk_scan"):
         getattr(lib, name).argtypes = [C.POINTER(pcs_delta_chunk_params), C.c_void_p]
     lib.pcs_head_norm_gate.argtypes = [C.POINTER(pcs_headnorm_params), C.c_void_p]
+    lib.pcs_delta_chunk_out.argtypes = [C.POINTER(pcs_delta_chunk_params), C.POINTER(pcs_headnorm_params), C.c_void_p]
     lib.pcs_side_boundary.argtypes = [C.POINTER(pcs_side_params), C.c_void_p]
     lib.pcs_side_gate.argtypes = [C.c_void_p, C.c_int64, C.c_void_p, C.c_int64, C.c_int, C.c_int, C.c_void_p, C.c_void_p, C.c_int, C.c_int, C.c_int, C.c_void_p]
     for name in EXPORTS[4:]:
@@ -1244,6 +1245,7 @@ def delta_inputs(proj: torch.Tensor, c_off: int, kv_heads: int, heads: int, dim:
 DELTA_CHUNK = 64          # PCS_DELTA_CHUNK
 DELTA_CHUNK_MIN_LEN = 32  # steps whose longest entry brings fewer tokens go token by token
 DELTA_CHUNK_MAX_DIM = 256
+DELTA_OUT_MAX_VDIM = 512  # value columns of a head that the read-out kernel holds
 
 
 def delta_takes_chunks(batch: Batch, dim: int, impl: int = 0) -> bool:
@@ -1285,6 +1287,8 @@ def delta_scan(qk: torch.Tensor, v: torch.Tensor, decay: Optional[torch.Tensor],
     if norm_w.dtype != dt or norm_w.numel() != V or tuple(gate.shape) != (T, H * V) or tuple(out.shape) != (T, H * V):
         raise NativeError("delta_scan: norm_w [vdim], gate and out [T, H * vdim] in the compute type")
     n = pcs_headnorm_params()
+    n.w, n.g, n.g_stride, n.out, n.out_stride = norm_w.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(), out.stride(0)
+    n.n_tokens, n.heads, n.vdim, n.eps, n.out_scale, n.dtype, n.silu = T, H, V, float(eps), float(out_scale), dtype_code(dt), 1 if gate_silu else 0
     if delta_takes_chunks(batch, D, impl):
         ch = DELTA_CHUNK
         plan = _gla_chunk_plan(batch, ch)
@@ -1300,6 +1304,9 @@ def delta_scan(qk: torch.Tensor, v: torch.Tensor, decay: Optional[torch.Tensor],
         p.seq_slot, p.seq_pos0, p.seq_chunk0, p.seq_chunks = batch.seq_slot.data_ptr(), batch.seq_pos0.data_ptr(), plan["seq0"].data_ptr(), plan["seqn"].data_ptr()
         _check(load().pcs_delta_chunk_prep(C.byref(p), _stream()), "pcs_delta_chunk_prep")
         _check(load().pcs_delta_chunk_scan(C.byref(p), _stream()), "pcs_delta_chunk_scan")   # u: every token's correction; s: the chunks' start states
+        if dt == torch.bfloat16 and V <= DELTA_OUT_MAX_VDIM:   # the read-out with its norm and gate in one launch
+            _check(load().pcs_delta_chunk_out(C.byref(p), C.byref(n), _stream()), "pcs_delta_chunk_out")
+            return
         o = torch.baddbmm(torch.bmm(a, u), qd, s)             # [chunks * H, chunk, vdim]
         n.tok_row, n.chunk_size = plan["tok_row"].data_ptr(), ch
     else:
@@ -1311,6 +1318,5 @@ def delta_scan(qk: torch.Tensor, v: torch.Tensor, decay: Optional[torch.Tensor],
         p.seq_slot, p.seq_pos0, p.seq_len, p.seq_off = (batch.seq_slot.data_ptr(), batch.seq_pos0.data_ptr(), batch.seq_len.data_ptr(), batch.seq_off.data_ptr())
         p.n_seqs, p.n_tokens, p.dtype, p.impl = batch.n_seqs, T, dtype_code(dt), 1 if impl == 1 else 0
         _check(load().pcs_delta_scan(C.byref(p), _stream()), "pcs_delta_scan")
-    n.o, n.w, n.g, n.g_stride, n.out, n.out_stride = o.data_ptr(), norm_w.data_ptr(), gate.data_ptr(), gate.stride(0), out.data_ptr(), out.stride(0)
-    n.n_tokens, n.heads, n.vdim, n.eps, n.out_scale, n.dtype, n.silu = T, H, V, float(eps), float(out_scale), dtype_code(dt), 1 if gate_silu else 0
+    n.o = o.data_ptr()
     _check(load().pcs_head_norm_gate(C.byref(n), _stream()), "pcs_head_norm_gate")

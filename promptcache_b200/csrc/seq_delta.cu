@@ -502,15 +502,9 @@ __device__ __forceinline__ int delta_kd_slot(int d) { return (d & ~63) + 4 * (d 
 // vdim columns of diag(beta) V.  `key(i, col)` gives row i of column col of K exp(B).
 template <typename T, typename Key>
 __device__ __forceinline__ void delta_chunk_solve(const pcs_delta_chunk_params& p, const float* As, const float* beta, long long base, int first, int n, int head, Key key) {
-  constexpr bool kFast = sizeof(T) == 2;
   const int D = p.dim, V = p.vdim, H = p.heads, tid = threadIdx.x;
-  const int D8 = (D + 7) & ~7;
-  float* wg = p.w + base * D8 * kC;
+  float* wg = p.w + base * ((D + 7) & ~7) * kC;
   float* ug = p.u + base * kC * V;
-  for (int e = tid; e < (D8 - D) * kC; e += kDpThreads) {   // channels that only pad the fragments
-    const int d = D + e / kC, i = e % kC;
-    if (kFast) wg[(((d >> 3) * 4 + (i >> 4)) * 32 + (i & 7) * 4 + (d & 3)) * 4 + ((i >> 3) & 1) + 2 * ((d >> 2) & 1)] = 0.f;
-  }
 #pragma unroll 1
   for (int col = tid; col < D + V; col += kDpThreads) {
     float x[kC];
@@ -538,20 +532,154 @@ __device__ __forceinline__ void delta_chunk_solve(const pcs_delta_chunk_params& 
       x[i] -= a0 + a1;
     }
     if (col < D) {
-      if (kFast) {
-        float* o = wg + ((col >> 3) * 4 * 32 + (col & 3)) * 4 + 2 * ((col >> 2) & 1);
+      float* o = wg + static_cast<long long>(col) * kC;
 #pragma unroll
-        for (int mt = 0; mt < 4; ++mt)
-#pragma unroll
-          for (int g = 0; g < 16; ++g) o[(mt * 32 + (g & 7) * 4) * 4 + (g >> 3)] = x[mt * 16 + g];   // (wider stores would pin register pairs)
-      } else {
-        float* o = wg + static_cast<long long>(col) * kC;
-#pragma unroll
-        for (int r = 0; r < 16; ++r) *reinterpret_cast<float4*>(o + 4 * r) = make_float4(x[r], x[r + 16], x[r + 32], x[r + 48]);
-      }
+      for (int r = 0; r < 16; ++r) *reinterpret_cast<float4*>(o + 4 * r) = make_float4(x[r], x[r + 16], x[r + 32], x[r + 48]);
     } else {
 #pragma unroll
       for (int i = 0; i < kC; ++i) ug[i * u_step + (col - D)] = x[i];
+    }
+  }
+}
+
+// The same in bfloat16 runs: M^-1 is formed once (a unit lower triangular 64 x 64 matrix: its four diagonal blocks of 16 by substitution, one
+// column per thread, then the blocks below them, diagonal by diagonal, all in 32-bit multiply-adds), and both results are products
+// M^-1 X with TF32 hi + lo operands, w written as the scan's operand fragments.  `inv` [64][kTi] shared memory.
+constexpr int kTi = kC + 4;
+
+template <typename Key>
+__device__ __forceinline__ void delta_chunk_solve_tc(const pcs_delta_chunk_params& p, const float* As, const float* beta, float* inv, long long base, int first, int n,
+                                                     int head, Key key) {
+  const int D = p.dim, V = p.vdim, H = p.heads, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  for (int e = tid; e < kC * kC; e += kDpThreads) {
+    const int i = e >> 6, j = e & 63;
+    if ((i >> 4) != (j >> 4)) inv[i * kTi + j] = 0.f;
+  }
+  if (tid < kC) {
+    const int b0 = tid & ~15, c = tid & 15;
+    float x[kCB];
+#pragma unroll
+    for (int i = 0; i < kCB; ++i) {
+      float a = 0.f;
+#pragma unroll
+      for (int j = 0; j < i; ++j) a = fmaf(As[(b0 + i) * kC + b0 + j], x[j], a);
+      x[i] = (i == c ? 1.f : 0.f) - a;    // (zero above the diagonal by itself)
+    }
+#pragma unroll
+    for (int i = 0; i < kCB; ++i) inv[(b0 + i) * kTi + b0 + c] = x[i];
+  }
+  __syncthreads();
+#pragma unroll 1
+  for (int d = 1; d < kNB; ++d) {   // blocks (I, I - d): first sum_K A[I, K] inv[K, J], kept in place, then -inv[I, I] times it
+    const int cnt = (kNB - d) * kCB * kCB;
+    for (int e = tid; e < cnt; e += kDpThreads) {
+      const int I = (e >> 8) + d, J = I - d, i = I * kCB + ((e >> 4) & 15), j = J * kCB + (e & 15);
+      float a0 = 0.f, a1 = 0.f;
+      for (int q = J * kCB; q < I * kCB; q += 2) {
+        a0 = fmaf(As[i * kC + q], inv[q * kTi + j], a0);
+        a1 = fmaf(As[i * kC + q + 1], inv[(q + 1) * kTi + j], a1);
+      }
+      inv[i * kTi + j] = a0 + a1;
+    }
+    __syncthreads();
+    float r[(kNB - 1) * kCB * kCB / kDpThreads];   // (two outputs per thread on the first diagonal)
+#pragma unroll
+    for (int m = 0; m < (kNB - 1) * kCB * kCB / kDpThreads; ++m) {
+      const int e = tid + m * kDpThreads;
+      r[m] = 0.f;
+      if (e < cnt) {
+        const int I = (e >> 8) + d, i = (e >> 4) & 15, j = (I - d) * kCB + (e & 15);
+        float a0 = 0.f, a1 = 0.f;
+#pragma unroll
+        for (int q = 0; q < kCB; q += 2) {
+          a0 = fmaf(inv[(I * kCB + i) * kTi + I * kCB + q], inv[(I * kCB + q) * kTi + j], a0);
+          a1 = fmaf(inv[(I * kCB + i) * kTi + I * kCB + q + 1], inv[(I * kCB + q + 1) * kTi + j], a1);
+        }
+        r[m] = -(a0 + a1);
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int m = 0; m < (kNB - 1) * kCB * kCB / kDpThreads; ++m) {
+      const int e = tid + m * kDpThreads;
+      if (e < cnt) {
+        const int I = (e >> 8) + d;
+        inv[(I * kCB + ((e >> 4) & 15)) * kTi + (I - d) * kCB + (e & 15)] = r[m];
+      }
+    }
+    __syncthreads();
+  }
+  // four tiles of 8 columns per warp and round.  In a tile of w column n of the product is channel (n >> 1) + 4 (n & 1): a lane's accumulators
+  // then are its operand fragment of the scan's w S
+  const int D8 = (D + 7) & ~7, NW = D8 / 8, tiles = NW + (V + 7) / 8;
+  float* wg = p.w + base * D8 * kC;
+  float* ug = p.u + base * kC * V;
+  const __nv_bfloat16* vb = static_cast<const __nv_bfloat16*>(p.v) + static_cast<long long>(first) * H * V + head * V;
+  const bool even = (V & 1) == 0;
+#pragma unroll 1
+  for (int t0 = warp * 4; t0 < tiles; t0 += (kDpThreads / 32) * 4) {
+    float acc[4][4][4];
+#pragma unroll
+    for (int a = 0; a < 4; ++a)
+#pragma unroll
+      for (int b = 0; b < 4; ++b) acc[a][b][0] = acc[a][b][1] = acc[a][b][2] = acc[a][b][3] = 0.f;
+#pragma unroll 1
+    for (int ks = 0; ks < kC / 8; ++ks) {
+      uint32_t bh[4][2], bl[4][2];
+#pragma unroll
+      for (int q = 0; q < 4; ++q)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int i = 8 * ks + t + 4 * h, tile = t0 + q;
+          float x = 0.f;
+          if (tile < NW) {
+            const int c = 8 * tile + (g >> 1) + 4 * (g & 1);
+            if (c < D) x = beta[i] * key(i, c);
+          } else {
+            const int c = 8 * (tile - NW) + g;
+            if (tile < tiles && c < V && i < n) x = beta[i] * ldf(vb + static_cast<long long>(i) * H * V + c);
+          }
+          split_tf32(x, bh[q][h], bl[q][h]);
+        }
+#pragma unroll
+      for (int mt = 0; mt < 4; ++mt) {
+        if (16 * mt + 15 < 8 * ks) continue;   // above the diagonal
+        const float* a = inv + (16 * mt + g) * kTi + 8 * ks + t;
+        uint32_t ah[4], al[4];
+        split_tf32(a[0], ah[0], al[0]);
+        split_tf32(a[8 * kTi], ah[1], al[1]);
+        split_tf32(a[4], ah[2], al[2]);
+        split_tf32(a[8 * kTi + 4], ah[3], al[3]);
+#pragma unroll
+        for (int q = 0; q < 4; ++q) mma_tf32(acc[q][mt], ah, bh[q][0], bh[q][1]);
+#pragma unroll
+        for (int q = 0; q < 4; ++q) mma_tf32(acc[q][mt], ah, bl[q][0], bl[q][1]);
+#pragma unroll
+        for (int q = 0; q < 4; ++q) mma_tf32(acc[q][mt], al, bh[q][0], bh[q][1]);
+      }
+    }
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      const int tile = t0 + q;
+      if (tile < NW) {
+#pragma unroll
+        for (int mt = 0; mt < 4; ++mt)
+          *reinterpret_cast<float4*>(wg + ((static_cast<long long>(tile) * 4 + mt) * 32 + lane) * 4) = make_float4(acc[q][mt][0], acc[q][mt][2], acc[q][mt][1], acc[q][mt][3]);
+      } else if (tile < tiles) {
+        const int c = 8 * (tile - NW) + 2 * t;
+#pragma unroll
+        for (int mt = 0; mt < 4; ++mt)
+#pragma unroll
+          for (int h = 0; h < 2; ++h) {
+            float* o = ug + static_cast<long long>(16 * mt + g + 8 * h) * V + c;
+            if (even) {
+              if (c < V) *reinterpret_cast<float2*>(o) = make_float2(acc[q][mt][2 * h], acc[q][mt][2 * h + 1]);
+            } else {
+              if (c < V) o[0] = acc[q][mt][2 * h];
+              if (c + 1 < V) o[1] = acc[q][mt][2 * h + 1];
+            }
+          }
+      }
     }
   }
 }
@@ -562,8 +690,8 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_
   const int D = p.dim, V = p.vdim, H = p.heads, D4 = (D + 3) & ~3, DP = D4 + 4, U = 2 * p.kv_heads * D, L = (D + 63) & ~63;
   float* qs = sm;              // [64][DP]: q, later scaled to its block's start
   float* ks = qs + kC * DP;    // [64][DP]: k, later scaled to its block's start
-  float* Bs = ks + kC * DP;    // [64][DP]: running sums, later the keys scaled to their block's end
-  float* f1 = Bs + kC * DP;    // [D4] each: the running sums at the blocks' ends, later exp(B_r(1)), exp(B_r(2) - B_r(1)), exp(B_r(3) - B_r(2))
+  float* Bs = ks + kC * DP;    // [64][DP]: running sums, later the keys scaled to their block's end; at last [64][kTi]
+  float* f1 = Bs + kC * (DP > kTi ? DP : kTi);    // [D4] each: the running sums at the blocks' ends, later exp(B_r(1)), exp(B_r(2) - B_r(1)), exp(B_r(3) - B_r(2))
   float* f2 = f1 + D4;
   float* f3 = f2 + D4;
   float* fe = f3 + D4;
@@ -742,10 +870,12 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_kernel(const pcs_
     As[(i + 8) * kC + s] = beta[i + 8] * k10; As[(i + 8) * kC + s + 8] = beta[i + 8] * k11;
   }
   __syncthreads();
-  delta_chunk_solve<T>(p, As, beta, base, first, n, head, [&](int i, int col) {
+  auto key = [&](int i, int col) {
     const float e1 = f1[col];
     return ks[i * DP + col] * (i < 16 ? 1.f : i < 32 ? e1 : i < 48 ? e1 * f2[col] : e1 * f2[col] * f3[col]);
-  });
+  };
+  if constexpr (kFast) delta_chunk_solve_tc(p, As, beta, Bs, base, first, n, head, key);   // (the keys scaled to their block's end have been used)
+  else delta_chunk_solve<T>(p, As, beta, base, first, n, head, key);
 }
 
 // One decay per head: the factor of a pair (i, s) is one number, exp(B_i - B_s) <= 1, so the sums over pairs are plain products q k^T and k k^T
@@ -761,6 +891,7 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_head_kernel(const
   float* Bs = beta + kC;
   float* eB = Bs + kC;
   float* eE = eB + kC;
+  float* inv = eE + kC;        // [64][kTi] (bfloat16 runs)
   const int cn = blockIdx.x, head = blockIdx.y, hk = head / (H / p.kv_heads), tid = threadIdx.x;
   const int first = p.chunk_first[cn], n = p.chunk_len[cn];
   const long long base = static_cast<long long>(cn) * H + head;
@@ -910,7 +1041,9 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_head_kernel(const
     for (int d = tid; d < D; d += kDpThreads) p.g[base * D + d] = eB[kC - 1];
   }
   __syncthreads();
-  delta_chunk_solve<T>(p, As, beta, base, first, n, head, [&](int i, int col) { return ks[i * DP + col] * eB[i]; });
+  auto key = [&](int i, int col) { return ks[i * DP + col] * eB[i]; };
+  if constexpr (kFast) delta_chunk_solve_tc(p, As, beta, inv, base, first, n, head, key);
+  else delta_chunk_solve<T>(p, As, beta, base, first, n, head, key);
 }
 
 // Block = (VS value columns, head, entry), 16 warps.  Both products split their sum over the warps and meet in `red`: u = u0 - w S over the
@@ -1361,6 +1494,150 @@ static int launch_delta_chunk_scan(const pcs_delta_chunk_params& p, size_t smem,
   return PCS_OK;
 }
 
+// ---- read-out of the chunks (bfloat16 runs) ---------------------------------------------------------------------------------------
+// Block = (chunk, head), a warp = 32 value columns: o = qd S + a u over dim + 64 terms (TF32 hi + lo operands; [qd | a] staged in shared memory,
+// S and u read once, a step ahead), then the head's norm and gate on the accumulators, and the result's rows.
+constexpr int kDoMaxWarps = 16;
+
+__global__ void __launch_bounds__(kDoMaxWarps * 32) delta_chunk_out_kernel(const pcs_delta_chunk_params p, const pcs_headnorm_params o) {
+  extern __shared__ __align__(16) float sm[];
+  const int D = p.dim, V = p.vdim, H = p.heads, D8 = (D + 7) & ~7, LD = ((D8 + kC + 31) & ~31) + 4;
+  float* A = sm;                   // [64][LD]
+  float* red = A + kC * LD;        // [warps][64], then [64]
+  const int cn = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
+  const long long base = static_cast<long long>(cn) * H + head;
+  const int first = p.chunk_first[cn], n = p.chunk_len[cn];
+  const float* qd = p.qd + base * kC * D;
+  const float* ag = p.a + base * kC * kC;
+  if (D % 4 == 0) {
+    for (int e = tid; e < kC * (D / 4); e += nthr) {
+      const int i = e / (D / 4), c = (e - i * (D / 4)) * 4;
+      cp_async16(A + i * LD + c, qd + i * D + c);
+    }
+  } else {
+    for (int e = tid; e < kC * D; e += nthr) {
+      const int i = e / D, c = e - i * D;
+      A[i * LD + c] = qd[e];
+    }
+  }
+  for (int e = tid; e < kC * (D8 - D); e += nthr) {
+    const int i = e / (D8 - D);
+    A[i * LD + D + (e - i * (D8 - D))] = 0.f;
+  }
+  for (int e = tid; e < kC * (kC / 4); e += nthr) cp_async16(A + (e >> 4) * LD + D8 + (e & 15) * 4, ag + e * 4);
+  cp_async_commit();
+  const int c0 = warp * 32 + g, KD = D8 / 8, KT = KD + kC / 8;
+  const float* sg = p.s + base * D * V;
+  const float* ug = p.u + base * kC * V;
+  auto load = [&](int kt, float (&b)[4][2]) {
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int r = 8 * (kt < KD ? kt : kt - KD) + t + 4 * h;
+      const float* src = (kt < KD ? sg : ug) + static_cast<long long>(r) * V;
+      const bool ok = kt < KT && (kt >= KD || r < D);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) b[q][h] = ok && c0 + 8 * q < V ? src[c0 + 8 * q] : 0.f;
+    }
+  };
+  float acc[4][4][4], nx[2][4][2];
+#pragma unroll
+  for (int q = 0; q < 4; ++q)
+#pragma unroll
+    for (int m = 0; m < 4; ++m) acc[q][m][0] = acc[q][m][1] = acc[q][m][2] = acc[q][m][3] = 0.f;
+  load(0, nx[0]);
+  load(1, nx[1]);
+  cp_async_wait<0>();
+  __syncthreads();
+  auto step = [&](int kt, float (&b)[4][2]) {
+    uint32_t bh[4][2], bl[4][2];
+#pragma unroll
+    for (int q = 0; q < 4; ++q) {
+      split_tf32(b[q][0], bh[q][0], bl[q][0]);
+      split_tf32(b[q][1], bh[q][1], bl[q][1]);
+    }
+    load(kt + 2, b);
+    if (kt >= KT) return;
+#pragma unroll
+    for (int m = 0; m < 4; ++m) {
+      if (kt >= KD && 16 * m + 15 < 8 * (kt - KD)) continue;   // `a` is zero above the diagonal
+      const float* a = A + (16 * m + g) * LD + 8 * kt + t;
+      uint32_t ah[4], al[4];
+      split_tf32(a[0], ah[0], al[0]);
+      split_tf32(a[8 * LD], ah[1], al[1]);
+      split_tf32(a[4], ah[2], al[2]);
+      split_tf32(a[8 * LD + 4], ah[3], al[3]);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) mma_tf32(acc[q][m], ah, bh[q][0], bh[q][1]);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) mma_tf32(acc[q][m], ah, bl[q][0], bl[q][1]);
+#pragma unroll
+      for (int q = 0; q < 4; ++q) mma_tf32(acc[q][m], al, bh[q][0], bh[q][1]);
+    }
+  };
+#pragma unroll 1
+  for (int kt = 0; kt < KT; kt += 2) {
+    step(kt, nx[0]);
+    step(kt + 1, nx[1]);
+  }
+  // the head's mean square per token: a row's columns are spread over 4 lanes and all warps
+#pragma unroll
+  for (int m = 0; m < 4; ++m)
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      float ss = 0.f;
+#pragma unroll
+      for (int q = 0; q < 4; ++q) ss = fmaf(acc[q][m][2 * h], acc[q][m][2 * h], fmaf(acc[q][m][2 * h + 1], acc[q][m][2 * h + 1], ss));
+      ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+      ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+      if (t == 0) red[warp * kC + 16 * m + g + 8 * h] = ss;
+    }
+  __syncthreads();
+  float inv = 0.f;
+  for (int i = tid; i < kC; i += nthr) {   // (at least two warps)
+    for (int w = 0; w < nthr / 32; ++w) inv += red[w * kC + i];
+    inv = o.out_scale / sqrtf(inv / static_cast<float>(V) + o.eps);
+  }
+  __syncthreads();
+  if (tid < kC) red[tid] = inv;
+  __syncthreads();
+  const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(o.g) + static_cast<long long>(first) * o.g_stride + head * V;
+  const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(o.w);
+  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(o.out) + static_cast<long long>(first) * o.out_stride + head * V;
+  const bool pairs = V % 2 == 0 && o.out_stride % 2 == 0 && o.g_stride % 2 == 0 && ((reinterpret_cast<uintptr_t>(o.g) | reinterpret_cast<uintptr_t>(o.out) | reinterpret_cast<uintptr_t>(o.w)) & 3) == 0;
+  auto gated = [&](float x, float f, float wv, float gv) { return x * f * wv * sigmoidf_(gv) * (o.silu ? gv : 1.f); };
+#pragma unroll
+  for (int q = 0; q < 4; ++q) {
+    const int c = warp * 32 + 8 * q + 2 * t;
+    if (c >= V) continue;
+    float w0, w1 = 0.f;
+    if (pairs) {
+      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(w + c));
+      w0 = f.x;
+      w1 = f.y;
+    } else {
+      w0 = ldf(w + c);
+      if (c + 1 < V) w1 = ldf(w + c + 1);
+    }
+#pragma unroll
+    for (int m = 0; m < 4; ++m)
+#pragma unroll
+      for (int h = 0; h < 2; ++h) {
+        const int i = 16 * m + g + 8 * h;
+        if (i >= n) continue;
+        const float f = red[i];
+        const __nv_bfloat16* gr = gate + static_cast<long long>(i) * o.g_stride + c;
+        __nv_bfloat16* r = out + static_cast<long long>(i) * o.out_stride + c;
+        if (pairs) {
+          const float2 gv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gr));
+          *reinterpret_cast<uint32_t*>(r) = pack_bf16(gated(acc[q][m][2 * h], f, w0, gv.x), gated(acc[q][m][2 * h + 1], f, w1, gv.y));
+        } else {
+          stf(r, gated(acc[q][m][2 * h], f, w0, ldf(gr)));
+          if (c + 1 < V) stf(r + 1, gated(acc[q][m][2 * h + 1], f, w1, ldf(gr + 1)));
+        }
+      }
+  }
+}
+
 // ---- per-head norm and gate ------------------------------------------------------------------------------------------------------
 template <typename T>
 __global__ void __launch_bounds__(256) head_norm_gate_kernel(const pcs_headnorm_params p) {
@@ -1492,10 +1769,10 @@ PCS_API int pcs_delta_chunk_prep(const pcs_delta_chunk_params* p, void* stream) 
   PCS_REQUIRE(p->heads > 0 && p->heads <= 65535 && p->kv_heads > 0 && p->heads % p->kv_heads == 0 && p->dim > 0 && p->dim <= 256 && p->vdim > 0,
               "pcs_delta_chunk_prep: bad sizes (dim %d of at most 256)", p->dim);
   const int D4 = (p->dim + 3) & ~3;
-  const size_t smem = (static_cast<size_t>(3) * pcs::kC * (D4 + 4) + 4 * D4 + pcs::kC * pcs::kC + pcs::kC) * sizeof(float);
+  const size_t smem = (static_cast<size_t>(2) * pcs::kC * (D4 + 4) + static_cast<size_t>(pcs::kC) * (D4 + 4 > pcs::kTi ? D4 + 4 : pcs::kTi) + 4 * D4 + pcs::kC * pcs::kC + pcs::kC) * sizeof(float);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (!p->ld) {
-    const size_t smem_h = (static_cast<size_t>(2) * pcs::kC * (((p->dim + 31) & ~31) + 4) + pcs::kC * pcs::kC + 4 * pcs::kC) * sizeof(float);
+    const size_t smem_h = (static_cast<size_t>(2) * pcs::kC * (((p->dim + 31) & ~31) + 4) + pcs::kC * pcs::kC + 4 * pcs::kC + pcs::kC * pcs::kTi) * sizeof(float);
     PCS_DISPATCH(p->dtype, PCS_CHECK_CUDA(cudaFuncSetAttribute(pcs::delta_chunk_prep_head_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024)));
     PCS_DISPATCH(p->dtype, pcs::delta_chunk_prep_head_kernel<T><<<dim3(p->n_chunks, p->heads), pcs::kDpThreads, smem_h, st>>>(*p));
     PCS_CHECK_CUDA(cudaGetLastError());
@@ -1529,6 +1806,22 @@ PCS_API int pcs_delta_chunk_scan(const pcs_delta_chunk_params* p, void* stream) 
   const bool two = smem(vs, 2) <= (one_wave ? 227u : 112u) * 1024u;
   if (narrow) return two ? pcs::launch_delta_chunk_scan<8, 2>(*p, smem(8, 2), st) : pcs::launch_delta_chunk_scan<8, 1>(*p, smem(8, 1), st);
   return two ? pcs::launch_delta_chunk_scan<16, 2>(*p, smem(16, 2), st) : pcs::launch_delta_chunk_scan<16, 1>(*p, smem(16, 1), st);
+}
+
+PCS_API int pcs_delta_chunk_out(const pcs_delta_chunk_params* p, const pcs_headnorm_params* o, void* stream) {
+  PCS_REQUIRE(p && o, "pcs_delta_chunk_out: null params");
+  if (p->n_chunks == 0) return PCS_OK;
+  PCS_REQUIRE(p->qd && p->a && p->s && p->u && p->chunk_first && p->chunk_len && o->w && o->g && o->out, "pcs_delta_chunk_out: null tensor");
+  PCS_REQUIRE(p->dtype == PCS_BF16 && p->heads > 0 && p->heads <= 65535 && p->dim > 0 && p->dim <= 256 && p->vdim > 0 && p->vdim <= 32 * pcs::kDoMaxWarps,
+              "pcs_delta_chunk_out: serves bfloat16, dim up to 256 and vdim up to %d", 32 * pcs::kDoMaxWarps);
+  PCS_REQUIRE(((reinterpret_cast<uintptr_t>(p->qd) | reinterpret_cast<uintptr_t>(p->a)) & 15) == 0, "pcs_delta_chunk_out: qd and a must be 16-byte aligned");
+  const int warps = (p->vdim + 31) / 32 < 2 ? 2 : (p->vdim + 31) / 32, D8 = (p->dim + 7) & ~7;
+  const size_t smem = (static_cast<size_t>(pcs::kC) * (((D8 + pcs::kC + 31) & ~31) + 4) + static_cast<size_t>(warps) * pcs::kC) * sizeof(float);
+  PCS_CHECK_CUDA(cudaFuncSetAttribute(pcs::delta_chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+  pcs::delta_chunk_out_kernel<<<dim3(p->n_chunks, p->heads), warps * 32, smem, static_cast<cudaStream_t>(stream)>>>(*p, *o);
+  PCS_CHECK_CUDA(cudaGetLastError());
+  pcs::count_launch();
+  return PCS_OK;
 }
 
 PCS_API int pcs_head_norm_gate(const pcs_headnorm_params* p, void* stream) {
