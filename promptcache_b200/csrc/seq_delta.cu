@@ -609,41 +609,69 @@ __device__ __forceinline__ void delta_chunk_solve_tc(const pcs_delta_chunk_param
     }
     __syncthreads();
   }
-  // four tiles of 8 columns per warp and round.  In a tile of w column n of the product is channel (n >> 1) + 4 (n & 1): a lane's accumulators
-  // then are its operand fragment of the scan's w S
-  const int D8 = (D + 7) & ~7, NW = D8 / 8, tiles = NW + (V + 7) / 8;
+  // A warp and round takes 32 columns as four tiles of 8, of w or of u.  Which column a tile's place stands for is free: in a tile of w place x is
+  // channel (x >> 1) + 4 (x & 1), so that a lane's accumulators are its operand fragment of the scan's w S; of u's 32 columns place x of tile q is
+  // column 4 x + q, so that a lane's four values of a row, read or written, are neighbours.
+  const int D8 = (D + 7) & ~7, NW = D8 / 8, GW = (NW + 3) / 4, groups = GW + (V + 31) / 32;
   float* wg = p.w + base * D8 * kC;
   float* ug = p.u + base * kC * V;
   const __nv_bfloat16* vb = static_cast<const __nv_bfloat16*>(p.v) + static_cast<long long>(first) * H * V + head * V;
-  const bool even = (V & 1) == 0;
+  const bool quads = (V & 3) == 0 && (reinterpret_cast<uintptr_t>(p.v) & 7) == 0;
 #pragma unroll 1
-  for (int t0 = warp * 4; t0 < tiles; t0 += (kDpThreads / 32) * 4) {
+  for (int grp = warp; grp < groups; grp += kDpThreads / 32) {
+    const bool of_w = grp < GW;
+    const int t0 = grp * 4, cu = (grp - GW) * 32 + 4 * g;   // first tile of w; this lane's four columns of u
+    uint2 vr[kC / 8][2];
+    if (!of_w) {   // the lane's values of all steps, requested at once
+#pragma unroll
+      for (int ks = 0; ks < kC / 8; ++ks)
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+          const int i = 8 * ks + t + 4 * h;
+          const __nv_bfloat16* r = vb + static_cast<long long>(i) * H * V + cu;
+          vr[ks][h] = make_uint2(0u, 0u);
+          if (i < n) {
+            if (quads) {
+              if (cu < V) vr[ks][h] = *reinterpret_cast<const uint2*>(r);
+            } else {
+              float x[4];
+#pragma unroll
+              for (int q = 0; q < 4; ++q) x[q] = cu + q < V ? ldf(r + q) : 0.f;
+              vr[ks][h] = make_uint2(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3]));
+            }
+          }
+        }
+    }
     float acc[4][4][4];
 #pragma unroll
     for (int a = 0; a < 4; ++a)
 #pragma unroll
       for (int b = 0; b < 4; ++b) acc[a][b][0] = acc[a][b][1] = acc[a][b][2] = acc[a][b][3] = 0.f;
-#pragma unroll 1
+#pragma unroll
     for (int ks = 0; ks < kC / 8; ++ks) {
       uint32_t bh[4][2], bl[4][2];
 #pragma unroll
-      for (int q = 0; q < 4; ++q)
+      for (int h = 0; h < 2; ++h) {
+        const int i = 8 * ks + t + 4 * h;
+        const float bt = beta[i];
+        float x[4];
+        if (of_w) {
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {
-          const int i = 8 * ks + t + 4 * h, tile = t0 + q;
-          float x = 0.f;
-          if (tile < NW) {
-            const int c = 8 * tile + (g >> 1) + 4 * (g & 1);
-            if (c < D) x = beta[i] * key(i, c);
-          } else {
-            const int c = 8 * (tile - NW) + g;
-            if (tile < tiles && c < V && i < n) x = beta[i] * ldf(vb + static_cast<long long>(i) * H * V + c);
+          for (int q = 0; q < 4; ++q) {
+            const int c = 8 * (t0 + q) + (g >> 1) + 4 * (g & 1);
+            x[q] = c < D ? key(i, c) : 0.f;
           }
-          split_tf32(x, bh[q][h], bl[q][h]);
+        } else {
+          x[0] = __uint_as_float(vr[ks][h].x << 16);
+          x[1] = __uint_as_float(vr[ks][h].x & 0xffff0000u);
+          x[2] = __uint_as_float(vr[ks][h].y << 16);
+          x[3] = __uint_as_float(vr[ks][h].y & 0xffff0000u);
         }
 #pragma unroll
-      for (int mt = 0; mt < 4; ++mt) {
-        if (16 * mt + 15 < 8 * ks) continue;   // above the diagonal
+        for (int q = 0; q < 4; ++q) split_tf32(bt * x[q], bh[q][h], bl[q][h]);
+      }
+#pragma unroll
+      for (int mt = ks / 2; mt < 4; ++mt) {   // (row tiles above the diagonal hold zeros)
         const float* a = inv + (16 * mt + g) * kTi + 8 * ks + t;
         uint32_t ah[4], al[4];
         split_tf32(a[0], ah[0], al[0]);
@@ -658,28 +686,29 @@ __device__ __forceinline__ void delta_chunk_solve_tc(const pcs_delta_chunk_param
         for (int q = 0; q < 4; ++q) mma_tf32(acc[q][mt], al, bh[q][0], bh[q][1]);
       }
     }
+    if (of_w) {
 #pragma unroll
-    for (int q = 0; q < 4; ++q) {
-      const int tile = t0 + q;
-      if (tile < NW) {
+      for (int q = 0; q < 4; ++q)
+        if (t0 + q < NW) {
 #pragma unroll
-        for (int mt = 0; mt < 4; ++mt)
-          *reinterpret_cast<float4*>(wg + ((static_cast<long long>(tile) * 4 + mt) * 32 + lane) * 4) = make_float4(acc[q][mt][0], acc[q][mt][2], acc[q][mt][1], acc[q][mt][3]);
-      } else if (tile < tiles) {
-        const int c = 8 * (tile - NW) + 2 * t;
+          for (int mt = 0; mt < 4; ++mt)
+            *reinterpret_cast<float4*>(wg + ((static_cast<long long>(t0 + q) * 4 + mt) * 32 + lane) * 4) = make_float4(acc[q][mt][0], acc[q][mt][2], acc[q][mt][1], acc[q][mt][3]);
+        }
+    } else {
 #pragma unroll
-        for (int mt = 0; mt < 4; ++mt)
+      for (int mt = 0; mt < 4; ++mt)
 #pragma unroll
-          for (int h = 0; h < 2; ++h) {
-            float* o = ug + static_cast<long long>(16 * mt + g + 8 * h) * V + c;
-            if (even) {
-              if (c < V) *reinterpret_cast<float2*>(o) = make_float2(acc[q][mt][2 * h], acc[q][mt][2 * h + 1]);
-            } else {
-              if (c < V) o[0] = acc[q][mt][2 * h];
-              if (c + 1 < V) o[1] = acc[q][mt][2 * h + 1];
-            }
+        for (int x = 0; x < 4; ++x) {   // place 2 t + (x & 1) of row 16 mt + g + 8 (x >> 1)
+          const int c = (grp - GW) * 32 + 4 * (2 * t + (x & 1));
+          float* o = ug + static_cast<long long>(16 * mt + g + 8 * (x >> 1)) * V + c;
+          if (quads) {
+            if (c < V) *reinterpret_cast<float4*>(o) = make_float4(acc[0][mt][x], acc[1][mt][x], acc[2][mt][x], acc[3][mt][x]);
+          } else {
+#pragma unroll
+            for (int q = 0; q < 4; ++q)
+              if (c + q < V) o[q] = acc[q][mt][x];
           }
-      }
+        }
     }
   }
 }
@@ -958,40 +987,53 @@ __global__ void __launch_bounds__(kDpThreads) delta_chunk_prep_head_kernel(const
   };
   if (kFast) {
     const int g = lane >> 2, t = lane & 3;
-    // 20 tiles of 16 x 8 pairs on and below the diagonal: row tile mi holds 2 (mi + 1) of them
-    for (int job = warp; job < 20; job += kWarps) {
-      const int mi = job < 2 ? 0 : job < 6 ? 1 : job < 12 ? 2 : 3, ni = job - mi * (mi + 1);
-      float q[3][4], k[3][4];
+    // ten tiles of 16 x 16 pairs on and below the diagonal, a warp each: (mi, nj) with nj <= mi
+    for (int job = warp; job < 10; job += kWarps) {
+      const int mi = job < 1 ? 0 : job < 3 ? 1 : job < 6 ? 2 : 3, nj = job - mi * (mi + 1) / 2;
+      float q[3][2][4], k[3][2][4];
 #pragma unroll
       for (int a = 0; a < 3; ++a)
 #pragma unroll
-        for (int x = 0; x < 4; ++x) q[a][x] = k[a][x] = 0.f;
+        for (int u = 0; u < 2; ++u)
+#pragma unroll
+          for (int x = 0; x < 4; ++x) q[a][u][x] = k[a][u][x] = 0.f;
       const float* qa = qs + (16 * mi + g) * DP + t;
       const float* ka = ks + (16 * mi + g) * DP + t;
-      const float* kn = ks + (8 * ni + g) * DP + t;
+      const float* kn = ks + (16 * nj + g) * DP + t;
 #pragma unroll 2
       for (int d = 0; d < D8; d += 8) {
-        uint32_t ah[4], al[4], h0, l0, h1, l1;
-        split_tf32(kn[d], h0, l0);
-        split_tf32(kn[d + 4], h1, l1);
+        uint32_t ah[4], al[4], bh[2][2], bl[2][2];
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          split_tf32(kn[8 * u * DP + d], bh[u][0], bl[u][0]);
+          split_tf32(kn[8 * u * DP + d + 4], bh[u][1], bl[u][1]);
+        }
         split_tf32(qa[d], ah[0], al[0]);
         split_tf32(qa[d + 8 * DP], ah[1], al[1]);
         split_tf32(qa[d + 4], ah[2], al[2]);
         split_tf32(qa[d + 8 * DP + 4], ah[3], al[3]);
-        mma_tf32(q[0], ah, h0, h1);
-        mma_tf32(q[1], ah, l0, l1);
-        mma_tf32(q[2], al, h0, h1);
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          mma_tf32(q[0][u], ah, bh[u][0], bh[u][1]);
+          mma_tf32(q[1][u], ah, bl[u][0], bl[u][1]);
+          mma_tf32(q[2][u], al, bh[u][0], bh[u][1]);
+        }
         split_tf32(ka[d], ah[0], al[0]);
         split_tf32(ka[d + 8 * DP], ah[1], al[1]);
         split_tf32(ka[d + 4], ah[2], al[2]);
         split_tf32(ka[d + 8 * DP + 4], ah[3], al[3]);
-        mma_tf32(k[0], ah, h0, h1);
-        mma_tf32(k[1], ah, l0, l1);
-        mma_tf32(k[2], al, h0, h1);
+#pragma unroll
+        for (int u = 0; u < 2; ++u) {
+          mma_tf32(k[0][u], ah, bh[u][0], bh[u][1]);
+          mma_tf32(k[1][u], ah, bl[u][0], bl[u][1]);
+          mma_tf32(k[2][u], al, bh[u][0], bh[u][1]);
+        }
       }
 #pragma unroll
-      for (int x = 0; x < 4; ++x)
-        put(16 * mi + g + 8 * (x >> 1), 8 * ni + 2 * t + (x & 1), q[0][x] + (q[1][x] + q[2][x]), k[0][x] + (k[1][x] + k[2][x]));
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int x = 0; x < 4; ++x)
+          put(16 * mi + g + 8 * (x >> 1), 16 * nj + 8 * u + 2 * t + (x & 1), q[0][u][x] + (q[1][u][x] + q[2][u][x]), k[0][u][x] + (k[1][u][x] + k[2][u][x]));
     }
   } else {
     for (int e = tid; e < (kC / 2) * (kC / 2 + 1) / 2; e += kDpThreads) {   // 2 x 2 pairs on and below the diagonal
@@ -1495,89 +1537,117 @@ static int launch_delta_chunk_scan(const pcs_delta_chunk_params& p, size_t smem,
 }
 
 // ---- read-out of the chunks (bfloat16 runs) ---------------------------------------------------------------------------------------
-// Block = (chunk, head), a warp = 32 value columns: o = qd S + a u over dim + 64 terms (TF32 hi + lo operands; [qd | a] staged in shared memory,
-// S and u read once, a step ahead), then the head's norm and gate on the accumulators, and the result's rows.
+// Block = (chunk, head), a warp = 32 value columns: o = qd S + a u over dim + 64 terms, then the head's norm and gate on the accumulators, and the
+// result's rows.  The result leaves in bfloat16, so the operands enter as hi + lo bfloat16 pairs (hi hi + hi lo + lo hi in 32-bit accumulators,
+// about 2^-16 of a product); the state itself stays as it is.  [qd | a] is staged in shared memory as such pairs, S and u are read once, a step ahead.
 constexpr int kDoMaxWarps = 16;
 
 __global__ void __launch_bounds__(kDoMaxWarps * 32) delta_chunk_out_kernel(const pcs_delta_chunk_params p, const pcs_headnorm_params o) {
   extern __shared__ __align__(16) float sm[];
-  const int D = p.dim, V = p.vdim, H = p.heads, D8 = (D + 7) & ~7, LD = ((D8 + kC + 31) & ~31) + 4;
-  float* A = sm;                   // [64][LD]
-  float* red = A + kC * LD;        // [warps][64], then [64]
+  const int D = p.dim, V = p.vdim, H = p.heads, D16 = (D + 15) & ~15, LD = D16 + kC + 8;   // (rows an odd number of 16-byte pieces apart)
+  __nv_bfloat16* Ah = reinterpret_cast<__nv_bfloat16*>(sm);   // [64][LD]
+  __nv_bfloat16* Al = Ah + kC * LD;                           // [64][LD]
+  float* red = reinterpret_cast<float*>(Al + kC * LD);        // [warps][64], then [64]
   const int cn = blockIdx.x, head = blockIdx.y, tid = threadIdx.x, nthr = blockDim.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t = lane & 3;
   const long long base = static_cast<long long>(cn) * H + head;
   const int first = p.chunk_first[cn], n = p.chunk_len[cn];
   const float* qd = p.qd + base * kC * D;
   const float* ag = p.a + base * kC * kC;
-  if (D % 4 == 0) {
-    for (int e = tid; e < kC * (D / 4); e += nthr) {
-      const int i = e / (D / 4), c = (e - i * (D / 4)) * 4;
-      cp_async16(A + i * LD + c, qd + i * D + c);
-    }
-  } else {
-    for (int e = tid; e < kC * D; e += nthr) {
-      const int i = e / D, c = e - i * D;
-      A[i * LD + c] = qd[e];
-    }
-  }
-  for (int e = tid; e < kC * (D8 - D); e += nthr) {
-    const int i = e / (D8 - D);
-    A[i * LD + D + (e - i * (D8 - D))] = 0.f;
-  }
-  for (int e = tid; e < kC * (kC / 4); e += nthr) cp_async16(A + (e >> 4) * LD + D8 + (e & 15) * 4, ag + e * 4);
-  cp_async_commit();
-  const int c0 = warp * 32 + g, KD = D8 / 8, KT = KD + kC / 8;
+  auto put = [&](int i, int c, const float (&x)[4]) {
+    uint2 hi, lo;
+    hi.x = split_pair(x[0], x[1], lo.x);
+    hi.y = split_pair(x[2], x[3], lo.y);
+    *reinterpret_cast<uint2*>(Ah + i * LD + c) = hi;
+    *reinterpret_cast<uint2*>(Al + i * LD + c) = lo;
+  };
+  // (place x of the warp's tile q is its column 4 x + q: a lane's four values of a row are neighbours)
+  const int c0 = warp * 32 + 4 * g, KD = D16 / 16, KT = KD + kC / 16;
   const float* sg = p.s + base * D * V;
   const float* ug = p.u + base * kC * V;
-  auto load = [&](int kt, float (&b)[4][2]) {
+  const bool quads = V % 4 == 0;
+  auto load = [&](int kt, float (&b)[4][4]) {   // rows 2t, 2t + 1, 2t + 8, 2t + 9 of the step's 16
+    const bool state = kt < KD;
+    const int r0 = 16 * (state ? kt : kt - KD) + 2 * t;
+    const float* src = (state ? sg : ug) + static_cast<long long>(r0) * V + c0;
 #pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      const int r = 8 * (kt < KD ? kt : kt - KD) + t + 4 * h;
-      const float* src = (kt < KD ? sg : ug) + static_cast<long long>(r) * V;
-      const bool ok = kt < KT && (kt >= KD || r < D);
-#pragma unroll
-      for (int q = 0; q < 4; ++q) b[q][h] = ok && c0 + 8 * q < V ? src[c0 + 8 * q] : 0.f;
+    for (int h = 0; h < 4; ++h) {
+      const int dr = (h & 1) + 8 * (h >> 1);
+      const bool ok = kt < KT && (!state || r0 + dr < D);
+      float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+      const float* r = src + static_cast<long long>(dr) * V;
+      if (ok && quads) {
+        if (c0 < V) x = *reinterpret_cast<const float4*>(r);
+      } else if (ok) {
+        if (c0 < V) x.x = r[0];
+        if (c0 + 1 < V) x.y = r[1];
+        if (c0 + 2 < V) x.z = r[2];
+        if (c0 + 3 < V) x.w = r[3];
+      }
+      b[0][h] = x.x;
+      b[1][h] = x.y;
+      b[2][h] = x.z;
+      b[3][h] = x.w;
     }
   };
-  float acc[4][4][4], nx[2][4][2];
+  float acc[4][4][4], nx[4][4];
 #pragma unroll
   for (int q = 0; q < 4; ++q)
 #pragma unroll
     for (int m = 0; m < 4; ++m) acc[q][m][0] = acc[q][m][1] = acc[q][m][2] = acc[q][m][3] = 0.f;
-  load(0, nx[0]);
-  load(1, nx[1]);
-  cp_async_wait<0>();
+  load(0, nx);
+  const int per = D16 / 4, pieces = kC * (per + kC / 4);   // a row's pieces of qd, then of a
+  for (int e0 = tid; e0 < pieces; e0 += 4 * nthr) {        // (four requests before the first is used)
+    float x[4][4];
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int e = e0 + k * nthr;
+      x[k][0] = x[k][1] = x[k][2] = x[k][3] = 0.f;
+      if (e < pieces) {
+        const int i = e / (per + kC / 4), c = e - i * (per + kC / 4);
+        if (c >= per) {
+          ldx(ag + i * kC + (c - per) * 4, x[k]);
+        } else if (D % 4 == 0) {
+          if (4 * c < D) ldx(qd + i * D + 4 * c, x[k]);
+        } else {
+#pragma unroll
+          for (int y = 0; y < 4; ++y)
+            if (4 * c + y < D) x[k][y] = qd[i * D + 4 * c + y];
+        }
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int e = e0 + k * nthr;
+      if (e < pieces) {
+        const int i = e / (per + kC / 4);
+        put(i, 4 * (e - i * (per + kC / 4)), x[k]);
+      }
+    }
+  }
   __syncthreads();
-  auto step = [&](int kt, float (&b)[4][2]) {
+  const uint32_t a_hi = static_cast<uint32_t>(__cvta_generic_to_shared(Ah)) + ((lane & 15) * LD + (lane >> 4) * 8) * 2, a_lo = a_hi + kC * LD * 2;
+#pragma unroll 1
+  for (int kt = 0; kt < KT; ++kt) {
     uint32_t bh[4][2], bl[4][2];
 #pragma unroll
     for (int q = 0; q < 4; ++q) {
-      split_tf32(b[q][0], bh[q][0], bl[q][0]);
-      split_tf32(b[q][1], bh[q][1], bl[q][1]);
+      bh[q][0] = split_pair(nx[q][0], nx[q][1], bl[q][0]);
+      bh[q][1] = split_pair(nx[q][2], nx[q][3], bl[q][1]);
     }
-    load(kt + 2, b);
-    if (kt >= KT) return;
+    load(kt + 1, nx);
 #pragma unroll
     for (int m = 0; m < 4; ++m) {
-      if (kt >= KD && 16 * m + 15 < 8 * (kt - KD)) continue;   // `a` is zero above the diagonal
-      const float* a = A + (16 * m + g) * LD + 8 * kt + t;
-      uint32_t ah[4], al[4];
-      split_tf32(a[0], ah[0], al[0]);
-      split_tf32(a[8 * LD], ah[1], al[1]);
-      split_tf32(a[4], ah[2], al[2]);
-      split_tf32(a[8 * LD + 4], ah[3], al[3]);
+      if (m < kt - KD) continue;   // `a` is zero above the diagonal
+      uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
+      ldsm_x4(a_hi + (m * 16 * LD + kt * 16) * 2, h0, h1, h2, h3);
+      ldsm_x4(a_lo + (m * 16 * LD + kt * 16) * 2, l0, l1, l2, l3);
 #pragma unroll
-      for (int q = 0; q < 4; ++q) mma_tf32(acc[q][m], ah, bh[q][0], bh[q][1]);
+      for (int q = 0; q < 4; ++q) mma_bf16(acc[q][m], h0, h1, h2, h3, bh[q][0], bh[q][1]);
 #pragma unroll
-      for (int q = 0; q < 4; ++q) mma_tf32(acc[q][m], ah, bl[q][0], bl[q][1]);
+      for (int q = 0; q < 4; ++q) mma_bf16(acc[q][m], h0, h1, h2, h3, bl[q][0], bl[q][1]);
 #pragma unroll
-      for (int q = 0; q < 4; ++q) mma_tf32(acc[q][m], al, bh[q][0], bh[q][1]);
+      for (int q = 0; q < 4; ++q) mma_bf16(acc[q][m], l0, l1, l2, l3, bh[q][0], bh[q][1]);
     }
-  };
-#pragma unroll 1
-  for (int kt = 0; kt < KT; kt += 2) {
-    step(kt, nx[0]);
-    step(kt + 1, nx[1]);
   }
   // the head's mean square per token: a row's columns are spread over 4 lanes and all warps
 #pragma unroll
@@ -1603,38 +1673,51 @@ __global__ void __launch_bounds__(kDoMaxWarps * 32) delta_chunk_out_kernel(const
   const __nv_bfloat16* gate = static_cast<const __nv_bfloat16*>(o.g) + static_cast<long long>(first) * o.g_stride + head * V;
   const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(o.w);
   __nv_bfloat16* out = static_cast<__nv_bfloat16*>(o.out) + static_cast<long long>(first) * o.out_stride + head * V;
-  const bool pairs = V % 2 == 0 && o.out_stride % 2 == 0 && o.g_stride % 2 == 0 && ((reinterpret_cast<uintptr_t>(o.g) | reinterpret_cast<uintptr_t>(o.out) | reinterpret_cast<uintptr_t>(o.w)) & 3) == 0;
+  const bool vec = quads && o.out_stride % 4 == 0 && o.g_stride % 4 == 0 && ((reinterpret_cast<uintptr_t>(o.g) | reinterpret_cast<uintptr_t>(o.out) | reinterpret_cast<uintptr_t>(o.w)) & 7) == 0;
+  auto unpack = [](const uint2& v, float (&f)[4]) {
+    f[0] = __uint_as_float(v.x << 16);
+    f[1] = __uint_as_float(v.x & 0xffff0000u);
+    f[2] = __uint_as_float(v.y << 16);
+    f[3] = __uint_as_float(v.y & 0xffff0000u);
+  };
   auto gated = [&](float x, float f, float wv, float gv) { return x * f * wv * sigmoidf_(gv) * (o.silu ? gv : 1.f); };
 #pragma unroll
-  for (int q = 0; q < 4; ++q) {
-    const int c = warp * 32 + 8 * q + 2 * t;
+  for (int e = 0; e < 2; ++e) {   // this lane's columns c .. c + 3 (places 2t + e), eight tokens: all gates are requested before the first result leaves
+    const int c = warp * 32 + 4 * (2 * t + e);
     if (c >= V) continue;
-    float w0, w1 = 0.f;
-    if (pairs) {
-      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(w + c));
-      w0 = f.x;
-      w1 = f.y;
-    } else {
-      w0 = ldf(w + c);
-      if (c + 1 < V) w1 = ldf(w + c + 1);
-    }
+    if (vec) {
+      uint2 gv[8];
 #pragma unroll
-    for (int m = 0; m < 4; ++m)
+      for (int k = 0; k < 8; ++k) {
+        const int i = 16 * (k >> 1) + g + 8 * (k & 1);
+        gv[k] = i < n ? *reinterpret_cast<const uint2*>(gate + static_cast<long long>(i) * o.g_stride + c) : make_uint2(0u, 0u);
+      }
+      float wv[4];
+      unpack(*reinterpret_cast<const uint2*>(w + c), wv);
 #pragma unroll
-      for (int h = 0; h < 2; ++h) {
-        const int i = 16 * m + g + 8 * h;
+      for (int k = 0; k < 8; ++k) {
+        const int m = k >> 1, x = 2 * (k & 1) + e, i = 16 * m + g + 8 * (k & 1);
         if (i >= n) continue;
         const float f = red[i];
-        const __nv_bfloat16* gr = gate + static_cast<long long>(i) * o.g_stride + c;
-        __nv_bfloat16* r = out + static_cast<long long>(i) * o.out_stride + c;
-        if (pairs) {
-          const float2 gv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gr));
-          *reinterpret_cast<uint32_t*>(r) = pack_bf16(gated(acc[q][m][2 * h], f, w0, gv.x), gated(acc[q][m][2 * h + 1], f, w1, gv.y));
-        } else {
-          stf(r, gated(acc[q][m][2 * h], f, w0, ldf(gr)));
-          if (c + 1 < V) stf(r + 1, gated(acc[q][m][2 * h + 1], f, w1, ldf(gr + 1)));
-        }
+        float gf[4];
+        unpack(gv[k], gf);
+        uint2 r;
+        r.x = pack_bf16(gated(acc[0][m][x], f, wv[0], gf[0]), gated(acc[1][m][x], f, wv[1], gf[1]));
+        r.y = pack_bf16(gated(acc[2][m][x], f, wv[2], gf[2]), gated(acc[3][m][x], f, wv[3], gf[3]));
+        *reinterpret_cast<uint2*>(out + static_cast<long long>(i) * o.out_stride + c) = r;
       }
+    } else {
+#pragma unroll
+      for (int k = 0; k < 8; ++k) {
+        const int m = k >> 1, x = 2 * (k & 1) + e, i = 16 * m + g + 8 * (k & 1);
+        if (i >= n) continue;
+        const float f = red[i];
+#pragma unroll
+        for (int q = 0; q < 4; ++q)
+          if (c + q < V)
+            stf(out + static_cast<long long>(i) * o.out_stride + c + q, gated(acc[q][m][x], f, ldf(w + c + q), ldf(gate + static_cast<long long>(i) * o.g_stride + c + q)));
+      }
+    }
   }
 }
 
@@ -1815,8 +1898,8 @@ PCS_API int pcs_delta_chunk_out(const pcs_delta_chunk_params* p, const pcs_headn
   PCS_REQUIRE(p->dtype == PCS_BF16 && p->heads > 0 && p->heads <= 65535 && p->dim > 0 && p->dim <= 256 && p->vdim > 0 && p->vdim <= 32 * pcs::kDoMaxWarps,
               "pcs_delta_chunk_out: serves bfloat16, dim up to 256 and vdim up to %d", 32 * pcs::kDoMaxWarps);
   PCS_REQUIRE(((reinterpret_cast<uintptr_t>(p->qd) | reinterpret_cast<uintptr_t>(p->a)) & 15) == 0, "pcs_delta_chunk_out: qd and a must be 16-byte aligned");
-  const int warps = (p->vdim + 31) / 32 < 2 ? 2 : (p->vdim + 31) / 32, D8 = (p->dim + 7) & ~7;
-  const size_t smem = (static_cast<size_t>(pcs::kC) * (((D8 + pcs::kC + 31) & ~31) + 4) + static_cast<size_t>(warps) * pcs::kC) * sizeof(float);
+  const int warps = (p->vdim + 31) / 32 < 2 ? 2 : (p->vdim + 31) / 32, D16 = (p->dim + 15) & ~15;
+  const size_t smem = static_cast<size_t>(2) * pcs::kC * (D16 + pcs::kC + 8) * sizeof(__nv_bfloat16) + static_cast<size_t>(warps) * pcs::kC * sizeof(float);
   PCS_CHECK_CUDA(cudaFuncSetAttribute(pcs::delta_chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
   pcs::delta_chunk_out_kernel<<<dim3(p->n_chunks, p->heads), warps * 32, smem, static_cast<cudaStream_t>(stream)>>>(*p, *o);
   PCS_CHECK_CUDA(cudaGetLastError());
