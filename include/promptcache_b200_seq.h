@@ -66,7 +66,7 @@
 extern "C" {
 #endif
 
-#define PCS_ABI_VERSION 5
+#define PCS_ABI_VERSION 6
 #define PCS_BF16 0
 #define PCS_F32 1
 

@@ -1,6 +1,6 @@
 // Gated delta rule over the slot pool.
 //
-// Per head, with a decay per key channel and a step size beta in (0, 1):
+// Per head, with a decay per key channel (or one per head, formed here from its pre-activation) and a step size beta in (0, 1):
 //     S <- diag(decay_t) S;   u = beta_t (v_t - S^T k_t);   S <- S + k_t u^T;   o_t = S^T q_t          (S: dim x vdim, 32-bit)
 // q, k and v come out of a short causal convolution with silu; q and k are unit vectors per head.
 //
@@ -11,7 +11,8 @@
 //                       (sequence, head, slice of columns): state in registers (dim <= 256, aligned) or in shared memory.
 // pcs_delta_chunk_prep  prompts: everything about a chunk of 64 tokens that does not need the state it starts from.
 // pcs_delta_chunk_scan  prompts: the chunks in order, two products per chunk on a slice of columns held in shared memory.
-// pcs_head_norm_gate    per-head norm and sigmoid gate of the recurrence's result.
+// pcs_delta_chunk_out   prompts in bfloat16: the read-out of the chunks with the per-head norm and gate.
+// pcs_head_norm_gate    per-head norm and sigmoid (or silu) gate of the recurrence's result.
 #include "seq_common.cuh"
 #include "seq_mma.cuh"
 
